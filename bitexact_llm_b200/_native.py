@@ -1,6 +1,7 @@
-"""ctypes binding of libbitexact_b200.so (C ABI in include/bitexact_b200.h).
+"""ctypes bindings of libbitexact_b200.so (`lib()`, C ABI in include/bitexact_b200.h: integer engines, sampler) and
+libbitexact_float.so (`float_lib()`, include/bitexact_float.h: float models).
 
-The library is built in-tree by `bitexact_llm_b200.build` (nvcc, sm_100a).  Loading fails loudly when it is
+The libraries are built in-tree by `bitexact_llm_b200.build` (nvcc, sm_100a).  Loading fails loudly when one is
 missing: there is deliberately no fallback path.
 """
 
@@ -9,15 +10,16 @@ import os
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "_lib", "libbitexact_b200.so")
+FLOAT_LIB_PATH = os.path.join(_HERE, "_lib", "libbitexact_float.so")
 
 BX_OK, BX_EARG, BX_ELAUNCH, BX_EDEVICE, BX_ELIMIT = 0, -1, -2, -3, -4
 _ERR = {BX_EARG: "argument contract violated (shape / alignment / null pointer)",
         BX_ELAUNCH: "CUDA launch or driver call failed", BX_EDEVICE: "a device-side wait timed out",
         BX_ELIMIT: "request exceeds the fixed capacity of this entry point"}
 
-_lib = None
+_libs = {}
 
-P, I, L, Z = ctypes.c_void_p, ctypes.c_int, ctypes.c_int64, ctypes.c_size_t
+P, I, L, Z, R = ctypes.c_void_p, ctypes.c_int, ctypes.c_int64, ctypes.c_size_t, ctypes.c_float
 
 _SIGNATURES = {
     "bx_version": (I, []),
@@ -83,22 +85,65 @@ _SIGNATURES = {
 }
 
 
-def lib():
-    global _lib
-    if _lib is None:
-        if not os.path.exists(LIB_PATH):
-            raise RuntimeError(f"{LIB_PATH} is missing: build it with `python -m bitexact_llm_b200.build` "
+
+class Epilogue(ctypes.Structure):
+    """bxf_epilogue."""
+    _fields_ = [("kind", I), ("out_type", I), ("act", I), ("n_main", I), ("act_p", R), ("act_q", R), ("out", P), ("ldo", L),
+                ("gso", L), ("side", P), ("lds", L), ("bias", P), ("gate", P), ("ldg", L), ("cs", P), ("rot_out", P),
+                ("ldr", L), ("hsr", L), ("rot_dim", I), ("pad_", I)]
+
+
+class Gru(ctypes.Structure):
+    """bxf_gru."""
+    _fields_ = [("bias_z", P), ("bias_x", P), ("state", P), ("flags", P), ("seq", P), ("out", P), ("ldo", L), ("decay", P),
+                ("local", P), ("mode", I), ("pad_", I)]
+
+
+_FLOAT_SIGNATURES = {
+    "bxf_version": (I, []),
+    "bxf_launch_count": (ctypes.c_longlong, []),
+    "bxf_device_status": (I, []),
+    "bxf_clear_device_status": (I, []),
+    "bxf_set_device_status": (I, [I]),
+    "bxf_linear": (I, [I, P, L, L, P, L, L, I, I, I, I, P, ctypes.POINTER(Epilogue), I, P]),
+    "bxf_gru_tile_rows": (I, [I]),
+    "bxf_gru_long_tile": (I, [I]),
+    "bxf_gru_linear": (I, [I, P, L, P, L, I, I, I, ctypes.POINTER(Gru), P]),
+    "bxf_gru_finish": (I, [I, I, I, ctypes.POINTER(Gru), P]),
+    "bxf_row_flags": (I, [P, P, P, P, I, P]),
+    "bxf_norm": (I, [I, P, P, P, L, P, P, P, I, P, P, R, P, L, P, I, I, I, P]),
+    "bxf_route": (I, [P, L, I, I, P, P, P, P, I, P]),
+    "bxf_gather": (I, [I, P, L, I, P, P, P, I, I, P, P, I, P]),
+    "bxf_latent_prepare": (I, [I, P, L, I, I, I, I, P, P, R, P, P, P, P, L, P, L, P, P, I, P]),
+    "bxf_latent_attention_scratch": (Z, [I, I, I]),
+    "bxf_latent_attention_tile": (I, [I]),
+    "bxf_latent_attention": (I, [I, P, L, I, I, I, I, P, L, I, I, P, I, L, I, P, P, P, I, I, P, R, P, L, P, Z, I, P]),
+}
+
+
+def _load(path, signatures):
+    if path not in _libs:
+        if not os.path.exists(path):
+            raise RuntimeError(f"{path} is missing: build it with `python -m bitexact_llm_b200.build` "
                                "(nvcc, sm_100a). There is no fallback path.")
-        h = ctypes.CDLL(LIB_PATH)
-        for name, (res, args) in _SIGNATURES.items():
+        h = ctypes.CDLL(path)
+        for name, (res, args) in signatures.items():
             fn = getattr(h, name)                       # AttributeError if the library is stale
             fn.restype, fn.argtypes = res, args
-        _lib = h
-    return _lib
+        _libs[path] = h
+    return _libs[path]
 
 
-def exported_symbols():
-    return sorted(_SIGNATURES)
+def lib():
+    return _load(LIB_PATH, _SIGNATURES)
+
+
+def float_lib():
+    return _load(FLOAT_LIB_PATH, _FLOAT_SIGNATURES)
+
+
+def exported_symbols(float_models=False):
+    return sorted(_FLOAT_SIGNATURES if float_models else _SIGNATURES)
 
 
 def check(rc, what):
@@ -121,6 +166,11 @@ def device_status():
     return lib().bx_device_status()
 
 
+def float_device_status():
+    """`device_status` of the float-model library."""
+    return float_lib().bxf_device_status()
+
+
 def clear_device_status():
     check(lib().bx_clear_device_status(), "bx_clear_device_status")
 
@@ -138,10 +188,10 @@ class DeviceWaitError(RuntimeError):
     """A bounded device-side wait gave up: kernels launched since then may have left their outputs unwritten."""
 
 
-def check_device_status():
+def check_device_status(status=device_status):
     """Raises DeviceWaitError when the device status word is non-zero (the state stays set until
     `clear_device_status`)."""
-    n = device_status()
+    n = status()
     if n != 0:
         raise DeviceWaitError(f"{n} device-side wait(s) timed out: results since then are not valid; "
                               "call clear_device_status() and rerun the step")

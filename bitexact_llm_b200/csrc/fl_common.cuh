@@ -1,0 +1,71 @@
+// Shared pieces of the float-model kernels: element types, scalar functions, row flags.
+#pragma once
+
+#include <cuda_bf16.h>
+#include <stdint.h>
+
+#include "bx_ptx.cuh"
+
+namespace bxf {
+
+using bf16 = __nv_bfloat16;
+using i64 = long long;
+
+template <class T>
+__device__ __forceinline__ float ld(const T* p);
+template <>
+__device__ __forceinline__ float ld<float>(const float* p) { return *p; }
+template <>
+__device__ __forceinline__ float ld<bf16>(const bf16* p) { return __bfloat162float(*p); }
+
+__device__ __forceinline__ void st(float* p, float v) { *p = v; }
+__device__ __forceinline__ void st(bf16* p, float v) { *p = __float2bfloat16(v); }
+
+// sigmoid(v) and 1 - sigmoid(v), both without cancellation.
+__device__ __forceinline__ void sigmoid_pair(float v, float& s, float& one_minus_s) {
+  const float e = expf(-fabsf(v)), r = 1.0f / (1.0f + e);
+  s = v >= 0.0f ? r : e * r;
+  one_minus_s = v >= 0.0f ? e * r : r;
+}
+
+__device__ __forceinline__ float sigmoid(float v) { return 1.0f / (1.0f + expf(-v)); }
+__device__ __forceinline__ float silu(float v) { return v / (1.0f + expf(-v)); }
+
+__device__ __forceinline__ float activate(int act, float z, float p, float q) {
+  if (act == BXF_ACT_RELU2) {
+    const float r = fmaxf(z, 0.0f);
+    return r * r;
+  }
+  if (act == BXF_ACT_XIELU) return (z > 0.0f ? p * z * z : q * (expm1f(z) - z)) + 0.5f * z;
+  return z;
+}
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
+
+__device__ __forceinline__ float warp_max(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
+  return v;
+}
+
+// Sum over the block (a multiple of 32 threads, at most 1024); `red` holds 33 floats.
+__device__ __forceinline__ float block_sum(float v, float* red) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  v = warp_sum(v);
+  __syncthreads();                                       // red may still be read from the previous sum
+  if (lane == 0) red[warp] = v;
+  __syncthreads();
+  if (warp == 0) {
+    float t = lane < warps ? red[lane] : 0.0f;
+    t = warp_sum(t);
+    if (lane == 0) red[32] = t;
+  }
+  __syncthreads();
+  return red[32];
+}
+
+}  // namespace bxf

@@ -1,0 +1,166 @@
+// Epilogues of the float products. A product kernel computes a tile of 128 weight rows x TA token rows; an epilogue
+// thread owns ONE weight row (output channel) n and walks token columns, so per-channel constants live in registers, a
+// warp stores 32 consecutive channels of a token, a rotated pair is two neighbouring lanes, and a recurrence over tokens
+// is a loop of one thread. The kernels hand the accumulators over through a `get` object:
+//   get.template load<W>(plane, column, v)   W consecutive token columns of one product plane
+// which reads TMEM, the summed partials of a K-split cluster, or registers. All calls are warp-collective.
+#pragma once
+
+#include "fl_common.cuh"
+
+namespace bxf {
+
+constexpr int NROWS = 128;           // weight rows of a tile
+constexpr int EPI_THREADS = 512;     // epilogue threads: 16 warps, four per quarter of the 128 rows when K is not split
+
+struct Tile {
+  int group, n0;                     // weight plane, first weight row
+  int row0, rows;                    // first token row, token rows that exist (<= TA)
+};
+
+__device__ __forceinline__ void epi_barrier() { asm volatile("bar.sync 1, 512;" ::: "memory"); }
+
+// ---- elementwise epilogues (bxf_epilogue) ----
+struct StageEpi {
+  using Params = bxf_epilogue;
+  static constexpr int PLANES = 1;
+  static __host__ __device__ constexpr int stash_bytes(int) { return 0; }
+
+  template <class T>
+  static __device__ __forceinline__ void chunk(const Params& p, int group, int n, int N, i64 row, int cnt,
+                                               const float (&v)[8]) {
+    if (p.kind == BXF_EPI_ROPE) {
+      const int r = n - p.n_main, j = r >= 0 ? r % p.rot_dim : 0, h = r >= 0 ? r / p.rot_dim : 0;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const float other = __shfl_xor_sync(0xffffffffu, v[i], 1);
+        if (i >= cnt || n >= N) continue;
+        if (r < 0) {
+          st(static_cast<T*>(p.out) + (row + i) * p.ldo + n, v[i]);
+        } else {
+          const float2 cs = *reinterpret_cast<const float2*>(p.cs + ((row + i) * (p.rot_dim / 2) + (j >> 1)) * 2);
+          st(static_cast<T*>(p.rot_out) + (row + i) * p.ldr + h * p.hsr + j,
+             (j & 1) ? v[i] * cs.x + other * cs.y : v[i] * cs.x - other * cs.y);
+        }
+      }
+      return;
+    }
+    if (n >= N) return;
+    if (p.kind == BXF_EPI_ADD) {
+      float* o = static_cast<float*>(p.out) + row * p.ldo + n;
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if (i < cnt) o[i * p.ldo] += v[i];
+    } else if (p.kind == BXF_EPI_GATE) {
+      T* o = static_cast<T*>(p.out) + group * p.gso + row * p.ldo + n;
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if (i < cnt) st(o + i * p.ldo, v[i] * p.gate[(row + i) * p.ldg + group]);
+    } else if (n >= p.n_main) {
+      const float b = p.bias ? p.bias[n - p.n_main] : 0.0f;
+      float* o = p.side + row * p.lds + (n - p.n_main);
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if (i < cnt) o[i * p.lds] = v[i] + b;
+    } else {
+      const i64 at = group * p.gso + row * p.ldo + n;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        if (i >= cnt) break;
+        const float y = activate(p.act, v[i], p.act_p, p.act_q);
+        if (p.out_type == BXF_OUT_T) st(static_cast<T*>(p.out) + at + i * p.ldo, y);
+        else if (p.out_type == BXF_OUT_F32) static_cast<float*>(p.out)[at + i * p.ldo] = y;
+        else static_cast<i64*>(p.out)[at + i * p.ldo] = __double2ll_rn((double)y * 16777216.0);
+      }
+    }
+  }
+
+  // groups: how many warps share a row (they take chunks of 8 columns in turn).
+  template <class T, int TA, int W, class Get>
+  static __device__ __forceinline__ void run(Get& get, const Params& p, const Tile& t, int N, int row, int group_index,
+                                             int groups, uint8_t*) {
+    for (int c = group_index * 8; c < TA && c < t.rows; c += groups * 8) {
+      float v[8];
+      get.template load<8>(0, c, v);
+      chunk<T>(p, t.group, t.n0 + row, N, (i64)t.row0 + c, min(8, t.rows - c), v);
+    }
+  }
+};
+
+// ---- minGRU: gates and recurrence along the token columns ----
+// The recurrence S_t = a_t S_(t-1) + b_t over a tile is a scan split over the warps of a row: every warp folds its
+// columns to one (a, b) pair, the pairs of the warps before it give its start, and a second walk produces the states.
+// At the first row of a sequence the state of its slot enters b and a becomes 0, so tiles need not know sequences.
+// a and b of the first walk stay in shared memory for the second one (the slots of `state` may be rewritten by then).
+struct GruEpi {
+  using Params = bxf_gru;
+  static constexpr int PLANES = 3;
+  static __host__ __device__ constexpr int stash_bytes(int ta) { return 2 * ta * NROWS * 4 + 16 * NROWS * 8; }
+
+  template <class T, int TA, int W, class Get>
+  static __device__ __forceinline__ void run(Get& get, const Params& p, const Tile& t, int N, int row, int group_index,
+                                             int groups, uint8_t* stash) {
+    float* sa = reinterpret_cast<float*>(stash);                        // [TA][128]
+    float* sb = sa + TA * NROWS;
+    float2* fold = reinterpret_cast<float2*>(sb + TA * NROWS);          // [warp of the row][128]
+    const int per = TA / groups, c_begin = group_index * per, c_end = min(c_begin + per, t.rows);
+    const int n = t.n0 + row;
+    const bool live = n < N;
+    const float bz = live ? p.bias_z[n] : 0.0f, bx = live ? p.bias_x[n] : 0.0f;
+    float A = 1.0f, B = 0.0f;
+    for (int c = c_begin; c < c_end; c += W) {
+      float z[W], u[W];
+      get.template load<W>(0, c, z);
+      get.template load<W>(1, c, u);
+#pragma unroll
+      for (int i = 0; i < W; ++i) {
+        if (c + i >= c_end) break;
+        float s, a;
+        sigmoid_pair(z[i] + bz, s, a);
+        const float x = u[i] + bx;
+        float b = s * (x >= 0.0f ? x + 0.5f : sigmoid(x));
+        const int f = p.flags[t.row0 + c + i];
+        if (f & BXF_ROW_FIRST) {
+          if (live && !(f & (BXF_ROW_START | BXF_ROW_PAD))) b += a * p.state[p.seq[t.row0 + c + i] * N + n];
+          a = 0.0f;
+        }
+        sa[(c + i) * NROWS + row] = a;
+        sb[(c + i) * NROWS + row] = b;
+        B = B * a + b;
+        A *= a;
+      }
+    }
+    fold[group_index * NROWS + row] = make_float2(A, B);
+    epi_barrier();
+    float P = 1.0f, S = 0.0f;
+    for (int k = 0; k < group_index; ++k) {
+      const float2 f = fold[k * NROWS + row];
+      S = S * f.x + f.y;
+      P *= f.x;
+    }
+    for (int c = c_begin; c < c_end; c += W) {
+      float g[W];
+      get.template load<W>(2, c, g);
+#pragma unroll
+      for (int i = 0; i < W; ++i) {
+        if (c + i >= c_end) break;
+        const float a = sa[(c + i) * NROWS + row];
+        S = S * a + sb[(c + i) * NROWS + row];
+        P *= a;
+        if (!live) continue;
+        const i64 m = t.row0 + c + i;
+        T* o = static_cast<T*>(p.out) + m * p.ldo + n;
+        if (p.mode == 0) {
+          st(o, S * silu(g[i]));
+          if (p.flags[m] & BXF_ROW_LAST) p.state[p.seq[m] * N + n] = S;
+        } else {
+          st(o, silu(g[i]));
+          p.decay[m * N + n] = P;
+          p.local[m * N + n] = S;
+        }
+      }
+    }
+  }
+};
+
+}  // namespace bxf

@@ -1,0 +1,212 @@
+// Memory-bound stages of the float models: row flags, embedding / expert combination + layer norm, expert routing and
+// gathering, the preparation of latent attention, the second pass of a long minGRU scan. All arithmetic is 32-bit.
+#pragma once
+
+#include "fl_common.cuh"
+
+namespace bxf {
+
+__global__ void fl_row_flags_kernel(const i64* seq, const i64* slot, const i64* pos, int* flags, int M) {
+  const int m = blockIdx.x * blockDim.x + threadIdx.x;
+  if (m >= M) return;
+  if (slot[m] < 0) {
+    flags[m] = BXF_ROW_PAD | BXF_ROW_FIRST;
+    return;
+  }
+  const bool first = m == 0 || seq[m - 1] != seq[m] || slot[m - 1] < 0;
+  const bool last = m == M - 1 || seq[m + 1] != seq[m] || slot[m + 1] < 0;
+  flags[m] = (first ? BXF_ROW_FIRST : 0) | (last ? BXF_ROW_LAST : 0) | (pos[m] == 0 ? BXF_ROW_START : 0);
+}
+
+constexpr int NORM_THREADS = 256;
+
+// One row per CTA; the row stays in shared memory between the passes.
+template <class T>
+__global__ void __launch_bounds__(NORM_THREADS)
+fl_norm_kernel(float* __restrict__ x, const i64* ids, const T* __restrict__ embed, i64 V, const float* __restrict__ y,
+               const int* __restrict__ place, const float* __restrict__ weight, int top, const float* __restrict__ w,
+               const float* __restrict__ b, float eps, T* __restrict__ h, i64 ldh, int* zero, int nzero, int D) {
+  extern __shared__ float row[];
+  __shared__ float red[33];
+  const i64 m = blockIdx.x;
+  float* xm = x + m * D;
+  if (blockIdx.x == 0)
+    for (int i = threadIdx.x; i < nzero; i += NORM_THREADS) zero[i] = 0;
+  const T* em = nullptr;
+  if (ids) {
+    const i64 id = ids[m];
+    em = embed + (id < 0 || id >= V ? 0 : id) * D;
+  }
+  float s = 0.0f;
+  if (D % 4 == 0) {
+    for (int d = threadIdx.x * 4; d < D; d += NORM_THREADS * 4) {
+      float4 v;
+      if (em) {
+        v = make_float4(ld(em + d), ld(em + d + 1), ld(em + d + 2), ld(em + d + 3));
+      } else {
+        v = *reinterpret_cast<const float4*>(xm + d);
+        for (int k = 0; k < top; ++k) {
+          const float wk = weight[m * top + k];
+          const float4 e = *reinterpret_cast<const float4*>(y + (i64)place[m * top + k] * D + d);
+          v.x += wk * e.x;
+          v.y += wk * e.y;
+          v.z += wk * e.z;
+          v.w += wk * e.w;
+        }
+      }
+      if (em || top) *reinterpret_cast<float4*>(xm + d) = v;
+      *reinterpret_cast<float4*>(row + d) = v;
+      s += (v.x + v.y) + (v.z + v.w);
+    }
+  } else {
+    for (int d = threadIdx.x; d < D; d += NORM_THREADS) {
+      float v = em ? ld(em + d) : xm[d];
+      if (!em)
+        for (int k = 0; k < top; ++k) v += weight[m * top + k] * y[(i64)place[m * top + k] * D + d];
+      if (em || top) xm[d] = v;
+      row[d] = v;
+      s += v;
+    }
+  }
+  if (!h) return;
+  const float mean = block_sum(s, red) / D;
+  float q = 0.0f;
+  for (int d = threadIdx.x; d < D; d += NORM_THREADS) {
+    const float c = row[d] - mean;
+    q += c * c;
+  }
+  const float r = 1.0f / sqrtf(block_sum(q, red) / D + eps);
+  for (int d = threadIdx.x; d < D; d += NORM_THREADS) st(h + m * ldh + d, (row[d] - mean) * r * w[d] + b[d]);
+}
+
+// One warp per row: `top` rounds of (largest, lowest index first).
+__global__ void fl_route_kernel(const float* __restrict__ logits, i64 ldl, int E, int top, int* chosen, float* weight,
+                                int* rank, int* counts, int M) {
+  const int m = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (m >= M) return;
+  const float* z = logits + m * ldl;
+  constexpr int PER = BXF_MAX_EXPERTS / 32;
+  uint32_t taken = 0;                                    // bit j: expert j * 32 + lane is chosen already
+  float mine = 0.0f, first = 0.0f, sum = 0.0f;           // lane k keeps the k-th choice
+  int pick = 0;
+  for (int k = 0; k < top; ++k) {
+    float best = -INFINITY;
+    int at = E;
+    for (int j = 0; j < PER && j * 32 + lane < E; ++j) {
+      const float v = z[j * 32 + lane];
+      if (!(taken >> j & 1) && (v > best || at == E)) {
+        best = v;
+        at = j * 32 + lane;
+      }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float bo = __shfl_xor_sync(0xffffffffu, best, o);
+      const int ao = __shfl_xor_sync(0xffffffffu, at, o);
+      if (ao < E && (at >= E || bo > best || (bo == best && ao < at))) {
+        best = bo;
+        at = ao;
+      }
+    }
+    if (k == 0) first = best;
+    const float e = expf(best - first);
+    sum += e;
+    if (lane == k) {
+      mine = e;
+      pick = at;
+    }
+    if (lane == (at & 31)) taken |= 1u << (at >> 5);
+  }
+  if (lane < top) {
+    chosen[m * top + lane] = pick;
+    weight[m * top + lane] = mine / sum;
+    rank[m * top + lane] = atomicAdd(counts + pick, 1);
+  }
+}
+
+// One CTA per (row, choice): its place in expert order, and the copy of the row.
+template <class T>
+__global__ void __launch_bounds__(128)
+fl_gather_kernel(const T* __restrict__ h, i64 ldh, int D, const int* chosen, const int* rank, const int* counts, int top,
+                 T* __restrict__ hp, int* place) {
+  __shared__ int base;
+  const int pair = blockIdx.x, e = chosen[pair];
+  if (threadIdx.x < 32) {
+    int s = 0;
+    for (int i = threadIdx.x; i < e; i += 32) s += counts[i];
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+    if (threadIdx.x == 0) {
+      base = s + rank[pair];
+      place[pair] = base;
+    }
+  }
+  __syncthreads();
+  const T* src = h + (i64)(pair / top) * ldh;
+  T* dst = hp + (i64)base * ldh;
+  constexpr int V = 16 / sizeof(T);
+  if (ldh % V == 0) {                                    // the tail of a row lies inside its leading dimension
+    for (int d = threadIdx.x * V; d < D; d += blockDim.x * V)
+      *reinterpret_cast<uint4*>(dst + d) = *reinterpret_cast<const uint4*>(src + d);
+  } else {
+    for (int d = threadIdx.x; d < D; d += blockDim.x) dst[d] = src[d];
+  }
+}
+
+constexpr int PREP_THREADS = 128;
+
+template <class T>
+__global__ void __launch_bounds__(PREP_THREADS)
+fl_latent_prepare_kernel(const float* __restrict__ y, i64 ldy, int q_rank, int R, int rot, int H,
+                         const float* __restrict__ wq, const float* __restrict__ wkv, float eps,
+                         const float* __restrict__ freq, const i64* pos, const i64* slot, T* __restrict__ cq, i64 ldcq,
+                         T* __restrict__ cache, i64 ldc, float* __restrict__ cs, float* __restrict__ gate) {
+  __shared__ float red[33];
+  const i64 m = blockIdx.x;
+  const float* ym = y + m * ldy;
+  const float* yc = ym + q_rank;
+  const float* yr = yc + R;
+  T* row = cache + (slot[m] < 0 ? 0 : slot[m]) * ldc;
+  float sq = 0.0f, sk = 0.0f;
+  for (int d = threadIdx.x; d < q_rank; d += PREP_THREADS) sq += ym[d] * ym[d];
+  for (int d = threadIdx.x; d < R; d += PREP_THREADS) sk += yc[d] * yc[d];
+  const float rq = 1.0f / sqrtf(block_sum(sq, red) / q_rank + eps);
+  const float rk = 1.0f / sqrtf(block_sum(sk, red) / R + eps);
+  for (int d = threadIdx.x; d < q_rank; d += PREP_THREADS) st(cq + m * ldcq + d, ym[d] * rq * wq[d]);
+  for (int d = threadIdx.x; d < R; d += PREP_THREADS) st(row + d, yc[d] * rk * wkv[d]);
+  const float p = (float)pos[m];
+  for (int i = threadIdx.x; i < rot / 2; i += PREP_THREADS) {
+    float s, c;
+    sincosf(p * freq[i], &s, &c);
+    cs[(m * (rot / 2) + i) * 2] = c;
+    cs[(m * (rot / 2) + i) * 2 + 1] = s;
+    const float u = yr[2 * i], v = yr[2 * i + 1];
+    st(row + R + 2 * i, u * c - v * s);
+    st(row + R + 2 * i + 1, v * c + u * s);
+  }
+  for (int i = threadIdx.x; i < H; i += PREP_THREADS) gate[m * H + i] = sigmoid(yr[rot + i]);
+}
+
+// Second pass of a minGRU scan longer than a tile: the state carried into a tile is folded from the last rows of the
+// tiles before it, then S = local + decay * carried. One thread per channel and CTA row; blockIdx.y = tile.
+template <class T>
+__global__ void __launch_bounds__(128)
+fl_gru_finish_kernel(const bxf_gru g, int M, int width, int tile) {
+  const int n = blockIdx.x * 128 + threadIdx.x, j = blockIdx.y;
+  if (n >= width) return;
+  float carry = 0.0f;
+  for (int i = 0; i < j; ++i) {
+    const i64 at = (i64)(i * tile + tile - 1) * width + n;
+    carry = g.local[at] + g.decay[at] * carry;
+  }
+  const int m1 = min(M, (j + 1) * tile);
+  for (int m = j * tile + blockIdx.z; m < m1; m += gridDim.z) {
+    const i64 at = (i64)m * width + n;
+    const float s = g.local[at] + g.decay[at] * carry;
+    T* o = static_cast<T*>(g.out) + (i64)m * g.ldo + n;
+    st(o, s * ld(o));
+    if (g.flags[m] & BXF_ROW_LAST) g.state[g.seq[m] * width + n] = s;
+  }
+}
+
+}  // namespace bxf

@@ -1,5 +1,5 @@
-"""A minimal decode loop over `ExactEngine`: paged-cache bookkeeping, chunked prompt processing, greedy /
-Gumbel-max sampling and per-position logits hashes (the reference's `generate` / `logits_sha`,
+"""A minimal decode loop over any token-row engine (`engine_base`): paged-cache bookkeeping, chunked prompt processing,
+greedy / Gumbel-max sampling and per-position logits hashes (the reference's `generate` / `logits_sha`,
 src/bitexact/generate.py:21-50, on a batch of sequences with one block-table row each)."""
 
 import hashlib
@@ -15,21 +15,94 @@ def logits_sha(row):
 
 
 class Session:
-    """B sequences, each with a contiguous run of cache blocks (block 0 is the null block)."""
+    """B sequences with one block-table row each (page 0 is the null page; a recurrent layer's state of sequence b is slot
+    b of its cache). By default every sequence owns a run of pages for max_len tokens. With `pages`, the cache has that
+    many pages for all sequences together: `feed` takes them as a sequence grows and `release` gives them back."""
 
-    def __init__(self, eng, B, max_len, bs=16, perm_seed=None):
+    def __init__(self, eng, B, max_len, bs=16, perm_seed=None, pages=None):
         self.eng, self.B, self.bs = eng, B, bs
         self.nblk = (max_len + bs - 1) // bs
-        nb = 1 + B * self.nblk
+        nb = 1 + (B * self.nblk if pages is None else pages)
         dev = eng.dev
-        self.kvs = [torch.zeros(nb, eng.HKV, bs, 8 * eng.HD, dtype=torch.int8, device=dev) for _ in range(eng.L)]
+        self.kvs = eng.new_cache(B, nb, bs)
         blocks = torch.arange(1, nb, dtype=torch.int64)
         if perm_seed is not None:                                  # scattered pages
             g = torch.Generator().manual_seed(perm_seed)
             blocks = blocks[torch.randperm(nb - 1, generator=g)]
-        self.bt = blocks.view(B, self.nblk).to(torch.int32).to(dev)
+        self.free = None
+        if pages is None:
+            self.bt = blocks.view(B, self.nblk).to(torch.int32).to(dev)
+        else:
+            self.bt = torch.zeros(B, self.nblk, dtype=torch.int32, device=dev)
+            self.free = blocks.tolist()[::-1]
+            self.held = [[] for _ in range(B)]
         self.lens = torch.zeros(B, dtype=torch.long, device=dev)
         self.rows = torch.arange(B, device=dev)
+
+    def _reserve(self, seq, n):
+        """Pages for positions 0 .. n - 1 of the sequence."""
+        need = (n + self.bs - 1) // self.bs
+        if need > self.nblk:
+            raise ValueError(f"sequence {seq}: {n} tokens are beyond the session's max_len")
+        if self.free is None or need <= len(self.held[seq]):
+            return
+        have = len(self.held[seq])
+        if need - have > len(self.free):
+            raise MemoryError("the session has no free pages")
+        new = [self.free.pop() for _ in range(need - have)]
+        self.held[seq] += new
+        self.bt[seq, have:need] = torch.tensor(new, dtype=torch.int32).to(self.bt.device)
+
+    def release(self, seq):
+        """The sequence is finished: its pages go back to the pool and its row may serve another one. Nothing is cleared:
+        keys beyond a sequence's length are never read, and a recurrent state starts from zero at position 0."""
+        if self.free is not None:
+            self.free += self.held[seq][::-1]
+            self.held[seq] = []
+            self.bt[seq] = 0
+        self.lens[seq] = 0
+
+    @torch.no_grad()
+    def feed(self, entries, chunk_rows=4096):
+        """entries: [(sequence, its next tokens)], every sequence at most once; any mix of prompt portions and single
+        decode tokens goes through one forward call per chunk_rows rows. Returns the residual rows [n, D] per entry."""
+        dev = self.eng.dev
+        lens = self.lens.tolist()
+        todo = [[int(s), torch.as_tensor(t, dtype=torch.long), lens[s]] for s, t in entries]
+        assert len({s for s, _, _ in todo}) == len(todo), "a sequence may appear once per call"
+        for s, t, n in todo:
+            self._reserve(s, n + len(t))
+        out, i = [[] for _ in todo], 0
+        while i < len(todo):
+            runs, at = [], 0                                       # (entry, sequence, first position, tokens)
+            while i < len(todo) and at < chunk_rows:
+                s, t, n = todo[i]
+                take = min(len(t), chunk_rows - at)
+                if take:
+                    runs.append((i, s, n, t[:take]))
+                    at += take
+                todo[i][1], todo[i][2] = t[take:], n + take
+                if take == len(t):
+                    i += 1
+            if not runs:
+                continue
+            seq = torch.cat([torch.full((len(t),), s) for _, s, _, t in runs]).to(dev)
+            pos = torch.cat([torch.arange(n, n + len(t)) for _, _, n, t in runs]).to(dev)
+            ids = torch.cat([t for _, _, _, t in runs]).to(dev)
+            tt, row = [], 0
+            for _, s, n, t in runs:
+                tt.append((s, row, len(t), n + len(t)))
+                row += len(t)
+            longest = max(c for _, _, q, c in tt if q > 1) if any(q > 1 for _, _, q, _ in tt) else 0
+            tt = self.eng.tile_table(tt, self.bs) if longest > self.eng.tiles_from else None
+            x = self.eng.forward(self.kvs, ids, pos, self._slots(seq, pos), self.bt, seq,
+                                 tiles=None if tt is None else tt.to(dev))
+            row = 0
+            for e, s, n, t in runs:
+                out[e].append(x[row:row + len(t)])
+                row += len(t)
+                self.lens[s] = n + len(t)
+        return [torch.cat(o) if o else torch.empty(0, self.eng.D, device=dev) for o in out]
 
     def _slots(self, seq, pos):
         return self.bt[seq, pos // self.bs].long() * self.bs + pos % self.bs
@@ -56,19 +129,17 @@ class Session:
         of a chunk runs on the prefill tile kernel (runs of 32 / G consecutive tokens share their K / V staging),
         else every token is a row of the decode kernel. Same integers either way. Returns the final residual row of
         each sequence [B, D]."""
-        from .vllm_plugin import tri_prefill
         B, P = prompts.shape
         dev = self.eng.dev
         prompts = prompts.to(dev)
         lens_host = [P] * B if lens is None else [int(v) for v in lens.tolist()]
         lens = torch.full((B,), P, dtype=torch.long, device=dev) if lens is None else lens.to(dev).long()
-        G = self.eng.H // self.eng.HKV
-        # the tile kernel pays for itself once a tile walks a few key blocks (measured: 0.83 x the row kernel on
-        # 128-token prompts, 1.7 x on 2048-token ones); short chunks at the start of a prompt stay on rows
-        use_tiles = tiles and self.eng.HD == 64 and tri_prefill.BM % G == 0 and self.bs in (8, 16, 32, 64, 128)
-        tile_from = 0 if tiles == "always" else 384
+        if self.free is not None:
+            for b in range(B):
+                self._reserve(b, lens_host[b])
+        tile_from = 0 if tiles == "always" else self.eng.tiles_from
         step = max(1, chunk_rows // B)
-        last = torch.zeros(B, self.eng.D, dtype=torch.long, device=dev)
+        last = None
         for p0 in range(0, P, step):
             p1 = min(P, p0 + step)
             grid = torch.arange(p0, p1, device=dev).expand(B, -1)
@@ -78,16 +149,19 @@ class Session:
             pos = grid[live]                                                      # sequence-major rows
             seq = self.rows[:, None].expand(-1, p1 - p0)[live]
             tt = None
-            if use_tiles and p1 > tile_from:                                    # sequence-major rows: runs per sequence
+            if tiles and p1 > tile_from:                                        # sequence-major rows: runs per sequence
                 pre, row0 = [], 0
                 for b in range(B):
                     n = max(0, min(p1, lens_host[b]) - p0)
                     if n:
                         pre.append((b, row0, n, p0 + n))
                     row0 += n
-                tt = tri_prefill.tile_table(pre, G, tri_prefill.ROWS).to(dev)
+                tt = self.eng.tile_table(pre, self.bs)
+                tt = None if tt is None else tt.to(dev)
             x = self.eng.forward(self.kvs, prompts[:, p0:p1][live], pos, self._slots(seq, pos), self.bt, seq, tiles=tt)
             fin = pos == lens[seq] - 1
+            if last is None:
+                last = torch.zeros(B, self.eng.D, dtype=x.dtype, device=dev)
             last[seq[fin]] = x[fin]
         self.lens += lens
         return last
@@ -95,7 +169,7 @@ class Session:
     @torch.no_grad()
     def step(self, tokens, pos=None):
         """One decode step: tokens int64 [B] at positions `pos` (default: the lengths tracked on the device).
-        Returns the residual rows [B, D]."""
+        Returns the residual rows [B, D]. (With a page pool the pages must be there: `feed` takes them as needed.)"""
         pos = self.lens.clone() if pos is None else pos
         x = self.eng.forward(self.kvs, tokens, pos, self._slots(self.rows, pos), self.bt, self.rows)
         self.lens += 1

@@ -6,11 +6,12 @@ qkv, attention, attn_out, linear, add_norm, linear, silu_quant, linear, add_norm
 import torch
 
 from .. import _native as nv
+from ..engine_base import TokenRowEngine
 from ..vllm_plugin import tri_fuse, tri_paged, tri_prefill
 from .gemm_skinny import linear_post
 
 
-class IntEngine:
+class IntEngine(TokenRowEngine):
     FR = 16
 
     def __init__(self, c, dev="cuda", n_layers=None, nl=2):

@@ -8,6 +8,7 @@ silu_quant, linear, add_norm), device tensors only, no host synchronisation insi
 import torch
 
 from .. import _native as nv
+from ..engine_base import TokenRowEngine
 from ..exact.model import Lin
 from . import exact_fuse, tri_exact_attn, tri_prefill
 from .exact_gemm import FusedLin
@@ -15,7 +16,7 @@ from .exact_gemm import FusedLin
 L2E28_HD = {64: 387270501, 128: 273841598}        # src/bitexact/exact/ops.py:19-20
 
 
-class ExactEngine:
+class ExactEngine(TokenRowEngine):
     FR = 24
 
     def __init__(self, c, dev="cuda", n_layers=None):

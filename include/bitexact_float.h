@@ -1,0 +1,146 @@
+/* C ABI of libbitexact_float.so: sm_100a kernels of the float models (hybrids of recurrent and attention layers served
+ * from bf16 weights, or in 32-bit throughout). Same conventions as bitexact_b200.h: device pointers unless said
+ * otherwise, BX_* status codes, `stream` is a cudaStream_t, calls are asynchronous and allocate nothing.
+ *
+ * Element type T of a call: dtype BXF_BF16 (bfloat16) or BXF_F32 (float, no reduced-precision product anywhere).
+ * "row" = one token of the step. Rows of one sequence are consecutive and in position order.
+ * Leading dimensions (ld*) and group strides (gs*) count elements. In bf16, operands of the products start on 16-byte
+ * boundaries and have leading dimensions and group strides that are multiples of 8; the extents themselves are free.
+ */
+#ifndef BITEXACT_FLOAT_H
+#define BITEXACT_FLOAT_H
+
+#include "bitexact_b200.h"
+
+#ifdef __cplusplus
+extern "C" {
+#endif
+
+#define BXF_BF16 0
+#define BXF_F32 1
+
+#define BXF_MAX_TOP 32          /* experts per token */
+#define BXF_MAX_EXPERTS 1024
+
+/* Row flags (bxf_row_flags): first / last row of its sequence in this step, first token of the sequence, padding. */
+#define BXF_ROW_FIRST 1
+#define BXF_ROW_LAST 2
+#define BXF_ROW_START 4
+#define BXF_ROW_PAD 8
+
+/* What a product does with its accumulators. */
+#define BXF_EPI_STORE 0         /* out[m, n] = act(acc); rows n >= n_main go to side[m, n - n_main] = acc + bias (float) */
+#define BXF_EPI_ADD 1           /* out (float) [m, n] += acc */
+#define BXF_EPI_ROPE 2          /* n < n_main: out[m, n] = acc; the others are rotated pairs, see rot_* */
+#define BXF_EPI_GATE 3          /* out[m, n] = acc * gate[m, group] */
+
+#define BXF_OUT_T 0
+#define BXF_OUT_F32 1
+#define BXF_OUT_I64 2           /* round(v * 2^24), the fixed-point logits of the integer sampler */
+
+#define BXF_ACT_NONE 0
+#define BXF_ACT_RELU2 1         /* max(z, 0)^2 */
+#define BXF_ACT_XIELU 2         /* z > 0: act_p z^2 + z / 2; else act_q (e^z - 1 - z) + z / 2 */
+
+typedef struct {
+  int kind, out_type, act, n_main;
+  float act_p, act_q;
+  void* out;                    /* T, float or int64 */
+  int64_t ldo, gso;
+  float* side;                  /* BXF_EPI_STORE, n >= n_main */
+  int64_t lds;
+  const float* bias;            /* [N - n_main] or NULL */
+  const float* gate;            /* BXF_EPI_GATE: float [M, groups], row stride ldg */
+  int64_t ldg;
+  const float* cs;              /* BXF_EPI_ROPE: (cos, sin) pairs float [M, rot_dim / 2, 2] */
+  void* rot_out;                /* T: row m, head h, entry j -> rot_out[m * ldr + h * hsr + j] */
+  int64_t ldr, hsr;
+  int rot_dim;
+  int pad_;
+} bxf_epilogue;
+
+/* The gates of a minGRU layer after its three products (update, candidate, output gate; planes 0, 1, 2). */
+typedef struct {
+  const float *bias_z, *bias_x; /* [width] */
+  float* state;                 /* [slots, width] */
+  const int* flags;             /* [M] row flags */
+  const int64_t* seq;           /* [M] state slot of each row */
+  void* out;                    /* T [M, ldo]: state * silu(gate) (mode 0) or silu(gate) alone (mode 1) */
+  int64_t ldo;
+  float *decay, *local;         /* mode 1: float [M, width] */
+  int mode;                     /* 0: rows fit one tile, finished here; 1: bxf_gru_finish follows */
+  int pad_;
+} bxf_gru;
+
+int bxf_version(void);
+long long bxf_launch_count(void);
+int bxf_device_status(void);            /* as bx_device_status, for the kernels of this library */
+int bxf_clear_device_status(void);
+int bxf_set_device_status(int value);
+
+/* acc[g][m, n] = sum_k x[g][m, k] w[g][n, k] in 32-bit accumulation, then the epilogue (HOST pointer, copied).
+ *   w T [groups, N, ldw] (group stride gsw), x T [groups, M, ldx] (group stride gsx)
+ *   counts NULL: every group has the M rows. Else int32 [groups]: the rows of x are ordered by group, group e has
+ *   counts[e] of the M rows (experts; gsx unused, and out's rows are the rows of x).
+ *   tile_rows 0 = automatic (else a row-tile size of the bf16 kernels); results do not depend on it beyond rounding. */
+int bxf_linear(int dtype, const void* w, int64_t ldw, int64_t gsw, const void* x, int64_t ldx, int64_t gsx, int groups,
+               int M, int N, int K, const int* counts, const bxf_epilogue* epi, int tile_rows, void* stream);
+
+/* The three products of a minGRU layer with its recurrence: w T [3, width, ldw] (planes z, x, g), x T [M, ldx].
+ * z = sigmoid(acc_0 + bias_z), u = acc_1 + bias_x, candidate = u + 1/2 (u >= 0) or sigmoid(u),
+ * S = (1 - z) S + z candidate along the rows of a sequence, from `state` (zero on BXF_ROW_START) and back into it.
+ * bxf_gru_tile_rows: the most rows mode 0 takes. Mode 1 leaves for every row the prefix product of (1 - z) and the
+ * state from a zero start, both within its tile of bxf_gru_long_tile rows, for bxf_gru_finish. */
+int bxf_gru_tile_rows(int dtype);
+int bxf_gru_long_tile(int dtype);
+int bxf_gru_linear(int dtype, const void* w, int64_t ldw, const void* x, int64_t ldx, int M, int width, int K,
+                   const bxf_gru* gru, void* stream);
+int bxf_gru_finish(int dtype, int M, int width, const bxf_gru* gru, void* stream);
+
+/* flags int32 [M] from seq / slot / pos int64 [M] (slot < 0: padding row). */
+int bxf_row_flags(const int64_t* seq, const int64_t* slot, const int64_t* pos, int* flags, int M, void* stream);
+
+/* x float [M, D]: ids != NULL: x = embed[ids] (embed T [V, D], vocab V); else, with top > 0,
+ * x += sum_k weight[m, k] y[place[m, k]] (y float [*, D]: the experts' outputs). Then, with h, the layer norm
+ * (w, b float [D]) of x as T [M, ldh]. zero / nzero: int32 words cleared on the way (expert counters). */
+int bxf_norm(int dtype, float* x, const int64_t* ids, const void* embed, int64_t V, const float* y, const int* place,
+             const float* weight, int top, const float* w, const float* b, float eps, void* h, int64_t ldh, int* zero,
+             int nzero, int M, int D, void* stream);
+
+/* Routing: logits float [M, ldl] over `experts` -> chosen int32 [M, top], weight float [M, top] (softmax over the
+ * chosen), rank int32 [M, top] (place within the expert); counts int32 [experts] must be zero and receives the sizes. */
+int bxf_route(const float* logits, int64_t ldl, int experts, int top, int* chosen, float* weight, int* rank, int* counts,
+              int M, void* stream);
+/* Rows of h T [M, ldh] gathered in expert order into hp T [M * top, ldh]; place int32 [M, top] = the row of each pair. */
+int bxf_gather(int dtype, const void* h, int64_t ldh, int D, const int* chosen, const int* rank, const int* counts,
+               int experts, int top, void* hp, int* place, int M, void* stream);
+
+/* After the first projection of a latent attention layer, y float [M, ldy] = [query latent (q_rank) | key latent
+ * (kv_rank) | rotated key part (rot_dim) | head gates (heads)]:
+ *   cq T [M, ldcq] = RMS norm of the query latent (weight wq), gate float [M, heads] = sigmoid of the gates,
+ *   cs float [M, rot_dim / 2, 2] = (cos, sin) of pos * freq, and the cache row of the token's slot (T [*, ldc]):
+ *   [RMS norm of the key latent (weight wkv) | rotated key part]. slot int64 [M] (negative: row 0). */
+int bxf_latent_prepare(int dtype, const float* y, int64_t ldy, int q_rank, int kv_rank, int rot_dim, int heads,
+                       const float* wq, const float* wkv, float eps, const float* freq, const int64_t* pos,
+                       const int64_t* slot, void* cq, int64_t ldcq, void* cache, int64_t ldc, float* cs, float* gate,
+                       int M, void* stream);
+
+/* Attention over the latent cache (keys and values are the cache rows themselves; the value part is the first kv_rank
+ * entries), one sliding window, a sink per head in the denominator.
+ *   q T [M, heads, ldq] (first kv_rank + rot_dim entries used), cache T [nb, bs, ldc], bt int32 / int64 [*, nblk],
+ *   seq int64 [M] table row of each query row, pos int64 [M]; window 0: none; sink float [heads] or NULL
+ *   tiles int32 [ntiles, 3] (table row, first query row, rows) or NULL (every row by itself)
+ *   out T [M, heads, ldo]; scratch of bxf_latent_attention_scratch bytes (may be NULL: no split over keys)
+ *   variant 0 automatic, 1 one CTA per (row, head), 2 tensor cores. */
+size_t bxf_latent_attention_scratch(int M, int heads, int kv_rank);
+int bxf_latent_attention_tile(int heads);     /* query rows of a tile of the tensor-core kernel (at least 1) */
+int bxf_latent_attention(int dtype, const void* q, int64_t ldq, int M, int heads, int kv_rank, int rot_dim,
+                         const void* cache, int64_t ldc, int bs, int nb, const void* bt, int bt_is64, int64_t bt_stride,
+                         int nblk, const int64_t* seq, const int64_t* pos, const int* tiles, int ntiles, int window,
+                         const float* sink, float scale, void* out, int64_t ldo, void* scratch, size_t scratch_bytes,
+                         int variant, void* stream);
+
+#ifdef __cplusplus
+}
+#endif
+#endif
