@@ -1,0 +1,363 @@
+// Latent attention on the tensor cores (bf16 cache, fp32 scores and softmax), one kernel for prompts and decoding.
+//
+// A tile is up to 128 query rows = (consecutive tokens of one sequence) x heads: all of them read the same latent rows, so
+// a block of 64 cache rows is staged once for 128 queries. Scores Q C^T: A = Q tile [128 x W] (W = latent + rotated part),
+// B = cache rows, both K-major. P V: the values are the first R entries of the SAME staged rows, read as an MN-major B
+// operand (their rows are the contraction index), so nothing is transposed or loaded twice; A = P comes from TMEM, where
+// the softmax warps leave it as bf16 in place of the scores. TMEM: two score buffers of 64 columns, then the output
+// accumulator (256 columns; a wider latent is cut into value slices over blockIdx.z).
+//
+// Warp 0 = TMA, warp 1 = MMA, warps 2 .. 5 = softmax, one thread per query row. The running maximum starts at the sink
+// (denominator 1); the accumulator is rescaled only when the maximum grows by more than 2^8 since the last time. Few
+// tiles (decoding): the keys of a tile are split over blockIdx.y, and a second kernel joins the parts.
+#pragma once
+
+#include "fl_attention.cuh"
+#include "fl_gemm.cuh"
+
+namespace bxf {
+
+constexpr int LT_KEYS = 64, LT_THREADS = 192, LT_MAX_STAGES = 4, LT_MAX_SPLIT = 4, LT_VCOLS = 256;
+constexpr int LT_O = 2 * LT_KEYS;                        // first TMEM column of the output accumulator
+constexpr float LT_LOG2E = 1.4426950408889634f;
+constexpr float LT_GROWTH = 8.0f;
+
+struct LatentTc {
+  int cols;                                              // 64-entry column blocks of a row, ceil(W / 64)
+  int stages, qrows;                                     // key stages of the ring, rows of the Q box
+  int row_blocks, vsplit;                                // blockIdx.z = value slice * row_blocks + row block
+  int splits;
+  float* part;                                           // splits > 1: [splits][M H][R] accumulators, then [splits][M H][2]
+};
+
+struct LatentShared {
+  uint64_t q_full, o_done;
+  uint64_t full[LT_MAX_STAGES], empty[LT_MAX_STAGES];
+  uint64_t s_full[2], p_full[2], pv_done[2];
+  uint32_t tmem_base, abort_flag;
+};
+
+// D (+)= A[tmem] * B[smem]; A: bf16 pairs, one row per lane.
+__device__ __forceinline__ void umma_bf16_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t b_desc, uint32_t idesc,
+                                             uint32_t accumulate) {
+  asm volatile(
+      "{\n\t"
+      ".reg .pred p;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t"
+      "}\n" ::"r"(d_tmem),
+      "r"(a_tmem), "l"(b_desc), "r"(idesc), "r"(accumulate)
+      : "memory");
+}
+
+// MN-major operand in 128-byte-swizzled boxes of 64 entries x LT_KEYS rows: 8 contraction rows are 1024 bytes apart, the
+// next 64 entries one box further on.
+__device__ __forceinline__ uint64_t umma_desc_mn(uint32_t addr) {
+  uint64_t d = umma_desc_sw128(addr);
+  d &= ~(static_cast<uint64_t>(0x3FFF) << 16);
+  return d | static_cast<uint64_t>((LT_KEYS * 128) >> 4) << 16;
+}
+
+__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
+  const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
+
+__global__ void __launch_bounds__(LT_THREADS, 1)
+fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mc,
+                              const LatentAttn a, const LatentTc c) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* qs = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* ring = qs + c.cols * 128 * 128;
+  const int stage_bytes = c.cols * LT_KEYS * 128;
+  LatentShared* sh = reinterpret_cast<LatentShared*>(ring + c.stages * stage_bytes);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+
+  // ---- the tile ----
+  int tok0, ntok;
+  i64 seq;
+  if (a.tiles) {
+    const int* t = a.tiles + (i64)blockIdx.x * 3;
+    seq = t[0];
+    tok0 = t[1];
+    ntok = t[2];
+  } else {
+    tok0 = blockIdx.x;
+    ntok = 1;
+    seq = a.seq[tok0];
+  }
+  const int row0 = (blockIdx.z % c.row_blocks) * 128, rows = min(128, ntok * a.H - row0);
+  const int v0 = (blockIdx.z / c.row_blocks) * LT_VCOLS, vn = min(LT_VCOLS, a.R - v0);
+  const i64 limit = (i64)a.nblk * a.bs - 1;
+  const i64 p_first = min(a.pos[tok0], limit), p_last = min(a.pos[tok0 + ntok - 1], limit);
+  const int b_lo = a.first_key(p_first) / LT_KEYS, b_hi = (int)(p_last / LT_KEYS) + 1;
+  const int b0 = b_lo + (b_hi - b_lo) * (int)blockIdx.y / c.splits, b1 = b_lo + (b_hi - b_lo) * ((int)blockIdx.y + 1) / c.splits;
+  const int nb = b1 - b0;
+  if (rows <= 0) return;
+  const int soft_warps = (rows + 31) / 32;
+
+  if (threadIdx.x == 0) {
+    mbar_init(&sh->q_full, 1);
+    mbar_init(&sh->o_done, 1);
+    for (int i = 0; i < c.stages; ++i) {
+      mbar_init(&sh->full[i], 1);
+      mbar_init(&sh->empty[i], 1);
+    }
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&sh->s_full[i], 1);
+      mbar_init(&sh->p_full[i], soft_warps);
+      mbar_init(&sh->pv_done[i], 1);
+    }
+    sh->abort_flag = *reinterpret_cast<volatile int*>(&g_wait_timeouts) != 0;
+    fence_barrier_init();
+    tma_prefetch_desc(&mq);
+    tma_prefetch_desc(&mc);
+  }
+  __syncthreads();
+  if (warp == 1) {
+    tmem_alloc(&sh->tmem_base, 512);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = sh->tmem_base;
+  const bool dead = sh->abort_flag != 0;
+  __syncthreads();
+
+  auto fail = [&] {
+    atomicAdd(&g_wait_timeouts, 1);
+    *reinterpret_cast<volatile uint32_t*>(&sh->abort_flag) = 1;
+  };
+
+  if (dead) {
+  } else if (warp == 0) {
+    if (lane == 0 && nb > 0) {
+      // ---- TMA: the queries once, then the key blocks page by page ----
+      mbar_arrive_expect_tx(&sh->q_full, c.cols * c.qrows * 128);
+      for (int j = 0; j < c.cols; ++j)
+        tma_load_3d(qs + j * 128 * 128, &mq, &sh->q_full, j * 64, tok0 * a.H + row0, 0);
+      const int box = min(a.bs, LT_KEYS), pages = LT_KEYS / box;
+      int i = 0;
+      bool ok = true;
+      for (; i < nb; ++i) {
+        const int s = i % c.stages, round = i / c.stages;
+        if (round > 0 && !(ok = mbar_wait(&sh->empty[s], (round - 1) & 1))) break;
+        uint8_t* st = ring + s * stage_bytes;
+        mbar_arrive_expect_tx(&sh->full[s], stage_bytes);
+        for (int p = 0; p < pages; ++p) {
+          const int key = (b0 + i) * LT_KEYS + p * box;
+          const int page = (int)(a.page_row(seq, min(key / a.bs, a.nblk - 1)) / a.bs);
+          for (int j = 0; j < c.cols; ++j)
+            tma_load_3d(st + j * LT_KEYS * 128 + p * box * 128, &mc, &sh->full[s], j * 64, key % a.bs, page);
+        }
+      }
+      if (!ok) {
+        fail();
+        mbar_wait(&sh->q_full, 0);
+        for (int k = i > c.stages ? i - c.stages : 0; k < i; ++k) mbar_wait(&sh->full[k % c.stages], (k / c.stages) & 1);
+      }
+    }
+  } else if (warp == 1) {
+    if (lane == 0 && nb > 0) {
+      // ---- MMA: scores of block i + 1 are issued before the values of block i ----
+      constexpr uint32_t ID_S = umma_idesc_bf16(LT_KEYS);
+      const uint32_t id_v = umma_idesc_bf16((vn + 15) / 16 * 16, true);
+      auto scores = [&](int i) {
+        const int s = i % c.stages, buf = i & 1;
+        if (!mbar_wait(&sh->full[s], (i / c.stages) & 1)) return false;
+        if (i >= 2 && !mbar_wait(&sh->pv_done[buf], ((i >> 1) - 1) & 1)) return false;   // P of block i - 2 is read
+        tc_fence_after();
+        const uint32_t qa = smem_u32(qs), ka = smem_u32(ring + s * stage_bytes);
+        for (int j = 0; j < c.cols; ++j)
+#pragma unroll
+          for (int ks = 0; ks < 4; ++ks)
+            umma_bf16(tmem + buf * LT_KEYS, umma_desc_sw128(qa + j * 128 * 128 + ks * 32),
+                      umma_desc_sw128(ka + j * LT_KEYS * 128 + ks * 32), ID_S, (j | ks) != 0);
+        umma_commit(&sh->s_full[buf]);
+        return true;
+      };
+      bool ok = mbar_wait(&sh->q_full, 0) && scores(0);
+      for (int i = 0; i < nb && ok; ++i) {
+        const int s = i % c.stages, buf = i & 1;
+        if (c.stages > 1 && i + 1 < nb && !(ok = scores(i + 1))) break;
+        if (!(ok = mbar_wait(&sh->p_full[buf], (i >> 1) & 1))) break;
+        tc_fence_after();
+        const uint32_t va = smem_u32(ring + s * stage_bytes) + (v0 / 64) * LT_KEYS * 128;
+#pragma unroll
+        for (int ks = 0; ks < LT_KEYS / 16; ++ks)
+          umma_bf16_ts(tmem + LT_O, tmem + buf * LT_KEYS + ks * 8, umma_desc_mn(va + ks * 2048), id_v, (i | ks) != 0);
+        umma_commit(&sh->pv_done[buf]);
+        umma_commit(&sh->empty[s]);
+        if (c.stages == 1 && i + 1 < nb) ok = scores(i + 1);             // one stage: nothing to run ahead into
+      }
+      if (ok) umma_commit(&sh->o_done);
+      else fail();
+    }
+  } else if (warp - 2 < 4) {
+    // ---- softmax: thread = query row (the TMEM lane quarter of the warp id) ----
+    const int quarter = warp & 3, r = quarter * 32 + lane;
+    if (quarter < soft_warps) {
+      const bool live = r < rows;
+      const int flat = row0 + (live ? r : 0), head = flat % a.H;
+      const int m = tok0 + flat / a.H;
+      const i64 pos = min(a.pos[m], limit);
+      const int lo = a.first_key(pos), hi = (int)pos;
+      const float scale = a.scale * LT_LOG2E;
+      const bool sink_here = a.sink && blockIdx.y == 0;
+      float ref = a.sink ? a.sink[head] * LT_LOG2E : -INFINITY, den = sink_here ? 1.0f : 0.0f;
+      const uint32_t lanes = (uint32_t)(quarter * 32) << 16;
+      bool ok = true;
+      for (int i = 0; i < nb; ++i) {
+        const int buf = i & 1;
+        ok = mbar_wait(&sh->s_full[buf], (i >> 1) & 1);
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
+        tc_fence_after();
+        float s[LT_KEYS];
+#pragma unroll
+        for (int q = 0; q < LT_KEYS; q += 16) {
+          uint32_t u[16];
+          tmem_ld16(tmem + lanes + buf * LT_KEYS + q, u);
+          tmem_ld_wait();
+#pragma unroll
+          for (int k = 0; k < 16; ++k) s[q + k] = __uint_as_float(u[k]);
+        }
+        const int k0 = (b0 + i) * LT_KEYS;
+        float mx = -INFINITY;
+        if (k0 >= lo && k0 + LT_KEYS - 1 <= hi) {
+#pragma unroll
+          for (int k = 0; k < LT_KEYS; ++k) {
+            s[k] *= scale;
+            mx = fmaxf(mx, s[k]);
+          }
+        } else {
+#pragma unroll
+          for (int k = 0; k < LT_KEYS; ++k) {
+            s[k] = k0 + k >= lo && k0 + k <= hi ? s[k] * scale : -INFINITY;
+            mx = fmaxf(mx, s[k]);
+          }
+        }
+        float f = 1.0f;
+        if (mx > ref + LT_GROWTH || ref == -INFINITY) {
+          f = ref == -INFINITY ? 0.0f : exp2f(ref - mx);
+          ref = mx;
+        }
+        if (__any_sync(0xffffffffu, f != 1.0f && live)) {
+          den *= f;
+          if (i > 0) {
+            // the accumulator may be touched once the values of block i - 1 are in
+            ok = mbar_wait(&sh->pv_done[buf ^ 1], ((i - 1) >> 1) & 1);
+            ok = __all_sync(0xffffffffu, ok);
+            if (!ok) break;
+            tc_fence_after();
+            for (int q = 0; q < vn; q += 16) {
+              uint32_t u[16];
+              tmem_ld16(tmem + lanes + LT_O + q, u);
+              tmem_ld_wait();
+#pragma unroll
+              for (int k = 0; k < 16; ++k) u[k] = __float_as_uint(__uint_as_float(u[k]) * f);
+              tmem_st16(tmem + lanes + LT_O + q, u);
+            }
+            tmem_st_wait();
+          }
+        }
+        const float base = ref == -INFINITY ? 0.0f : ref;            // no visible key yet: every weight is 0
+        float d0 = 0.0f, d1 = 0.0f;
+#pragma unroll
+        for (int q = 0; q < LT_KEYS; q += 32) {
+          uint32_t u[16];
+#pragma unroll
+          for (int k = 0; k < 16; ++k) {
+            const float e0 = exp2f(s[q + 2 * k] - base), e1 = exp2f(s[q + 2 * k + 1] - base);
+            d0 += e0;
+            d1 += e1;
+            u[k] = pack_bf16(e0, e1);
+          }
+          tmem_st16(tmem + lanes + buf * LT_KEYS + q / 2, u);
+        }
+        den += d0 + d1;
+        tmem_st_wait();
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&sh->p_full[buf]);
+      }
+      if (ok && nb > 0) ok = mbar_wait(&sh->o_done, 0);
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) {
+        if (lane == 0) fail();
+      } else {
+        tc_fence_after();
+        const i64 at = (i64)tok0 * a.H + row0 + r;
+        const float inv = 1.0f / den;
+        float* part = c.part + ((i64)blockIdx.y * a.M * a.H + at) * a.R + v0;
+        bf16* out = static_cast<bf16*>(a.out) + at * a.ldo + v0;
+        for (int q = 0; q < vn; q += 16) {
+          uint32_t u[16] = {};
+          if (nb > 0) {
+            tmem_ld16(tmem + lanes + LT_O + q, u);
+            tmem_ld_wait();
+          }
+          if (!live) continue;
+          const int n = min(16, vn - q);
+          if (c.splits == 1) {
+            if (n == 16) {                                               // out rows start on 16-byte boundaries
+              uint32_t w[8];
+#pragma unroll
+              for (int k = 0; k < 8; ++k)
+                w[k] = pack_bf16(__uint_as_float(u[2 * k]) * inv, __uint_as_float(u[2 * k + 1]) * inv);
+              *reinterpret_cast<uint4*>(out + q) = make_uint4(w[0], w[1], w[2], w[3]);
+              *reinterpret_cast<uint4*>(out + q + 8) = make_uint4(w[4], w[5], w[6], w[7]);
+            } else {
+#pragma unroll
+              for (int k = 0; k < 16; ++k)
+                if (k < n) st(out + q + k, __uint_as_float(u[k]) * inv);
+            }
+          } else {
+#pragma unroll
+            for (int k = 0; k < 16; ++k)
+              if (k < n) part[q + k] = __uint_as_float(u[k]);
+          }
+        }
+        if (c.splits > 1 && live && v0 == 0) {
+          float* ml = c.part + (i64)c.splits * a.M * a.H * a.R + ((i64)blockIdx.y * a.M * a.H + at) * 2;
+          ml[0] = ref;
+          ml[1] = den;
+        }
+      }
+    }
+  }
+
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    __syncwarp();
+    tc_fence_after();
+    tmem_dealloc(tmem, 512);
+  }
+}
+
+// Joins the key splits: one CTA per query row (token, head).
+__global__ void __launch_bounds__(128) fl_latent_join_kernel(const LatentAttn a, const float* part, int splits) {
+  const i64 at = blockIdx.x, n = (i64)a.M * a.H;
+  const float* ml = part + splits * n * a.R;
+  float mx = -INFINITY, f[LT_MAX_SPLIT], den = 0.0f;
+  for (int s = 0; s < splits; ++s)
+    if (ml[(s * n + at) * 2 + 1] > 0.0f) mx = fmaxf(mx, ml[(s * n + at) * 2]);
+#pragma unroll
+  for (int s = 0; s < LT_MAX_SPLIT; ++s) {
+    f[s] = s < splits && ml[(s * n + at) * 2 + 1] > 0.0f ? exp2f(ml[(s * n + at) * 2] - mx) : 0.0f;
+    if (f[s] > 0.0f) den += f[s] * ml[(s * n + at) * 2 + 1];
+  }
+  const float inv = 1.0f / den;
+  bf16* out = static_cast<bf16*>(a.out) + at * a.ldo;
+  for (int d = threadIdx.x; d < a.R; d += 128) {
+    float o = 0.0f;
+#pragma unroll
+    for (int s = 0; s < LT_MAX_SPLIT; ++s)
+      if (f[s] > 0.0f) o += f[s] * part[(s * n + at) * a.R + d];
+    st(out + d, o * inv);
+  }
+}
+
+}  // namespace bxf

@@ -7,6 +7,7 @@
 #include "../../include/bitexact_float.h"
 #include "host_util.cuh"
 #include "fl_attention.cuh"
+#include "fl_attention_tc.cuh"
 #include "fl_gemm.cuh"
 #include "fl_gemm_simt.cuh"
 #include "fl_stages.cuh"
@@ -14,6 +15,8 @@
 namespace {
 
 using namespace bxf;
+
+static_assert(sizeof(bxf_epilogue) == 128 && sizeof(bxf_gru) == 80, "layouts of the callers' structs");
 
 inline cudaStream_t stream_of(void* s) { return static_cast<cudaStream_t>(s); }
 inline bool dtype_ok(int d) { return d == BXF_BF16 || d == BXF_F32; }
@@ -146,6 +149,52 @@ int run_bf16(const Operands& o, const GemmShape& s, const typename Epi::Params& 
     case 256: return launch_persistent<256, Epi>(o, s, ep, st);
     default: return BX_EARG;
   }
+}
+
+// The tensor-core attention kernel takes pages of 8, 16, .. keys, rows of at most 9 column blocks (shared memory).
+bool latent_tc_fits(int dtype, const LatentAttn& a) {
+  return dtype == BXF_BF16 && a.bs >= 8 && (a.bs & (a.bs - 1)) == 0 && ceil_div(a.R + a.rot, 64) <= 9 && aligned16(a.q) &&
+         aligned16(a.cache) && aligned16(a.out) && a.ldq % 8 == 0 && a.ldc % 8 == 0 && a.ldo % 8 == 0;
+}
+
+size_t latent_scratch(i64 rows, int R, int splits) { return (size_t)splits * rows * (R + 2) * sizeof(float); }
+
+int launch_latent_tc(const LatentAttn& a, void* scratch, size_t scratch_bytes, cudaStream_t st) {
+  constexpr int SMEM_MAX = 227 * 1024;
+  static PerDevice configured;
+  if (once_per_device(configured, [] {
+        return cudaFuncSetAttribute(fl_latent_attention_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MAX);
+      }) != BX_OK)
+    return BX_ELAUNCH;
+  LatentTc c = {};
+  const int W = a.R + a.rot;
+  c.cols = ceil_div(W, 64);
+  const int fixed = 1024 + c.cols * 128 * 128 + (int)sizeof(LatentShared);
+  c.stages = (SMEM_MAX - fixed) / (c.cols * LT_KEYS * 128);
+  if (c.stages > LT_MAX_STAGES) c.stages = LT_MAX_STAGES;
+  const int tokens = a.tiles ? bxf_latent_attention_tile(a.H) : 1, tiles = a.tiles ? a.ntiles : a.M;
+  const int rows = tokens * a.H;
+  c.qrows = rows >= 128 ? 128 : ceil_div(rows, 8) * 8;
+  c.row_blocks = ceil_div(rows, 128);
+  c.vsplit = ceil_div(a.R, LT_VCOLS);
+  c.splits = 1;
+  const i64 span = a.window > 0 && a.window + tokens < (i64)a.nblk * a.bs ? a.window + tokens : (i64)a.nblk * a.bs;
+  const i64 blocks = span / LT_KEYS + 1, ctas = (i64)tiles * c.row_blocks * c.vsplit;
+  const int sms = device_sms();
+  if (sms <= 0) return BX_ELAUNCH;
+  while (c.splits < LT_MAX_SPLIT && ctas * c.splits * 2 <= sms && blocks >= c.splits * 4 && scratch &&
+         scratch_bytes >= latent_scratch((i64)a.M * a.H, a.R, c.splits * 2))
+    c.splits *= 2;
+  c.part = static_cast<float*>(scratch);
+  CUtensorMap mq, mc;
+  if (!make_map_bf16(&mq, a.q, W, (i64)a.M * a.H, 1, a.ldq, 0, c.qrows, 1) ||
+      !make_map_bf16(&mc, a.cache, W, a.bs, a.nb, a.ldc, (i64)a.bs * a.ldc, a.bs < LT_KEYS ? a.bs : LT_KEYS, 1))
+    return BX_ELAUNCH;
+  const dim3 grid(tiles, c.splits, c.row_blocks * c.vsplit);
+  fl_latent_attention_tc_kernel<<<grid, LT_THREADS, fixed + c.stages * c.cols * LT_KEYS * 128, st>>>(mq, mc, a, c);
+  if (c.splits == 1) return launched(1);
+  fl_latent_join_kernel<<<(unsigned)(a.M * a.H), 128, 0, st>>>(a, c.part, c.splits);
+  return launched(2);
 }
 
 constexpr int GRU_TILE = 64, GRU_LONG_TILE = 128;        // bf16; the 32-bit kernel has tiles of SIMT_TA rows
@@ -287,7 +336,12 @@ int bxf_latent_prepare(int dtype, const float* y, int64_t ldy, int q_rank, int k
   return launched(1);
 }
 
-size_t bxf_latent_attention_scratch(int M, int heads, int kv_rank) { return 0; }
+// Key splits only happen while the query tiles leave SMs idle.
+size_t bxf_latent_attention_scratch(int M, int heads, int kv_rank) {
+  if (M < 1 || heads < 1 || kv_rank < 1 || M > 148) return 0;
+  return latent_scratch((i64)M * heads, kv_rank, LT_MAX_SPLIT);
+}
+
 int bxf_latent_attention_tile(int heads) { return heads >= 128 ? 1 : 128 / (heads < 1 ? 1 : heads); }
 
 int bxf_latent_attention(int dtype, const void* q, int64_t ldq, int M, int heads, int kv_rank, int rot_dim,
@@ -305,6 +359,9 @@ int bxf_latent_attention(int dtype, const void* q, int64_t ldq, int M, int heads
   const LatentAttn a{q, ldq, M, heads, kv_rank, rot_dim, cache, ldc, bs, nb, bt, bt_is64, bt_stride, nblk,
                      reinterpret_cast<const i64*>(seq), reinterpret_cast<const i64*>(pos), tiles, ntiles, window, sink,
                      scale, out, ldo};
+  if (variant == 2 && !latent_tc_fits(dtype, a)) return BX_ELIMIT;
+  if (variant != 1 && latent_tc_fits(dtype, a) && (!tiles || ntiles > 0))
+    return launch_latent_tc(a, scratch, scratch_bytes, stream_of(stream));
   const dim3 grid(M, heads);
   const int smem = (kv_rank + rot_dim) * 4;
   if (dtype == BXF_F32) fl_latent_attention_kernel<float><<<grid, LA_THREADS, smem, stream_of(stream)>>>(a);
