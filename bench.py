@@ -2,8 +2,9 @@
 """Benchmark of the exact-mode decode path: random-init Llama-3.2-1B, 512-token prompts, batched decode.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--repeats R] [--batch B] [--prompt P] [--mode exact|int8]
-                    [--impl reference]
+                    [--impl reference] [--workload llama|hybrid]
 
+`--workload hybrid` measures the hybrid float models beside the integer Llama instead (bench_hybrid.py). Otherwise:
 A step is one decode step of the whole batch: 16 layers (4 limb GEMMs, RoPE/KV store, paged attention, attention
 division, two RMSNorms, SiLU per layer), final norm, LM head and the integer Gumbel-max sampler at T = 0.7.
 One process per GPU; with N > 1 (torchrun) every rank decodes its own B sequences (sequence sharding, no
@@ -47,6 +48,8 @@ def parse():
     ap.add_argument("--mode", default="exact", choices=["exact", "int8"],
                     help="exact: original bf16 weights as 3 limbs (the headline); int8: int8 weights, 2-limb activations")
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
+    ap.add_argument("--workload", default="llama", choices=["llama", "hybrid"],
+                    help="hybrid: prefill and decode throughput of the hybrid float models beside the integer Llama")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-int8-extra", action="store_true", help="skip the int8-mode pass reported under `extra`")
     ap.add_argument("--no-column-sharded", action="store_true",
@@ -729,6 +732,11 @@ def main():
     world = int(os.environ.get("WORLD_SIZE", 1))
     if args.impl == "reference":
         run_reference(args, rank)
+        return
+    if args.workload == "hybrid":
+        import bench_hybrid
+        if rank == 0:
+            bench_hybrid.run(args)
         return
     if world > 1:
         import torch

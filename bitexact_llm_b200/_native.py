@@ -96,7 +96,7 @@ class Epilogue(ctypes.Structure):
 class Gru(ctypes.Structure):
     """bxf_gru."""
     _fields_ = [("bias_z", P), ("bias_x", P), ("state", P), ("flags", P), ("seq", P), ("out", P), ("ldo", L), ("decay", P),
-                ("local", P), ("mode", I), ("pad_", I)]
+                ("local", P), ("mode", I), ("tile", I)]
 
 
 _FLOAT_SIGNATURES = {
@@ -106,8 +106,7 @@ _FLOAT_SIGNATURES = {
     "bxf_clear_device_status": (I, []),
     "bxf_set_device_status": (I, [I]),
     "bxf_linear": (I, [I, P, L, L, P, L, L, I, I, I, I, P, ctypes.POINTER(Epilogue), I, P]),
-    "bxf_gru_tile_rows": (I, [I]),
-    "bxf_gru_long_tile": (I, [I]),
+    "bxf_gru_tile": (I, [I, I, I]),
     "bxf_gru_linear": (I, [I, P, L, P, L, I, I, I, ctypes.POINTER(Gru), P]),
     "bxf_gru_finish": (I, [I, I, I, ctypes.POINTER(Gru), P]),
     "bxf_row_flags": (I, [P, P, P, P, I, P]),

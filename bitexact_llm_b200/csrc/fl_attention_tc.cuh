@@ -7,9 +7,11 @@
 // the softmax warps leave it as bf16 in place of the scores. TMEM: two score buffers of 64 columns, then the output
 // accumulator (256 columns; a wider latent is cut into value slices over blockIdx.z).
 //
-// Warp 0 = TMA, warp 1 = MMA, warps 2 .. 5 = softmax, one thread per query row. The running maximum starts at the sink
-// (denominator 1); the accumulator is rescaled only when the maximum grows by more than 2^8 since the last time. Few
-// tiles (decoding): the keys of a tile are split over blockIdx.y, and a second kernel joins the parts.
+// Warp 0 = TMA, warp 1 = MMA, warps 2 .. 17 = softmax: a query row is shared by four threads (one per warp of its TMEM lane
+// quarter), 16 of the 64 keys each; a decoding tile fills one quarter only, and a single warp per row would be bound by its
+// own latency. The running maximum starts at the sink (denominator 1); the accumulator is rescaled only when the maximum
+// grows by more than 2^8 since the last time. Few tiles (decoding): the keys of a tile are split over blockIdx.y, and a
+// second kernel joins the parts.
 #pragma once
 
 #include "fl_attention.cuh"
@@ -17,7 +19,7 @@
 
 namespace bxf {
 
-constexpr int LT_KEYS = 64, LT_THREADS = 192, LT_MAX_STAGES = 4, LT_MAX_SPLIT = 4, LT_VCOLS = 256;
+constexpr int LT_KEYS = 64, LT_THREADS = 64 + 512, LT_MAX_STAGES = 4, LT_MAX_SPLIT = 8, LT_VCOLS = 256;
 constexpr int LT_O = 2 * LT_KEYS;                        // first TMEM column of the output accumulator
 constexpr float LT_LOG2E = 1.4426950408889634f;
 constexpr float LT_GROWTH = 8.0f;
@@ -34,8 +36,18 @@ struct LatentShared {
   uint64_t q_full, o_done;
   uint64_t full[LT_MAX_STAGES], empty[LT_MAX_STAGES];
   uint64_t s_full[2], p_full[2], pv_done[2];
+  float row_max[2][4][128], row_den[4][128];
   uint32_t tmem_base, abort_flag;
 };
+
+__device__ __forceinline__ float exp2_fast(float v) {
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+  return r;
+}
+
+// The four warps of a lane quarter.
+__device__ __forceinline__ void quarter_barrier(int quarter) { asm volatile("bar.sync %0, 128;" ::"r"(1 + quarter) : "memory"); }
 
 // D (+)= A[tmem] * B[smem]; A: bf16 pairs, one row per lane.
 __device__ __forceinline__ void umma_bf16_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t b_desc, uint32_t idesc,
@@ -68,10 +80,13 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
                               const LatentAttn a, const LatentTc c) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* qs = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint8_t* ring = qs + c.cols * 128 * 128;
+  const int q_box = c.qrows * 128;                       // bytes of a column block of the queries
+  uint8_t* ring = qs + c.cols * q_box;
   const int stage_bytes = c.cols * LT_KEYS * 128;
   LatentShared* sh = reinterpret_cast<LatentShared*>(ring + c.stages * stage_bytes);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+
+  wait_previous();
 
   // ---- the tile ----
   int tok0, ntok;
@@ -94,7 +109,7 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
   const int b0 = b_lo + (b_hi - b_lo) * (int)blockIdx.y / c.splits, b1 = b_lo + (b_hi - b_lo) * ((int)blockIdx.y + 1) / c.splits;
   const int nb = b1 - b0;
   if (rows <= 0) return;
-  const int soft_warps = (rows + 31) / 32;
+  const int quarters = (rows + 31) / 32;                 // TMEM lane quarters in use
 
   if (threadIdx.x == 0) {
     mbar_init(&sh->q_full, 1);
@@ -105,7 +120,7 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
     }
     for (int i = 0; i < 2; ++i) {
       mbar_init(&sh->s_full[i], 1);
-      mbar_init(&sh->p_full[i], soft_warps);
+      mbar_init(&sh->p_full[i], 4 * quarters);
       mbar_init(&sh->pv_done[i], 1);
     }
     sh->abort_flag = *reinterpret_cast<volatile int*>(&g_wait_timeouts) != 0;
@@ -121,6 +136,7 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
+  launch_next();                                         // after the TMEM allocation
   const uint32_t tmem = sh->tmem_base;
   const bool dead = sh->abort_flag != 0;
   __syncthreads();
@@ -134,9 +150,9 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
   } else if (warp == 0) {
     if (lane == 0 && nb > 0) {
       // ---- TMA: the queries once, then the key blocks page by page ----
-      mbar_arrive_expect_tx(&sh->q_full, c.cols * c.qrows * 128);
+      mbar_arrive_expect_tx(&sh->q_full, c.cols * q_box);
       for (int j = 0; j < c.cols; ++j)
-        tma_load_3d(qs + j * 128 * 128, &mq, &sh->q_full, j * 64, tok0 * a.H + row0, 0);
+        tma_load_3d(qs + j * q_box, &mq, &sh->q_full, j * 64, tok0 * a.H + row0, 0);
       const int box = min(a.bs, LT_KEYS), pages = LT_KEYS / box;
       int i = 0;
       bool ok = true;
@@ -160,7 +176,8 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
     }
   } else if (warp == 1) {
     if (lane == 0 && nb > 0) {
-      // ---- MMA: scores of block i + 1 are issued before the values of block i ----
+      // ---- MMA: scores of block i + 1 are issued before the values of block i. A query box of fewer than 128 rows is
+      //      read on into what follows it in shared memory: those accumulator lanes belong to no query ----
       constexpr uint32_t ID_S = umma_idesc_bf16(LT_KEYS);
       const uint32_t id_v = umma_idesc_bf16((vn + 15) / 16 * 16, true);
       auto scores = [&](int i) {
@@ -172,7 +189,7 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
         for (int j = 0; j < c.cols; ++j)
 #pragma unroll
           for (int ks = 0; ks < 4; ++ks)
-            umma_bf16(tmem + buf * LT_KEYS, umma_desc_sw128(qa + j * 128 * 128 + ks * 32),
+            umma_bf16(tmem + buf * LT_KEYS, umma_desc_sw128(qa + j * q_box + ks * 32),
                       umma_desc_sw128(ka + j * LT_KEYS * 128 + ks * 32), ID_S, (j | ks) != 0);
         umma_commit(&sh->s_full[buf]);
         return true;
@@ -194,136 +211,126 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
       if (ok) umma_commit(&sh->o_done);
       else fail();
     }
-  } else if (warp - 2 < 4) {
-    // ---- softmax: thread = query row (the TMEM lane quarter of the warp id) ----
-    const int quarter = warp & 3, r = quarter * 32 + lane;
-    if (quarter < soft_warps) {
-      const bool live = r < rows;
-      const int flat = row0 + (live ? r : 0), head = flat % a.H;
-      const int m = tok0 + flat / a.H;
-      const i64 pos = min(a.pos[m], limit);
-      const int lo = a.first_key(pos), hi = (int)pos;
-      const float scale = a.scale * LT_LOG2E;
-      const bool sink_here = a.sink && blockIdx.y == 0;
-      float ref = a.sink ? a.sink[head] * LT_LOG2E : -INFINITY, den = sink_here ? 1.0f : 0.0f;
-      const uint32_t lanes = (uint32_t)(quarter * 32) << 16;
-      bool ok = true;
-      for (int i = 0; i < nb; ++i) {
-        const int buf = i & 1;
-        ok = mbar_wait(&sh->s_full[buf], (i >> 1) & 1);
-        ok = __all_sync(0xffffffffu, ok);
-        if (!ok) break;
-        tc_fence_after();
-        float s[LT_KEYS];
+  } else if ((warp & 3) < quarters) {
+    // ---- softmax. A wait that gives up is remembered and the loop goes on (the quarter's barriers count every warp) ----
+    constexpr int KW = LT_KEYS / 4;
+    const int quarter = warp & 3, part = (warp - 2) >> 2, r = quarter * 32 + lane;
+    const bool live = r < rows;
+    const int flat = row0 + (live ? r : 0), head = flat % a.H;
+    const i64 pos = min(a.pos[tok0 + flat / a.H], limit);
+    const int lo = a.first_key(pos), hi = (int)pos;
+    const float scale = a.scale * LT_LOG2E;
+    float ref = a.sink ? a.sink[head] * LT_LOG2E : -INFINITY;
+    float den = a.sink && blockIdx.y == 0 && part == 0 ? 1.0f : 0.0f;
+    const uint32_t lanes = (uint32_t)(quarter * 32) << 16;
+    bool ok = true;
+    for (int i = 0; i < nb; ++i) {
+      const int buf = i & 1;
+      ok = ok && mbar_wait(&sh->s_full[buf], (i >> 1) & 1);
+      __syncwarp();
+      tc_fence_after();
+      uint32_t u[KW];
+      tmem_ld16(tmem + lanes + buf * LT_KEYS + part * KW, u);
+      tmem_ld_wait();
+      const int k0 = (b0 + i) * LT_KEYS + part * KW;
+      float s[KW], mx = -INFINITY;
+      if (k0 >= lo && k0 + KW - 1 <= hi) {
 #pragma unroll
-        for (int q = 0; q < LT_KEYS; q += 16) {
-          uint32_t u[16];
-          tmem_ld16(tmem + lanes + buf * LT_KEYS + q, u);
-          tmem_ld_wait();
-#pragma unroll
-          for (int k = 0; k < 16; ++k) s[q + k] = __uint_as_float(u[k]);
+        for (int k = 0; k < KW; ++k) {
+          s[k] = __uint_as_float(u[k]) * scale;
+          mx = fmaxf(mx, s[k]);
         }
-        const int k0 = (b0 + i) * LT_KEYS;
-        float mx = -INFINITY;
-        if (k0 >= lo && k0 + LT_KEYS - 1 <= hi) {
+      } else {
 #pragma unroll
-          for (int k = 0; k < LT_KEYS; ++k) {
-            s[k] *= scale;
-            mx = fmaxf(mx, s[k]);
+        for (int k = 0; k < KW; ++k) {
+          s[k] = k0 + k >= lo && k0 + k <= hi ? __uint_as_float(u[k]) * scale : -INFINITY;
+          mx = fmaxf(mx, s[k]);
+        }
+      }
+      sh->row_max[buf][part][r] = mx;
+      tc_fence_before();
+      quarter_barrier(quarter);                            // the quarter's scores are in registers: P may replace them
+      tc_fence_after();
+      mx = fmaxf(fmaxf(sh->row_max[buf][0][r], sh->row_max[buf][1][r]), fmaxf(sh->row_max[buf][2][r], sh->row_max[buf][3][r]));
+      float f = 1.0f;
+      if (mx > ref + LT_GROWTH || ref == -INFINITY) {
+        f = ref == -INFINITY ? 0.0f : exp2_fast(ref - mx);
+        ref = mx;
+      }
+      if (__any_sync(0xffffffffu, f != 1.0f && live)) {    // the same in the four warps of the quarter
+        den *= f;
+        if (i > 0) {
+          // the accumulator may be touched once the values of block i - 1 are in
+          ok = ok && mbar_wait(&sh->pv_done[buf ^ 1], ((i - 1) >> 1) & 1);
+          __syncwarp();
+          tc_fence_after();
+          for (int q = part * 16; q < vn; q += 64) {
+            uint32_t o[16];
+            tmem_ld16(tmem + lanes + LT_O + q, o);
+            tmem_ld_wait();
+#pragma unroll
+            for (int k = 0; k < 16; ++k) o[k] = __float_as_uint(__uint_as_float(o[k]) * f);
+            tmem_st16(tmem + lanes + LT_O + q, o);
           }
+        }
+      }
+      const float base = ref == -INFINITY ? 0.0f : ref;    // no visible key yet: every weight is 0
+      float d0 = 0.0f, d1 = 0.0f;
+      uint32_t w[KW / 2];
+#pragma unroll
+      for (int k = 0; k < KW / 2; ++k) {
+        const float e0 = exp2_fast(s[2 * k] - base), e1 = exp2_fast(s[2 * k + 1] - base);
+        d0 += e0;
+        d1 += e1;
+        w[k] = pack_bf16(e0, e1);
+      }
+      den += d0 + d1;
+      tmem_st8(tmem + lanes + buf * LT_KEYS + part * (KW / 2), w);
+      tmem_st_wait();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&sh->p_full[buf]);
+    }
+    if (nb > 0) ok = ok && mbar_wait(&sh->o_done, 0);
+    ok = __all_sync(0xffffffffu, ok);
+    sh->row_den[part][r] = den;
+    quarter_barrier(quarter);
+    den = (sh->row_den[0][r] + sh->row_den[1][r]) + (sh->row_den[2][r] + sh->row_den[3][r]);
+    if (!ok) {
+      if (lane == 0) fail();
+    } else {
+      tc_fence_after();
+      const i64 at = (i64)tok0 * a.H + row0 + r;
+      const float inv = 1.0f / den;
+      float* acc = c.part + ((i64)blockIdx.y * a.M * a.H + at) * a.R + v0;
+      bf16* out = static_cast<bf16*>(a.out) + at * a.ldo + v0;
+      for (int q = part * 16; q < vn; q += 64) {
+        uint32_t u[16] = {};
+        if (nb > 0) {
+          tmem_ld16(tmem + lanes + LT_O + q, u);
+          tmem_ld_wait();
+        }
+        if (!live) continue;
+        const int n = min(16, vn - q);
+        float v[16];
+#pragma unroll
+        for (int k = 0; k < 16; ++k) v[k] = __uint_as_float(u[k]) * (c.splits == 1 ? inv : 1.0f);
+        if (n == 16) {
+          if (c.splits == 1) store_run<16>(out + q, v);
+          else store_run<16>(acc + q, v);
         } else {
 #pragma unroll
-          for (int k = 0; k < LT_KEYS; ++k) {
-            s[k] = k0 + k >= lo && k0 + k <= hi ? s[k] * scale : -INFINITY;
-            mx = fmaxf(mx, s[k]);
-          }
-        }
-        float f = 1.0f;
-        if (mx > ref + LT_GROWTH || ref == -INFINITY) {
-          f = ref == -INFINITY ? 0.0f : exp2f(ref - mx);
-          ref = mx;
-        }
-        if (__any_sync(0xffffffffu, f != 1.0f && live)) {
-          den *= f;
-          if (i > 0) {
-            // the accumulator may be touched once the values of block i - 1 are in
-            ok = mbar_wait(&sh->pv_done[buf ^ 1], ((i - 1) >> 1) & 1);
-            ok = __all_sync(0xffffffffu, ok);
-            if (!ok) break;
-            tc_fence_after();
-            for (int q = 0; q < vn; q += 16) {
-              uint32_t u[16];
-              tmem_ld16(tmem + lanes + LT_O + q, u);
-              tmem_ld_wait();
-#pragma unroll
-              for (int k = 0; k < 16; ++k) u[k] = __float_as_uint(__uint_as_float(u[k]) * f);
-              tmem_st16(tmem + lanes + LT_O + q, u);
+          for (int k = 0; k < 16; ++k)
+            if (k < n) {
+              if (c.splits == 1) st(out + q + k, v[k]);
+              else acc[q + k] = v[k];
             }
-            tmem_st_wait();
-          }
         }
-        const float base = ref == -INFINITY ? 0.0f : ref;            // no visible key yet: every weight is 0
-        float d0 = 0.0f, d1 = 0.0f;
-#pragma unroll
-        for (int q = 0; q < LT_KEYS; q += 32) {
-          uint32_t u[16];
-#pragma unroll
-          for (int k = 0; k < 16; ++k) {
-            const float e0 = exp2f(s[q + 2 * k] - base), e1 = exp2f(s[q + 2 * k + 1] - base);
-            d0 += e0;
-            d1 += e1;
-            u[k] = pack_bf16(e0, e1);
-          }
-          tmem_st16(tmem + lanes + buf * LT_KEYS + q / 2, u);
-        }
-        den += d0 + d1;
-        tmem_st_wait();
-        tc_fence_before();
-        __syncwarp();
-        if (lane == 0) mbar_arrive(&sh->p_full[buf]);
       }
-      if (ok && nb > 0) ok = mbar_wait(&sh->o_done, 0);
-      ok = __all_sync(0xffffffffu, ok);
-      if (!ok) {
-        if (lane == 0) fail();
-      } else {
-        tc_fence_after();
-        const i64 at = (i64)tok0 * a.H + row0 + r;
-        const float inv = 1.0f / den;
-        float* part = c.part + ((i64)blockIdx.y * a.M * a.H + at) * a.R + v0;
-        bf16* out = static_cast<bf16*>(a.out) + at * a.ldo + v0;
-        for (int q = 0; q < vn; q += 16) {
-          uint32_t u[16] = {};
-          if (nb > 0) {
-            tmem_ld16(tmem + lanes + LT_O + q, u);
-            tmem_ld_wait();
-          }
-          if (!live) continue;
-          const int n = min(16, vn - q);
-          if (c.splits == 1) {
-            if (n == 16) {                                               // out rows start on 16-byte boundaries
-              uint32_t w[8];
-#pragma unroll
-              for (int k = 0; k < 8; ++k)
-                w[k] = pack_bf16(__uint_as_float(u[2 * k]) * inv, __uint_as_float(u[2 * k + 1]) * inv);
-              *reinterpret_cast<uint4*>(out + q) = make_uint4(w[0], w[1], w[2], w[3]);
-              *reinterpret_cast<uint4*>(out + q + 8) = make_uint4(w[4], w[5], w[6], w[7]);
-            } else {
-#pragma unroll
-              for (int k = 0; k < 16; ++k)
-                if (k < n) st(out + q + k, __uint_as_float(u[k]) * inv);
-            }
-          } else {
-#pragma unroll
-            for (int k = 0; k < 16; ++k)
-              if (k < n) part[q + k] = __uint_as_float(u[k]);
-          }
-        }
-        if (c.splits > 1 && live && v0 == 0) {
-          float* ml = c.part + (i64)c.splits * a.M * a.H * a.R + ((i64)blockIdx.y * a.M * a.H + at) * 2;
-          ml[0] = ref;
-          ml[1] = den;
-        }
+      if (c.splits > 1 && live && v0 == 0 && part == 0) {
+        float* ml = c.part + (i64)c.splits * a.M * a.H * a.R + ((i64)blockIdx.y * a.M * a.H + at) * 2;
+        ml[0] = ref;
+        ml[1] = den;
       }
     }
   }
@@ -339,6 +346,8 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
 
 // Joins the key splits: one CTA per query row (token, head).
 __global__ void __launch_bounds__(128) fl_latent_join_kernel(const LatentAttn a, const float* part, int splits) {
+  launch_next();
+  wait_previous();
   const i64 at = blockIdx.x, n = (i64)a.M * a.H;
   const float* ml = part + splits * n * a.R;
   float mx = -INFINITY, f[LT_MAX_SPLIT], den = 0.0f;

@@ -11,6 +11,15 @@ namespace bxf {
 using bf16 = __nv_bfloat16;
 using i64 = long long;
 
+// Programmatic dependent launch: the kernels of a step are launched so that the next one may start (barriers, TMEM, the
+// first weight tiles) while the last CTAs of the one before it are still running. `launch_next` permits that, as soon as
+// every CTA has come this far; `wait_previous` returns when the previous kernel has completed and its writes are visible,
+// and stands before the first access to anything another kernel of the step reads or writes. Weights are exempt. A
+// kernel that allocates TMEM calls `launch_next` after the allocation: a CTA of the next kernel on the same SM could
+// otherwise take the columns first and wait, holding them, for the CTA that needs them.
+__device__ __forceinline__ void launch_next() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
+__device__ __forceinline__ void wait_previous() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+
 template <class T>
 __device__ __forceinline__ float ld(const T* p);
 template <>

@@ -1,8 +1,11 @@
-// Epilogues of the float products. A product kernel computes a tile of 128 weight rows x TA token rows; an epilogue
-// thread owns ONE weight row (output channel) n and walks token columns, so per-channel constants live in registers, a
-// warp stores 32 consecutive channels of a token, a rotated pair is two neighbouring lanes, and a recurrence over tokens
-// is a loop of one thread. The kernels hand the accumulators over through a `get` object:
-//   get.template load<W>(plane, column, v)   W consecutive token columns of one product plane
+// Epilogues of the float products, for both orientations of a tile.
+// Weight-major (`run`): 128 weight rows x TA token rows; a thread owns ONE weight row (output channel) n and walks token
+// columns, so per-channel constants live in registers, a warp stores 32 consecutive channels of a token, a rotated pair
+// is two neighbouring lanes, and a recurrence over tokens is a loop of one thread.
+// Token-major (`run_rows`, long prompts): 128 token rows x TN weight rows; a thread owns one token and stores runs of
+// consecutive channels with 16-byte stores.
+// The kernels hand the accumulators over through a `get` object:
+//   get.template load<W>(plane, column, v)   W consecutive columns of one product plane
 // which reads TMEM, the summed partials of a K-split cluster, or registers. All calls are warp-collective.
 #pragma once
 
@@ -10,13 +13,61 @@
 
 namespace bxf {
 
-constexpr int NROWS = 128;           // weight rows of a tile
+constexpr int NROWS = 128;           // rows of the 128-row operand of a tile
 constexpr int EPI_THREADS = 512;     // epilogue threads: 16 warps, four per quarter of the 128 rows when K is not split
 
 struct Tile {
   int group, n0;                     // weight plane, first weight row
-  int row0, rows;                    // first token row, token rows that exist (<= TA)
+  int row0, rows;                    // first token row, token rows that exist
 };
+
+// N consecutive values to memory: 16-byte stores when the address allows them.
+template <int N>
+__device__ __forceinline__ void store_run(bf16* p, const float (&v)[N]) {
+  if ((reinterpret_cast<uintptr_t>(p) & 15) == 0) {
+#pragma unroll
+    for (int i = 0; i < N; i += 8) {
+      uint32_t w[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const __nv_bfloat162 b = __floats2bfloat162_rn(v[i + 2 * k], v[i + 2 * k + 1]);
+        w[k] = *reinterpret_cast<const uint32_t*>(&b);
+      }
+      *reinterpret_cast<uint4*>(p + i) = make_uint4(w[0], w[1], w[2], w[3]);
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; ++i) st(p + i, v[i]);
+  }
+}
+
+template <int N>
+__device__ __forceinline__ void store_run(float* p, const float (&v)[N]) {
+  if ((reinterpret_cast<uintptr_t>(p) & 15) == 0) {
+#pragma unroll
+    for (int i = 0; i < N; i += 4) *reinterpret_cast<float4*>(p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; ++i) p[i] = v[i];
+  }
+}
+
+template <int N>
+__device__ __forceinline__ void load_run(const float* p, float (&v)[N]) {
+  if ((reinterpret_cast<uintptr_t>(p) & 15) == 0) {
+#pragma unroll
+    for (int i = 0; i < N; i += 4) {
+      const float4 f = *reinterpret_cast<const float4*>(p + i);
+      v[i] = f.x;
+      v[i + 1] = f.y;
+      v[i + 2] = f.z;
+      v[i + 3] = f.w;
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] = p[i];
+  }
+}
 
 __device__ __forceinline__ void epi_barrier() { asm volatile("bar.sync 1, 512;" ::: "memory"); }
 
@@ -48,9 +99,12 @@ struct StageEpi {
     if (n >= N) return;
     if (p.kind == BXF_EPI_ADD) {
       float* o = static_cast<float*>(p.out) + row * p.ldo + n;
+      float old[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) old[i] = i < cnt ? o[i * p.ldo] : 0.0f;
 #pragma unroll
       for (int i = 0; i < 8; ++i)
-        if (i < cnt) o[i * p.ldo] += v[i];
+        if (i < cnt) o[i * p.ldo] = old[i] + v[i];
     } else if (p.kind == BXF_EPI_GATE) {
       T* o = static_cast<T*>(p.out) + group * p.gso + row * p.ldo + n;
 #pragma unroll
@@ -71,6 +125,102 @@ struct StageEpi {
         if (p.out_type == BXF_OUT_T) st(static_cast<T*>(p.out) + at + i * p.ldo, y);
         else if (p.out_type == BXF_OUT_F32) static_cast<float*>(p.out)[at + i * p.ldo] = y;
         else static_cast<i64*>(p.out)[at + i * p.ldo] = __double2ll_rn((double)y * 16777216.0);
+      }
+    }
+  }
+
+  static constexpr int RW = 8;                   // channels a thread takes at a time in `run_rows`
+
+  // Channels n .. n + cnt - 1 of token row m; v holds their accumulators.
+  template <class T>
+  static __device__ __forceinline__ void chunk_rows(const Params& p, int group, i64 m, int n, int cnt, float (&v)[RW]) {
+    const bool full = cnt == RW;
+    if (p.kind == BXF_EPI_ADD) {
+      float* o = static_cast<float*>(p.out) + m * p.ldo + n;
+      if (full) {
+        float old[RW];
+        load_run<RW>(o, old);
+#pragma unroll
+        for (int i = 0; i < RW; ++i) old[i] += v[i];
+        store_run<RW>(o, old);
+      } else {
+        for (int i = 0; i < RW; ++i)
+          if (i < cnt) o[i] += v[i];
+      }
+      return;
+    }
+    if (p.kind == BXF_EPI_ROPE && n >= p.n_main) {                      // n and n_main are even: whole pairs
+#pragma unroll
+      for (int i = 0; i < RW; i += 2) {
+        if (i >= cnt) break;
+        const int r = n + i - p.n_main, j = r % p.rot_dim;
+        const float2 cs = *reinterpret_cast<const float2*>(p.cs + (m * (p.rot_dim / 2) + (j >> 1)) * 2);
+        T* o = static_cast<T*>(p.rot_out) + m * p.ldr + r / p.rot_dim * p.hsr + j;
+        st(o, v[i] * cs.x - v[i + 1] * cs.y);
+        st(o + 1, v[i + 1] * cs.x + v[i] * cs.y);
+      }
+      return;
+    }
+    if (p.kind == BXF_EPI_GATE) {
+      const float g = p.gate[m * p.ldg + group];
+#pragma unroll
+      for (int i = 0; i < RW; ++i) v[i] *= g;
+    } else if (p.kind == BXF_EPI_STORE) {
+#pragma unroll
+      for (int i = 0; i < RW; ++i) {
+        if (i < cnt && n + i >= p.n_main)
+          p.side[m * p.lds + (n + i - p.n_main)] = v[i] + (p.bias ? p.bias[n + i - p.n_main] : 0.0f);
+      }
+      if (n >= p.n_main) return;
+      if (p.act == BXF_ACT_RELU2) {
+#pragma unroll
+        for (int i = 0; i < RW; ++i) v[i] = activate(BXF_ACT_RELU2, v[i], 0.0f, 0.0f);
+      } else if (p.act == BXF_ACT_XIELU) {
+#pragma unroll
+        for (int i = 0; i < RW; ++i) v[i] = activate(BXF_ACT_XIELU, v[i], p.act_p, p.act_q);
+      }
+      cnt = min(cnt, p.n_main - n);
+    }
+    const i64 at = group * p.gso + m * p.ldo + n;
+    if (p.out_type == BXF_OUT_I64) {
+#pragma unroll
+      for (int i = 0; i < RW; ++i)
+        if (i < cnt) static_cast<i64*>(p.out)[at + i] = __double2ll_rn((double)v[i] * 16777216.0);
+    } else if (p.out_type == BXF_OUT_F32) {
+      float* o = static_cast<float*>(p.out) + at;
+      if (cnt == RW) {
+        store_run<RW>(o, v);
+      } else {
+#pragma unroll
+        for (int i = 0; i < RW; ++i)
+          if (i < cnt) o[i] = v[i];
+      }
+    } else {
+      T* o = static_cast<T*>(p.out) + at;
+      if (cnt == RW) {
+        store_run<RW>(o, v);
+      } else {
+#pragma unroll
+        for (int i = 0; i < RW; ++i)
+          if (i < cnt) st(o + i, v[i]);
+      }
+    }
+  }
+
+  // row: the thread's token row of the tile; the four warps of a lane quarter take 16 columns in turn.
+  template <class T, int TN, class Get>
+  static __device__ __forceinline__ void run_rows(Get& get, const Params& p, const Tile& t, int N, int row, int group_index) {
+    for (int c = group_index * 16; c < TN && t.n0 + c < N; c += 64) {
+      float v[16];
+      get.template load<16>(0, c, v);
+      if (row >= t.rows) continue;
+#pragma unroll
+      for (int h = 0; h < 16; h += RW) {
+        const int n = t.n0 + c + h, cnt = min(RW, N - n);
+        float w[RW];
+#pragma unroll
+        for (int i = 0; i < RW; ++i) w[i] = v[h + i];
+        if (cnt > 0) chunk_rows<T>(p, t.group, (i64)t.row0 + row, n, cnt, w);
       }
     }
   }

@@ -1,12 +1,13 @@
-// bf16 products on tcgen05 (kind::f16, fp32 accumulators in TMEM), weights on the MMA M side like the limb GEMM: 128
-// weight rows per tile (TMEM lanes), TA token rows as the MMA N side, so a decode batch of 1 .. 16 rows streams the
-// weights once with TA = 16 and a prompt runs tiles of 128 x 256. NP product planes (the three projections of a minGRU
-// layer) share one token tile: plane p accumulates into TMEM columns [p TA, (p + 1) TA).
+// bf16 products on tcgen05 (kind::f16, fp32 accumulators in TMEM).
 //
 // Warp roles as in limb_gemm.cuh: warp 0 = TMA producer, warp 1 = TMEM allocation + MMA issue, warps 2 .. 17 = epilogue.
-// Two kernels: one tile per cluster with K split over its S CTAs (short tile lists; the fp32 partials are exchanged
-// through distributed shared memory and every CTA finishes 128 / S weight rows), and a persistent one with two TMEM
-// buffers (long tile lists; the epilogue of a tile runs behind the MMAs of the next).
+// fl_gemm_kernel (short tile lists: decoding, short portions) has the weights on the MMA M side like the limb GEMM: 128
+// weight rows (TMEM lanes) x TA token rows, so a batch of 1 .. 16 rows streams the weights once with TA = 16. A cluster of S
+// CTAs shares a tile with K split between them; the fp32 partials are exchanged through distributed shared memory and
+// every CTA finishes 128 / S weight rows. NP product planes (the three projections of a minGRU layer) share one token
+// tile: plane p accumulates into TMEM columns [p TA, (p + 1) TA).
+// fl_gemm_persistent_kernel (long tile lists: prompts) has the tokens on the M side: 128 token rows x TN weight rows, two
+// TMEM buffers, so that the epilogue of a tile (16-byte stores of consecutive channels) runs behind the MMAs of the next.
 // Every wait is bounded; a timeout raises the device status word and the CTA leaves without storing.
 #pragma once
 
@@ -72,7 +73,8 @@ struct TmemGet {
   template <int W>
   __device__ __forceinline__ void load(int plane, int c, float (&v)[W]) const {
     uint32_t r[W];
-    tmem_ldn<W>(base + plane * ta + c, r);
+    if constexpr (W == 16) tmem_ld16(base + plane * ta + c, r);
+    else tmem_ldn<W>(base + plane * ta + c, r);
     tmem_ld_wait();
 #pragma unroll
     for (int i = 0; i < W; ++i) v[i] = __uint_as_float(r[i]);
@@ -98,19 +100,39 @@ struct ClusterGet {
 };
 
 // ---- the two asynchronous roles; `it` counts stages over the life of the CTA ----
-template <int NP, int TA>
+// TOKENS_M: the 128-row operand is the token tile (one plane), else the weight tile. Of the CTA's first tile, `ahead`
+// stages have their weights under way already (feed_weights).
+template <int NP, int TA, bool TOKENS_M = false>
 __device__ __forceinline__ bool feed_tile(FlShared* sh, uint8_t* ring, const CUtensorMap* mw, const CUtensorMap* mx,
-                                          const Tile& t, bool ragged, int kb0, int nkb, int& it) {
+                                          const Tile& t, bool ragged, int kb0, int nkb, int& it, int ahead = 0) {
   using Cfg = FlCfg<NP, TA>;
   for (int i = 0; i < nkb; ++i, ++it) {
     const int s = it % Cfg::STAGES, round = it / Cfg::STAGES;
     if (round > 0 && !mbar_wait(&sh->empty[s], (round - 1) & 1)) return false;
     uint8_t* st = ring + s * Cfg::STAGE_BYTES;
-    mbar_arrive_expect_tx(&sh->full[s], Cfg::STAGE_BYTES);
-    tma_load_3d(st, mw, &sh->full[s], (kb0 + i) * KE, t.n0, NP == 1 ? t.group : 0);
-    tma_load_3d(st + Cfg::W_BYTES, mx, &sh->full[s], (kb0 + i) * KE, t.row0, ragged ? 0 : t.group);
+    uint8_t* w_tile = TOKENS_M ? st + Cfg::W_BYTES : st;
+    uint8_t* x_tile = TOKENS_M ? st : st + Cfg::W_BYTES;
+    if (i >= ahead) {
+      mbar_arrive_expect_tx(&sh->full[s], Cfg::STAGE_BYTES);
+      tma_load_3d(w_tile, mw, &sh->full[s], (kb0 + i) * KE, t.n0, NP == 1 ? t.group : 0);
+    }
+    tma_load_3d(x_tile, mx, &sh->full[s], (kb0 + i) * KE, t.row0, ragged ? 0 : t.group);
   }
   return true;
+}
+
+// The weight tiles of the first stages of the CTA's first tile, ahead of the previous kernel's end; returns how many.
+template <int NP, int TA, bool TOKENS_M = false>
+__device__ __forceinline__ int feed_weights(FlShared* sh, uint8_t* ring, const CUtensorMap* mw, const Tile& t, int kb0,
+                                            int nkb) {
+  using Cfg = FlCfg<NP, TA>;
+  const int n = min(nkb, Cfg::STAGES);
+  for (int s = 0; s < n; ++s) {
+    mbar_arrive_expect_tx(&sh->full[s], Cfg::STAGE_BYTES);
+    tma_load_3d(ring + s * Cfg::STAGE_BYTES + (TOKENS_M ? Cfg::W_BYTES : 0), mw, &sh->full[s], (kb0 + s) * KE, t.n0,
+                NP == 1 ? t.group : 0);
+  }
+  return n;
 }
 
 template <int NP, int TA>
@@ -173,6 +195,7 @@ __device__ __forceinline__ uint32_t open_cta(FlShared* sh, int stages, const CUt
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
+  launch_next();                        // after the TMEM allocation: the next kernel's CTAs allocate too
   return sh->tmem_base;
 }
 
@@ -205,6 +228,7 @@ fl_gemm_kernel(const __grid_constant__ CUtensorMap mw, const __grid_constant__ C
   const int S = (int)cluster.num_blocks(), rank = (int)cluster.block_rank();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   Tile t;
+  if (s.counts) wait_previous();                                        // the group sizes are the previous kernels' work
   if (!locate_tile(s, TA, blockIdx.x / S, t)) return;                  // the same for every CTA of the cluster
   const int nkb_all = (s.K + KE - 1) / KE;
   const int kb0 = rank * nkb_all / S, nkb = (rank + 1) * nkb_all / S - kb0;
@@ -216,7 +240,9 @@ fl_gemm_kernel(const __grid_constant__ CUtensorMap mw, const __grid_constant__ C
   if (warp == 0) {
     if (lane == 0 && !dead) {
       int it = 0;
-      if (!feed_tile<NP, TA>(sh, ring, &mw, &mx, t, s.counts != nullptr, kb0, nkb, it)) {
+      const int ahead = feed_weights<NP, TA>(sh, ring, &mw, t, kb0, nkb);
+      wait_previous();
+      if (!feed_tile<NP, TA>(sh, ring, &mw, &mx, t, s.counts != nullptr, kb0, nkb, it, ahead)) {
         give_up(sh);
         drain_ring<Cfg::STAGES>(sh, it);
       }
@@ -228,6 +254,7 @@ fl_gemm_kernel(const __grid_constant__ CUtensorMap mw, const __grid_constant__ C
       else give_up(sh);
     }
   } else if (!dead) {
+    wait_previous();
     if (nkb > 0) ok = mbar_wait(&sh->acc_full[0], 0);
     ok = ok && !aborted(sh);
     ok = __all_sync(0xffffffffu, ok);
@@ -277,13 +304,12 @@ fl_gemm_kernel(const __grid_constant__ CUtensorMap mw, const __grid_constant__ C
 }
 
 // ---- persistent: every CTA walks the tile list, two TMEM buffers ----
-template <int TA, class Epi>
+template <int TN, class Epi>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
 fl_gemm_persistent_kernel(const __grid_constant__ CUtensorMap mw, const __grid_constant__ CUtensorMap mx,
                           const GemmShape s, const __grid_constant__ typename Epi::Params ep) {
-  constexpr int NP = Epi::PLANES;
-  using Cfg = FlCfg<NP, TA>;
-  static_assert(2 * Cfg::COLS <= 512 && Epi::stash_bytes(TA) == 0, "two accumulator buffers, no stash");
+  using Cfg = FlCfg<1, TN>;
+  static_assert(2 * Cfg::COLS <= 512 && Epi::PLANES == 1, "two accumulator buffers");
   constexpr int TCOLS = Cfg::tmem_cols(2 * Cfg::COLS);
   extern __shared__ uint8_t smem_raw[];
   uint8_t* ring = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -295,14 +321,15 @@ fl_gemm_persistent_kernel(const __grid_constant__ CUtensorMap mw, const __grid_c
   const uint32_t tmem = open_cta<TCOLS>(sh, Cfg::STAGES, &mw, &mx);
   const bool dead = sh->abort_flag != 0;
   __syncthreads();
+  wait_previous();
   Tile t;
   if (!dead) {
     if (warp == 0) {
       int it = 0;
       bool ok = true;
       for (int tile = blockIdx.x; tile < total && ok; tile += gridDim.x) {
-        if (!locate_tile(s, TA, tile, t)) continue;
-        if (lane == 0) ok = feed_tile<NP, TA>(sh, ring, &mw, &mx, t, ragged, 0, nkb, it);
+        if (!locate_tile(s, NROWS, tile, t, TN)) continue;
+        if (lane == 0) ok = feed_tile<1, TN, true>(sh, ring, &mw, &mx, t, ragged, 0, nkb, it);
         ok = __all_sync(0xffffffffu, ok);
       }
       if (!ok && lane == 0) {
@@ -313,12 +340,12 @@ fl_gemm_persistent_kernel(const __grid_constant__ CUtensorMap mw, const __grid_c
       int it = 0, count = 0;
       bool ok = true;
       for (int tile = blockIdx.x; tile < total && ok; tile += gridDim.x) {
-        if (!locate_tile(s, TA, tile, t)) continue;
+        if (!locate_tile(s, NROWS, tile, t, TN)) continue;
         const int buf = count & 1, use = count >> 1;
         if (lane == 0) {
           if (use > 0) ok = mbar_wait(&sh->acc_empty[buf], (use - 1) & 1);
           tc_fence_after();
-          ok = ok && multiply_tile<NP, TA>(sh, ring, tmem + buf * Cfg::COLS, nkb, it);
+          ok = ok && multiply_tile<1, TN>(sh, ring, tmem + buf * Cfg::COLS, nkb, it);
           if (ok) umma_commit(&sh->acc_full[buf]);
         }
         ok = __all_sync(0xffffffffu, ok);
@@ -330,14 +357,14 @@ fl_gemm_persistent_kernel(const __grid_constant__ CUtensorMap mw, const __grid_c
       int count = 0;
       bool ok = true;
       for (int tile = blockIdx.x; tile < total; tile += gridDim.x) {
-        if (!locate_tile(s, TA, tile, t)) continue;
+        if (!locate_tile(s, NROWS, tile, t, TN)) continue;
         const int buf = count & 1, use = count >> 1;
         ok = mbar_wait(&sh->acc_full[buf], use & 1) && !aborted(sh);
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
         tc_fence_after();
-        TmemGet get{tmem + buf * Cfg::COLS + ((uint32_t)(quarter * 32) << 16), TA};
-        Epi::template run<bf16, TA, 8>(get, ep, t, s.N, quarter * 32 + lane, we >> 2, 4, nullptr);
+        TmemGet get{tmem + buf * Cfg::COLS + ((uint32_t)(quarter * 32) << 16), TN};
+        Epi::template run_rows<bf16, TN>(get, ep, t, s.N, quarter * 32 + lane, we >> 2);
         tc_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive(&sh->acc_empty[buf]);

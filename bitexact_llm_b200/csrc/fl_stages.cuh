@@ -7,6 +7,8 @@
 namespace bxf {
 
 __global__ void fl_row_flags_kernel(const i64* seq, const i64* slot, const i64* pos, int* flags, int M) {
+  launch_next();
+  wait_previous();
   const int m = blockIdx.x * blockDim.x + threadIdx.x;
   if (m >= M) return;
   if (slot[m] < 0) {
@@ -26,6 +28,8 @@ __global__ void __launch_bounds__(NORM_THREADS)
 fl_norm_kernel(float* __restrict__ x, const i64* ids, const T* __restrict__ embed, i64 V, const float* __restrict__ y,
                const int* __restrict__ place, const float* __restrict__ weight, int top, const float* __restrict__ w,
                const float* __restrict__ b, float eps, T* __restrict__ h, i64 ldh, int* zero, int nzero, int D) {
+  launch_next();
+  wait_previous();
   extern __shared__ float row[];
   __shared__ float red[33];
   const i64 m = blockIdx.x;
@@ -82,6 +86,8 @@ fl_norm_kernel(float* __restrict__ x, const i64* ids, const T* __restrict__ embe
 // One warp per row: `top` rounds of (largest, lowest index first).
 __global__ void fl_route_kernel(const float* __restrict__ logits, i64 ldl, int E, int top, int* chosen, float* weight,
                                 int* rank, int* counts, int M) {
+  launch_next();
+  wait_previous();
   const int m = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (m >= M) return;
   const float* z = logits + m * ldl;
@@ -129,6 +135,8 @@ template <class T>
 __global__ void __launch_bounds__(128)
 fl_gather_kernel(const T* __restrict__ h, i64 ldh, int D, const int* chosen, const int* rank, const int* counts, int top,
                  T* __restrict__ hp, int* place) {
+  launch_next();
+  wait_previous();
   __shared__ int base;
   const int pair = blockIdx.x, e = chosen[pair];
   if (threadIdx.x < 32) {
@@ -161,6 +169,8 @@ fl_latent_prepare_kernel(const float* __restrict__ y, i64 ldy, int q_rank, int R
                          const float* __restrict__ wq, const float* __restrict__ wkv, float eps,
                          const float* __restrict__ freq, const i64* pos, const i64* slot, T* __restrict__ cq, i64 ldcq,
                          T* __restrict__ cache, i64 ldc, float* __restrict__ cs, float* __restrict__ gate) {
+  launch_next();
+  wait_previous();
   __shared__ float red[33];
   const i64 m = blockIdx.x;
   const float* ym = y + m * ldy;
@@ -192,6 +202,8 @@ fl_latent_prepare_kernel(const float* __restrict__ y, i64 ldy, int q_rank, int R
 template <class T>
 __global__ void __launch_bounds__(128)
 fl_gru_finish_kernel(const bxf_gru g, int M, int width, int tile) {
+  launch_next();
+  wait_previous();
   const int n = blockIdx.x * 128 + threadIdx.x, j = blockIdx.y;
   if (n >= width) return;
   float carry = 0.0f;

@@ -45,10 +45,11 @@ __device__ __forceinline__ bool locate_ragged(const int* counts, int groups, int
   return false;
 }
 
-// Token tiles are the fastest index, so consecutive CTAs share a weight tile. Warp-collective.
-__device__ __forceinline__ bool locate_tile(const GemmShape& s, int ta, int tile, Tile& t) {
+// Tile number `tile` of tiles of ta token rows x tn weight rows. Token tiles are the fastest index, so consecutive CTAs
+// share a weight tile. Warp-collective.
+__device__ __forceinline__ bool locate_tile(const GemmShape& s, int ta, int tile, Tile& t, int tn = NROWS) {
   const int mt = tile % s.m_tiles, rest = tile / s.m_tiles;
-  t.n0 = (rest % s.n_tiles) * NROWS;
+  t.n0 = (rest % s.n_tiles) * tn;
   if (s.counts) return locate_ragged(s.counts, s.groups, ta, mt, t);
   t.group = rest / s.n_tiles;
   t.row0 = mt * ta;

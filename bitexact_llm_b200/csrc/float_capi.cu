@@ -37,6 +37,28 @@ bool make_map_bf16(CUtensorMap* m, const void* base, i64 K, i64 rows, i64 planes
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
+// Launch with the permission to start before the previous kernel of the stream has ended (every kernel launched this way
+// calls wait_previous before it touches dependent memory).
+template <class... P, class... A>
+int launch_chained(void (*kernel)(P...), dim3 grid, int threads, int smem, cudaStream_t st, int cluster, A&&... args) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = grid;
+  cfg.blockDim = dim3(threads, 1, 1);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = st;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = 1;
+  attr[1].id = cudaLaunchAttributeClusterDimension;
+  attr[1].val.clusterDim.x = cluster;
+  attr[1].val.clusterDim.y = 1;
+  attr[1].val.clusterDim.z = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = cluster > 0 ? 2 : 1;
+  if (cudaLaunchKernelEx(&cfg, kernel, static_cast<P>(args)...) != cudaSuccess) return BX_ELAUNCH;
+  return launched(1);
+}
+
 struct Operands {
   const void *w, *x;
   i64 ldw, gsw, ldx, gsx;
@@ -58,73 +80,101 @@ int launch_simt(const Operands& o, GemmShape s, const typename Epi::Params& ep, 
   return launched(1);
 }
 
+// Token tiles of `rows` rows: exact for dense lists, an upper bound for ragged ones (the sizes are on the device).
+int token_tiles(const GemmShape& s, int rows) {
+  return s.counts ? s.M / rows + (s.groups < s.M ? s.groups : s.M) : ceil_div(s.M, rows);
+}
+
+// ---- which kernel and tile: the estimated cycles of the slowest SM ----
+struct Plan {
+  int tile;                    // token rows (16, 32, 64: fl_gemm_kernel) or weight rows (128, 256: persistent kernel)
+  int split;                   // CTAs that share K
+  double cycles;
+};
+
+// Expected token tiles; experts' sizes vary, so their tiles are counted at 1.3 times the mean size.
+double expected_tiles(const GemmShape& s, int rows) {
+  if (!s.counts) return ceil_div(s.M, rows);
+  const int used = s.groups < s.M ? s.groups : s.M;
+  return (double)used * ceil_div((int)(1.3 * s.M / used + 0.5), rows);
+}
+
+// A K block of a tile of R + C rows moves (R + C) x 128 bytes into shared memory and reads them once for the MMAs, at 128
+// bytes a cycle; the constants are the measured prologue, epilogue and cluster exchange.
+Plan tile_plan(const GemmShape& s, int planes, int ta, int max_split, int sms) {
+  const double tiles = expected_tiles(s, ta) * ceil_div(s.N, NROWS) * (s.counts || planes > 1 ? 1 : s.groups);
+  const int nkb = ceil_div(s.K, KE);
+  Plan best = {ta, 1, 1e300};
+  for (int split = 1; split <= max_split && (split == 1 || nkb >= 2 * split); split *= 2) {
+    const double waves = (double)(i64)((tiles * split + sms - 1) / sms);
+    const double per = ceil_div(nkb, split) * 2.3 * (planes * NROWS + ta) + 3000 + 20.0 * planes * ta + (split > 1 ? 1800 : 0);
+    if (waves * per < best.cycles) best = {ta, split, waves * per};
+  }
+  return best;
+}
+
+Plan persistent_plan(const GemmShape& s, int tn, int sms) {
+  const double tiles = expected_tiles(s, NROWS) * ceil_div(s.N, tn) * (s.counts ? 1 : s.groups);
+  const double waves = (double)(i64)((tiles + sms - 1) / sms);
+  const double loop = ceil_div(s.K, KE) * 2.3 * (NROWS + tn), epilogue = 25.0 * tn;
+  return {tn, 1, waves * (loop > epilogue ? loop : epilogue) + 3000 + epilogue};
+}
+
+Plan plan_linear(const GemmShape& s, int sms) {
+  Plan best = tile_plan(s, 1, 16, FL_SPLIT_MAX, sms);
+  const auto consider = [&](const Plan& p) {
+    if (p.cycles < best.cycles) best = p;
+  };
+  consider(tile_plan(s, 1, 32, FL_SPLIT_MAX, sms));
+  consider(tile_plan(s, 1, 64, FL_SPLIT_MAX, sms));
+  consider(persistent_plan(s, 128, sms));
+  consider(persistent_plan(s, 256, sms));
+  return best;
+}
+
+// One tile per cluster of `split` CTAs.
 template <int TA, class Epi>
-int maps_for(const Operands& o, const GemmShape& s, CUtensorMap* mw, CUtensorMap* mx) {
+int launch_tiles(const Operands& o, GemmShape s, const typename Epi::Params& ep, int split, cudaStream_t st) {
   constexpr int NP = Epi::PLANES;
-  const bool ok = make_map_bf16(mw, o.w, s.K, s.N, NP > 1 ? NP : s.groups, o.ldw, o.gsw, NROWS, NP) &&
-                  make_map_bf16(mx, o.x, s.K, s.M, NP > 1 || s.counts ? 1 : s.groups, o.ldx, o.gsx, TA, 1);
-  return ok ? BX_OK : BX_ELAUNCH;
-}
-
-template <int TA, class Epi>
-void tile_counts(GemmShape& s) {
-  s.n_tiles = ceil_div(s.N, NROWS);
-  s.m_tiles = s.counts ? s.M / TA + (s.groups < s.M ? s.groups : s.M) : ceil_div(s.M, TA);
-}
-
-// One tile per cluster; K is split while the tile list leaves most SMs idle and every slice keeps a few K blocks.
-template <int TA, class Epi>
-int launch_tiles(const Operands& o, GemmShape s, const typename Epi::Params& ep, cudaStream_t st) {
-  using Cfg = FlCfg<Epi::PLANES, TA>;
+  using Cfg = FlCfg<NP, TA>;
   static PerDevice configured;
   if (once_per_device(configured, [] {
         return cudaFuncSetAttribute(fl_gemm_kernel<TA, Epi>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                     Cfg::SMEM_BYTES);
       }) != BX_OK)
     return BX_ELAUNCH;
-  tile_counts<TA, Epi>(s);
+  s.n_tiles = ceil_div(s.N, NROWS);
+  s.m_tiles = token_tiles(s, TA);
   CUtensorMap mw, mx;
-  if (int rc = maps_for<TA, Epi>(o, s, &mw, &mx)) return rc;
-  const i64 tiles = (i64)s.n_tiles * s.m_tiles * (s.counts || Epi::PLANES > 1 ? 1 : s.groups);
-  const int sms = device_sms(), nkb = ceil_div(s.K, KE);
-  if (sms <= 0 || tiles > (1 << 24)) return BX_ELAUNCH;
-  int split = 1;
-  if (Cfg::PARTIAL_BYTES + Epi::stash_bytes(TA) <= Cfg::RING_BYTES)
-    while (split < FL_SPLIT_MAX && tiles * split * 2 <= sms && nkb >= split * 4) split *= 2;
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3((unsigned)(tiles * split), 1, 1);
-  cfg.blockDim = dim3(GEMM_THREADS, 1, 1);
-  cfg.dynamicSmemBytes = Cfg::SMEM_BYTES;
-  cfg.stream = st;
-  cudaLaunchAttribute attr[1];
-  attr[0].id = cudaLaunchAttributeClusterDimension;
-  attr[0].val.clusterDim.x = split;
-  attr[0].val.clusterDim.y = 1;
-  attr[0].val.clusterDim.z = 1;
-  cfg.attrs = attr;
-  cfg.numAttrs = 1;
-  if (cudaLaunchKernelEx(&cfg, fl_gemm_kernel<TA, Epi>, mw, mx, s, ep) != cudaSuccess) return BX_ELAUNCH;
-  return launched(1);
+  if (!make_map_bf16(&mw, o.w, s.K, s.N, NP > 1 ? NP : s.groups, o.ldw, o.gsw, NROWS, NP) ||
+      !make_map_bf16(&mx, o.x, s.K, s.M, NP > 1 || s.counts ? 1 : s.groups, o.ldx, o.gsx, TA, 1))
+    return BX_ELAUNCH;
+  const i64 tiles = (i64)s.n_tiles * s.m_tiles * (s.counts || NP > 1 ? 1 : s.groups);
+  if (tiles > (1 << 24)) return BX_ELIMIT;
+  if (Cfg::PARTIAL_BYTES + Epi::stash_bytes(TA) > Cfg::RING_BYTES) split = 1;
+  return launch_chained(fl_gemm_kernel<TA, Epi>, dim3((unsigned)(tiles * split)), GEMM_THREADS, Cfg::SMEM_BYTES, st, split,
+                        mw, mx, s, ep);
 }
 
-template <int TA, class Epi>
-int launch_persistent(const Operands& o, GemmShape s, const typename Epi::Params& ep, cudaStream_t st) {
-  using Cfg = FlCfg<Epi::PLANES, TA>;
+template <int TN, class Epi>
+int launch_persistent(const Operands& o, GemmShape s, const typename Epi::Params& ep, int sms, cudaStream_t st) {
+  using Cfg = FlCfg<1, TN>;
   static PerDevice configured;
   if (once_per_device(configured, [] {
-        return cudaFuncSetAttribute(fl_gemm_persistent_kernel<TA, Epi>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        return cudaFuncSetAttribute(fl_gemm_persistent_kernel<TN, Epi>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                     Cfg::SMEM_BYTES);
       }) != BX_OK)
     return BX_ELAUNCH;
-  tile_counts<TA, Epi>(s);
+  s.n_tiles = ceil_div(s.N, TN);
+  s.m_tiles = token_tiles(s, NROWS);
   CUtensorMap mw, mx;
-  if (int rc = maps_for<TA, Epi>(o, s, &mw, &mx)) return rc;
+  if (!make_map_bf16(&mw, o.w, s.K, s.N, s.groups, o.ldw, o.gsw, TN, 1) ||
+      !make_map_bf16(&mx, o.x, s.K, s.M, s.counts ? 1 : s.groups, o.ldx, o.gsx, NROWS, 1))
+    return BX_ELAUNCH;
   const i64 tiles = (i64)s.n_tiles * s.m_tiles * (s.counts ? 1 : s.groups);
-  const int sms = device_sms();
-  if (sms <= 0 || tiles > (1 << 24)) return BX_ELAUNCH;
-  fl_gemm_persistent_kernel<TA, Epi><<<(unsigned)(tiles < sms ? tiles : sms), GEMM_THREADS, Cfg::SMEM_BYTES, st>>>(mw, mx,
-                                                                                                                s, ep);
-  return launched(1);
+  if (tiles > (1 << 24)) return BX_ELIMIT;
+  return launch_chained(fl_gemm_persistent_kernel<TN, Epi>, dim3((unsigned)(tiles < sms ? tiles : sms)), GEMM_THREADS,
+                        Cfg::SMEM_BYTES, st, 0, mw, mx, s, ep);
 }
 
 bool operand_ok(const void* p, i64 ld, i64 gs, bool grouped, int K, int dtype) {
@@ -132,21 +182,18 @@ bool operand_ok(const void* p, i64 ld, i64 gs, bool grouped, int K, int dtype) {
   return dtype == BXF_F32 || (aligned16(p) && ld % 8 == 0 && (!grouped || gs % 8 == 0));
 }
 
-// Rows of a token tile when the caller leaves it open: the smallest that holds a group's rows (for experts: twice the
-// mean, their sizes vary).
-int pick_tile(const GemmShape& s) {
-  const int rows = s.counts ? ceil_div(2 * s.M, s.groups) : s.M;
-  return rows <= 16 ? 16 : rows <= 32 ? 32 : rows <= 64 ? 64 : rows <= 128 ? 128 : 256;
-}
-
-template <class Epi>
-int run_bf16(const Operands& o, const GemmShape& s, const typename Epi::Params& ep, int ta, cudaStream_t st) {
-  switch (ta ? ta : pick_tile(s)) {
-    case 16: return launch_tiles<16, Epi>(o, s, ep, st);
-    case 32: return launch_tiles<32, Epi>(o, s, ep, st);
-    case 64: return launch_tiles<64, Epi>(o, s, ep, st);
-    case 128: return launch_persistent<128, Epi>(o, s, ep, st);
-    case 256: return launch_persistent<256, Epi>(o, s, ep, st);
+int run_bf16(const Operands& o, const GemmShape& s, const bxf_epilogue& ep, int tile, cudaStream_t st) {
+  const int sms = device_sms();
+  if (sms <= 0) return BX_ELAUNCH;
+  Plan p = {tile, 1, 0};
+  if (tile == 0) p = plan_linear(s, sms);
+  else if (tile <= 64) p = tile_plan(s, 1, tile, FL_SPLIT_MAX, sms);
+  switch (p.tile) {
+    case 16: return launch_tiles<16, StageEpi>(o, s, ep, p.split, st);
+    case 32: return launch_tiles<32, StageEpi>(o, s, ep, p.split, st);
+    case 64: return launch_tiles<64, StageEpi>(o, s, ep, p.split, st);
+    case 128: return launch_persistent<128, StageEpi>(o, s, ep, sms, st);
+    case 256: return launch_persistent<256, StageEpi>(o, s, ep, sms, st);
     default: return BX_EARG;
   }
 }
@@ -169,12 +216,12 @@ int launch_latent_tc(const LatentAttn& a, void* scratch, size_t scratch_bytes, c
   LatentTc c = {};
   const int W = a.R + a.rot;
   c.cols = ceil_div(W, 64);
-  const int fixed = 1024 + c.cols * 128 * 128 + (int)sizeof(LatentShared);
-  c.stages = (SMEM_MAX - fixed) / (c.cols * LT_KEYS * 128);
-  if (c.stages > LT_MAX_STAGES) c.stages = LT_MAX_STAGES;
   const int tokens = a.tiles ? bxf_latent_attention_tile(a.H) : 1, tiles = a.tiles ? a.ntiles : a.M;
   const int rows = tokens * a.H;
   c.qrows = rows >= 128 ? 128 : ceil_div(rows, 8) * 8;
+  const int fixed = 1024 + c.cols * c.qrows * 128 + (int)sizeof(LatentShared);
+  c.stages = (SMEM_MAX - fixed) / (c.cols * LT_KEYS * 128);
+  if (c.stages > LT_MAX_STAGES) c.stages = LT_MAX_STAGES;
   c.row_blocks = ceil_div(rows, 128);
   c.vsplit = ceil_div(a.R, LT_VCOLS);
   c.splits = 1;
@@ -191,13 +238,11 @@ int launch_latent_tc(const LatentAttn& a, void* scratch, size_t scratch_bytes, c
       !make_map_bf16(&mc, a.cache, W, a.bs, a.nb, a.ldc, (i64)a.bs * a.ldc, a.bs < LT_KEYS ? a.bs : LT_KEYS, 1))
     return BX_ELAUNCH;
   const dim3 grid(tiles, c.splits, c.row_blocks * c.vsplit);
-  fl_latent_attention_tc_kernel<<<grid, LT_THREADS, fixed + c.stages * c.cols * LT_KEYS * 128, st>>>(mq, mc, a, c);
-  if (c.splits == 1) return launched(1);
-  fl_latent_join_kernel<<<(unsigned)(a.M * a.H), 128, 0, st>>>(a, c.part, c.splits);
-  return launched(2);
+  const int rc = launch_chained(fl_latent_attention_tc_kernel, grid, LT_THREADS, fixed + c.stages * c.cols * LT_KEYS * 128, st,
+                                0, mq, mc, a, c);
+  if (rc != BX_OK || c.splits == 1) return rc;
+  return launch_chained(fl_latent_join_kernel, dim3((unsigned)(a.M * a.H)), 128, 0, st, 0, a, c.part, c.splits);
 }
-
-constexpr int GRU_TILE = 64, GRU_LONG_TILE = 128;        // bf16; the 32-bit kernel has tiles of SIMT_TA rows
 
 }  // namespace
 
@@ -210,7 +255,7 @@ int bxf_clear_device_status(void) { return status_clear(); }
 int bxf_set_device_status(int value) { return status_write(value); }
 
 int bxf_linear(int dtype, const void* w, int64_t ldw, int64_t gsw, const void* x, int64_t ldx, int64_t gsx, int groups,
-               int M, int N, int K, const int* counts, const bxf_epilogue* epi, int tile_rows, void* stream) {
+               int M, int N, int K, const int* counts, const bxf_epilogue* epi, int tile, void* stream) {
   if (!dtype_ok(dtype) || !epi || groups < 1 || M < 0 || N < 1 || K < 1) return BX_EARG;
   if (!operand_ok(w, ldw, gsw, groups > 1, K, dtype) || !operand_ok(x, ldx, gsx, groups > 1 && !counts, K, dtype))
     return BX_EARG;
@@ -218,53 +263,61 @@ int bxf_linear(int dtype, const void* w, int64_t ldw, int64_t gsw, const void* x
   if (epi->kind == BXF_EPI_STORE && epi->n_main < N && (!epi->side || groups > 1)) return BX_EARG;
   if (epi->kind == BXF_EPI_GATE && !epi->gate) return BX_EARG;
   if (epi->kind == BXF_EPI_ROPE &&
-      (!epi->rot_out || !epi->cs || epi->rot_dim < 2 || epi->rot_dim % 2 || epi->n_main % 2 || groups > 1))
+      (!epi->rot_out || !epi->cs || epi->rot_dim < 2 || epi->rot_dim % 2 || epi->n_main % 8 || groups > 1))
     return BX_EARG;
   if (g_status_seen.load() != 0) return BX_EDEVICE;
   if (M == 0) return BX_OK;
   const Operands o{w, x, ldw, gsw, ldx, gsx};
   const GemmShape s{M, N, K, groups, 0, 0, counts};
   if (dtype == BXF_F32) return launch_simt<StageEpi>(o, s, *epi, stream_of(stream));
-  return run_bf16<StageEpi>(o, s, *epi, tile_rows, stream_of(stream));
+  return run_bf16(o, s, *epi, tile, stream_of(stream));
 }
 
-int bxf_gru_tile_rows(int dtype) { return dtype == BXF_F32 ? SIMT_TA : GRU_TILE; }
-int bxf_gru_long_tile(int dtype) { return dtype == BXF_F32 ? SIMT_TA : GRU_LONG_TILE; }
+// Small tiles while the list of large ones leaves SMs idle.
+int bxf_gru_tile(int dtype, int M, int width) {
+  if (dtype == BXF_F32) return SIMT_TA;
+  if (M <= 16) return 16;
+  return M <= 64 || (i64)ceil_div(M, 128) * ceil_div(width, NROWS) < 128 ? 64 : 128;
+}
 
 int bxf_gru_linear(int dtype, const void* w, int64_t ldw, const void* x, int64_t ldx, int M, int width, int K,
                    const bxf_gru* gru, void* stream) {
   if (!dtype_ok(dtype) || !gru || M < 0 || width < 1 || K < 1) return BX_EARG;
   if (!operand_ok(w, ldw, (i64)width * ldw, true, K, dtype) || !operand_ok(x, ldx, 0, false, K, dtype)) return BX_EARG;
   if (!gru->bias_z || !gru->bias_x || !gru->state || !gru->flags || !gru->seq || !gru->out) return BX_EARG;
-  if (gru->mode == 0 ? M > bxf_gru_tile_rows(dtype) : (gru->mode != 1 || !gru->decay || !gru->local)) return BX_EARG;
+  if (dtype == BXF_F32 ? gru->tile != SIMT_TA : gru->tile != 16 && gru->tile != 64 && gru->tile != 128) return BX_EARG;
+  if (gru->mode == 0 ? M > gru->tile || gru->tile == 128 : (gru->mode != 1 || !gru->decay || !gru->local)) return BX_EARG;
   if (g_status_seen.load() != 0) return BX_EDEVICE;
   if (M == 0) return BX_OK;
   const Operands o{w, x, ldw, (i64)width * ldw, ldx, 0};
   const GemmShape s{M, width, K, 1, 0, 0, nullptr};
   cudaStream_t st = stream_of(stream);
   if (dtype == BXF_F32) return launch_simt<GruEpi>(o, s, *gru, st);
-  if (gru->mode == 1) return launch_tiles<GRU_LONG_TILE, GruEpi>(o, s, *gru, st);
-  if (M <= 16) return launch_tiles<16, GruEpi>(o, s, *gru, st);
-  return launch_tiles<GRU_TILE, GruEpi>(o, s, *gru, st);
+  const int sms = device_sms();
+  if (sms <= 0) return BX_ELAUNCH;
+  const int split = gru->tile == 128 ? 1 : tile_plan(s, 3, gru->tile, FL_SPLIT_MAX, sms).split;
+  if (gru->tile == 16) return launch_tiles<16, GruEpi>(o, s, *gru, split, st);
+  if (gru->tile == 64) return launch_tiles<64, GruEpi>(o, s, *gru, split, st);
+  return launch_tiles<128, GruEpi>(o, s, *gru, 1, st);
 }
 
 int bxf_gru_finish(int dtype, int M, int width, const bxf_gru* gru, void* stream) {
   if (!dtype_ok(dtype) || !gru || gru->mode != 1 || M < 0 || width < 1 || !gru->decay || !gru->local || !gru->out)
     return BX_EARG;
   if (M == 0) return BX_OK;
-  const int tile = bxf_gru_long_tile(dtype);
+  const int tile = gru->tile;
+  if (tile < 16) return BX_EARG;
   const dim3 grid(ceil_div(width, 128), ceil_div(M, tile), tile / 16);
-  if (dtype == BXF_F32) fl_gru_finish_kernel<float><<<grid, 128, 0, stream_of(stream)>>>(*gru, M, width, tile);
-  else fl_gru_finish_kernel<bf16><<<grid, 128, 0, stream_of(stream)>>>(*gru, M, width, tile);
-  return launched(1);
+  return launch_chained(dtype == BXF_F32 ? fl_gru_finish_kernel<float> : fl_gru_finish_kernel<bf16>, grid, 128, 0,
+                        stream_of(stream), 0, *gru, M, width, tile);
 }
 
 int bxf_row_flags(const int64_t* seq, const int64_t* slot, const int64_t* pos, int* flags, int M, void* stream) {
   if (!seq || !slot || !pos || !flags || M < 0) return BX_EARG;
   if (M == 0) return BX_OK;
-  fl_row_flags_kernel<<<ceil_div(M, 256), 256, 0, stream_of(stream)>>>(
-      reinterpret_cast<const i64*>(seq), reinterpret_cast<const i64*>(slot), reinterpret_cast<const i64*>(pos), flags, M);
-  return launched(1);
+  return launch_chained(fl_row_flags_kernel, dim3(ceil_div(M, 256)), 256, 0, stream_of(stream), 0,
+                        reinterpret_cast<const i64*>(seq), reinterpret_cast<const i64*>(slot),
+                        reinterpret_cast<const i64*>(pos), flags, M);
 }
 
 int bxf_norm(int dtype, float* x, const int64_t* ids, const void* embed, int64_t V, const float* y, const int* place,
@@ -283,9 +336,8 @@ int bxf_norm(int dtype, float* x, const int64_t* ids, const void* embed, int64_t
           return cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 32768 * 4);
         }) != BX_OK)
       return BX_ELAUNCH;
-    kernel<<<M, NORM_THREADS, smem, stream_of(stream)>>>(x, ids_, static_cast<const T*>(embed), V, y, place, weight, top, w,
-                                                         b, eps, static_cast<T*>(h), ldh, zero, nzero, D);
-    return launched(1);
+    return launch_chained(kernel, dim3(M), NORM_THREADS, smem, stream_of(stream), 0, x, ids_, static_cast<const T*>(embed), V,
+                          y, place, weight, top, w, b, eps, static_cast<T*>(h), ldh, zero, nzero, D);
   };
   static PerDevice conf16, conf32;
   return dtype == BXF_F32 ? go(fl_norm_kernel<float>, (float*)nullptr, conf32) : go(fl_norm_kernel<bf16>, (bf16*)nullptr, conf16);
@@ -296,8 +348,8 @@ int bxf_route(const float* logits, int64_t ldl, int experts, int top, int* chose
   if (!logits || !chosen || !weight || !rank || !counts || M < 0) return BX_EARG;
   if (experts < 1 || experts > BXF_MAX_EXPERTS || top < 1 || top > BXF_MAX_TOP || top > experts) return BX_ELIMIT;
   if (M == 0) return BX_OK;
-  fl_route_kernel<<<ceil_div(M, 8), 256, 0, stream_of(stream)>>>(logits, ldl, experts, top, chosen, weight, rank, counts, M);
-  return launched(1);
+  return launch_chained(fl_route_kernel, dim3(ceil_div(M, 8)), 256, 0, stream_of(stream), 0, logits, ldl, experts, top, chosen,
+                        weight, rank, counts, M);
 }
 
 int bxf_gather(int dtype, const void* h, int64_t ldh, int D, const int* chosen, const int* rank, const int* counts,
@@ -306,12 +358,10 @@ int bxf_gather(int dtype, const void* h, int64_t ldh, int D, const int* chosen, 
   if (experts < 1 || experts > BXF_MAX_EXPERTS || top < 1 || top > BXF_MAX_TOP) return BX_ELIMIT;
   if (M == 0) return BX_OK;
   if (dtype == BXF_F32)
-    fl_gather_kernel<float><<<M * top, 128, 0, stream_of(stream)>>>(static_cast<const float*>(h), ldh, D, chosen, rank,
-                                                                    counts, top, static_cast<float*>(hp), place);
-  else
-    fl_gather_kernel<bf16><<<M * top, 128, 0, stream_of(stream)>>>(static_cast<const bf16*>(h), ldh, D, chosen, rank, counts,
-                                                                   top, static_cast<bf16*>(hp), place);
-  return launched(1);
+    return launch_chained(fl_gather_kernel<float>, dim3(M * top), 128, 0, stream_of(stream), 0, static_cast<const float*>(h),
+                          ldh, D, chosen, rank, counts, top, static_cast<float*>(hp), place);
+  return launch_chained(fl_gather_kernel<bf16>, dim3(M * top), 128, 0, stream_of(stream), 0, static_cast<const bf16*>(h), ldh,
+                        D, chosen, rank, counts, top, static_cast<bf16*>(hp), place);
 }
 
 int bxf_latent_prepare(int dtype, const float* y, int64_t ldy, int q_rank, int kv_rank, int rot_dim, int heads,
@@ -326,20 +376,19 @@ int bxf_latent_prepare(int dtype, const float* y, int64_t ldy, int q_rank, int k
   if (M == 0) return BX_OK;
   const i64 *pos_ = reinterpret_cast<const i64*>(pos), *slot_ = reinterpret_cast<const i64*>(slot);
   if (dtype == BXF_F32)
-    fl_latent_prepare_kernel<float><<<M, PREP_THREADS, 0, stream_of(stream)>>>(
-        y, ldy, q_rank, kv_rank, rot_dim, heads, wq, wkv, eps, freq, pos_, slot_, static_cast<float*>(cq), ldcq,
-        static_cast<float*>(cache), ldc, cs, gate);
-  else
-    fl_latent_prepare_kernel<bf16><<<M, PREP_THREADS, 0, stream_of(stream)>>>(
-        y, ldy, q_rank, kv_rank, rot_dim, heads, wq, wkv, eps, freq, pos_, slot_, static_cast<bf16*>(cq), ldcq,
-        static_cast<bf16*>(cache), ldc, cs, gate);
-  return launched(1);
+    return launch_chained(fl_latent_prepare_kernel<float>, dim3(M), PREP_THREADS, 0, stream_of(stream), 0, y, ldy, q_rank,
+                          kv_rank, rot_dim, heads, wq, wkv, eps, freq, pos_, slot_, static_cast<float*>(cq), ldcq,
+                          static_cast<float*>(cache), ldc, cs, gate);
+  return launch_chained(fl_latent_prepare_kernel<bf16>, dim3(M), PREP_THREADS, 0, stream_of(stream), 0, y, ldy, q_rank,
+                        kv_rank, rot_dim, heads, wq, wkv, eps, freq, pos_, slot_, static_cast<bf16*>(cq), ldcq,
+                        static_cast<bf16*>(cache), ldc, cs, gate);
 }
 
-// Key splits only happen while the query tiles leave SMs idle.
+// Key splits only happen while the query tiles leave SMs idle (148 of them).
 size_t bxf_latent_attention_scratch(int M, int heads, int kv_rank) {
   if (M < 1 || heads < 1 || kv_rank < 1 || M > 148) return 0;
-  return latent_scratch((i64)M * heads, kv_rank, LT_MAX_SPLIT);
+  const int splits = 148 / M < 2 ? 2 : 148 / M > LT_MAX_SPLIT ? LT_MAX_SPLIT : 148 / M;
+  return latent_scratch((i64)M * heads, kv_rank, splits);
 }
 
 int bxf_latent_attention_tile(int heads) { return heads >= 128 ? 1 : 128 / (heads < 1 ? 1 : heads); }

@@ -23,7 +23,7 @@ class HybridEngine(TokenRowEngine):
 
     def __init__(self, spec, weights, dev="cuda", dtype="bfloat16", n_layers=None):
         """spec: ModelSpec; weights: {'embed', 'head', 'final': (w, b), 'layers': [{'norm1', 'norm2': (w, b), 'mixer',
-        'ff': dicts of the mechanism}]} as CPU tensors (a design's `read_weights`)."""
+        'ff': dicts of the mechanism}]} as tensors (a design's `read_weights`)."""
         self.dev, self.spec = torch.device(dev), spec
         self.dtype, _ = ops.DTYPES[dtype]
         self.D, self.V = spec.width, spec.vocab

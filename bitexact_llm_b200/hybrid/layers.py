@@ -61,7 +61,7 @@ class LatentAttention:
         # query rows: every head's unrotated part (padded to 8), then every head's rotated part
         uq = w["uq"].view(H, dn + dr, spec.q_rank)
         self.dnp = ops.pad8(dn)
-        nope = torch.zeros(H, self.dnp, spec.q_rank, dtype=uq.dtype)
+        nope = torch.zeros(H, self.dnp, spec.q_rank, dtype=uq.dtype, device=uq.device)
         nope[:, :dn] = uq[:, :dn]
         self.uq = ops.pack(torch.cat([nope.view(-1, spec.q_rank), uq[:, dn:].reshape(-1, spec.q_rank)]), dtype, dev)
         self.uk = ops.pack(w["uk"].view(H, dn, R).transpose(1, 2), dtype, dev)          # [H, R, dn]

@@ -30,10 +30,10 @@ def code(t):
     return 1 if t.dtype == torch.float32 else 0
 
 
-def linear(w, x, M, N, K, epi, groups=1, gsw=0, ldx=None, gsx=0, counts=None, tile_rows=0):
+def linear(w, x, M, N, K, epi, groups=1, gsw=0, ldx=None, gsx=0, counts=None, tile=0):
     """w [(groups,) N, ldw] and x [M, ldx] tensors of one element type; epi: nv.Epilogue."""
     rc = nv.float_lib().bxf_linear(code(w), w.data_ptr(), w.shape[-1], gsw, x.data_ptr(), x.stride(0) if ldx is None else ldx,
-                                   gsx, groups, M, N, K, nv.ptr(counts), ctypes.byref(epi), tile_rows, nv.stream())
+                                   gsx, groups, M, N, K, nv.ptr(counts), ctypes.byref(epi), tile, nv.stream())
     nv.check(rc, "bxf_linear")
 
 
@@ -76,7 +76,8 @@ def min_gru(w, bias_z, bias_x, h, width, K, state, flags, seq):
     M, lib, dt = h.shape[0], nv.float_lib(), code(w)
     out = torch.empty(M, pad8(width), dtype=w.dtype, device=h.device)
     g = nv.Gru(bias_z=bias_z.data_ptr(), bias_x=bias_x.data_ptr(), state=state.data_ptr(), flags=flags.data_ptr(),
-               seq=seq.data_ptr(), out=out.data_ptr(), ldo=out.stride(0), mode=int(M > lib.bxf_gru_tile_rows(dt)))
+               seq=seq.data_ptr(), out=out.data_ptr(), ldo=out.stride(0), tile=lib.bxf_gru_tile(dt, M, width))
+    g.mode = int(M > g.tile)
     if g.mode:
         scan = torch.empty(2, M, width, dtype=torch.float32, device=h.device)
         g.decay, g.local = scan[0].data_ptr(), scan[1].data_ptr()

@@ -69,7 +69,7 @@ typedef struct {
   int64_t ldo;
   float *decay, *local;         /* mode 1: float [M, width] */
   int mode;                     /* 0: rows fit one tile, finished here; 1: bxf_gru_finish follows */
-  int pad_;
+  int tile;                     /* rows of a tile (bxf_gru_tile) */
 } bxf_gru;
 
 int bxf_version(void);
@@ -82,17 +82,17 @@ int bxf_set_device_status(int value);
  *   w T [groups, N, ldw] (group stride gsw), x T [groups, M, ldx] (group stride gsx)
  *   counts NULL: every group has the M rows. Else int32 [groups]: the rows of x are ordered by group, group e has
  *   counts[e] of the M rows (experts; gsx unused, and out's rows are the rows of x).
- *   tile_rows 0 = automatic (else a row-tile size of the bf16 kernels); results do not depend on it beyond rounding. */
+ *   tile 0 = automatic; bf16: 16, 32, 64 = token rows of a weight-major tile, 128, 256 = weight rows of a token-major
+ *   tile (128 tokens). Results do not depend on it beyond rounding. */
 int bxf_linear(int dtype, const void* w, int64_t ldw, int64_t gsw, const void* x, int64_t ldx, int64_t gsx, int groups,
-               int M, int N, int K, const int* counts, const bxf_epilogue* epi, int tile_rows, void* stream);
+               int M, int N, int K, const int* counts, const bxf_epilogue* epi, int tile, void* stream);
 
 /* The three products of a minGRU layer with its recurrence: w T [3, width, ldw] (planes z, x, g), x T [M, ldx].
  * z = sigmoid(acc_0 + bias_z), u = acc_1 + bias_x, candidate = u + 1/2 (u >= 0) or sigmoid(u),
  * S = (1 - z) S + z candidate along the rows of a sequence, from `state` (zero on BXF_ROW_START) and back into it.
- * bxf_gru_tile_rows: the most rows mode 0 takes. Mode 1 leaves for every row the prefix product of (1 - z) and the
- * state from a zero start, both within its tile of bxf_gru_long_tile rows, for bxf_gru_finish. */
-int bxf_gru_tile_rows(int dtype);
-int bxf_gru_long_tile(int dtype);
+ * bxf_gru_tile: the tile for M rows; mode 0 when they fit it. Mode 1 leaves for every row the prefix product of (1 - z)
+ * and the state from a zero start, both within its tile, for bxf_gru_finish. */
+int bxf_gru_tile(int dtype, int M, int width);
 int bxf_gru_linear(int dtype, const void* w, int64_t ldw, const void* x, int64_t ldx, int M, int width, int K,
                    const bxf_gru* gru, void* stream);
 int bxf_gru_finish(int dtype, int M, int width, const bxf_gru* gru, void* stream);

@@ -7,7 +7,11 @@
     python microbench.py prefill [--batch 4] [--ctx 2048] [--iters 10]
     python microbench.py prompt [--batch 4] [--ctx 2048] [--chunk 4096] [--iters 3]
     python microbench.py bmm [--ctx 2048] [--iters 5]
+    python microbench.py hybrid [--m 1,16,256,4096] [--iters 10]
 
+hybrid: every kernel of the hybrid float models at the sizes of bench_hybrid.py's w2048 (bytes and FLOPs of the algorithm,
+      inputs beyond L2; fractions of the copy bandwidth and of the bf16 GEMM rate in MEASURED_PEAKS.json, else of
+      6.65 TB/s and 1.59 PFLOP/s).
 gemm: the exact-mode fused linear on the projection shapes of one Llama-3.2-1B layer and the LM head
       (int8-equivalent ops = 2 * 9 * M * N * K; algorithmic bytes = 3 N K + 4 M K + 8 M N).
 gemmr: the fused projections of one layer with REAL constants (bf16 weights from N(0, 0.02^2), decomposed into limbs
@@ -423,9 +427,165 @@ def stages(args):
     return out
 
 
+def peaks():
+    path = os.path.join(os.path.dirname(os.path.abspath(__file__)), "MEASURED_PEAKS.json")
+    if os.path.exists(path):
+        with open(path) as f:
+            d = json.load(f)
+        return d["hbm_gbs"] * 1e9, d["bf16_tflops"] * 1e12
+    return 6.65e12, 1.59e15
+
+
+def hybrid(args):
+    from types import SimpleNamespace
+
+    from bitexact_llm_b200.hybrid import ops
+    from bitexact_llm_b200.hybrid.spec import LatentAttentionSpec
+    dev, D, BF = "cuda", 2048, torch.bfloat16
+    hbm, mma = peaks()
+    only = set(args.proj.split(",")) if args.proj else None
+    W = lambda *s: torch.randn(*s, device=dev, dtype=BF) * 0.02
+    X = lambda *s: torch.randn(*s, device=dev, dtype=BF)
+    F = lambda *s: torch.randn(*s, device=dev)
+
+    def report(name, M, make, flops, byts, per_set):
+        """make() -> a call on a fresh set of inputs, which must keep every tensor alive whose address it passes on;
+        per_set: bytes of one set."""
+        if only and name not in only:
+            return
+        n = max(1, min(24, int((200 << 20) // per_set) + 1))
+        calls = [make() for _ in range(n)]
+        us = _graph_time(lambda i: calls[i](), n, args.iters) * 1e3
+        rec = {"kernel": name, "M": M, "us": round(us, 2), "tflops": round(flops / us / 1e6, 1), "GBps": round(byts / us / 1e3, 1),
+               "roofline_us": round(max(flops / mma, byts / hbm) * 1e6, 2)}
+        rec["frac"] = round(rec["roofline_us"] / us, 3)
+        print(json.dumps(rec), flush=True)
+
+    def linear(name, M, N, K, kind, groups=1, act="none"):
+        def make():
+            w, x = W(groups, N, K) if groups > 1 else W(N, K), X(M, groups * K)
+            if kind == "add":
+                out = F(M, N)
+                epi = ops.add(out)
+            elif kind == "i64":
+                out = torch.empty(M, N, device=dev, dtype=torch.long)
+                epi = ops.store(out, N, N, out_type=ops.OUT_I64)
+            else:
+                out = torch.empty(M, groups * N, device=dev, dtype=BF if kind == "bf16" else torch.float32)
+                epi = ops.store(out, groups * N, N, act, 0.3, 0.8, ops.OUT_T if kind == "bf16" else ops.OUT_F32, gso=N)
+            return lambda: (out, ops.linear(w, x, M, N, K, epi, groups=groups, gsw=N * K, ldx=groups * K, gsx=K))
+        out_b = {"add": 8, "i64": 8, "bf16": 2, "f32": 4}[kind]
+        report(name, M, make, 2.0 * groups * M * N * K, groups * (2.0 * N * K + 2.0 * M * K + out_b * M * N),
+               groups * (2 * N * K + 2 * M * K + out_b * M * N))
+
+    def experts(name, M, N, K, E, top, kind):
+        rows = M * top
+        used = min(E, rows)
+
+        def make():
+            w, x = W(E, N, K), X(rows, K)
+            counts = torch.full((E,), rows // E, dtype=torch.int32, device=dev)
+            counts[: rows % E] += 1
+            out = torch.empty(rows, N, device=dev, dtype=BF if kind == "bf16" else torch.float32)
+            epi = ops.store(out, N, N, "relu2" if kind == "bf16" else "none", out_type=ops.OUT_T if kind == "bf16" else ops.OUT_F32)
+            return lambda: (out, ops.linear(w, x, rows, N, K, epi, groups=E, gsw=N * K, counts=counts))
+        byts = 2.0 * used * N * K + 2.0 * rows * K + (2 if kind == "bf16" else 4) * rows * N
+        report(name, M, make, 2.0 * rows * N * K, byts, byts)
+
+    def gru(M):
+        width = D
+
+        def make():
+            w, x = W(3, width, D), X(M, D)
+            b, state = F(width), torch.zeros(min(M, 256), width, device=dev)
+            flags = torch.full((M,), 3 if M <= 256 else 0, dtype=torch.int32, device=dev)
+            flags[0] |= 1
+            flags[-1] |= 2
+            seq = torch.arange(M, device=dev) if M <= 256 else torch.zeros(M, dtype=torch.long, device=dev)
+            return lambda: ops.min_gru(w, b, b, x, width, D, state, flags, seq)
+        report("min_gru", M, make, 6.0 * M * width * D, 6.0 * width * D + 2.0 * M * D + 2.0 * M * width + (8.0 * M * width if M <= 256 else 0),
+               6 * width * D + 4 * M * D)
+
+    def attention(name, B, ctx, tokens, window, H=32, R=256, rot=32):
+        sp = LatentAttentionSpec(H, 64, rot, 64, 768, R, 1e6, 0.1, window, 1e-6)
+        M, bs = B * tokens, 16
+        nblk = (ctx + bs - 1) // bs
+
+        def make():
+            cache = X(1 + B * nblk, bs, R + rot)
+            bt = (torch.randperm(B * nblk, device=dev) + 1).view(B, nblk).int()
+            seq = torch.arange(B, device=dev).repeat_interleave(tokens)
+            pos = torch.arange(ctx - tokens, ctx, device=dev).repeat(B)
+            q, sink = X(M, H, R + rot), F(H)
+            n = nv.float_lib().bxf_latent_attention_tile(H)
+            tiles = None
+            if tokens > 1:
+                tiles = torch.tensor([(b, b * tokens + t, min(n, tokens - t)) for b in range(B) for t in range(0, tokens, n)],
+                                     dtype=torch.int32, device=dev)
+            return lambda: ops.latent_attention(q, sp, cache, bt, seq, pos, sink, tiles)
+        keys = sum(min(p + 1, window or p + 1) for p in range(ctx - tokens, ctx)) * B
+        kv = B * min(ctx, (window or ctx) + tokens - 1) * (R + rot) * 2.0
+        report(name, M, make, 2.0 * keys * H * (2 * R + rot), kv + 2.0 * M * H * (2 * R + rot), kv + 2 * M * H * (R + rot))
+
+    for M in [int(v) for v in args.m.split(",")]:
+        linear("dense_up", M, 6 * D, D, "bf16", act="xielu")
+        linear("shared_up", M, 2 * D, D, "bf16", act="relu2")
+        linear("down", M, D, 2 * D, "add")
+        linear("mixer_out", M, D, D, "add")
+        linear("latent_first", M, 768 + 288 + 32, D, "f32")
+        linear("latent_q", M, 32 * 96, 768, "bf16")
+        linear("latent_uk", M, 256, 64, "bf16", groups=32)
+        linear("latent_uv", M, 64, 256, "bf16", groups=32)
+        if M <= 256:
+            linear("head", M, 128256, D, "i64")
+        experts("experts_up", M, 2 * D, D, 8, 2, "bf16")
+        experts("experts_down", M, D, 2 * D, 8, 2, "f32")
+        gru(M)
+        if M <= 256:
+            attention("attention_decode", M, 1040, 1, 1024)
+            attention("attention_decode_8k", M, 8192, 1, 0)
+        else:
+            attention("attention_prompt", 2, M // 2, M // 2, 1024)
+            attention("attention_prompt_full", 2, M // 2, M // 2, 0)
+        norm_sets = lambda: (F(M, D), X(M, D), F(D), F(D))
+
+        def norm_call(a):
+            return lambda: ops.norm(a[0], a[2], a[3], 1e-6, a[1])
+        report("norm", M, lambda: norm_call(norm_sets()), 0, 6.0 * M * D, 6 * M * D)
+
+        def combine():
+            x, h, w, b = norm_sets()
+            y, wt = F(2 * M, D), torch.rand(M, 2, device=dev)
+            place = torch.randperm(2 * M, device=dev).int().view(M, 2)
+            return lambda: ops.norm(x, w, b, 1e-6, h, experts=(y, place, wt))
+        report("norm_combine", M, combine, 0, 18.0 * M * D, 18 * M * D)
+
+        def route_call():
+            lg, counts = F(M, 8), torch.zeros(8, dtype=torch.int32, device=dev)
+            return lambda: ops.route(lg, 8, 2, counts)
+        report("route", M, route_call, 0, M * (8 * 4 + 2 * 12.0), 1 << 24)
+
+        def gather_call():
+            h = X(M, D)
+            counts = torch.zeros(8, dtype=torch.int32, device=dev)
+            chosen, _, rank = ops.route(F(M, 8), 8, 2, counts)
+            return lambda: ops.gather(h, D, chosen, rank, counts)
+        report("gather", M, gather_call, 0, 6.0 * M * D, 6 * M * D)
+
+        def prepare_call():
+            sp = SimpleNamespace(q_rank=768, kv_rank=256, rot_dim=32, heads=32, eps=1e-6)
+            y, cache = F(M, 768 + 288 + 32), X(M // 16 + 2, 16, 288)
+            a, b, c = F(768), F(256), F(16)
+            pos = torch.arange(M, device=dev)
+            return lambda: ops.latent_prepare(y, sp, a, b, c, pos, pos, cache)
+        report("latent_prepare", M, prepare_call, 0, M * (4.0 * 1088 + 2 * 768 + 2 * 288 + 4 * 64), M * 8000)
+    if nv.float_device_status() != 0:
+        raise SystemExit("device-side wait timed out")
+
+
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("what", choices=["gemm", "gemmr", "gemm8", "attn", "stages", "prefill", "prompt", "bmm"])
+    ap.add_argument("what", choices=["gemm", "gemmr", "gemm8", "attn", "stages", "prefill", "prompt", "bmm", "hybrid"])
     ap.add_argument("--m", default="1,16,256,4096")
     ap.add_argument("--tile", type=int, default=0)
     ap.add_argument("--iters", type=int, default=10)
@@ -436,11 +596,12 @@ def main():
     ap.add_argument("--variant", type=int, default=0)
     ap.add_argument("--no-scratch", action="store_true", help="attn: no scratch buffer (long contexts: cluster kernels)")
     ap.add_argument("--fixed", action="store_true", help="attn: every request has exactly --ctx keys")
-    ap.add_argument("--proj", default="", help="gemmr / gemm8: only this projection (wqkv, wo, wgu, wd, lm)")
+    ap.add_argument("--proj", default="", help="gemmr / gemm8: only this projection (wqkv, wo, wgu, wd, lm); hybrid: only these kernels")
     ap.add_argument("--eager", action="store_true", help="gemmr / gemm8: one plain launch per weight set, no timing")
     ap.add_argument("--chunk", type=int, default=4096, help="prompt: token rows per forward call")
     args = ap.parse_args()
-    {"gemm": gemm, "gemmr": gemmr, "gemm8": gemm8, "attn": attn, "stages": stages, "prefill": prefill, "prompt": prompt, "bmm": bmm_bench}[args.what](args)
+    {"gemm": gemm, "gemmr": gemmr, "gemm8": gemm8, "attn": attn, "stages": stages, "prefill": prefill, "prompt": prompt, "bmm": bmm_bench,
+     "hybrid": hybrid}[args.what](args)
     if nv.device_status() != 0:
         raise SystemExit("device-side wait timed out")
 

@@ -86,13 +86,13 @@ def test_linear_sizes_and_tiles(M, N, K, tile, dtype):
     w, x = rounded(rng.randn(N, K), dtype), rounded(rng.randn(M, K), dtype)
     W, X = packed(w, dtype), packed(x, dtype)
     out = torch.full((M, N + 3), 7.0, device="cuda")
-    ops.linear(W, X, M, N, K, ops.store(out, N + 3, N, out_type=ops.OUT_F32), tile_rows=tile)
+    ops.linear(W, X, M, N, K, ops.store(out, N + 3, N, out_type=ops.OUT_F32), tile=tile)
     close(out[:, :N].cpu(), x @ w.T, "float32")
     assert (out[:, N:] == 7.0).all()                                  # nothing beside the output
     fix = torch.zeros(M, N, dtype=torch.long, device="cuda")
-    ops.linear(W, X, M, N, K, ops.store(fix, N, N, out_type=ops.OUT_I64), tile_rows=tile)
+    ops.linear(W, X, M, N, K, ops.store(fix, N, N, out_type=ops.OUT_I64), tile=tile)
     assert torch.equal(fix, torch.round(out[:, :N].double() * 2 ** 24).long())
-    ops.linear(W, X, M, N, K, ops.add(out), tile_rows=tile)
+    ops.linear(W, X, M, N, K, ops.add(out), tile=tile)
     close(out[:, :N].cpu(), 2 * (x @ w.T), "float32")
 
 
@@ -110,7 +110,7 @@ def test_ragged_groups(counts, dtype):
     ref = np.einsum("mk,mnk->mn", x, w[group])
     for tile in ((0,) if dtype == "float32" else (0, 16, 64, 128, 256)):
         out.fill_(7.0)
-        ops.linear(W, X, M, N, K, ops.store(out, N, N, out_type=ops.OUT_F32), groups=G, gsw=N * W.shape[2], counts=c, tile_rows=tile)
+        ops.linear(W, X, M, N, K, ops.store(out, N, N, out_type=ops.OUT_F32), groups=G, gsw=N * W.shape[2], counts=c, tile=tile)
         close(out.cpu(), ref, "float32")
 
 
@@ -543,7 +543,7 @@ def test_padding_rows_touch_nothing():
 # ---------------------------------------------------------------- commands
 
 def test_trace_run_and_generate_commands(tmp_path):
-    cfg = hm.CONFIGS["odd"]
+    cfg = hm.settled(hm.CONFIGS["odd"])
     t = hm.weights(cfg, 3)
     w64 = hm.as_numpy(t)
     folder = hm.save_folder(tmp_path / "m", cfg, t)
