@@ -70,11 +70,6 @@ __device__ __forceinline__ uint64_t umma_desc_mn(uint32_t addr) {
   return d | static_cast<uint64_t>((LT_KEYS * 128) >> 4) << 16;
 }
 
-__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
-  const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-  return *reinterpret_cast<const uint32_t*>(&v);
-}
-
 __global__ void __launch_bounds__(LT_THREADS, 1)
 fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mc,
                               const LatentAttn a, const LatentTc c) {
@@ -148,27 +143,38 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
 
   if (dead) {
   } else if (warp == 0) {
-    if (lane == 0 && nb > 0) {
-      // ---- TMA: the queries once, then the key blocks page by page ----
-      mbar_arrive_expect_tx(&sh->q_full, c.cols * q_box);
-      for (int j = 0; j < c.cols; ++j)
-        tma_load_3d(qs + j * q_box, &mq, &sh->q_full, j * 64, tok0 * a.H + row0, 0);
-      const int box = min(a.bs, LT_KEYS), pages = LT_KEYS / box;
-      int i = 0;
+    // ---- TMA: the queries once, then the key blocks in boxes that lie in one page. The warp reads the block table for 32
+    //      boxes at a time; one lane issues the copies ----
+    if (nb > 0) {
+      if (lane == 0) {
+        mbar_arrive_expect_tx(&sh->q_full, c.cols * q_box);
+        for (int j = 0; j < c.cols; ++j)
+          tma_load_3d(qs + j * q_box, &mq, &sh->q_full, j * 64, tok0 * a.H + row0, 0);
+      }
+      const int box = min(a.bs, LT_KEYS), boxes = LT_KEYS / box;
+      int i = 0, held = 0;
       bool ok = true;
       for (; i < nb; ++i) {
         const int s = i % c.stages, round = i / c.stages;
-        if (round > 0 && !(ok = mbar_wait(&sh->empty[s], (round - 1) & 1))) break;
+        if (round > 0) ok = mbar_wait(&sh->empty[s], (round - 1) & 1);
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
         uint8_t* st = ring + s * stage_bytes;
-        mbar_arrive_expect_tx(&sh->full[s], stage_bytes);
-        for (int p = 0; p < pages; ++p) {
-          const int key = (b0 + i) * LT_KEYS + p * box;
-          const int page = (int)(a.page_row(seq, min(key / a.bs, a.nblk - 1)) / a.bs);
-          for (int j = 0; j < c.cols; ++j)
-            tma_load_3d(st + j * LT_KEYS * 128 + p * box * 128, &mc, &sh->full[s], j * 64, key % a.bs, page);
+        if (lane == 0) mbar_arrive_expect_tx(&sh->full[s], stage_bytes);
+        for (int p = 0; p < boxes; ++p) {
+          const int nth = i * boxes + p;                             // box of this CTA
+          if ((nth & 31) == 0) {
+            const int page = (b0 * LT_KEYS + (nth + lane) * box) / a.bs;
+            held = (int)(a.page_row(seq, min(page, a.nblk - 1)) / a.bs);
+          }
+          const int page = __shfl_sync(0xffffffffu, held, nth & 31);
+          if (lane == 0)
+            for (int j = 0; j < c.cols; ++j)
+              tma_load_3d(st + j * LT_KEYS * 128 + p * box * 128, &mc, &sh->full[s], j * 64,
+                          (b0 * LT_KEYS + nth * box) % a.bs, page);
         }
       }
-      if (!ok) {
+      if (!ok && lane == 0) {
         fail();
         mbar_wait(&sh->q_full, 0);
         for (int k = i > c.stages ? i - c.stages : 0; k < i; ++k) mbar_wait(&sh->full[k % c.stages], (k / c.stages) & 1);
@@ -315,17 +321,8 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
         float v[16];
 #pragma unroll
         for (int k = 0; k < 16; ++k) v[k] = __uint_as_float(u[k]) * (c.splits == 1 ? inv : 1.0f);
-        if (n == 16) {
-          if (c.splits == 1) store_run<16>(out + q, v);
-          else store_run<16>(acc + q, v);
-        } else {
-#pragma unroll
-          for (int k = 0; k < 16; ++k)
-            if (k < n) {
-              if (c.splits == 1) st(out + q + k, v[k]);
-              else acc[q + k] = v[k];
-            }
-        }
+        if (c.splits == 1) store_run(out + q, v, n);
+        else store_run(acc + q, v, n);
       }
       if (c.splits > 1 && live && v0 == 0 && part == 0) {
         float* ml = c.part + (i64)c.splits * a.M * a.H * a.R + ((i64)blockIdx.y * a.M * a.H + at) * 2;

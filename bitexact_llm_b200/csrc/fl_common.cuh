@@ -30,15 +30,52 @@ __device__ __forceinline__ float ld<bf16>(const bf16* p) { return __bfloat162flo
 __device__ __forceinline__ void st(float* p, float v) { *p = v; }
 __device__ __forceinline__ void st(bf16* p, float v) { *p = __float2bfloat16(v); }
 
+__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
+  const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
+
+// Four consecutive values at an address that is aligned to all four.
+__device__ __forceinline__ void st4(float* p, float a, float b, float c, float d) {
+  *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d);
+}
+__device__ __forceinline__ void st4(bf16* p, float a, float b, float c, float d) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(a, b), pack_bf16(c, d));
+}
+
+// e^v and 1 / v: the library's full-precision forms for the 32-bit kernels, the hardware's approximations (a few units in the
+// last place of a float) for the bf16 ones.
+template <class T>
+__device__ __forceinline__ float exp_of(float v);
+template <>
+__device__ __forceinline__ float exp_of<float>(float v) { return expf(v); }
+template <>
+__device__ __forceinline__ float exp_of<bf16>(float v) { return __expf(v); }
+
+template <class T>
+__device__ __forceinline__ float recip(float v);
+template <>
+__device__ __forceinline__ float recip<float>(float v) { return 1.0f / v; }
+template <>
+__device__ __forceinline__ float recip<bf16>(float v) { return __fdividef(1.0f, v); }
+
 // sigmoid(v) and 1 - sigmoid(v), both without cancellation.
+template <class T>
 __device__ __forceinline__ void sigmoid_pair(float v, float& s, float& one_minus_s) {
-  const float e = expf(-fabsf(v)), r = 1.0f / (1.0f + e);
+  const float e = exp_of<T>(-fabsf(v)), r = recip<T>(1.0f + e);
   s = v >= 0.0f ? r : e * r;
   one_minus_s = v >= 0.0f ? e * r : r;
 }
 
-__device__ __forceinline__ float sigmoid(float v) { return 1.0f / (1.0f + expf(-v)); }
-__device__ __forceinline__ float silu(float v) { return v / (1.0f + expf(-v)); }
+// 1 / (1 + e^-v) = e^v / (1 + e^v): the exponent is kept below zero, so nothing overflows.
+template <class T>
+__device__ __forceinline__ float sigmoid(float v) {
+  const float e = exp_of<T>(-fabsf(v)), r = recip<T>(1.0f + e);
+  return v >= 0.0f ? r : e * r;
+}
+
+template <class T>
+__device__ __forceinline__ float silu(float v) { return v * sigmoid<T>(v); }
 
 __device__ __forceinline__ float activate(int act, float z, float p, float q) {
   if (act == BXF_ACT_RELU2) {

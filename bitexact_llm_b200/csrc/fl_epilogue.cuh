@@ -21,51 +21,82 @@ struct Tile {
   int row0, rows;                    // first token row, token rows that exist
 };
 
-// N consecutive values to memory: 16-byte stores when the address allows them.
-template <int N>
-__device__ __forceinline__ void store_run(bf16* p, const float (&v)[N]) {
-  if ((reinterpret_cast<uintptr_t>(p) & 15) == 0) {
+// Runs of 32 bytes: one store (load) of a whole sector per thread when the address allows it.
+__device__ __forceinline__ bool aligned32(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 31) == 0; }
+
+__device__ __forceinline__ void store32(void* p, const uint32_t (&w)[8]) {
+  asm volatile("st.global.v8.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(p), "r"(w[0]), "r"(w[1]), "r"(w[2]), "r"(w[3]),
+               "r"(w[4]), "r"(w[5]), "r"(w[6]), "r"(w[7])
+               : "memory");
+}
+
+__device__ __forceinline__ void load32(const void* p, uint32_t (&w)[8]) {
+  asm volatile("ld.global.v8.b32 {%0, %1, %2, %3, %4, %5, %6, %7}, [%8];"
+               : "=r"(w[0]), "=r"(w[1]), "=r"(w[2]), "=r"(w[3]), "=r"(w[4]), "=r"(w[5]), "=r"(w[6]), "=r"(w[7])
+               : "l"(p)
+               : "memory");
+}
+
+// The first n of 16 consecutive values.
+__device__ __forceinline__ void store_run(bf16* p, const float (&v)[16], int n) {
+  if (n == 16 && aligned32(p)) {
+    uint32_t w[8];
 #pragma unroll
-    for (int i = 0; i < N; i += 8) {
-      uint32_t w[4];
-#pragma unroll
-      for (int k = 0; k < 4; ++k) {
-        const __nv_bfloat162 b = __floats2bfloat162_rn(v[i + 2 * k], v[i + 2 * k + 1]);
-        w[k] = *reinterpret_cast<const uint32_t*>(&b);
-      }
-      *reinterpret_cast<uint4*>(p + i) = make_uint4(w[0], w[1], w[2], w[3]);
-    }
+    for (int k = 0; k < 8; ++k) w[k] = pack_bf16(v[2 * k], v[2 * k + 1]);
+    store32(p, w);
   } else {
 #pragma unroll
-    for (int i = 0; i < N; ++i) st(p + i, v[i]);
+    for (int i = 0; i < 16; ++i)
+      if (i < n) st(p + i, v[i]);
   }
 }
 
-template <int N>
-__device__ __forceinline__ void store_run(float* p, const float (&v)[N]) {
-  if ((reinterpret_cast<uintptr_t>(p) & 15) == 0) {
+__device__ __forceinline__ void store_run(float* p, const float (&v)[16], int n) {
+  if (n == 16 && aligned32(p)) {
 #pragma unroll
-    for (int i = 0; i < N; i += 4) *reinterpret_cast<float4*>(p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
-  } else {
+    for (int h = 0; h < 16; h += 8) {
+      uint32_t w[8];
 #pragma unroll
-    for (int i = 0; i < N; ++i) p[i] = v[i];
-  }
-}
-
-template <int N>
-__device__ __forceinline__ void load_run(const float* p, float (&v)[N]) {
-  if ((reinterpret_cast<uintptr_t>(p) & 15) == 0) {
-#pragma unroll
-    for (int i = 0; i < N; i += 4) {
-      const float4 f = *reinterpret_cast<const float4*>(p + i);
-      v[i] = f.x;
-      v[i + 1] = f.y;
-      v[i + 2] = f.z;
-      v[i + 3] = f.w;
+      for (int k = 0; k < 8; ++k) w[k] = __float_as_uint(v[h + k]);
+      store32(p + h, w);
     }
   } else {
 #pragma unroll
-    for (int i = 0; i < N; ++i) v[i] = p[i];
+    for (int i = 0; i < 16; ++i)
+      if (i < n) p[i] = v[i];
+  }
+}
+
+// Fixed point at 24 bits.
+__device__ __forceinline__ void store_run(i64* p, const float (&v)[16], int n) {
+  i64 q[16];
+#pragma unroll
+  for (int i = 0; i < 16; ++i) q[i] = __double2ll_rn((double)v[i] * 16777216.0);
+  if (n == 16 && aligned32(p)) {
+#pragma unroll
+    for (int h = 0; h < 16; h += 4) bx::st_global_v4(p + h, q[h], q[h + 1], q[h + 2], q[h + 3]);
+  } else {
+#pragma unroll
+    for (int i = 0; i < 16; ++i)
+      if (i < n) p[i] = q[i];
+  }
+}
+
+__device__ __forceinline__ void add_run(float* p, const float (&v)[16], int n) {
+  if (n == 16 && aligned32(p)) {
+    uint32_t w[2][8];
+    load32(p, w[0]);
+    load32(p + 8, w[1]);
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+#pragma unroll
+      for (int k = 0; k < 8; ++k) w[h][k] = __float_as_uint(__uint_as_float(w[h][k]) + v[8 * h + k]);
+      store32(p + 8 * h, w[h]);
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < 16; ++i)
+      if (i < n) p[i] += v[i];
   }
 }
 
@@ -129,82 +160,51 @@ struct StageEpi {
     }
   }
 
-  static constexpr int RW = 8;                   // channels a thread takes at a time in `run_rows`
-
-  // Channels n .. n + cnt - 1 of token row m; v holds their accumulators.
+  // Channels n .. n + cnt - 1 (n a multiple of 16) of token row m; v holds their accumulators.
   template <class T>
-  static __device__ __forceinline__ void chunk_rows(const Params& p, int group, i64 m, int n, int cnt, float (&v)[RW]) {
-    const bool full = cnt == RW;
+  static __device__ __forceinline__ void chunk_rows(const Params& p, int group, i64 m, int n, int cnt, float (&v)[16]) {
     if (p.kind == BXF_EPI_ADD) {
-      float* o = static_cast<float*>(p.out) + m * p.ldo + n;
-      if (full) {
-        float old[RW];
-        load_run<RW>(o, old);
-#pragma unroll
-        for (int i = 0; i < RW; ++i) old[i] += v[i];
-        store_run<RW>(o, old);
-      } else {
-        for (int i = 0; i < RW; ++i)
-          if (i < cnt) o[i] += v[i];
-      }
+      add_run(static_cast<float*>(p.out) + m * p.ldo + n, v, cnt);
       return;
     }
-    if (p.kind == BXF_EPI_ROPE && n >= p.n_main) {                      // n and n_main are even: whole pairs
-#pragma unroll
-      for (int i = 0; i < RW; i += 2) {
-        if (i >= cnt) break;
-        const int r = n + i - p.n_main, j = r % p.rot_dim;
-        const float2 cs = *reinterpret_cast<const float2*>(p.cs + (m * (p.rot_dim / 2) + (j >> 1)) * 2);
-        T* o = static_cast<T*>(p.rot_out) + m * p.ldr + r / p.rot_dim * p.hsr + j;
-        st(o, v[i] * cs.x - v[i + 1] * cs.y);
-        st(o + 1, v[i + 1] * cs.x + v[i] * cs.y);
-      }
-      return;
-    }
+    int main_cnt = cnt;                                                 // of them, below n_main
     if (p.kind == BXF_EPI_GATE) {
       const float g = p.gate[m * p.ldg + group];
 #pragma unroll
-      for (int i = 0; i < RW; ++i) v[i] *= g;
-    } else if (p.kind == BXF_EPI_STORE) {
+      for (int i = 0; i < 16; ++i) v[i] *= g;
+    } else {
+      main_cnt = min(cnt, p.n_main - n);
+      if (main_cnt < cnt) {
 #pragma unroll
-      for (int i = 0; i < RW; ++i) {
-        if (i < cnt && n + i >= p.n_main)
-          p.side[m * p.lds + (n + i - p.n_main)] = v[i] + (p.bias ? p.bias[n + i - p.n_main] : 0.0f);
+        for (int i = 0; i < 16; i += 2) {                               // n_main is even where channels are rotated
+          const int r = n + i - p.n_main;
+          if (p.kind == BXF_EPI_ROPE) {
+            if (i >= cnt || r < 0) continue;
+            const int j = r % p.rot_dim;
+            const float2 cs = *reinterpret_cast<const float2*>(p.cs + (m * (p.rot_dim / 2) + (j >> 1)) * 2);
+            T* o = static_cast<T*>(p.rot_out) + m * p.ldr + r / p.rot_dim * p.hsr + j;
+            st(o, v[i] * cs.x - v[i + 1] * cs.y);
+            st(o + 1, v[i + 1] * cs.x + v[i] * cs.y);
+          } else {
+#pragma unroll
+            for (int k = 0; k < 2; ++k)
+              if (i + k < cnt && r + k >= 0) p.side[m * p.lds + r + k] = v[i + k] + (p.bias ? p.bias[r + k] : 0.0f);
+          }
+        }
       }
-      if (n >= p.n_main) return;
+      if (main_cnt <= 0) return;
       if (p.act == BXF_ACT_RELU2) {
 #pragma unroll
-        for (int i = 0; i < RW; ++i) v[i] = activate(BXF_ACT_RELU2, v[i], 0.0f, 0.0f);
+        for (int i = 0; i < 16; ++i) v[i] = activate(BXF_ACT_RELU2, v[i], 0.0f, 0.0f);
       } else if (p.act == BXF_ACT_XIELU) {
 #pragma unroll
-        for (int i = 0; i < RW; ++i) v[i] = activate(BXF_ACT_XIELU, v[i], p.act_p, p.act_q);
+        for (int i = 0; i < 16; ++i) v[i] = activate(BXF_ACT_XIELU, v[i], p.act_p, p.act_q);
       }
-      cnt = min(cnt, p.n_main - n);
     }
     const i64 at = group * p.gso + m * p.ldo + n;
-    if (p.out_type == BXF_OUT_I64) {
-#pragma unroll
-      for (int i = 0; i < RW; ++i)
-        if (i < cnt) static_cast<i64*>(p.out)[at + i] = __double2ll_rn((double)v[i] * 16777216.0);
-    } else if (p.out_type == BXF_OUT_F32) {
-      float* o = static_cast<float*>(p.out) + at;
-      if (cnt == RW) {
-        store_run<RW>(o, v);
-      } else {
-#pragma unroll
-        for (int i = 0; i < RW; ++i)
-          if (i < cnt) o[i] = v[i];
-      }
-    } else {
-      T* o = static_cast<T*>(p.out) + at;
-      if (cnt == RW) {
-        store_run<RW>(o, v);
-      } else {
-#pragma unroll
-        for (int i = 0; i < RW; ++i)
-          if (i < cnt) st(o + i, v[i]);
-      }
-    }
+    if (p.out_type == BXF_OUT_I64) store_run(static_cast<i64*>(p.out) + at, v, main_cnt);
+    else if (p.out_type == BXF_OUT_F32) store_run(static_cast<float*>(p.out) + at, v, main_cnt);
+    else store_run(static_cast<T*>(p.out) + at, v, main_cnt);
   }
 
   // row: the thread's token row of the tile; the four warps of a lane quarter take 16 columns in turn.
@@ -213,15 +213,7 @@ struct StageEpi {
     for (int c = group_index * 16; c < TN && t.n0 + c < N; c += 64) {
       float v[16];
       get.template load<16>(0, c, v);
-      if (row >= t.rows) continue;
-#pragma unroll
-      for (int h = 0; h < 16; h += RW) {
-        const int n = t.n0 + c + h, cnt = min(RW, N - n);
-        float w[RW];
-#pragma unroll
-        for (int i = 0; i < RW; ++i) w[i] = v[h + i];
-        if (cnt > 0) chunk_rows<T>(p, t.group, (i64)t.row0 + row, n, cnt, w);
-      }
+      if (row < t.rows) chunk_rows<T>(p, t.group, (i64)t.row0 + row, t.n0 + c, min(16, N - t.n0 - c), v);
     }
   }
 
@@ -266,9 +258,9 @@ struct GruEpi {
       for (int i = 0; i < W; ++i) {
         if (c + i >= c_end) break;
         float s, a;
-        sigmoid_pair(z[i] + bz, s, a);
+        sigmoid_pair<T>(z[i] + bz, s, a);
         const float x = u[i] + bx;
-        float b = s * (x >= 0.0f ? x + 0.5f : sigmoid(x));
+        float b = s * (x >= 0.0f ? x + 0.5f : sigmoid<T>(x));
         const int f = p.flags[t.row0 + c + i];
         if (f & BXF_ROW_FIRST) {
           if (live && !(f & (BXF_ROW_START | BXF_ROW_PAD))) b += a * p.state[p.seq[t.row0 + c + i] * N + n];
@@ -301,10 +293,10 @@ struct GruEpi {
         const i64 m = t.row0 + c + i;
         T* o = static_cast<T*>(p.out) + m * p.ldo + n;
         if (p.mode == 0) {
-          st(o, S * silu(g[i]));
+          st(o, S * silu<T>(g[i]));
           if (p.flags[m] & BXF_ROW_LAST) p.state[p.seq[m] * N + n] = S;
         } else {
-          st(o, silu(g[i]));
+          st(o, silu<T>(g[i]));
           p.decay[m * N + n] = P;
           p.local[m * N + n] = S;
         }

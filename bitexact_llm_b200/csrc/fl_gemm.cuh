@@ -81,20 +81,25 @@ struct TmemGet {
   }
 };
 
-constexpr int FL_SPLIT_MAX = 4;
+constexpr int FL_SPLIT_MAX = 4;         // clusters of 2 or 4 CTAs
 
-struct ClusterGet {
-  const float* part[FL_SPLIT_MAX];      // [plane][column][128] of every CTA of the cluster
-  int splits, ta, row;
+// The partial sums of the S CTAs of a cluster for the rows this one finishes: [S][column][128 / S] in its own shared memory.
+template <int S, int COLS>
+struct PartialGet {
+  const float* part;
+  int ta, row;                          // row among the 128 / S
   template <int W>
   __device__ __forceinline__ void load(int plane, int c, float (&v)[W]) const {
+    float t[S][W];
+#pragma unroll
+    for (int r = 0; r < S; ++r)
+#pragma unroll
+      for (int i = 0; i < W; ++i) t[r][i] = part[(r * COLS + plane * ta + c + i) * (NROWS / S) + row];
 #pragma unroll
     for (int i = 0; i < W; ++i) {
-      float t = 0.0f;
+      v[i] = t[0][i];
 #pragma unroll
-      for (int r = 0; r < FL_SPLIT_MAX; ++r)
-        if (r < splits) t += part[r][(plane * ta + c + i) * NROWS + row];
-      v[i] = t;
+      for (int r = 1; r < S; ++r) v[i] += t[r][i];
     }
   }
 };
@@ -273,32 +278,38 @@ fl_gemm_kernel(const __grid_constant__ CUtensorMap mw, const __grid_constant__ C
       Epi::template run<bf16, TA, (TA / 4 >= 8 ? 8 : 4)>(get, ep, t, s.N, quarter * 32 + lane, we >> 2, 4, ring);
     }
   } else if constexpr (Cfg::PARTIAL_BYTES + Epi::stash_bytes(TA) <= Cfg::RING_BYTES) {
-    float* part = reinterpret_cast<float*>(ring);                       // the ring is idle: every MMA has completed
+    float* part = reinterpret_cast<float*>(ring);
+    __syncthreads();
+    cluster.sync();                                                     // every ring of the cluster is idle
     if (warp >= 2) {
+      // lane quarter q goes to CTA q mod S, slot of this rank
       const int quarter = warp & 3;
+      float* to = cluster.map_shared_rank(part, quarter % S) +
+                  (size_t)rank * Cfg::COLS * (NROWS / S) + quarter / S * 32 + lane;
       const TmemGet get{tmem + ((uint32_t)(quarter * 32) << 16), TA};
       for (int c = (we >> 2) * 8; c < Cfg::COLS; c += 32) {
+        if (c % TA >= t.rows) continue;                                 // columns of no token
         float v[8];
 #pragma unroll
         for (int i = 0; i < 8; ++i) v[i] = 0.0f;
         if (ok && nkb > 0) get.load<8>(0, c, v);
 #pragma unroll
-        for (int i = 0; i < 8; ++i) part[(c + i) * NROWS + quarter * 32 + lane] = v[i];
+        for (int i = 0; i < 8; ++i) to[(c + i) * (NROWS / S)] = v[i];
       }
     }
-    cluster.sync();
+    cluster.sync();                                                     // every partial is in its owner's ring
     if (warp >= 2) {
       // this CTA finishes quarters rank, rank + S, ..: 4 / S of them, 4 S warps each
-      const int quarters = 4 / S, row = (rank + S * (we % quarters)) * 32 + lane;
-      ClusterGet get;
-      get.splits = S;
-      get.ta = TA;
-      get.row = row;
-#pragma unroll
-      for (int r = 0; r < FL_SPLIT_MAX; ++r) get.part[r] = r < S ? cluster.map_shared_rank(part, r) : part;
-      Epi::template run<bf16, TA, 1>(get, ep, t, s.N, row, we / quarters, 4 * S, ring + Cfg::PARTIAL_BYTES);
+      const int quarters = 4 / S, qi = we % quarters, row = (rank + S * qi) * 32 + lane;
+      uint8_t* stash = ring + Cfg::PARTIAL_BYTES;
+      if (S == 2) {
+        PartialGet<2, Cfg::COLS> get{part, TA, qi * 32 + lane};
+        Epi::template run<bf16, TA, (TA / 8 >= 8 ? 8 : TA / 8)>(get, ep, t, s.N, row, we / quarters, 8, stash);
+      } else {
+        PartialGet<4, Cfg::COLS> get{part, TA, qi * 32 + lane};
+        Epi::template run<bf16, TA, (TA / 16 >= 8 ? 8 : TA / 16)>(get, ep, t, s.N, row, we / quarters, 16, stash);
+      }
     }
-    cluster.sync();                                                     // nobody leaves while its partials are read
   }
   close_cta<TCOLS>(tmem);
 }

@@ -75,12 +75,29 @@ fl_norm_kernel(float* __restrict__ x, const i64* ids, const T* __restrict__ embe
   if (!h) return;
   const float mean = block_sum(s, red) / D;
   float q = 0.0f;
-  for (int d = threadIdx.x; d < D; d += NORM_THREADS) {
-    const float c = row[d] - mean;
-    q += c * c;
+  if (D % 4 == 0) {                                      // every thread meets its own entries again: no barrier needed
+    for (int d = threadIdx.x * 4; d < D; d += NORM_THREADS * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(row + d);
+      const float c0 = v.x - mean, c1 = v.y - mean, c2 = v.z - mean, c3 = v.w - mean;
+      q += (c0 * c0 + c1 * c1) + (c2 * c2 + c3 * c3);
+    }
+  } else {
+    for (int d = threadIdx.x; d < D; d += NORM_THREADS) {
+      const float c = row[d] - mean;
+      q += c * c;
+    }
   }
   const float r = 1.0f / sqrtf(block_sum(q, red) / D + eps);
-  for (int d = threadIdx.x; d < D; d += NORM_THREADS) st(h + m * ldh + d, (row[d] - mean) * r * w[d] + b[d]);
+  if (D % 4 == 0) {
+    for (int d = threadIdx.x * 4; d < D; d += NORM_THREADS * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(row + d), g = *reinterpret_cast<const float4*>(w + d),
+                   c = *reinterpret_cast<const float4*>(b + d);
+      st4(h + m * ldh + d, (v.x - mean) * r * g.x + c.x, (v.y - mean) * r * g.y + c.y, (v.z - mean) * r * g.z + c.z,
+          (v.w - mean) * r * g.w + c.w);
+    }
+  } else {
+    for (int d = threadIdx.x; d < D; d += NORM_THREADS) st(h + m * ldh + d, (row[d] - mean) * r * w[d] + b[d]);
+  }
 }
 
 // One warp per row: `top` rounds of (largest, lowest index first).
@@ -163,6 +180,15 @@ fl_gather_kernel(const T* __restrict__ h, i64 ldh, int D, const int* chosen, con
 
 constexpr int PREP_THREADS = 128;
 
+// Two sums over the block of PREP_THREADS threads in one exchange.
+__device__ __forceinline__ float2 block_sum2(float a, float b, float2* red) {
+  a = warp_sum(a);
+  b = warp_sum(b);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = make_float2(a, b);
+  __syncthreads();
+  return make_float2((red[0].x + red[1].x) + (red[2].x + red[3].x), (red[0].y + red[1].y) + (red[2].y + red[3].y));
+}
+
 template <class T>
 __global__ void __launch_bounds__(PREP_THREADS)
 fl_latent_prepare_kernel(const float* __restrict__ y, i64 ldy, int q_rank, int R, int rot, int H,
@@ -171,7 +197,7 @@ fl_latent_prepare_kernel(const float* __restrict__ y, i64 ldy, int q_rank, int R
                          T* __restrict__ cache, i64 ldc, float* __restrict__ cs, float* __restrict__ gate) {
   launch_next();
   wait_previous();
-  __shared__ float red[33];
+  __shared__ float2 red[4];
   const i64 m = blockIdx.x;
   const float* ym = y + m * ldy;
   const float* yc = ym + q_rank;
@@ -180,8 +206,8 @@ fl_latent_prepare_kernel(const float* __restrict__ y, i64 ldy, int q_rank, int R
   float sq = 0.0f, sk = 0.0f;
   for (int d = threadIdx.x; d < q_rank; d += PREP_THREADS) sq += ym[d] * ym[d];
   for (int d = threadIdx.x; d < R; d += PREP_THREADS) sk += yc[d] * yc[d];
-  const float rq = 1.0f / sqrtf(block_sum(sq, red) / q_rank + eps);
-  const float rk = 1.0f / sqrtf(block_sum(sk, red) / R + eps);
+  const float2 sums = block_sum2(sq, sk, red);
+  const float rq = 1.0f / sqrtf(sums.x / q_rank + eps), rk = 1.0f / sqrtf(sums.y / R + eps);
   for (int d = threadIdx.x; d < q_rank; d += PREP_THREADS) st(cq + m * ldcq + d, ym[d] * rq * wq[d]);
   for (int d = threadIdx.x; d < R; d += PREP_THREADS) st(row + d, yc[d] * rk * wkv[d]);
   const float p = (float)pos[m];
@@ -194,7 +220,7 @@ fl_latent_prepare_kernel(const float* __restrict__ y, i64 ldy, int q_rank, int R
     st(row + R + 2 * i, u * c - v * s);
     st(row + R + 2 * i + 1, v * c + u * s);
   }
-  for (int i = threadIdx.x; i < H; i += PREP_THREADS) gate[m * H + i] = sigmoid(yr[rot + i]);
+  for (int i = threadIdx.x; i < H; i += PREP_THREADS) gate[m * H + i] = sigmoid<float>(yr[rot + i]);
 }
 
 // Second pass of a minGRU scan longer than a tile: the state carried into a tile is folded from the last rows of the

@@ -19,7 +19,8 @@ class Session:
     b of its cache). By default every sequence owns a run of pages for max_len tokens. With `pages`, the cache has that
     many pages for all sequences together: `feed` takes them as a sequence grows and `release` gives them back."""
 
-    def __init__(self, eng, B, max_len, bs=16, perm_seed=None, pages=None):
+    def __init__(self, eng, B, max_len, bs=None, perm_seed=None, pages=None):
+        bs = eng.page if bs is None else bs
         self.eng, self.B, self.bs = eng, B, bs
         self.nblk = (max_len + bs - 1) // bs
         nb = 1 + (B * self.nblk if pages is None else pages)

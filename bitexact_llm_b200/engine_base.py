@@ -8,6 +8,7 @@ import torch
 class TokenRowEngine:
     """Engines with D, V, L, FR, ln, dev and forward(caches, ids, pos, slot, bt, rmap, tiles=None)."""
 
+    page = 16               # tokens per cache page of a session
     tiles_from = 384        # prompt portions that end before this position attend row by row
     # (the integer tile kernel pays for itself once a tile walks a few key blocks: 0.83 x the row kernel on 128-token
     # prompts, 1.7 x on 2048-token ones)

@@ -19,6 +19,7 @@ FEED_FORWARDS = {DenseSpec: DenseFF, ExpertsSpec: ExpertsFF}
 
 class HybridEngine(TokenRowEngine):
     FR = 24
+    page = 64               # the attention kernel's key block: one copy per page and column block
     tiles_from = 0
 
     def __init__(self, spec, weights, dev="cuda", dtype="bfloat16", n_layers=None):

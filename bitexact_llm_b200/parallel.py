@@ -18,6 +18,8 @@ import contextlib
 import torch
 import torch.distributed as dist
 
+from .engine_base import TokenRowEngine
+
 # Optional timing of the collectives: set TIMER to an object with a context-manager method
 # `span(name, payload_bytes)` (bench.py does, to report the per-step time of each exchange); None = no timing.
 TIMER = None
@@ -333,7 +335,7 @@ class ShardedMLPInt8:
         return gather_columns(linear_post(af, self.wd, self.md, self.fm_d, mant2, e2, flag, True), self.group)
 
 
-class ColumnShardedIntEngine:
+class ColumnShardedIntEngine(TokenRowEngine):
     """int8 mode over `world` GPUs with BOTH shardings of the 8-GPU configuration: every rank owns a block of the
     sequences (its KV cache, attention, the attention-side linears and every row-local stage), while the MLP and the
     LM head + sampler run on ALL ranks' rows with the weights split by output column. Per layer: one all-gather of the

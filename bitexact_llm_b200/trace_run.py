@@ -65,8 +65,7 @@ def main(argv=None):
     from .decode import Session
     n = max(1, args.max_tokens)
     eng = registry.load(args.model, dtype=dtype, max_len=n)
-    bs = 16
-    replay = Replay(Session(eng, SLOTS, n, bs, pages=(n + bs - 1) // bs + SLOTS))
+    replay = Replay(Session(eng, SLOTS, n, pages=(n + eng.page - 1) // eng.page + SLOTS))
     for line in sys.stdin:
         if not line.strip():
             continue

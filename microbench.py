@@ -508,7 +508,7 @@ def hybrid(args):
 
     def attention(name, B, ctx, tokens, window, H=32, R=256, rot=32):
         sp = LatentAttentionSpec(H, 64, rot, 64, 768, R, 1e6, 0.1, window, 1e-6)
-        M, bs = B * tokens, 16
+        M, bs = B * tokens, 64
         nblk = (ctx + bs - 1) // bs
 
         def make():

@@ -425,7 +425,7 @@ def test_portions_and_decoding(name, cut, dtype):
     cfg, _, eng = model(name, dtype)
     toks = hm.tokens(cfg, 260, 1)
     want = want_logits(name, dtype, toks)
-    ses = session(eng, 3, 272, perm_seed=4)
+    ses = session(eng, 3, 272, bs=16 if cut == "pages" else None, perm_seed=4)
     at, rows = 0, []
     for n in PORTIONS[cut]:
         rows += ses.feed([(1, toks[at:at + n])])
@@ -442,7 +442,7 @@ def test_mixed_batches_match_each_request_alone(name, dtype):
     toks = {k: hm.tokens(cfg, n, i + 10) for i, (k, n) in enumerate(lens.items())}
     plan = [[("a", 40), ("b", 1), ("c", 2)], [("a", 2), ("c", 33)], [("a", 1), ("c", 1), ("d", 3)], [("c", 31), ("a", 57)],
             [("e", 100), ("a", 1)], [("a", 49), ("e", 1)]] + [[("e", 1)]] * 3 + [[("e", 96)]]
-    ses = session(eng, 3, 208, pages=26)
+    ses = session(eng, 3, 208, bs=16, pages=26)
     slot, at, got, idle = {}, {k: 0 for k in lens}, {k: [] for k in lens}, [2, 0, 1]
     for entries in plan:
         for k, _ in entries:
