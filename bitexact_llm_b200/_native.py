@@ -95,8 +95,7 @@ class Epilogue(ctypes.Structure):
 
 class Gru(ctypes.Structure):
     """bxf_gru."""
-    _fields_ = [("bias_z", P), ("bias_x", P), ("state", P), ("flags", P), ("seq", P), ("out", P), ("ldo", L), ("decay", P),
-                ("local", P), ("mode", I), ("tile", I)]
+    _fields_ = [("bias_z", P), ("bias_x", P), ("state", P), ("flags", P), ("seq", P), ("out", P), ("ldo", L)]
 
 
 _FLOAT_SIGNATURES = {
@@ -106,9 +105,10 @@ _FLOAT_SIGNATURES = {
     "bxf_clear_device_status": (I, []),
     "bxf_set_device_status": (I, [I]),
     "bxf_linear": (I, [I, P, L, L, P, L, L, I, I, I, I, P, ctypes.POINTER(Epilogue), I, P]),
-    "bxf_gru_tile": (I, [I, I, I]),
+    "bxf_gru_rows": (I, [I]),
+    "bxf_gru_chunks": (I, [I]),
     "bxf_gru_linear": (I, [I, P, L, P, L, I, I, I, ctypes.POINTER(Gru), P]),
-    "bxf_gru_finish": (I, [I, I, I, ctypes.POINTER(Gru), P]),
+    "bxf_gru_scan": (I, [I, P, P, I, I, ctypes.POINTER(Gru), P]),
     "bxf_row_flags": (I, [P, P, P, P, I, P]),
     "bxf_norm": (I, [I, P, P, P, L, P, P, P, I, P, P, R, P, L, P, I, I, I, P]),
     "bxf_route": (I, [P, L, I, I, P, P, P, P, I, P]),

@@ -14,7 +14,7 @@
 namespace bxf {
 
 constexpr int NROWS = 128;           // rows of the 128-row operand of a tile
-constexpr int EPI_THREADS = 512;     // epilogue threads: 16 warps, four per quarter of the 128 rows when K is not split
+constexpr int EPI_THREADS = 512;     // epilogue threads of the kernels with one CTA per SM (16 warps)
 
 struct Tile {
   int group, n0;                     // weight plane, first weight row
@@ -106,6 +106,10 @@ __device__ __forceinline__ void epi_barrier() { asm volatile("bar.sync 1, 512;" 
 struct StageEpi {
   using Params = bxf_epilogue;
   static constexpr int PLANES = 1;
+  // Small token tiles: 8 epilogue warps and half of an SM's shared memory, so that a CTA of the next tile or of the next
+  // kernel of the step fetches its first weights while this one finishes.
+  static __host__ __device__ constexpr int warps(int ta) { return ta <= 32 ? 8 : 16; }
+  static __host__ __device__ constexpr int ctas(int ta) { return ta <= 32 ? 2 : 1; }
   static __host__ __device__ constexpr int stash_bytes(int) { return 0; }
 
   template <class T>
@@ -217,6 +221,15 @@ struct StageEpi {
     }
   }
 
+  // Into L1 while the products run: the residual lines this thread's warp will add to.
+  template <int TA>
+  static __device__ __forceinline__ void prefetch(const Params& p, const Tile& t, int N, int row, int group_index, int groups) {
+    if (p.kind != BXF_EPI_ADD || t.n0 + row >= N) return;
+    for (int c = group_index * 8; c < TA && c < t.rows; c += groups * 8)
+      for (int i = 0; i < min(8, t.rows - c); ++i)
+        bx::prefetch_l1(static_cast<const float*>(p.out) + ((i64)t.row0 + c + i) * p.ldo + t.n0 + row);
+  }
+
   // groups: how many warps share a row (they take chunks of 8 columns in turn).
   template <class T, int TA, int W, class Get>
   static __device__ __forceinline__ void run(Get& get, const Params& p, const Tile& t, int N, int row, int group_index,
@@ -229,7 +242,20 @@ struct StageEpi {
   }
 };
 
-// ---- minGRU: gates and recurrence along the token columns ----
+// One minGRU gate pair: S_t = a S_(t-1) + b from the update and candidate pre-activations.
+template <class T>
+__device__ __forceinline__ void gru_gate(float z, float u, float& a, float& b) {
+  float s;
+  sigmoid_pair<T>(z, s, a);
+  b = s * (u >= 0.0f ? u + 0.5f : sigmoid<T>(u));
+}
+
+// The first row of a sequence that does not start here: its state slot is read.
+__device__ __forceinline__ bool gru_resumes(int flags) {
+  return (flags & (BXF_ROW_FIRST | BXF_ROW_START | BXF_ROW_PAD)) == BXF_ROW_FIRST;
+}
+
+// ---- minGRU: gates and recurrence along the token columns, for rows that fit one tile ----
 // The recurrence S_t = a_t S_(t-1) + b_t over a tile is a scan split over the warps of a row: every warp folds its
 // columns to one (a, b) pair, the pairs of the warps before it give its start, and a second walk produces the states.
 // At the first row of a sequence the state of its slot enters b and a becomes 0, so tiles need not know sequences.
@@ -237,7 +263,18 @@ struct StageEpi {
 struct GruEpi {
   using Params = bxf_gru;
   static constexpr int PLANES = 3;
+  static __host__ __device__ constexpr int warps(int) { return 16; }
+  static __host__ __device__ constexpr int ctas(int) { return 1; }
   static __host__ __device__ constexpr int stash_bytes(int ta) { return 2 * ta * NROWS * 4 + 16 * NROWS * 8; }
+
+  // Into L1 while the products run: the states that the first rows of sequences start from.
+  template <int TA>
+  static __device__ __forceinline__ void prefetch(const Params& p, const Tile& t, int N, int row, int group_index, int groups) {
+    const int per = TA / groups, c0 = group_index * per;
+    for (int c = c0; c < min(c0 + per, t.rows); ++c)
+      if (gru_resumes(p.flags[t.row0 + c]) && t.n0 + row < N)
+        bx::prefetch_l1(p.state + p.seq[t.row0 + c] * N + t.n0 + row);
+  }
 
   template <class T, int TA, int W, class Get>
   static __device__ __forceinline__ void run(Get& get, const Params& p, const Tile& t, int N, int row, int group_index,
@@ -251,19 +288,22 @@ struct GruEpi {
     const float bz = live ? p.bias_z[n] : 0.0f, bx = live ? p.bias_x[n] : 0.0f;
     float A = 1.0f, B = 0.0f;
     for (int c = c_begin; c < c_end; c += W) {
-      float z[W], u[W];
+      float z[W], u[W], start[W];
+      int f[W];
+#pragma unroll
+      for (int i = 0; i < W; ++i) f[i] = c + i < c_end ? p.flags[t.row0 + c + i] : BXF_ROW_PAD;
+#pragma unroll
+      for (int i = 0; i < W; ++i)
+        start[i] = live && gru_resumes(f[i]) ? p.state[p.seq[t.row0 + c + i] * N + n] : 0.0f;
       get.template load<W>(0, c, z);
       get.template load<W>(1, c, u);
 #pragma unroll
       for (int i = 0; i < W; ++i) {
         if (c + i >= c_end) break;
-        float s, a;
-        sigmoid_pair<T>(z[i] + bz, s, a);
-        const float x = u[i] + bx;
-        float b = s * (x >= 0.0f ? x + 0.5f : sigmoid<T>(x));
-        const int f = p.flags[t.row0 + c + i];
-        if (f & BXF_ROW_FIRST) {
-          if (live && !(f & (BXF_ROW_START | BXF_ROW_PAD))) b += a * p.state[p.seq[t.row0 + c + i] * N + n];
+        float a, b;
+        gru_gate<T>(z[i] + bz, u[i] + bx, a, b);
+        if (f[i] & BXF_ROW_FIRST) {
+          b += a * start[i];
           a = 0.0f;
         }
         sa[(c + i) * NROWS + row] = a;
@@ -274,11 +314,10 @@ struct GruEpi {
     }
     fold[group_index * NROWS + row] = make_float2(A, B);
     epi_barrier();
-    float P = 1.0f, S = 0.0f;
+    float S = 0.0f;
     for (int k = 0; k < group_index; ++k) {
       const float2 f = fold[k * NROWS + row];
       S = S * f.x + f.y;
-      P *= f.x;
     }
     for (int c = c_begin; c < c_end; c += W) {
       float g[W];
@@ -286,20 +325,11 @@ struct GruEpi {
 #pragma unroll
       for (int i = 0; i < W; ++i) {
         if (c + i >= c_end) break;
-        const float a = sa[(c + i) * NROWS + row];
-        S = S * a + sb[(c + i) * NROWS + row];
-        P *= a;
+        S = S * sa[(c + i) * NROWS + row] + sb[(c + i) * NROWS + row];
         if (!live) continue;
         const i64 m = t.row0 + c + i;
-        T* o = static_cast<T*>(p.out) + m * p.ldo + n;
-        if (p.mode == 0) {
-          st(o, S * silu<T>(g[i]));
-          if (p.flags[m] & BXF_ROW_LAST) p.state[p.seq[m] * N + n] = S;
-        } else {
-          st(o, silu<T>(g[i]));
-          p.decay[m * N + n] = P;
-          p.local[m * N + n] = S;
-        }
+        st(static_cast<T*>(p.out) + m * p.ldo + n, S * silu<T>(g[i]));
+        if (p.flags[m] & BXF_ROW_LAST) p.state[p.seq[m] * N + n] = S;
       }
     }
   }

@@ -22,7 +22,8 @@ using namespace bx;
 
 constexpr int KE = 64;                  // K elements per stage (128 bytes: one swizzle atom per row)
 
-template <int NP, int TA>
+// CTAS: CTAs that share an SM (shared memory is cut accordingly).
+template <int NP, int TA, int CTAS = 1>
 struct FlCfg {
   static_assert(TA % 16 == 0 && TA >= 16 && TA <= 256, "MMA N");
   static constexpr int COLS = NP * TA;
@@ -30,7 +31,7 @@ struct FlCfg {
   static constexpr int W_BYTES = NP * NROWS * BKB;
   static constexpr int X_BYTES = TA * BKB;
   static constexpr int STAGE_BYTES = W_BYTES + X_BYTES;
-  static constexpr int STAGES_MAX = (227 * 1024 - 2048) / STAGE_BYTES;
+  static constexpr int STAGES_MAX = (227 * 1024 / CTAS - 3072) / STAGE_BYTES;
   static constexpr int STAGES = STAGES_MAX > 8 ? 8 : STAGES_MAX;
   static_assert(STAGES >= 2, "at least two stages");
   static constexpr int RING_BYTES = STAGES * STAGE_BYTES;
@@ -107,10 +108,9 @@ struct PartialGet {
 // ---- the two asynchronous roles; `it` counts stages over the life of the CTA ----
 // TOKENS_M: the 128-row operand is the token tile (one plane), else the weight tile. Of the CTA's first tile, `ahead`
 // stages have their weights under way already (feed_weights).
-template <int NP, int TA, bool TOKENS_M = false>
+template <class Cfg, int NP, bool TOKENS_M = false>
 __device__ __forceinline__ bool feed_tile(FlShared* sh, uint8_t* ring, const CUtensorMap* mw, const CUtensorMap* mx,
                                           const Tile& t, bool ragged, int kb0, int nkb, int& it, int ahead = 0) {
-  using Cfg = FlCfg<NP, TA>;
   for (int i = 0; i < nkb; ++i, ++it) {
     const int s = it % Cfg::STAGES, round = it / Cfg::STAGES;
     if (round > 0 && !mbar_wait(&sh->empty[s], (round - 1) & 1)) return false;
@@ -127,22 +127,19 @@ __device__ __forceinline__ bool feed_tile(FlShared* sh, uint8_t* ring, const CUt
 }
 
 // The weight tiles of the first stages of the CTA's first tile, ahead of the previous kernel's end; returns how many.
-template <int NP, int TA, bool TOKENS_M = false>
+template <class Cfg, int NP>
 __device__ __forceinline__ int feed_weights(FlShared* sh, uint8_t* ring, const CUtensorMap* mw, const Tile& t, int kb0,
                                             int nkb) {
-  using Cfg = FlCfg<NP, TA>;
   const int n = min(nkb, Cfg::STAGES);
   for (int s = 0; s < n; ++s) {
     mbar_arrive_expect_tx(&sh->full[s], Cfg::STAGE_BYTES);
-    tma_load_3d(ring + s * Cfg::STAGE_BYTES + (TOKENS_M ? Cfg::W_BYTES : 0), mw, &sh->full[s], (kb0 + s) * KE, t.n0,
-                NP == 1 ? t.group : 0);
+    tma_load_3d(ring + s * Cfg::STAGE_BYTES, mw, &sh->full[s], (kb0 + s) * KE, t.n0, NP == 1 ? t.group : 0);
   }
   return n;
 }
 
-template <int NP, int TA>
+template <class Cfg, int NP, int TA>
 __device__ __forceinline__ bool multiply_tile(FlShared* sh, uint8_t* ring, uint32_t acc, int nkb, int& it) {
-  using Cfg = FlCfg<NP, TA>;
   constexpr uint32_t ID = umma_idesc_bf16(TA);
   for (int i = 0; i < nkb; ++i, ++it) {
     const int s = it % Cfg::STAGES;
@@ -217,12 +214,12 @@ __device__ __forceinline__ void close_cta(uint32_t tmem) {
 
 // ---- one tile per cluster, K split over the cluster's CTAs ----
 template <int TA, class Epi>
-__global__ void __launch_bounds__(GEMM_THREADS, 1)
+__global__ void __launch_bounds__(64 + 32 * Epi::warps(TA), Epi::ctas(TA))
 fl_gemm_kernel(const __grid_constant__ CUtensorMap mw, const __grid_constant__ CUtensorMap mx, const GemmShape s,
                const __grid_constant__ typename Epi::Params ep) {
   namespace cg = cooperative_groups;
-  constexpr int NP = Epi::PLANES;
-  using Cfg = FlCfg<NP, TA>;
+  constexpr int NP = Epi::PLANES, EW = Epi::warps(TA);
+  using Cfg = FlCfg<NP, TA, Epi::ctas(TA)>;
   constexpr int TCOLS = Cfg::tmem_cols(Cfg::COLS);
   static_assert(Epi::stash_bytes(TA) <= Cfg::RING_BYTES, "the epilogue's stash lies in the idle ring");
   extern __shared__ uint8_t smem_raw[];
@@ -242,12 +239,16 @@ fl_gemm_kernel(const __grid_constant__ CUtensorMap mw, const __grid_constant__ C
   const bool dead = sh->abort_flag != 0;                                // an earlier timeout: no work, all barriers
   __syncthreads();
   bool ok = !dead;
+  // What an epilogue thread finishes: straight from TMEM its lane quarter (S = 1), else quarters rank, rank + S, .. of
+  // the tile, 4 / S of them
+  const int we = warp - 2, quarters = 4 / S, qi = S == 1 ? warp & 3 : we % quarters, group = we / quarters;
+  const int row = (rank + S * qi) * 32 + lane, groups = EW / quarters;
   if (warp == 0) {
     if (lane == 0 && !dead) {
       int it = 0;
-      const int ahead = feed_weights<NP, TA>(sh, ring, &mw, t, kb0, nkb);
+      const int ahead = feed_weights<Cfg, NP>(sh, ring, &mw, t, kb0, nkb);
       wait_previous();
-      if (!feed_tile<NP, TA>(sh, ring, &mw, &mx, t, s.counts != nullptr, kb0, nkb, it, ahead)) {
+      if (!feed_tile<Cfg, NP>(sh, ring, &mw, &mx, t, s.counts != nullptr, kb0, nkb, it, ahead)) {
         give_up(sh);
         drain_ring<Cfg::STAGES>(sh, it);
       }
@@ -255,11 +256,12 @@ fl_gemm_kernel(const __grid_constant__ CUtensorMap mw, const __grid_constant__ C
   } else if (warp == 1) {
     if (lane == 0 && !dead) {
       int it = 0;
-      if (multiply_tile<NP, TA>(sh, ring, tmem, nkb, it)) umma_commit(&sh->acc_full[0]);
+      if (multiply_tile<Cfg, NP, TA>(sh, ring, tmem, nkb, it)) umma_commit(&sh->acc_full[0]);
       else give_up(sh);
     }
   } else if (!dead) {
     wait_previous();
+    Epi::template prefetch<TA>(ep, t, s.N, row, group, groups);
     if (nkb > 0) ok = mbar_wait(&sh->acc_full[0], 0);
     ok = ok && !aborted(sh);
     ok = __all_sync(0xffffffffu, ok);
@@ -267,15 +269,11 @@ fl_gemm_kernel(const __grid_constant__ CUtensorMap mw, const __grid_constant__ C
     else if (lane == 0) atomicAdd(&g_wait_timeouts, 1);
   }
 
-  const int we = warp - 2;                                              // epilogue warp 0 .. 15
   if (S == 1) {
-    // accumulators straight from TMEM: a warp reads the lane quarter of its warp id
     __syncthreads();
-    const bool go = !dead && !aborted(sh) && nkb > 0;
-    if (warp >= 2 && go) {
-      const int quarter = warp & 3;
-      TmemGet get{tmem + ((uint32_t)(quarter * 32) << 16), TA};
-      Epi::template run<bf16, TA, (TA / 4 >= 8 ? 8 : 4)>(get, ep, t, s.N, quarter * 32 + lane, we >> 2, 4, ring);
+    if (warp >= 2 && !dead && !aborted(sh) && nkb > 0) {
+      TmemGet get{tmem + ((uint32_t)(qi * 32) << 16), TA};
+      Epi::template run<bf16, TA, (TA * 4 / EW >= 8 ? 8 : 4)>(get, ep, t, s.N, row, group, groups, ring);
     }
   } else if constexpr (Cfg::PARTIAL_BYTES + Epi::stash_bytes(TA) <= Cfg::RING_BYTES) {
     float* part = reinterpret_cast<float*>(ring);
@@ -287,7 +285,7 @@ fl_gemm_kernel(const __grid_constant__ CUtensorMap mw, const __grid_constant__ C
       float* to = cluster.map_shared_rank(part, quarter % S) +
                   (size_t)rank * Cfg::COLS * (NROWS / S) + quarter / S * 32 + lane;
       const TmemGet get{tmem + ((uint32_t)(quarter * 32) << 16), TA};
-      for (int c = (we >> 2) * 8; c < Cfg::COLS; c += 32) {
+      for (int c = (we >> 2) * 8; c < Cfg::COLS; c += EW * 2) {
         if (c % TA >= t.rows) continue;                                 // columns of no token
         float v[8];
 #pragma unroll
@@ -299,15 +297,15 @@ fl_gemm_kernel(const __grid_constant__ CUtensorMap mw, const __grid_constant__ C
     }
     cluster.sync();                                                     // every partial is in its owner's ring
     if (warp >= 2) {
-      // this CTA finishes quarters rank, rank + S, ..: 4 / S of them, 4 S warps each
-      const int quarters = 4 / S, qi = we % quarters, row = (rank + S * qi) * 32 + lane;
       uint8_t* stash = ring + Cfg::PARTIAL_BYTES;
       if (S == 2) {
+        constexpr int PER = TA * 2 / EW;                                // columns of a thread
         PartialGet<2, Cfg::COLS> get{part, TA, qi * 32 + lane};
-        Epi::template run<bf16, TA, (TA / 8 >= 8 ? 8 : TA / 8)>(get, ep, t, s.N, row, we / quarters, 8, stash);
+        Epi::template run<bf16, TA, (PER >= 8 ? 8 : PER)>(get, ep, t, s.N, row, group, groups, stash);
       } else {
+        constexpr int PER = TA / EW;
         PartialGet<4, Cfg::COLS> get{part, TA, qi * 32 + lane};
-        Epi::template run<bf16, TA, (TA / 16 >= 8 ? 8 : TA / 16)>(get, ep, t, s.N, row, we / quarters, 16, stash);
+        Epi::template run<bf16, TA, (PER >= 8 ? 8 : PER)>(get, ep, t, s.N, row, group, groups, stash);
       }
     }
   }
@@ -340,7 +338,7 @@ fl_gemm_persistent_kernel(const __grid_constant__ CUtensorMap mw, const __grid_c
       bool ok = true;
       for (int tile = blockIdx.x; tile < total && ok; tile += gridDim.x) {
         if (!locate_tile(s, NROWS, tile, t, TN)) continue;
-        if (lane == 0) ok = feed_tile<1, TN, true>(sh, ring, &mw, &mx, t, ragged, 0, nkb, it);
+        if (lane == 0) ok = feed_tile<Cfg, 1, true>(sh, ring, &mw, &mx, t, ragged, 0, nkb, it);
         ok = __all_sync(0xffffffffu, ok);
       }
       if (!ok && lane == 0) {
@@ -356,7 +354,7 @@ fl_gemm_persistent_kernel(const __grid_constant__ CUtensorMap mw, const __grid_c
         if (lane == 0) {
           if (use > 0) ok = mbar_wait(&sh->acc_empty[buf], (use - 1) & 1);
           tc_fence_after();
-          ok = ok && multiply_tile<1, TN>(sh, ring, tmem + buf * Cfg::COLS, nkb, it);
+          ok = ok && multiply_tile<Cfg, 1, TN>(sh, ring, tmem + buf * Cfg::COLS, nkb, it);
           if (ok) umma_commit(&sh->acc_full[buf]);
         }
         ok = __all_sync(0xffffffffu, ok);

@@ -1,8 +1,8 @@
 // Memory-bound stages of the float models: row flags, embedding / expert combination + layer norm, expert routing and
-// gathering, the preparation of latent attention, the second pass of a long minGRU scan. All arithmetic is 32-bit.
+// gathering, the preparation of latent attention, long minGRU scans. All arithmetic is 32-bit.
 #pragma once
 
-#include "fl_common.cuh"
+#include "fl_epilogue.cuh"
 
 namespace bxf {
 
@@ -223,28 +223,85 @@ fl_latent_prepare_kernel(const float* __restrict__ y, i64 ldy, int q_rank, int R
   for (int i = threadIdx.x; i < H; i += PREP_THREADS) gate[m * H + i] = sigmoid<float>(yr[rot + i]);
 }
 
-// Second pass of a minGRU scan longer than a tile: the state carried into a tile is folded from the last rows of the
-// tiles before it, then S = local + decay * carried. One thread per channel and CTA row; blockIdx.y = tile.
+// ---- minGRU over more rows than a product tile takes: y float [M, 3 width] holds the three products, the rows are scanned
+// in chunks side by side. The first kernel folds every chunk to S -> A S + B; the second folds the chunks before its own to
+// the state it starts from and produces the outputs. Only the first kernel reads state slots: it leaves a first row's
+// finished b in place of the row's update pre-activation, since the second kernel's last rows rewrite the slots.
+// One thread per channel; rows are read ahead in batches. ----
+constexpr int GRU_BATCH = 8;
+
+template <class T, bool APPLY>
+__device__ __forceinline__ void gru_rows(const bxf_gru& g, float* __restrict__ y, int width, int n, int m0, int m1,
+                                         float& A, float& S) {
+  const float bz = g.bias_z[n], bx = g.bias_x[n];
+  const i64 ldy = 3 * (i64)width;
+  for (int m = m0; m < m1; m += GRU_BATCH) {
+    float z[GRU_BATCH], u[GRU_BATCH], x[GRU_BATCH];                     // x: output gate, or the state a first row resumes
+    int f[GRU_BATCH];
+#pragma unroll
+    for (int i = 0; i < GRU_BATCH; ++i) {
+      const bool in = m + i < m1;
+      const float* row = y + (m + i) * ldy + n;
+      f[i] = in ? g.flags[m + i] : 0;
+      z[i] = in ? row[0] : 0.0f;
+      u[i] = in ? row[width] : 0.0f;
+      if (APPLY) x[i] = in ? row[2 * width] : 0.0f;
+    }
+    if (!APPLY) {
+#pragma unroll
+      for (int i = 0; i < GRU_BATCH; ++i) x[i] = gru_resumes(f[i]) ? g.state[g.seq[m + i] * width + n] : 0.0f;
+    }
+#pragma unroll
+    for (int i = 0; i < GRU_BATCH; ++i) {
+      if (m + i >= m1) break;
+      float a, b;
+      if (APPLY && (f[i] & BXF_ROW_FIRST)) {
+        a = 0.0f;
+        b = z[i];
+      } else {
+        gru_gate<T>(z[i] + bz, u[i] + bx, a, b);
+        if (f[i] & BXF_ROW_FIRST) {
+          b += a * x[i];
+          a = 0.0f;
+          y[(m + i) * ldy + n] = b;
+        }
+      }
+      S = S * a + b;
+      A *= a;
+      if (APPLY) {
+        st(static_cast<T*>(g.out) + (i64)(m + i) * g.ldo + n, S * silu<T>(x[i]));
+        if (f[i] & BXF_ROW_LAST) g.state[g.seq[m + i] * width + n] = S;
+      }
+    }
+  }
+}
+
 template <class T>
 __global__ void __launch_bounds__(128)
-fl_gru_finish_kernel(const bxf_gru g, int M, int width, int tile) {
+fl_gru_fold_kernel(const bxf_gru g, float* y, float2* fold, int M, int width, int chunk) {
   launch_next();
   wait_previous();
   const int n = blockIdx.x * 128 + threadIdx.x, j = blockIdx.y;
   if (n >= width) return;
-  float carry = 0.0f;
-  for (int i = 0; i < j; ++i) {
-    const i64 at = (i64)(i * tile + tile - 1) * width + n;
-    carry = g.local[at] + g.decay[at] * carry;
-  }
-  const int m1 = min(M, (j + 1) * tile);
-  for (int m = j * tile + blockIdx.z; m < m1; m += gridDim.z) {
-    const i64 at = (i64)m * width + n;
-    const float s = g.local[at] + g.decay[at] * carry;
-    T* o = static_cast<T*>(g.out) + (i64)m * g.ldo + n;
-    st(o, s * ld(o));
-    if (g.flags[m] & BXF_ROW_LAST) g.state[g.seq[m] * width + n] = s;
-  }
+  float A = 1.0f, S = 0.0f;
+  gru_rows<T, false>(g, y, width, n, j * chunk, min(M, (j + 1) * chunk), A, S);
+  fold[(i64)j * width + n] = make_float2(A, S);
+}
+
+template <class T>
+__global__ void __launch_bounds__(128)
+fl_gru_apply_kernel(const bxf_gru g, float* y, const float2* fold, int M, int width, int chunk) {
+  launch_next();
+  wait_previous();
+  const int n = blockIdx.x * 128 + threadIdx.x, j = blockIdx.y;
+  if (n >= width) return;
+  float A = 1.0f, S = 0.0f;
+  if (!(g.flags[j * chunk] & BXF_ROW_FIRST))
+    for (int i = 0; i < j; ++i) {
+      const float2 f = fold[(i64)i * width + n];
+      S = S * f.x + f.y;
+    }
+  gru_rows<T, true>(g, y, width, n, j * chunk, min(M, (j + 1) * chunk), A, S);
 }
 
 }  // namespace bxf

@@ -16,7 +16,7 @@ namespace {
 
 using namespace bxf;
 
-static_assert(sizeof(bxf_epilogue) == 128 && sizeof(bxf_gru) == 80, "layouts of the callers' structs");
+static_assert(sizeof(bxf_epilogue) == 128 && sizeof(bxf_gru) == 56, "layouts of the callers' structs");
 
 inline cudaStream_t stream_of(void* s) { return static_cast<cudaStream_t>(s); }
 inline bool dtype_ok(int d) { return d == BXF_BF16 || d == BXF_F32; }
@@ -99,6 +99,10 @@ double expected_tiles(const GemmShape& s, int rows) {
   return (double)used * ceil_div((int)(1.3 * s.M / used + 0.5), rows);
 }
 
+// Clusters of `split` CTAs of the tile kernels that the device holds at a time (a cluster lies within one group of SMs, so
+// fewer than SMs / split), cached per device.
+int resident_clusters(int split, int sms);
+
 // A K block of a tile of R + C rows moves (R + C) x 128 bytes into shared memory and reads them once for the MMAs, at 128
 // bytes a cycle; the constants are the measured prologue, epilogue and cluster exchange.
 Plan tile_plan(const GemmShape& s, int planes, int ta, int max_split, int sms) {
@@ -106,7 +110,8 @@ Plan tile_plan(const GemmShape& s, int planes, int ta, int max_split, int sms) {
   const int nkb = ceil_div(s.K, KE);
   Plan best = {ta, 1, 1e300};
   for (int split = 1; split <= max_split && (split == 1 || nkb >= 2 * split); split *= 2) {
-    const double waves = (double)(i64)((tiles * split + sms - 1) / sms);
+    const int slots = split == 1 ? sms : resident_clusters(split, sms);
+    const double waves = (double)(i64)((tiles + slots - 1) / slots);
     const double per = ceil_div(nkb, split) * 2.3 * (planes * NROWS + ta) + 3000 + 20.0 * planes * ta + (split > 1 ? 1800 : 0);
     if (waves * per < best.cycles) best = {ta, split, waves * per};
   }
@@ -132,11 +137,40 @@ Plan plan_linear(const GemmShape& s, int sms) {
   return best;
 }
 
+int resident_clusters(int split, int sms) {
+  static PerDevice cache[2];
+  const int dev = current_device();
+  if (dev < 0) return sms / split;
+  std::atomic<int>& slot = cache[split == 2 ? 0 : 1].v[dev];
+  int n = slot.load(std::memory_order_acquire);
+  if (n > 0) return n;
+  using Cfg = FlCfg<3, 64>;                              // one CTA per SM
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(4 * 148, 1, 1);
+  cfg.blockDim = dim3(64 + 32 * GruEpi::warps(64), 1, 1);
+  cfg.dynamicSmemBytes = Cfg::SMEM_BYTES;
+  cudaLaunchAttribute attr[1];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = split;
+  attr[0].val.clusterDim.y = 1;
+  attr[0].val.clusterDim.z = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = 1;
+  if (cudaFuncSetAttribute(fl_gemm_kernel<64, GruEpi>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES) !=
+          cudaSuccess ||
+      cudaOccupancyMaxActiveClusters(&n, fl_gemm_kernel<64, GruEpi>, &cfg) != cudaSuccess || n <= 0) {
+    cudaGetLastError();
+    return sms / split;
+  }
+  slot.store(n, std::memory_order_release);
+  return n;
+}
+
 // One tile per cluster of `split` CTAs.
 template <int TA, class Epi>
 int launch_tiles(const Operands& o, GemmShape s, const typename Epi::Params& ep, int split, cudaStream_t st) {
   constexpr int NP = Epi::PLANES;
-  using Cfg = FlCfg<NP, TA>;
+  using Cfg = FlCfg<NP, TA, Epi::ctas(TA)>;
   static PerDevice configured;
   if (once_per_device(configured, [] {
         return cudaFuncSetAttribute(fl_gemm_kernel<TA, Epi>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -152,8 +186,8 @@ int launch_tiles(const Operands& o, GemmShape s, const typename Epi::Params& ep,
   const i64 tiles = (i64)s.n_tiles * s.m_tiles * (s.counts || NP > 1 ? 1 : s.groups);
   if (tiles > (1 << 24)) return BX_ELIMIT;
   if (Cfg::PARTIAL_BYTES + Epi::stash_bytes(TA) > Cfg::RING_BYTES) split = 1;
-  return launch_chained(fl_gemm_kernel<TA, Epi>, dim3((unsigned)(tiles * split)), GEMM_THREADS, Cfg::SMEM_BYTES, st, split,
-                        mw, mx, s, ep);
+  return launch_chained(fl_gemm_kernel<TA, Epi>, dim3((unsigned)(tiles * split)), 64 + 32 * Epi::warps(TA), Cfg::SMEM_BYTES,
+                        st, split, mw, mx, s, ep);
 }
 
 template <int TN, class Epi>
@@ -244,6 +278,13 @@ int launch_latent_tc(const LatentAttn& a, void* scratch, size_t scratch_bytes, c
   return launch_chained(fl_latent_join_kernel, dim3((unsigned)(a.M * a.H)), 128, 0, st, 0, a, c.part, c.splits);
 }
 
+bool gru_ok(const bxf_gru* g, int M, int width) {
+  return g && M >= 0 && width >= 1 && g->bias_z && g->bias_x && g->state && g->flags && g->seq && g->out && g->ldo >= width;
+}
+
+// Rows of a scan chunk: short ones while there are few rows to spread over the SMs.
+int gru_chunk(int M) { return M <= 512 ? 16 : 64; }
+
 }  // namespace
 
 extern "C" {
@@ -273,20 +314,13 @@ int bxf_linear(int dtype, const void* w, int64_t ldw, int64_t gsw, const void* x
   return run_bf16(o, s, *epi, tile, stream_of(stream));
 }
 
-// Small tiles while the list of large ones leaves SMs idle.
-int bxf_gru_tile(int dtype, int M, int width) {
-  if (dtype == BXF_F32) return SIMT_TA;
-  if (M <= 16) return 16;
-  return M <= 64 || (i64)ceil_div(M, 128) * ceil_div(width, NROWS) < 128 ? 64 : 128;
-}
+int bxf_gru_rows(int dtype) { return dtype == BXF_F32 ? SIMT_TA : 64; }
+int bxf_gru_chunks(int M) { return ceil_div(M, gru_chunk(M)); }
 
 int bxf_gru_linear(int dtype, const void* w, int64_t ldw, const void* x, int64_t ldx, int M, int width, int K,
                    const bxf_gru* gru, void* stream) {
-  if (!dtype_ok(dtype) || !gru || M < 0 || width < 1 || K < 1) return BX_EARG;
+  if (!dtype_ok(dtype) || !gru_ok(gru, M, width) || K < 1 || M > bxf_gru_rows(dtype)) return BX_EARG;
   if (!operand_ok(w, ldw, (i64)width * ldw, true, K, dtype) || !operand_ok(x, ldx, 0, false, K, dtype)) return BX_EARG;
-  if (!gru->bias_z || !gru->bias_x || !gru->state || !gru->flags || !gru->seq || !gru->out) return BX_EARG;
-  if (dtype == BXF_F32 ? gru->tile != SIMT_TA : gru->tile != 16 && gru->tile != 64 && gru->tile != 128) return BX_EARG;
-  if (gru->mode == 0 ? M > gru->tile || gru->tile == 128 : (gru->mode != 1 || !gru->decay || !gru->local)) return BX_EARG;
   if (g_status_seen.load() != 0) return BX_EDEVICE;
   if (M == 0) return BX_OK;
   const Operands o{w, x, ldw, (i64)width * ldw, ldx, 0};
@@ -295,21 +329,23 @@ int bxf_gru_linear(int dtype, const void* w, int64_t ldw, const void* x, int64_t
   if (dtype == BXF_F32) return launch_simt<GruEpi>(o, s, *gru, st);
   const int sms = device_sms();
   if (sms <= 0) return BX_ELAUNCH;
-  const int split = gru->tile == 128 ? 1 : tile_plan(s, 3, gru->tile, FL_SPLIT_MAX, sms).split;
-  if (gru->tile == 16) return launch_tiles<16, GruEpi>(o, s, *gru, split, st);
-  if (gru->tile == 64) return launch_tiles<64, GruEpi>(o, s, *gru, split, st);
-  return launch_tiles<128, GruEpi>(o, s, *gru, 1, st);
+  const int tile = M <= 16 ? 16 : 64;
+  const int split = tile_plan(s, 3, tile, FL_SPLIT_MAX, sms).split;
+  return tile == 16 ? launch_tiles<16, GruEpi>(o, s, *gru, split, st) : launch_tiles<64, GruEpi>(o, s, *gru, split, st);
 }
 
-int bxf_gru_finish(int dtype, int M, int width, const bxf_gru* gru, void* stream) {
-  if (!dtype_ok(dtype) || !gru || gru->mode != 1 || M < 0 || width < 1 || !gru->decay || !gru->local || !gru->out)
-    return BX_EARG;
+int bxf_gru_scan(int dtype, float* y, float* fold, int M, int width, const bxf_gru* gru, void* stream) {
+  if (!dtype_ok(dtype) || !gru_ok(gru, M, width) || !y || !fold) return BX_EARG;
   if (M == 0) return BX_OK;
-  const int tile = gru->tile;
-  if (tile < 16) return BX_EARG;
-  const dim3 grid(ceil_div(width, 128), ceil_div(M, tile), tile / 16);
-  return launch_chained(dtype == BXF_F32 ? fl_gru_finish_kernel<float> : fl_gru_finish_kernel<bf16>, grid, 128, 0,
-                        stream_of(stream), 0, *gru, M, width, tile);
+  const int chunk = gru_chunk(M);
+  if (ceil_div(M, chunk) > 65535) return BX_ELIMIT;
+  const dim3 grid(ceil_div(width, 128), ceil_div(M, chunk));
+  float2* f = reinterpret_cast<float2*>(fold);
+  const int rc = launch_chained(dtype == BXF_F32 ? fl_gru_fold_kernel<float> : fl_gru_fold_kernel<bf16>, grid, 128, 0,
+                                stream_of(stream), 0, *gru, y, f, M, width, chunk);
+  if (rc != BX_OK) return rc;
+  return launch_chained(dtype == BXF_F32 ? fl_gru_apply_kernel<float> : fl_gru_apply_kernel<bf16>, grid, 128, 0,
+                        stream_of(stream), 0, *gru, y, f, M, width, chunk);
 }
 
 int bxf_row_flags(const int64_t* seq, const int64_t* slot, const int64_t* pos, int* flags, int M, void* stream) {

@@ -72,20 +72,21 @@ def row_flags(seq, slot, pos):
 
 def min_gru(w, bias_z, bias_x, h, width, K, state, flags, seq):
     """-> state * silu(gate) [M, pad8(width)]; `state` float [slots, width] is advanced by the rows of every sequence.
-    One kernel when the rows fit a tile (decoding, short portions), two otherwise."""
+    w [3, width, pad8(K)]. One kernel when the rows fit a tile (decoding, short portions), else product and scan."""
     M, lib, dt = h.shape[0], nv.float_lib(), code(w)
     out = torch.empty(M, pad8(width), dtype=w.dtype, device=h.device)
     g = nv.Gru(bias_z=bias_z.data_ptr(), bias_x=bias_x.data_ptr(), state=state.data_ptr(), flags=flags.data_ptr(),
-               seq=seq.data_ptr(), out=out.data_ptr(), ldo=out.stride(0), tile=lib.bxf_gru_tile(dt, M, width))
-    g.mode = int(M > g.tile)
-    if g.mode:
-        scan = torch.empty(2, M, width, dtype=torch.float32, device=h.device)
-        g.decay, g.local = scan[0].data_ptr(), scan[1].data_ptr()
-    rc = lib.bxf_gru_linear(dt, w.data_ptr(), w.shape[-1], h.data_ptr(), h.stride(0), M, width, K, ctypes.byref(g),
-                            nv.stream())
-    nv.check(rc, "bxf_gru_linear")
-    if g.mode:
-        nv.check(lib.bxf_gru_finish(dt, M, width, ctypes.byref(g), nv.stream()), "bxf_gru_finish")
+               seq=seq.data_ptr(), out=out.data_ptr(), ldo=out.stride(0))
+    if M <= lib.bxf_gru_rows(dt):
+        rc = lib.bxf_gru_linear(dt, w.data_ptr(), w.shape[-1], h.data_ptr(), h.stride(0), M, width, K, ctypes.byref(g),
+                                nv.stream())
+        nv.check(rc, "bxf_gru_linear")
+        return out
+    y = torch.empty(M, 3 * width, dtype=torch.float32, device=h.device)
+    linear(w, h, M, 3 * width, K, store(y, 3 * width, 3 * width, out_type=OUT_F32))
+    fold = torch.empty(lib.bxf_gru_chunks(M), width, 2, dtype=torch.float32, device=h.device)
+    rc = lib.bxf_gru_scan(dt, y.data_ptr(), fold.data_ptr(), M, width, ctypes.byref(g), nv.stream())
+    nv.check(rc, "bxf_gru_scan")
     return out
 
 

@@ -59,17 +59,14 @@ typedef struct {
   int pad_;
 } bxf_epilogue;
 
-/* The gates of a minGRU layer after its three products (update, candidate, output gate; planes 0, 1, 2). */
+/* The recurrence of a minGRU layer after its three products (update, candidate, output gate). */
 typedef struct {
   const float *bias_z, *bias_x; /* [width] */
   float* state;                 /* [slots, width] */
   const int* flags;             /* [M] row flags */
   const int64_t* seq;           /* [M] state slot of each row */
-  void* out;                    /* T [M, ldo]: state * silu(gate) (mode 0) or silu(gate) alone (mode 1) */
+  void* out;                    /* T [M, ldo]: state * silu(gate) */
   int64_t ldo;
-  float *decay, *local;         /* mode 1: float [M, width] */
-  int mode;                     /* 0: rows fit one tile, finished here; 1: bxf_gru_finish follows */
-  int tile;                     /* rows of a tile (bxf_gru_tile) */
 } bxf_gru;
 
 int bxf_version(void);
@@ -87,15 +84,18 @@ int bxf_set_device_status(int value);
 int bxf_linear(int dtype, const void* w, int64_t ldw, int64_t gsw, const void* x, int64_t ldx, int64_t gsx, int groups,
                int M, int N, int K, const int* counts, const bxf_epilogue* epi, int tile, void* stream);
 
-/* The three products of a minGRU layer with its recurrence: w T [3, width, ldw] (planes z, x, g), x T [M, ldx].
- * z = sigmoid(acc_0 + bias_z), u = acc_1 + bias_x, candidate = u + 1/2 (u >= 0) or sigmoid(u),
- * S = (1 - z) S + z candidate along the rows of a sequence, from `state` (zero on BXF_ROW_START) and back into it.
- * bxf_gru_tile: the tile for M rows; mode 0 when they fit it. Mode 1 leaves for every row the prefix product of (1 - z)
- * and the state from a zero start, both within its tile, for bxf_gru_finish. */
-int bxf_gru_tile(int dtype, int M, int width);
+/* minGRU: acc_z, acc_x, acc_g = three products of the normed row; z = sigmoid(acc_z + bias_z), u = acc_x + bias_x,
+ * candidate = u + 1/2 (u >= 0) or sigmoid(u), S = (1 - z) S + z candidate along the rows of a sequence, from `state` (zero
+ * on BXF_ROW_START) and back into it; out = S silu(acc_g).
+ *   bxf_gru_linear  products and recurrence in one kernel, for at most bxf_gru_rows(dtype) rows (decoding, short portions):
+ *                   w T [3, width, ldw] (planes z, x, g), x T [M, ldx]
+ *   bxf_gru_scan    the recurrence alone, any M: y float [M, 3 width] = [acc_z | acc_x | acc_g] (overwritten); fold: scratch
+ *                   float [bxf_gru_chunks(M), width, 2] */
+int bxf_gru_rows(int dtype);
+int bxf_gru_chunks(int M);
 int bxf_gru_linear(int dtype, const void* w, int64_t ldw, const void* x, int64_t ldx, int M, int width, int K,
                    const bxf_gru* gru, void* stream);
-int bxf_gru_finish(int dtype, int M, int width, const bxf_gru* gru, void* stream);
+int bxf_gru_scan(int dtype, float* y, float* fold, int M, int width, const bxf_gru* gru, void* stream);
 
 /* flags int32 [M] from seq / slot / pos int64 [M] (slot < 0: padding row). */
 int bxf_row_flags(const int64_t* seq, const int64_t* slot, const int64_t* pos, int* flags, int M, void* stream);

@@ -139,10 +139,10 @@ def test_float_library_exports_every_declared_symbol_and_checks_arguments():
     assert lib.bxf_linear(0, 16, 12, 0, 16, 8, 0, 1, 1, 8, 8, None, ctypes.byref(epi), 0, None) == nv.BX_EARG   # ld % 8
     assert lib.bxf_linear(0, 16, 8, 0, 16, 8, 0, 1, 1, 9, 8, None, ctypes.byref(epi), 0, None) == nv.BX_EARG    # no side
     assert lib.bxf_route(16, 8, 8, 9, 16, 16, 16, 16, 1, None) == nv.BX_ELIMIT
-    g = nv.Gru(mode=0)
+    g = nv.Gru()
     assert lib.bxf_gru_linear(0, 16, 8, 16, 8, 4, 8, 8, ctypes.byref(g), None) == nv.BX_EARG
     assert lib.bxf_latent_attention_tile(12) == 10 and lib.bxf_latent_attention_tile(200) == 1
-    assert ctypes.sizeof(nv.Epilogue) == 128 and ctypes.sizeof(nv.Gru) == 80      # as asserted in float_capi.cu
+    assert ctypes.sizeof(nv.Epilogue) == 128 and ctypes.sizeof(nv.Gru) == 56      # as asserted in float_capi.cu
 
 
 def test_sources_of_the_targets_are_separate():
