@@ -56,7 +56,7 @@ class Session:
 
     def release(self, seq):
         """The sequence is finished: its pages go back to the pool and its row may serve another one. Nothing is cleared:
-        keys beyond a sequence's length are never read, and a recurrent state starts from zero at position 0."""
+        keys beyond a sequence's length carry no weight, and a recurrent state starts from zero at position 0."""
         if self.free is not None:
             self.free += self.held[seq][::-1]
             self.held[seq] = []
