@@ -27,6 +27,7 @@ class Head:
         """The int64 logits [R, V] at 16 fractional bits."""
         if self.c.dtype == torch.int64:
             return self.c[:self.R]
+        assert self.c.dtype == torch.int32 and self.c.shape[0] >= 2 * self.M and self.c.is_contiguous()   # limb products
         y = torch.empty(self.M, self.V, dtype=torch.long, device=self.c.device)
         flag = torch.zeros(1, dtype=torch.int32, device=self.c.device)
         if self.M:

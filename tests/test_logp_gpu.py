@@ -93,7 +93,7 @@ def test_tri_logp_from_the_head():
     from bitexact_llm_b200.vllm_plugin import rl, tri_logp, tri_sample
     g = torch.Generator().manual_seed(9)
     M, V = 6, 5000
-    c = torch.randint(-(1 << 24), 1 << 24, (M, V), generator=g, dtype=torch.int32).cuda()
+    c = torch.randint(-(1 << 24), 1 << 24, (2 * M, V), generator=g, dtype=torch.int32).cuda()   # two limb planes
     m = torch.randint(1 << 20, 1 << 23, (V,), generator=g).cuda()
     mant = torch.randint(1 << 23, 1 << 24, (M,), generator=g).cuda()
     e = torch.randint(-6, 2, (M,), generator=g).cuda()
