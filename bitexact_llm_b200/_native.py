@@ -90,12 +90,45 @@ class Epilogue(ctypes.Structure):
     """bxf_epilogue."""
     _fields_ = [("kind", I), ("out_type", I), ("act", I), ("n_main", I), ("act_p", R), ("act_q", R), ("out", P), ("ldo", L),
                 ("gso", L), ("side", P), ("lds", L), ("bias", P), ("gate", P), ("ldg", L), ("cs", P), ("rot_out", P),
-                ("ldr", L), ("hsr", L), ("rot_dim", I), ("pad_", I)]
+                ("ldr", L), ("hsr", L), ("rot_dim", I), ("pad_", I), ("main_bias", P)]
 
 
 class Gru(ctypes.Structure):
     """bxf_gru."""
     _fields_ = [("bias_z", P), ("bias_x", P), ("state", P), ("flags", P), ("seq", P), ("out", P), ("ldo", L)]
+
+
+class StreamsStep(ctypes.Structure):
+    """bxf_streams_step."""
+    _fields_ = [("x", P), ("ids", P), ("embed", P), ("vocab", L), ("y", P), ("out", P), ("mix", P), ("in_", P), ("w", P),
+                ("h", P), ("ldh", L), ("sum", P), ("eps", R), ("streams", I), ("D", I), ("pad_", I)]
+
+
+class GqaRows(ctypes.Structure):
+    """bxf_gqa_rows."""
+    _fields_ = [("y", P), ("ldy", L), ("heads", I), ("kv_heads", I), ("dim", I), ("vdim", I), ("rot_dims", I), ("page", I),
+                ("q_norm", P), ("k_norm", P), ("cs", P), ("slot", P), ("q", P), ("ldq", L), ("cache", P), ("ldc", L),
+                ("voff", L), ("eps", R), ("pad_", I)]
+
+
+class Conv(ctypes.Structure):
+    """bxf_conv."""
+    _fields_ = [("u", P), ("ldu", L), ("w", P), ("b", P), ("state", P), ("flags", P), ("seq", P), ("pos", P),
+                ("channels", I), ("taps", I)]
+
+
+class RecurrenceRows(ctypes.Structure):
+    """bxf_recurrence_rows."""
+    _fields_ = [("kind", I), ("heads", I), ("groups", I), ("K", I), ("V", I), ("rank", I), ("q0", I), ("k0", I), ("v0", I),
+                ("pad_", I), ("y", P), ("ldy", L), ("side", P), ("lds", L), ("a2", P), ("a2_b", P), ("inv_tau", R),
+                ("q_scale", R), ("A_log", P), ("skip", P), ("conv", Conv), ("state", P), ("flags", P), ("seq", P), ("out", P),
+                ("ldo", L)]
+
+
+class GateRows(ctypes.Structure):
+    """bxf_gate_rows."""
+    _fields_ = [("o", P), ("z", P), ("ldo", L), ("ldz", L), ("w", P), ("out", P), ("ldout", L), ("n", I), ("parts", I),
+                ("wn", I), ("gate_first", I), ("eps", R), ("pad_", I), ("conv", Conv)]
 
 
 _FLOAT_SIGNATURES = {
@@ -117,6 +150,14 @@ _FLOAT_SIGNATURES = {
     "bxf_latent_attention_scratch": (Z, [I, I, I]),
     "bxf_latent_attention_tile": (I, [I]),
     "bxf_latent_attention": (I, [I, P, L, I, I, I, I, P, L, I, I, P, I, L, I, P, P, P, I, I, P, R, P, L, P, Z, I, P]),
+    "bxf_angles": (I, [P, I, P, P, I, P]),
+    "bxf_gqa_prepare": (I, [I, ctypes.POINTER(GqaRows), I, P]),
+    "bxf_gqa_attention_scratch": (Z, [I, I, I, I]),
+    "bxf_gqa_attention": (I, [I, P, L, I, I, I, I, I, P, L, L, I, I, P, I, L, I, P, P, P, I, I, P, R, P, L, P, Z, I, P]),
+    "bxf_streams": (I, [I, ctypes.POINTER(StreamsStep), I, P]),
+    "bxf_causal_conv": (I, [I, ctypes.POINTER(Conv), P, L, I, P]),
+    "bxf_recurrence": (I, [I, ctypes.POINTER(RecurrenceRows), I, P]),
+    "bxf_gated_norm": (I, [I, ctypes.POINTER(GateRows), I, P]),
 }
 
 

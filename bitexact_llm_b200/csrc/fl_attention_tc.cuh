@@ -1,9 +1,10 @@
-// Latent attention on the tensor cores (bf16 cache, fp32 scores and softmax), one kernel for prompts and decoding.
+// Attention over a paged cache on the tensor cores (bf16 cache, fp32 scores and softmax), one kernel for prompts and decoding.
 //
-// A tile is up to 128 query rows = (consecutive tokens of one sequence) x heads: all of them read the same latent rows, so
-// a block of 64 cache rows is staged once for 128 queries. Scores Q C^T: A = Q tile [128 x W] (W = latent + rotated part),
-// B = cache rows, both K-major. P V: the values are the first R entries of the SAME staged rows, read as an MN-major B
-// operand (their rows are the contraction index), so nothing is transposed or loaded twice; A = P comes from TMEM, where
+// A tile is up to 128 query rows = (consecutive tokens of one sequence) x (heads of one group): all of them read the same
+// cache rows, so a block of 64 rows is staged once for 128 queries. Scores Q K^T: A = Q tile [128 x W], B = the rows' keys,
+// both K-major. P V: the values are staged row by row like the keys and read as an MN-major B operand (their rows are the
+// contraction index), so nothing is transposed; in latent attention they are the first R entries of the staged keys
+// themselves and nothing is loaded twice. A = P comes from TMEM, where
 // the softmax warps leave it as bf16 in place of the scores. TMEM: two score buffers of 64 columns, then the output
 // accumulator (256 columns; a wider latent is cut into value slices over blockIdx.z).
 //
@@ -25,11 +26,11 @@ constexpr float LT_LOG2E = 1.4426950408889634f;
 constexpr float LT_GROWTH = 8.0f;
 
 struct LatentTc {
-  int cols;                                              // 64-entry column blocks of a row, ceil(W / 64)
+  int cols, kcols, vbox;                                 // 64-entry column blocks of a staged row, of its key; first one of its value
   int stages, qrows;                                     // key stages of the ring, rows of the Q box
-  int row_blocks, vsplit;                                // blockIdx.z = value slice * row_blocks + row block
+  int row_blocks, vsplit;                                // blockIdx.z = (group * vsplit + value slice) * row_blocks + row block
   int splits;
-  float* part;                                           // splits > 1: [splits][M H][R] accumulators, then [splits][M H][2]
+  float* part;                                           // splits > 1: [splits][M G H][R] accumulators, then [splits][M G H][2]
 };
 
 struct LatentShared {
@@ -71,12 +72,12 @@ __device__ __forceinline__ uint64_t umma_desc_mn(uint32_t addr) {
 }
 
 __global__ void __launch_bounds__(LT_THREADS, 1)
-fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mc,
-                              const LatentAttn a, const LatentTc c) {
+fl_paged_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mc,
+                             const PagedAttn a, const LatentTc c) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* qs = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int q_box = c.qrows * 128;                       // bytes of a column block of the queries
-  uint8_t* ring = qs + c.cols * q_box;
+  uint8_t* ring = qs + c.kcols * q_box;
   const int stage_bytes = c.cols * LT_KEYS * 128;
   LatentShared* sh = reinterpret_cast<LatentShared*>(ring + c.stages * stage_bytes);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -97,7 +98,8 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
     seq = a.seq[tok0];
   }
   const int row0 = (blockIdx.z % c.row_blocks) * 128, rows = min(128, ntok * a.H - row0);
-  const int v0 = (blockIdx.z / c.row_blocks) * LT_VCOLS, vn = min(LT_VCOLS, a.R - v0);
+  const int slice = blockIdx.z / c.row_blocks, group = slice / c.vsplit;
+  const int v0 = slice % c.vsplit * LT_VCOLS, vn = min(LT_VCOLS, a.R - v0);
   const i64 limit = (i64)a.nblk * a.bs - 1;
   const i64 p_first = min(a.pos[tok0], limit), p_last = min(a.pos[tok0 + ntok - 1], limit);
   const int b_lo = a.first_key(p_first) / LT_KEYS, b_hi = (int)(p_last / LT_KEYS) + 1;
@@ -147,9 +149,9 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
     //      boxes at a time; one lane issues the copies ----
     if (nb > 0) {
       if (lane == 0) {
-        mbar_arrive_expect_tx(&sh->q_full, c.cols * q_box);
-        for (int j = 0; j < c.cols; ++j)
-          tma_load_3d(qs + j * q_box, &mq, &sh->q_full, j * 64, tok0 * a.H + row0, 0);
+        mbar_arrive_expect_tx(&sh->q_full, c.kcols * q_box);
+        for (int j = 0; j < c.kcols; ++j)
+          tma_load_3d(qs + j * q_box, &mq, &sh->q_full, j * 64, tok0 * a.H + row0, group);
       }
       const int box = min(a.bs, LT_KEYS), boxes = LT_KEYS / box;
       int i = 0, held = 0;
@@ -165,13 +167,13 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
           const int nth = i * boxes + p;                             // box of this CTA
           if ((nth & 31) == 0) {
             const int page = (b0 * LT_KEYS + (nth + lane) * box) / a.bs;
-            held = (int)(a.page_row(seq, min(page, a.nblk - 1)) / a.bs);
+            held = (int)a.page_of(seq, min(page, a.nblk - 1)) * a.G + group;
           }
           const int page = __shfl_sync(0xffffffffu, held, nth & 31);
           if (lane == 0)
             for (int j = 0; j < c.cols; ++j)
-              tma_load_3d(st + j * LT_KEYS * 128 + p * box * 128, &mc, &sh->full[s], j * 64,
-                          (b0 * LT_KEYS + nth * box) % a.bs, page);
+              tma_load_3d(st + j * LT_KEYS * 128 + p * box * 128, &mc, &sh->full[s],
+                          j < c.kcols ? j * 64 : a.voff + (j - c.kcols) * 64, (b0 * LT_KEYS + nth * box) % a.bs, page);
         }
       }
       if (!ok && lane == 0) {
@@ -192,7 +194,7 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
         if (i >= 2 && !mbar_wait(&sh->pv_done[buf], ((i >> 1) - 1) & 1)) return false;   // P of block i - 2 is read
         tc_fence_after();
         const uint32_t qa = smem_u32(qs), ka = smem_u32(ring + s * stage_bytes);
-        for (int j = 0; j < c.cols; ++j)
+        for (int j = 0; j < c.kcols; ++j)
 #pragma unroll
           for (int ks = 0; ks < 4; ++ks)
             umma_bf16(tmem + buf * LT_KEYS, umma_desc_sw128(qa + j * q_box + ks * 32),
@@ -206,7 +208,7 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
         if (c.stages > 1 && i + 1 < nb && !(ok = scores(i + 1))) break;
         if (!(ok = mbar_wait(&sh->p_full[buf], (i >> 1) & 1))) break;
         tc_fence_after();
-        const uint32_t va = smem_u32(ring + s * stage_bytes) + (v0 / 64) * LT_KEYS * 128;
+        const uint32_t va = smem_u32(ring + s * stage_bytes) + (c.vbox + v0 / 64) * LT_KEYS * 128;
 #pragma unroll
         for (int ks = 0; ks < LT_KEYS / 16; ++ks)
           umma_bf16_ts(tmem + LT_O, tmem + buf * LT_KEYS + ks * 8, umma_desc_mn(va + ks * 2048), id_v, (i | ks) != 0);
@@ -222,8 +224,8 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
     constexpr int KW = LT_KEYS / 4;
     const int quarter = warp & 3, part = (warp - 2) >> 2, r = quarter * 32 + lane;
     const bool live = r < rows;
-    const int flat = row0 + (live ? r : 0), head = flat % a.H;
-    const i64 pos = min(a.pos[tok0 + flat / a.H], limit);
+    const int flat = row0 + (live ? r : 0), token = tok0 + flat / a.H, head = group * a.H + flat % a.H;
+    const i64 pos = min(a.pos[token], limit);
     const int lo = a.first_key(pos), hi = (int)pos;
     const float scale = a.scale * LT_LOG2E;
     float ref = a.sink ? a.sink[head] * LT_LOG2E : -INFINITY;
@@ -306,10 +308,10 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
       if (lane == 0) fail();
     } else {
       tc_fence_after();
-      const i64 at = (i64)tok0 * a.H + row0 + r;
+      const i64 n = (i64)a.M * a.H * a.G, at = (i64)token * a.H * a.G + head;
       const float inv = 1.0f / den;
-      float* acc = c.part + ((i64)blockIdx.y * a.M * a.H + at) * a.R + v0;
-      bf16* out = static_cast<bf16*>(a.out) + at * a.ldo + v0;
+      float* acc = c.part + (blockIdx.y * n + at) * a.R + v0;
+      bf16* out = static_cast<bf16*>(a.out) + token * a.out_tok + head * a.out_head + v0;
       for (int q = part * 16; q < vn; q += 64) {
         uint32_t u[16] = {};
         if (nb > 0) {
@@ -317,15 +319,15 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
           tmem_ld_wait();
         }
         if (!live) continue;
-        const int n = min(16, vn - q);
+        const int cnt = min(16, vn - q);
         float v[16];
 #pragma unroll
         for (int k = 0; k < 16; ++k) v[k] = __uint_as_float(u[k]) * (c.splits == 1 ? inv : 1.0f);
-        if (c.splits == 1) store_run(out + q, v, n);
-        else store_run(acc + q, v, n);
+        if (c.splits == 1) store_run(out + q, v, cnt);
+        else store_run(acc + q, v, cnt);
       }
       if (c.splits > 1 && live && v0 == 0 && part == 0) {
-        float* ml = c.part + (i64)c.splits * a.M * a.H * a.R + ((i64)blockIdx.y * a.M * a.H + at) * 2;
+        float* ml = c.part + c.splits * n * a.R + (blockIdx.y * n + at) * 2;
         ml[0] = ref;
         ml[1] = den;
       }
@@ -342,10 +344,10 @@ fl_latent_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gr
 }
 
 // Joins the key splits: one CTA per query row (token, head).
-__global__ void __launch_bounds__(128) fl_latent_join_kernel(const LatentAttn a, const float* part, int splits) {
+__global__ void __launch_bounds__(128) fl_attention_join_kernel(const PagedAttn a, const float* part, int splits) {
   launch_next();
   wait_previous();
-  const i64 at = blockIdx.x, n = (i64)a.M * a.H;
+  const i64 at = blockIdx.x, heads = a.H * a.G, n = a.M * heads;
   const float* ml = part + splits * n * a.R;
   float mx = -INFINITY, f[LT_MAX_SPLIT], den = 0.0f;
   for (int s = 0; s < splits; ++s)
@@ -356,7 +358,7 @@ __global__ void __launch_bounds__(128) fl_latent_join_kernel(const LatentAttn a,
     if (f[s] > 0.0f) den += f[s] * ml[(s * n + at) * 2 + 1];
   }
   const float inv = 1.0f / den;
-  bf16* out = static_cast<bf16*>(a.out) + at * a.ldo;
+  bf16* out = static_cast<bf16*>(a.out) + at / heads * a.out_tok + at % heads * a.out_head;
   for (int d = threadIdx.x; d < a.R; d += 128) {
     float o = 0.0f;
 #pragma unroll

@@ -77,12 +77,17 @@ __device__ __forceinline__ float sigmoid(float v) {
 template <class T>
 __device__ __forceinline__ float silu(float v) { return v * sigmoid<T>(v); }
 
+template <class T>
 __device__ __forceinline__ float activate(int act, float z, float p, float q) {
   if (act == BXF_ACT_RELU2) {
     const float r = fmaxf(z, 0.0f);
     return r * r;
   }
   if (act == BXF_ACT_XIELU) return (z > 0.0f ? p * z * z : q * (expm1f(z) - z)) + 0.5f * z;
+  // (1 + tanh(a)) / 2 = sigmoid(2 a), a = sqrt(2 / pi) (z + 0.044715 z^3)
+  if (act == BXF_ACT_GELU) return z * sigmoid<T>(1.5957691216057308f * (z + 0.044715f * z * z * z));
+  if (act == BXF_ACT_SCALE) return p * z;
+  if (act == BXF_ACT_SOFTCAP) return q * tanhf(p * z);
   return z;
 }
 

@@ -67,6 +67,23 @@ __device__ __forceinline__ void store_run(float* p, const float (&v)[16], int n)
   }
 }
 
+// Eight consecutive values.
+__device__ __forceinline__ void store_run8(bf16* p, const float (&v)[8], int n) {
+  if (n == 8 && (reinterpret_cast<uintptr_t>(p) & 15) == 0) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+  } else {
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+      if (i < n) st(p + i, v[i]);
+  }
+}
+
+__device__ __forceinline__ void store_run8(float* p, const float (&v)[8], int n) {
+#pragma unroll
+  for (int i = 0; i < 8; ++i)
+    if (i < n) p[i] = v[i];
+}
+
 // Fixed point at 24 bits.
 __device__ __forceinline__ void store_run(i64* p, const float (&v)[16], int n) {
   i64 q[16];
@@ -131,6 +148,15 @@ struct StageEpi {
       }
       return;
     }
+    if (p.kind == BXF_EPI_GLU) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const float up = __shfl_xor_sync(0xffffffffu, v[i], 1);
+        if (i < cnt && n < N && !(n & 1))
+          st(static_cast<T*>(p.out) + (row + i) * p.ldo + (n >> 1), activate<T>(p.act, v[i], p.act_p, p.act_q) * up);
+      }
+      return;
+    }
     if (n >= N) return;
     if (p.kind == BXF_EPI_ADD) {
       float* o = static_cast<float*>(p.out) + row * p.ldo + n;
@@ -153,10 +179,11 @@ struct StageEpi {
         if (i < cnt) o[i * p.lds] = v[i] + b;
     } else {
       const i64 at = group * p.gso + row * p.ldo + n;
+      const float b = p.main_bias ? p.main_bias[n] : 0.0f;
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         if (i >= cnt) break;
-        const float y = activate(p.act, v[i], p.act_p, p.act_q);
+        const float y = activate<T>(p.act, v[i] + b, p.act_p, p.act_q);
         if (p.out_type == BXF_OUT_T) st(static_cast<T*>(p.out) + at + i * p.ldo, y);
         else if (p.out_type == BXF_OUT_F32) static_cast<float*>(p.out)[at + i * p.ldo] = y;
         else static_cast<i64*>(p.out)[at + i * p.ldo] = __double2ll_rn((double)y * 16777216.0);
@@ -169,6 +196,13 @@ struct StageEpi {
   static __device__ __forceinline__ void chunk_rows(const Params& p, int group, i64 m, int n, int cnt, float (&v)[16]) {
     if (p.kind == BXF_EPI_ADD) {
       add_run(static_cast<float*>(p.out) + m * p.ldo + n, v, cnt);
+      return;
+    }
+    if (p.kind == BXF_EPI_GLU) {
+      float o[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) o[i] = activate<T>(p.act, v[2 * i], p.act_p, p.act_q) * v[2 * i + 1];
+      store_run8(static_cast<T*>(p.out) + m * p.ldo + (n >> 1), o, cnt >> 1);
       return;
     }
     int main_cnt = cnt;                                                 // of them, below n_main
@@ -197,12 +231,14 @@ struct StageEpi {
         }
       }
       if (main_cnt <= 0) return;
-      if (p.act == BXF_ACT_RELU2) {
+      if (p.main_bias) {
 #pragma unroll
-        for (int i = 0; i < 16; ++i) v[i] = activate(BXF_ACT_RELU2, v[i], 0.0f, 0.0f);
-      } else if (p.act == BXF_ACT_XIELU) {
+        for (int i = 0; i < 16; ++i)
+          if (i < main_cnt) v[i] += p.main_bias[n + i];
+      }
+      if (p.act != BXF_ACT_NONE) {
 #pragma unroll
-        for (int i = 0; i < 16; ++i) v[i] = activate(BXF_ACT_XIELU, v[i], p.act_p, p.act_q);
+        for (int i = 0; i < 16; ++i) v[i] = activate<T>(p.act, v[i], p.act_p, p.act_q);
       }
     }
     const i64 at = group * p.gso + m * p.ldo + n;

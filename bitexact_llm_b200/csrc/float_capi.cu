@@ -10,13 +10,15 @@
 #include "fl_attention_tc.cuh"
 #include "fl_gemm.cuh"
 #include "fl_gemm_simt.cuh"
+#include "fl_recurrence.cuh"
 #include "fl_stages.cuh"
+#include "fl_streams.cuh"
 
 namespace {
 
 using namespace bxf;
 
-static_assert(sizeof(bxf_epilogue) == 128 && sizeof(bxf_gru) == 56, "layouts of the callers' structs");
+static_assert(sizeof(bxf_epilogue) == 136 && sizeof(bxf_gru) == 56, "layouts of the callers' structs");
 
 inline cudaStream_t stream_of(void* s) { return static_cast<cudaStream_t>(s); }
 inline bool dtype_ok(int d) { return d == BXF_BF16 || d == BXF_F32; }
@@ -233,53 +235,142 @@ int run_bf16(const Operands& o, const GemmShape& s, const bxf_epilogue& ep, int 
 }
 
 // The tensor-core attention kernel takes pages of 8, 16, .. keys, rows of at most 9 column blocks (shared memory).
-bool latent_tc_fits(int dtype, const LatentAttn& a) {
-  return dtype == BXF_BF16 && a.bs >= 8 && (a.bs & (a.bs - 1)) == 0 && ceil_div(a.R + a.rot, 64) <= 9 && aligned16(a.q) &&
-         aligned16(a.cache) && aligned16(a.out) && a.ldq % 8 == 0 && a.ldc % 8 == 0 && a.ldo % 8 == 0;
+bool paged_tc_fits(int dtype, const PagedAttn& a) {
+  const int cols = ceil_div(a.W, 64) + (a.voff > 0 ? ceil_div(a.R, 64) : 0);
+  return dtype == BXF_BF16 && a.bs >= 8 && (a.bs & (a.bs - 1)) == 0 && cols <= 9 && aligned16(a.q) && aligned16(a.cache) &&
+         a.ldq % 8 == 0 && a.ldc % 8 == 0 && a.voff % 8 == 0;
 }
 
-size_t latent_scratch(i64 rows, int R, int splits) { return (size_t)splits * rows * (R + 2) * sizeof(float); }
+size_t attention_scratch(i64 rows, int R, int splits) { return (size_t)splits * rows * (R + 2) * sizeof(float); }
 
-int launch_latent_tc(const LatentAttn& a, void* scratch, size_t scratch_bytes, cudaStream_t st) {
+// Key splits only happen while the query tiles leave SMs idle (148 of them).
+size_t attention_scratch_for(int M, int groups, int heads, int R) {
+  if (M < 1 || groups < 1 || heads < 1 || R < 1 || (i64)M * groups > 148) return 0;
+  const int free = 148 / (M * groups), splits = free < 2 ? 2 : free > LT_MAX_SPLIT ? LT_MAX_SPLIT : free;
+  return attention_scratch((i64)M * groups * heads, R, splits);
+}
+
+int launch_paged_tc(const PagedAttn& a, void* scratch, size_t scratch_bytes, cudaStream_t st) {
   constexpr int SMEM_MAX = 227 * 1024;
   static PerDevice configured;
   if (once_per_device(configured, [] {
-        return cudaFuncSetAttribute(fl_latent_attention_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MAX);
+        return cudaFuncSetAttribute(fl_paged_attention_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MAX);
       }) != BX_OK)
     return BX_ELAUNCH;
   LatentTc c = {};
-  const int W = a.R + a.rot;
-  c.cols = ceil_div(W, 64);
+  c.kcols = ceil_div(a.W, 64);
+  c.vbox = a.voff > 0 ? c.kcols : 0;
+  c.cols = c.kcols + (a.voff > 0 ? ceil_div(a.R, 64) : 0);
   const int tokens = a.tiles ? bxf_latent_attention_tile(a.H) : 1, tiles = a.tiles ? a.ntiles : a.M;
   const int rows = tokens * a.H;
   c.qrows = rows >= 128 ? 128 : ceil_div(rows, 8) * 8;
-  const int fixed = 1024 + c.cols * c.qrows * 128 + (int)sizeof(LatentShared);
+  const int fixed = 1024 + c.kcols * c.qrows * 128 + (int)sizeof(LatentShared);
   c.stages = (SMEM_MAX - fixed) / (c.cols * LT_KEYS * 128);
   if (c.stages > LT_MAX_STAGES) c.stages = LT_MAX_STAGES;
   c.row_blocks = ceil_div(rows, 128);
   c.vsplit = ceil_div(a.R, LT_VCOLS);
   c.splits = 1;
   const i64 span = a.window > 0 && a.window + tokens < (i64)a.nblk * a.bs ? a.window + tokens : (i64)a.nblk * a.bs;
-  const i64 blocks = span / LT_KEYS + 1, ctas = (i64)tiles * c.row_blocks * c.vsplit;
+  const i64 blocks = span / LT_KEYS + 1, ctas = (i64)tiles * c.row_blocks * c.vsplit * a.G;
+  if ((i64)c.row_blocks * c.vsplit * a.G > 65535) return BX_ELIMIT;
   const int sms = device_sms();
   if (sms <= 0) return BX_ELAUNCH;
   while (c.splits < LT_MAX_SPLIT && ctas * c.splits * 2 <= sms && blocks >= c.splits * 4 && scratch &&
-         scratch_bytes >= latent_scratch((i64)a.M * a.H, a.R, c.splits * 2))
+         scratch_bytes >= attention_scratch((i64)a.M * a.H * a.G, a.R, c.splits * 2))
     c.splits *= 2;
   c.part = static_cast<float*>(scratch);
   CUtensorMap mq, mc;
-  if (!make_map_bf16(&mq, a.q, W, (i64)a.M * a.H, 1, a.ldq, 0, c.qrows, 1) ||
-      !make_map_bf16(&mc, a.cache, W, a.bs, a.nb, a.ldc, (i64)a.bs * a.ldc, a.bs < LT_KEYS ? a.bs : LT_KEYS, 1))
+  if (!make_map_bf16(&mq, a.q, a.W, (i64)a.M * a.H, a.G, a.ldq, (i64)a.M * a.H * a.ldq, c.qrows, 1) ||
+      !make_map_bf16(&mc, a.cache, a.voff > 0 ? a.voff + a.R : a.W, a.bs, (i64)a.nb * a.G, a.ldc, (i64)a.bs * a.ldc,
+                     a.bs < LT_KEYS ? a.bs : LT_KEYS, 1))
     return BX_ELAUNCH;
-  const dim3 grid(tiles, c.splits, c.row_blocks * c.vsplit);
-  const int rc = launch_chained(fl_latent_attention_tc_kernel, grid, LT_THREADS, fixed + c.stages * c.cols * LT_KEYS * 128, st,
+  const dim3 grid(tiles, c.splits, c.row_blocks * c.vsplit * a.G);
+  const int rc = launch_chained(fl_paged_attention_tc_kernel, grid, LT_THREADS, fixed + c.stages * c.cols * LT_KEYS * 128, st,
                                 0, mq, mc, a, c);
   if (rc != BX_OK || c.splits == 1) return rc;
-  return launch_chained(fl_latent_join_kernel, dim3((unsigned)(a.M * a.H)), 128, 0, st, 0, a, c.part, c.splits);
+  return launch_chained(fl_attention_join_kernel, dim3((unsigned)(a.M * a.H * a.G)), 128, 0, st, 0, a, c.part, c.splits);
+}
+
+int run_attention(int dtype, const PagedAttn& a, void* scratch, size_t scratch_bytes, int variant, cudaStream_t st) {
+  if (a.R > LA_MAX_R || a.W > 8192 || (i64)a.H * a.G > 65535) return BX_ELIMIT;
+  if (g_status_seen.load() != 0) return BX_EDEVICE;
+  if (a.M == 0) return BX_OK;
+  if (variant == 2 && !paged_tc_fits(dtype, a)) return BX_ELIMIT;
+  if (variant != 1 && paged_tc_fits(dtype, a) && (!a.tiles || a.ntiles > 0)) return launch_paged_tc(a, scratch, scratch_bytes, st);
+  const dim3 grid(a.M, a.H * a.G);
+  if (dtype == BXF_F32) fl_paged_attention_kernel<float><<<grid, LA_THREADS, a.W * 4, st>>>(a);
+  else fl_paged_attention_kernel<bf16><<<grid, LA_THREADS, a.W * 4, st>>>(a);
+  return launched(1);
 }
 
 bool gru_ok(const bxf_gru* g, int M, int width) {
   return g && M >= 0 && width >= 1 && g->bias_z && g->bias_x && g->state && g->flags && g->seq && g->out && g->ldo >= width;
+}
+
+template <class T>
+int launch_streams(const bxf_streams_step& p, int M, bool vec, cudaStream_t st) {
+  const int S = p.streams;
+  auto* kernel = S <= 2 ? (vec ? fl_streams_kernel<T, 2, 4> : fl_streams_kernel<T, 2, 1>)
+               : S <= 4 ? (vec ? fl_streams_kernel<T, 4, 4> : fl_streams_kernel<T, 4, 1>)
+                        : (vec ? fl_streams_kernel<T, BXF_MAX_STREAMS, 4> : fl_streams_kernel<T, BXF_MAX_STREAMS, 1>);
+  const int smem = p.h ? p.D * 4 : 0;
+  if (smem > 40 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
+    return BX_ELAUNCH;
+  return launch_chained(kernel, dim3(M), NORM_THREADS, smem, st, 0, p);
+}
+
+bool conv_ok(const bxf_conv* c) {
+  return c && c->u && c->w && c->b && c->state && c->flags && c->seq && c->pos && c->channels >= 1 && c->taps >= 1 &&
+         c->taps <= BXF_MAX_TAPS && c->ldu >= c->channels;
+}
+
+bool recurrence_ok(const bxf_recurrence_rows* p) {
+  if (!p || !p->y || !p->side || !p->state || !p->flags || !p->seq || !p->out || p->heads < 1 || p->groups < 1 ||
+      p->heads % p->groups || p->K < 1 || p->V < 1 || p->ldo < (i64)p->heads * p->V)
+    return false;
+  if (p->kind == BXF_DECAY_CHANNEL) return p->rank >= 1 && p->a2 && p->a2_b && p->groups == p->heads;
+  return p->kind == BXF_DECAY_HEAD && p->A_log && p->skip;
+}
+
+template <class T, bool CHANNEL, int KR>
+int launch_recurrence_as(const bxf_recurrence_rows& p, int M, cudaStream_t st) {
+  const int smem = recurrence_smem(p.K, CHANNEL);
+  static PerDevice configured;
+  if (once_per_device(configured, [] {
+        return cudaFuncSetAttribute(fl_recurrence_kernel<T, CHANNEL, KR>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                    recurrence_smem(REC_LANES * KR, CHANNEL));
+      }) != BX_OK)
+    return BX_ELAUNCH;
+  return launch_chained(fl_recurrence_kernel<T, CHANNEL, KR>, dim3(M, p.heads, ceil_div(p.V, REC_COLS)), REC_THREADS, smem, st, 0,
+                        p, M);
+}
+
+template <class T>
+int launch_recurrence(const bxf_recurrence_rows& p, int M, cudaStream_t st) {
+  const int kr = ceil_div(p.K, REC_LANES);
+  auto go = [&](auto channel) {
+    constexpr bool C = decltype(channel)::value;
+    if (kr <= 1) return launch_recurrence_as<T, C, 1>(p, M, st);
+    if (kr <= 2) return launch_recurrence_as<T, C, 2>(p, M, st);
+    if (kr <= 4) return launch_recurrence_as<T, C, 4>(p, M, st);
+    if (kr <= 8) return launch_recurrence_as<T, C, 8>(p, M, st);
+    return launch_recurrence_as<T, C, 16>(p, M, st);
+  };
+  return p.kind == BXF_DECAY_CHANNEL ? go(std::true_type{}) : go(std::false_type{});
+}
+
+template <class T>
+int launch_gated_norm(const bxf_gate_rows& p, int M, cudaStream_t st) {
+  const int size = p.n / p.parts;
+  const bool vec = size % 8 == 0 && p.wn % 8 == 0 && p.ldo % 8 == 0 && p.ldz % 8 == 0 && p.ldout % 8 == 0 && aligned16(p.o) &&
+                   aligned16(p.z) && aligned16(p.out) && aligned16(p.w);
+  const bool warp = size <= 512;                         // a warp per part, or a CTA
+  const int part_ctas = warp ? ceil_div(p.parts, GATE_THREADS / 32) : p.parts;
+  if (part_ctas >= 65535) return BX_ELIMIT;
+  const dim3 grid(M, part_ctas + (p.conv.w && p.conv.taps > 1 ? 1 : 0));
+  auto* kernel = warp ? (vec ? fl_gated_norm_kernel<T, true, 8> : fl_gated_norm_kernel<T, true, 1>)
+                      : (vec ? fl_gated_norm_kernel<T, false, 8> : fl_gated_norm_kernel<T, false, 1>);
+  return launch_chained(kernel, grid, GATE_THREADS, 0, st, 0, p, part_ctas);
 }
 
 // Rows of a scan chunk: short ones while there are few rows to spread over the SMs.
@@ -300,9 +391,10 @@ int bxf_linear(int dtype, const void* w, int64_t ldw, int64_t gsw, const void* x
   if (!dtype_ok(dtype) || !epi || groups < 1 || M < 0 || N < 1 || K < 1) return BX_EARG;
   if (!operand_ok(w, ldw, gsw, groups > 1, K, dtype) || !operand_ok(x, ldx, gsx, groups > 1 && !counts, K, dtype))
     return BX_EARG;
-  if (epi->kind < BXF_EPI_STORE || epi->kind > BXF_EPI_GATE || !epi->out) return BX_EARG;
+  if (epi->kind < BXF_EPI_STORE || epi->kind > BXF_EPI_GLU || !epi->out) return BX_EARG;
   if (epi->kind == BXF_EPI_STORE && epi->n_main < N && (!epi->side || groups > 1)) return BX_EARG;
   if (epi->kind == BXF_EPI_GATE && !epi->gate) return BX_EARG;
+  if (epi->kind == BXF_EPI_GLU && (N % 2 || groups > 1)) return BX_EARG;
   if (epi->kind == BXF_EPI_ROPE &&
       (!epi->rot_out || !epi->cs || epi->rot_dim < 2 || epi->rot_dim % 2 || epi->n_main % 8 || groups > 1))
     return BX_EARG;
@@ -420,12 +512,7 @@ int bxf_latent_prepare(int dtype, const float* y, int64_t ldy, int q_rank, int k
                         static_cast<bf16*>(cache), ldc, cs, gate);
 }
 
-// Key splits only happen while the query tiles leave SMs idle (148 of them).
-size_t bxf_latent_attention_scratch(int M, int heads, int kv_rank) {
-  if (M < 1 || heads < 1 || kv_rank < 1 || M > 148) return 0;
-  const int splits = 148 / M < 2 ? 2 : 148 / M > LT_MAX_SPLIT ? LT_MAX_SPLIT : 148 / M;
-  return latent_scratch((i64)M * heads, kv_rank, splits);
-}
+size_t bxf_latent_attention_scratch(int M, int heads, int kv_rank) { return attention_scratch_for(M, 1, heads, kv_rank); }
 
 int bxf_latent_attention_tile(int heads) { return heads >= 128 ? 1 : 128 / (heads < 1 ? 1 : heads); }
 
@@ -438,20 +525,92 @@ int bxf_latent_attention(int dtype, const void* q, int64_t ldq, int M, int heads
   if (kv_rank < 1 || rot_dim < 0 || ldq < kv_rank + rot_dim || ldc < kv_rank + rot_dim || ldo < kv_rank || bs < 1 || nb < 1 ||
       nblk < 1 || window < 0 || heads > 65535)
     return BX_EARG;
-  if (kv_rank > LA_MAX_R || kv_rank + rot_dim > 8192) return BX_ELIMIT;
-  if (g_status_seen.load() != 0) return BX_EDEVICE;
+  const PagedAttn a{q, ldq, M, heads, 1, kv_rank + rot_dim, kv_rank, 0, cache, ldc, bs, nb, bt, bt_is64, bt_stride, nblk,
+                    reinterpret_cast<const i64*>(seq), reinterpret_cast<const i64*>(pos), tiles, ntiles, window, sink,
+                    scale, out, heads * ldo, ldo};
+  return run_attention(dtype, a, scratch, scratch_bytes, variant, stream_of(stream));
+}
+
+int bxf_angles(const double* freq, int half, const int64_t* pos, float* cs, int M, void* stream) {
+  if (!freq || !pos || !cs || half < 1 || M < 0) return BX_EARG;
   if (M == 0) return BX_OK;
-  const LatentAttn a{q, ldq, M, heads, kv_rank, rot_dim, cache, ldc, bs, nb, bt, bt_is64, bt_stride, nblk,
-                     reinterpret_cast<const i64*>(seq), reinterpret_cast<const i64*>(pos), tiles, ntiles, window, sink,
-                     scale, out, ldo};
-  if (variant == 2 && !latent_tc_fits(dtype, a)) return BX_ELIMIT;
-  if (variant != 1 && latent_tc_fits(dtype, a) && (!tiles || ntiles > 0))
-    return launch_latent_tc(a, scratch, scratch_bytes, stream_of(stream));
-  const dim3 grid(M, heads);
-  const int smem = (kv_rank + rot_dim) * 4;
-  if (dtype == BXF_F32) fl_latent_attention_kernel<float><<<grid, LA_THREADS, smem, stream_of(stream)>>>(a);
-  else fl_latent_attention_kernel<bf16><<<grid, LA_THREADS, smem, stream_of(stream)>>>(a);
-  return launched(1);
+  const i64 n = (i64)M * half;
+  return launch_chained(fl_angles_kernel, dim3((unsigned)((n + 255) / 256)), 256, 0, stream_of(stream), 0, freq, half,
+                        reinterpret_cast<const i64*>(pos), cs, n);
+}
+
+int bxf_gqa_prepare(int dtype, const bxf_gqa_rows* p, int M, void* stream) {
+  if (!dtype_ok(dtype) || !p || M < 0) return BX_EARG;
+  if (p->heads < 1 || p->kv_heads < 1 || p->heads % p->kv_heads || p->dim < 1 || p->vdim < 1 || p->rot_dims < 0 ||
+      p->rot_dims % 2 || p->rot_dims > p->dim || (p->rot_dims > 0 && !p->cs) || !p->y || !p->slot || !p->q || !p->cache ||
+      p->page < 1)
+    return BX_EARG;
+  const i64 nq = (i64)p->heads * p->dim, nk = (i64)p->kv_heads * p->dim, nv = (i64)p->kv_heads * p->vdim;
+  if (p->ldy < nq + nk + nv || p->ldq < p->dim || p->voff < p->dim || p->ldc < p->voff + p->vdim) return BX_EARG;
+  if (M == 0) return BX_OK;
+  const bool vec = p->dim % 8 == 0 && p->vdim % 8 == 0 && p->rot_dims % 16 == 0 && p->ldy % 8 == 0 && p->ldq % 8 == 0 &&
+                   p->ldc % 8 == 0 && p->voff % 8 == 0 && aligned16(p->y) && aligned16(p->q) && aligned16(p->cache);
+  cudaStream_t st = stream_of(stream);
+  if (dtype == BXF_F32)
+    return launch_chained(fl_gqa_prepare_kernel<float, 1>, dim3(M), PREP_THREADS, 0, st, 0, *p, M);
+  return launch_chained(vec ? fl_gqa_prepare_kernel<bf16, 8> : fl_gqa_prepare_kernel<bf16, 1>, dim3(M), PREP_THREADS, 0, st, 0,
+                        *p, M);
+}
+
+size_t bxf_gqa_attention_scratch(int M, int heads, int kv_heads, int vdim) {
+  return kv_heads < 1 ? 0 : attention_scratch_for(M, kv_heads, heads / kv_heads, vdim);
+}
+
+int bxf_gqa_attention(int dtype, const void* q, int64_t ldq, int M, int heads, int kv_heads, int dim, int vdim,
+                      const void* cache, int64_t ldc, int64_t voff, int bs, int nb, const void* bt, int bt_is64,
+                      int64_t bt_stride, int nblk, const int64_t* seq, const int64_t* pos, const int* tiles, int ntiles,
+                      int window, const float* sink, float scale, void* out, int64_t ldo, void* scratch,
+                      size_t scratch_bytes, int variant, void* stream) {
+  if (!dtype_ok(dtype) || !q || !cache || !bt || !seq || !pos || !out || M < 0 || heads < 1 || kv_heads < 1) return BX_EARG;
+  if (heads % kv_heads || dim < 1 || vdim < 1 || ldq < dim || voff < dim || ldc < voff + vdim ||
+      ldo < (int64_t)heads * vdim || bs < 1 || nb < 1 || nblk < 1 || window < 0)
+    return BX_EARG;
+  const PagedAttn a{q, ldq, M, heads / kv_heads, kv_heads, dim, vdim, (int)voff, cache, ldc, bs, nb, bt, bt_is64, bt_stride,
+                    nblk, reinterpret_cast<const i64*>(seq), reinterpret_cast<const i64*>(pos), tiles, ntiles, window, sink,
+                    scale, out, ldo, vdim};
+  return run_attention(dtype, a, scratch, scratch_bytes, variant, stream_of(stream));
+}
+
+int bxf_streams(int dtype, const bxf_streams_step* p, int M, void* stream) {
+  if (!dtype_ok(dtype) || !p || M < 0 || !p->x || p->streams < 1 || p->streams > BXF_MAX_STREAMS || p->D < 1 || p->D > 32768)
+    return BX_EARG;
+  if ((p->ids && (!p->embed || p->vocab < 1)) || (p->y && (!p->out || !p->mix)) || (p->h && (!p->w || p->ldh < p->D)) ||
+      (!p->h && !p->sum))
+    return BX_EARG;
+  if (M == 0) return BX_OK;
+  const bool vec = p->D % 4 == 0 && (!p->h || p->ldh % 4 == 0);
+  return dtype == BXF_F32 ? launch_streams<float>(*p, M, vec, stream_of(stream)) : launch_streams<bf16>(*p, M, vec, stream_of(stream));
+}
+
+int bxf_causal_conv(int dtype, const bxf_conv* c, void* out, int64_t ldo, int M, void* stream) {
+  if (!dtype_ok(dtype) || !conv_ok(c) || !out || ldo < c->channels || M < 0) return BX_EARG;
+  if (M == 0) return BX_OK;
+  if (ceil_div(M, CONV_ROWS) > 65535) return BX_ELIMIT;
+  const dim3 grid(ceil_div(c->channels, 256), ceil_div(M, CONV_ROWS));
+  if (dtype == BXF_F32)
+    return launch_chained(fl_causal_conv_kernel<float>, grid, 128, 0, stream_of(stream), 0, *c, static_cast<float*>(out), ldo, M);
+  return launch_chained(fl_causal_conv_kernel<bf16>, grid, 128, 0, stream_of(stream), 0, *c, static_cast<bf16*>(out), ldo, M);
+}
+
+int bxf_recurrence(int dtype, const bxf_recurrence_rows* p, int M, void* stream) {
+  if (!dtype_ok(dtype) || !recurrence_ok(p) || M < 0 || (p->conv.w && !conv_ok(&p->conv))) return BX_EARG;
+  if (p->K > BXF_MAX_STATE || p->heads > 65535 || ceil_div(p->V, REC_COLS) > 65535) return BX_ELIMIT;
+  if (M == 0) return BX_OK;
+  return dtype == BXF_F32 ? launch_recurrence<float>(*p, M, stream_of(stream)) : launch_recurrence<bf16>(*p, M, stream_of(stream));
+}
+
+int bxf_gated_norm(int dtype, const bxf_gate_rows* p, int M, void* stream) {
+  if (!dtype_ok(dtype) || !p || M < 0 || !p->o || !p->z || !p->w || !p->out || p->n < 1 || p->parts < 1 || p->n % p->parts ||
+      p->wn < 1 || p->ldo < p->n || p->ldz < p->n || p->ldout < p->n)
+    return BX_EARG;
+  if (p->conv.w && !conv_ok(&p->conv)) return BX_EARG;
+  if (M == 0) return BX_OK;
+  return dtype == BXF_F32 ? launch_gated_norm<float>(*p, M, stream_of(stream)) : launch_gated_norm<bf16>(*p, M, stream_of(stream));
 }
 
 }  // extern "C"

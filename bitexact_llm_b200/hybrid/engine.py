@@ -2,19 +2,21 @@
 `forward` / `logits` / `check`), so `decode.Session`, `generate`, the CUDA-graph decoders and the integer sampler serve
 it unchanged. Logits leave as fixed-point integers at 24 bits, rounded once from the 32-bit accumulators.
 
-The residual stream is float [rows, D]. Caches per layer: pages of latent rows (attention) or one float state per
-sequence (recurrent layers), indexed by the block table and its row number."""
+The residual (`residual.py`) is float: one stream or several. Caches per layer run: pages of rows (attention) or float states
+and convolution inputs per sequence (recurrent layers), indexed by the block table and its row number. A layer that runs
+several times in a row shares its weights and has a cache per run."""
 
 import torch
 
 from .. import _native as nv
 from ..engine_base import TokenRowEngine
 from . import ops
-from .layers import DenseFF, ExpertsFF, LatentAttention, MinGRU, Step
-from .spec import DenseSpec, ExpertsSpec, LatentAttentionSpec, MinGRUSpec
+from .layers import GLA, Attention, DenseFF, ExpertsFF, GatedFF, LatentAttention, Mamba2, MinGRU, Step, Tiles
+from .residual import LayerNormResidual, StreamsResidual
+from .spec import (AttentionSpec, DenseSpec, ExpertsSpec, GatedSpec, GLASpec, LatentAttentionSpec, Mamba2Spec, MinGRUSpec)
 
-MIXERS = {MinGRUSpec: MinGRU, LatentAttentionSpec: LatentAttention}
-FEED_FORWARDS = {DenseSpec: DenseFF, ExpertsSpec: ExpertsFF}
+MIXERS = {MinGRUSpec: MinGRU, LatentAttentionSpec: LatentAttention, AttentionSpec: Attention, Mamba2Spec: Mamba2, GLASpec: GLA}
+FEED_FORWARDS = {DenseSpec: DenseFF, GatedSpec: GatedFF, ExpertsSpec: ExpertsFF}
 
 
 class HybridEngine(TokenRowEngine):
@@ -23,21 +25,26 @@ class HybridEngine(TokenRowEngine):
     tiles_from = 0
 
     def __init__(self, spec, weights, dev="cuda", dtype="bfloat16", n_layers=None):
-        """spec: ModelSpec; weights: {'embed', 'head', 'final': (w, b), 'layers': [{'norm1', 'norm2': (w, b), 'mixer',
-        'ff': dicts of the mechanism}]} as tensors (a design's `read_weights`)."""
+        """spec: ModelSpec; weights: {'embed', 'head', 'final', 'layers': [{'norm1', 'norm2', 'mixer', 'ff': dicts of the
+        mechanism, 'hc1', 'hc2'}]} as tensors (a design's `read_weights`). Norms are (w, b), with streams w around zero;
+        'hc<q>' are the dicts 'in', 'out', 'mix' of a sublayer's streams. n_layers: only the first runs."""
         self.dev, self.spec = torch.device(dev), spec
         self.dtype, _ = ops.DTYPES[dtype]
         self.D, self.V = spec.width, spec.vocab
-        self.L = len(spec.layers) if n_layers is None else n_layers
-        vec = lambda pair: tuple(t.to(self.dev).float().contiguous() for t in pair)
+        runs = (tuple(range(len(spec.layers))) if spec.runs is None else spec.runs)[:n_layers]
+        self.L = len(runs)
+        self.residual = StreamsResidual if spec.streams else LayerNormResidual
+        sub = lambda w, q: self.residual.prepare(w[f"norm{q}"], w.get(f"hc{q}"), self.dev)
         make = lambda table, s, w: None if s is None else table[type(s)](w, s, self.D, self.dtype, self.dev)
         self.embed = weights["embed"].to(self.dev).to(self.dtype).contiguous()
         self.head = ops.pack(weights["head"], self.dtype, self.dev)
-        self.final = vec(weights["final"])
-        self.layers = []
-        for s, w in zip(spec.layers[: self.L], weights["layers"]):
-            self.layers.append((vec(w["norm1"]), make(MIXERS, s.mixer, w["mixer"]),
-                                vec(w["norm2"]) if s.ff is not None else None, make(FEED_FORWARDS, s.ff, w["ff"])))
+        self.final = self.residual.prepare(weights["final"], None, self.dev)
+        made = {}
+        for i in set(runs):
+            s, w = spec.layers[i], weights["layers"][i]
+            made[i] = (sub(w, 1), make(MIXERS, s.mixer, w["mixer"]), sub(w, 2) if s.ff is not None else None,
+                       make(FEED_FORWARDS, s.ff, w["ff"]))
+        self.layers = [made[i] for i in runs]
         counters = max([ff.counters for _, _, _, ff in self.layers if ff is not None], default=0)
         self.counts = torch.zeros(max(1, counters), dtype=torch.int32, device=self.dev)
         self._ln = None
@@ -58,12 +65,10 @@ class HybridEngine(TokenRowEngine):
         return [mixer.new_cache(n_seqs, n_blocks, bs) for _, mixer, _, _ in self.layers]
 
     def tile_table(self, runs, bs):
-        per = [mixer.spec.heads for _, mixer, _, _ in self.layers if isinstance(mixer, LatentAttention)]
-        if not per or self.dtype != torch.bfloat16:
+        if self.dtype != torch.bfloat16:
             return None
-        n = min(nv.float_lib().bxf_latent_attention_tile(h) for h in per)
-        return torch.tensor([[r, t0 + s, min(n, ql - s)] for r, t0, ql, _ in runs for s in range(0, ql, n)],
-                            dtype=torch.int32).reshape(-1, 3)
+        heads = {mixer.tile_heads for _, mixer, _, _ in self.layers if isinstance(mixer, (LatentAttention, Attention))}
+        return Tiles.of(runs, {nv.float_lib().bxf_latent_attention_tile(h) for h in heads})
 
     def forward(self, caches, ids, pos, slot, bt, rmap, tiles=None):
         """ids, pos, slot [N]: the step's tokens (slot < 0: padding, written to page 0); caches: `new_cache`; bt
@@ -73,26 +78,25 @@ class HybridEngine(TokenRowEngine):
         ids, pos, slot, seq = ids.long().contiguous(), pos.long().contiguous(), slot.long().contiguous(), rmap.long().contiguous()
         M = ids.shape[0]
         step = Step(pos, slot, seq, bt, ops.row_flags(seq, slot, pos), tiles)
-        x = torch.empty(M, self.D, dtype=torch.float32, device=self.dev)
-        h = torch.empty(M, ops.pad8(self.D), dtype=self.dtype, device=self.dev)
-        due, start = None, dict(ids=ids, embed=self.embed)
-        for (norm1, mixer, norm2, ff), cache in zip(self.layers, caches):
-            ops.norm(x, *norm1, self.spec.eps, h, experts=due, **start)
-            due, start = None, {}
-            mixer.run(step, h, x, cache)
+        res = self.residual(self, M, ids)
+        for (sub1, mixer, sub2, ff), cache in zip(self.layers, caches):
+            h = res.open(sub1)
+            x, add = res.target()
+            mixer.run(step, h, x, cache, add)
             if ff is not None:
                 counts = self.counts[: ff.counters] if ff.counters else None
-                ops.norm(x, *norm2, self.spec.eps, h, zero=counts)
-                due = ff.run(h, x, counts)
-        if due is not None or start:
-            ops.norm(x, None, None, self.spec.eps, experts=due, **start)
-        return x
+                h = res.open(sub2, counts)
+                x, add = res.target()
+                res.due(ff.run(h, x, counts, add))
+        return res.close()
 
     def _head(self, x, out_type, dtype):
         h = torch.empty(x.shape[0], ops.pad8(self.D), dtype=self.dtype, device=self.dev)
-        ops.norm(x, *self.final, self.spec.eps, h)
+        self.residual.final_norm(x, self.final, self.spec.eps, h)
         out = torch.empty(x.shape[0], self.V, dtype=dtype, device=self.dev)
-        ops.linear(self.head, h, x.shape[0], self.V, self.D, ops.store(out, self.V, self.V, out_type=out_type))
+        scale, cap = self.spec.logit_scale, self.spec.logit_softcap
+        act = ("softcap", scale / cap, cap) if cap else ("none", 0.0, 0.0) if scale == 1.0 else ("scale", scale, 0.0)
+        ops.linear(self.head, h, x.shape[0], self.V, self.D, ops.store(out, self.V, self.V, *act, out_type=out_type))
         return out
 
     def logits(self, x):

@@ -1,12 +1,13 @@
-"""The layer mechanisms of the hybrid float models: mixers (minGRU, latent attention) and feed-forwards (dense, experts).
+"""The layer mechanisms of the hybrid float models: mixers (minGRU, latent attention, grouped-query attention, Mamba-2, gated
+linear attention) and feed-forwards (dense, gated, experts).
 
-A mixer owns its packed weights and the shape of its per-layer cache; `run(step, h, x, cache)` reads the normed rows h
-and adds its output to the residual rows x. A feed-forward's `run(h, x, counts)` does the same and returns what is still
-due to x (the experts' outputs, folded into the next norm) or None. Weights arrive as a dict name -> tensor with the
+A mixer owns its packed weights and the shape of its per-layer cache; `run(step, h, x, cache, add)` reads the normed rows h
+and adds its output to the rows x, or stores it there. A feed-forward's `run(h, x, counts, add)` does the same and returns
+what is still due to x (the experts' outputs, folded into the next norm) or None. Weights arrive as a dict name -> tensor with the
 mechanism's own names ('z', 'dq.norm', 'e0.up', ...)."""
 
 import math
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 
 import torch
 
@@ -22,11 +23,48 @@ class Step:
     seq: torch.Tensor           # int64 [M] block-table row = state slot
     bt: torch.Tensor            # [slots, blocks]
     flags: torch.Tensor         # int32 [M] bxf_row_flags
-    tiles: torch.Tensor = None  # int32 [T, 3] attention tiles of a prompt portion
+    tiles: object = None        # Tiles of a prompt portion
+    turned: dict = field(default_factory=dict)
+
+    def angles(self, freq):
+        """(cos, sin) of every row's position times freq, computed once per step and set of frequencies."""
+        key = freq.data_ptr()
+        if key not in self.turned:
+            self.turned[key] = ops.angles(freq, self.pos)
+        return self.turned[key]
+
+
+class Tiles:
+    """What the tile kernels of a prompt portion walk: attention tiles int32 [T, 3] (table row, first row, rows) by their
+    number of tokens, and the runs int32 [R, 2] (first row, rows) of its sequences."""
+
+    def __init__(self, attention, runs):
+        self.attention, self.runs = attention, runs
+
+    @classmethod
+    def of(cls, runs, sizes):
+        """runs = [(table row, first token row, tokens, context length)], sizes: the tile heights in use."""
+        table = lambda n: torch.tensor([[r, t0 + s, min(n, ql - s)] for r, t0, ql, _ in runs for s in range(0, ql, n)],
+                                       dtype=torch.int32).reshape(-1, 3)
+        return cls({n: table(n) for n in sizes}, torch.tensor([[t0, ql] for _, t0, ql, _ in runs], dtype=torch.int32).reshape(-1, 2))
+
+    def to(self, dev):
+        return Tiles({n: t.to(dev) for n, t in self.attention.items()}, self.runs.to(dev))
+
+    def for_heads(self, heads):
+        return self.attention.get(nv.float_lib().bxf_latent_attention_tile(heads))
 
 
 def _vec(t, dev):
     return t.to(dev).float().contiguous()
+
+
+def _frequencies(base, dims, dev, made={}):
+    """base^(-2 i / dims) in double; layers with the same rotation share the tensor."""
+    key = (base, dims, str(dev))
+    if key not in made:
+        made[key] = torch.tensor([base ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64, device=dev)
+    return made[key]
 
 
 class MinGRU:
@@ -42,9 +80,9 @@ class MinGRU:
     def new_cache(self, n_seqs, n_blocks, bs):
         return torch.zeros(n_seqs, self.spec.width, dtype=torch.float32, device=self.w.device)
 
-    def run(self, step, h, x, cache):
+    def run(self, step, h, x, cache, add=True):
         s = ops.min_gru(self.w, self.bz, self.bx, h, self.spec.width, self.D, cache, step.flags, step.seq)
-        ops.linear(self.o, s, x.shape[0], self.D, self.spec.width, ops.add(x))
+        ops.linear(self.o, s, x.shape[0], self.D, self.spec.width, ops.sublayer_output(x, add))
 
 
 class LatentAttention:
@@ -74,7 +112,11 @@ class LatentAttention:
         return torch.zeros(n_blocks, bs, ops.pad8(self.spec.kv_rank + self.spec.rot_dim), dtype=self.dtype,
                            device=self.first.device)
 
-    def run(self, step, h, x, cache):
+    @property
+    def tile_heads(self):
+        return self.spec.heads
+
+    def run(self, step, h, x, cache, add=True):
         sp, M, dev = self.spec, x.shape[0], x.device
         H, R, dnp = sp.heads, sp.kv_rank, self.dnp
         n1 = self.first.shape[0]
@@ -88,13 +130,132 @@ class LatentAttention:
                    nv.Epilogue(kind=ops.ROPE, n_main=H * dnp, out=qn.data_ptr(), ldo=H * dnp, cs=cs.data_ptr(),
                                rot_out=q.data_ptr() + R * q.element_size(), ldr=H * ldq, hsr=ldq, rot_dim=sp.rot_dim))
         ops.linear(self.uk, qn, M, R, sp.dim, ops.store(q, H * ldq, R, gso=ldq), groups=H, gsw=R * self.uk.shape[2], gsx=dnp)
-        o = ops.latent_attention(q, sp, cache, step.bt, step.seq, step.pos, self.sink, step.tiles)
+        o = ops.latent_attention(q, sp, cache, step.bt, step.seq, step.pos, self.sink,
+                                 step.tiles.for_heads(H) if step.tiles is not None else None)
         og = torch.empty(M, ops.pad8(H * sp.vdim), dtype=self.dtype, device=dev)
         ops.linear(self.uv, o, M, sp.vdim, R,
                    nv.Epilogue(kind=ops.GATE, n_main=sp.vdim, out=og.data_ptr(), ldo=og.shape[1], gso=sp.vdim,
                                gate=gate.data_ptr(), ldg=H),
                    groups=H, gsw=sp.vdim * self.uv.shape[2], ldx=H * o.shape[2], gsx=o.shape[2])
-        ops.linear(self.o, og, M, self.D, H * sp.vdim, ops.add(x))
+        ops.linear(self.o, og, M, self.D, H * sp.vdim, ops.sublayer_output(x, add))
+
+
+class Attention:
+    """Grouped-query attention with rotated halves, a sliding window and a sink per head; queries and keys normed over their
+    whole projections. A token's cache row holds [key | value] of every key/value head."""
+
+    def __init__(self, w, spec, D, dtype, dev):
+        self.spec, self.D, self.dtype = spec, D, dtype
+        if spec.heads % spec.kv_heads or spec.rot_dims % 2 or spec.rot_dims > spec.dim:
+            raise ValueError("attention: heads in equal groups, an even number of rotated entries within a head")
+        self.qkv = ops.pack(torch.cat([w["q"], w["k"], w["v"]]), dtype, dev)
+        biases = [w.get(n + ".b") for n in "qkv"]
+        self.bias = None
+        if any(b is not None for b in biases):
+            self.bias = _vec(torch.cat([torch.zeros(w[n].shape[0]) if b is None else b.float().cpu() for n, b in zip("qkv", biases)]), dev)
+        self.q_norm, self.k_norm, self.sink = (_vec(w[n], dev) if n in w else None for n in ("q.norm", "k.norm", "sink"))
+        self.o = ops.pack(w["o"], dtype, dev)
+        half = spec.rot_dims // 2
+        self.freq = _frequencies(spec.rot_base, spec.rot_dims, dev) if half else None
+
+    @property
+    def tile_heads(self):
+        return self.spec.heads // self.spec.kv_heads
+
+    def new_cache(self, n_seqs, n_blocks, bs):
+        sp = self.spec
+        return torch.zeros(n_blocks, sp.kv_heads, bs, ops.pad8(sp.dim) + ops.pad8(sp.vdim), dtype=self.dtype, device=self.o.device)
+
+    def run(self, step, h, x, cache, add=True):
+        sp, M = self.spec, x.shape[0]
+        n = self.qkv.shape[0]
+        y = torch.empty(M, ops.pad8(n), dtype=self.dtype, device=x.device)
+        ops.linear(self.qkv, h, M, n, self.D, ops.store(y, y.shape[1], n, main_bias=self.bias))
+        cs = step.angles(self.freq) if self.freq is not None else None
+        q = ops.gqa_prepare(y, sp, self.q_norm, self.k_norm, cs, step.slot, cache)
+        o = ops.gqa_attention(q, sp, cache, step.bt, step.seq, step.pos, self.sink,
+                              step.tiles.for_heads(self.tile_heads) if step.tiles is not None else None)
+        ops.linear(self.o, o, M, self.D, sp.heads * sp.vdim, ops.sublayer_output(x, add))
+
+
+class GLA:
+    """Gated linear attention: state [dim, vdim] per head with a decay per key channel, sigmoid(z)^(1 / tau) through a product
+    of low rank; outputs normed per head, gated. State: float [slots, heads, dim, vdim]."""
+
+    def __init__(self, w, spec, D, dtype, dev):
+        self.spec, self.D = spec, D
+        self.first = ops.pack(torch.cat([w["q"], w["k"], w["v"], w["g"], w["a1"]]), dtype, dev)
+        self.rank = w["a1"].shape[0]
+        self.a2, self.a2_b, self.norm = (_vec(w[n], dev) for n in ("a2", "a2.b", "norm"))
+        self.o = ops.pack(w["o"], dtype, dev)
+
+    def new_cache(self, n_seqs, n_blocks, bs):
+        sp = self.spec
+        return torch.zeros(n_seqs, sp.heads, sp.dim, sp.vdim, dtype=torch.float32, device=self.o.device)
+
+    def run(self, step, h, x, cache, add=True):
+        sp, M = self.spec, x.shape[0]
+        nk, nv_ = sp.heads * sp.dim, sp.heads * sp.vdim
+        n = 2 * nk + 2 * nv_
+        y = torch.empty(M, ops.pad8(n), dtype=h.dtype, device=x.device)
+        a1 = torch.empty(M, self.rank, dtype=torch.float32, device=x.device)
+        ops.linear(self.first, h, M, n + self.rank, self.D, ops.store(y, y.shape[1], n, side=a1))
+        o = ops.recurrence(ops.DECAY_CHANNEL, y, a1, cache, step, sp.heads, (0, nk, 2 * nk), a2=self.a2, a2_b=self.a2_b,
+                           inv_tau=1.0 / sp.tau, q_scale=sp.dim ** -0.5)
+        o = ops.gated_norm(o, y[:, 2 * nk + nv_:], nv_, sp.heads, self.norm, sp.eps, gate_first=False)
+        ops.linear(self.o, o, M, self.D, nv_, ops.sublayer_output(x, add))
+
+
+class Mamba2:
+    """Mamba-2: a causal convolution over x, B, C, a state [N, vdim] per head with a scalar decay, gate before the grouped norm.
+    Cache: (state float [slots, heads, N, vdim], the convolution's last inputs T [slots, taps - 1, channels])."""
+
+    def __init__(self, w, spec, D, dtype, dev):
+        self.spec, self.D, self.dtype = spec, D, dtype
+        self.first = ops.pack(w["in"], dtype, dev)
+        self.conv, self.conv_b, self.dt_bias, self.A_log, self.skip, self.norm = (
+            _vec(w[n], dev) for n in ("conv", "conv.b", "dt_bias", "A_log", "D", "norm"))
+        self.o = ops.pack(w["o"], dtype, dev)
+        self.channels = self.conv.shape[0]
+        inner = spec.heads * spec.vdim
+        if self.channels != inner + 2 * spec.groups * spec.state or self.conv.shape[1] != spec.taps or inner % spec.norm_groups:
+            raise ValueError("mamba2: sizes of the convolution or the norm groups do not fit")
+
+    def new_cache(self, n_seqs, n_blocks, bs):
+        sp, dev = self.spec, self.o.device
+        return (torch.zeros(n_seqs, sp.heads, sp.state, sp.vdim, dtype=torch.float32, device=dev),
+                torch.zeros(n_seqs, max(1, sp.taps - 1), self.channels, dtype=self.dtype, device=dev))
+
+    def run(self, step, h, x, cache, add=True):
+        sp, M = self.spec, x.shape[0]
+        inner, gn = sp.heads * sp.vdim, sp.groups * sp.state
+        n = inner + self.channels
+        y = torch.empty(M, ops.pad8(n), dtype=h.dtype, device=x.device)
+        dt = torch.empty(M, sp.heads, dtype=torch.float32, device=x.device)
+        ops.linear(self.first, h, M, n + sp.heads, self.D, ops.store(y, y.shape[1], n, side=dt, bias=self.dt_bias))
+        conv = ops.conv_of(y[:, inner:], self.conv, self.conv_b, cache[1], step)
+        o = ops.recurrence(ops.DECAY_HEAD, y, dt, cache[0], step, sp.groups, (2 * inner + gn, 2 * inner, inner), conv=conv,
+                           A_log=self.A_log, skip=self.skip)
+        o = ops.gated_norm(o, y, inner, sp.norm_groups, self.norm, sp.eps, gate_first=True, conv=conv)
+        ops.linear(self.o, o, M, self.D, inner, ops.sublayer_output(x, add))
+
+
+class GatedFF:
+    """W_down(act(W_gate h) * (W_up h)); the two first products are one, their rows in turn."""
+
+    counters = 0
+
+    def __init__(self, w, spec, D, dtype, dev):
+        self.spec, self.D = spec, D
+        self.first = ops.pack(ops.interleave(w["gate"], w["up"]), dtype, dev)
+        self.down = ops.pack(w["down"], dtype, dev)
+
+    def run(self, h, x, counts, add=True):
+        M, ff = x.shape[0], self.spec.ff
+        a = torch.empty(M, ops.pad8(ff), dtype=h.dtype, device=h.device)
+        ops.linear(self.first, h, M, 2 * ff, self.D, ops.glu(a, self.spec.act))
+        ops.linear(self.down, a, M, self.D, ff, ops.sublayer_output(x, add))
+        return None
 
 
 class DenseFF:
@@ -108,11 +269,11 @@ class DenseFF:
 
     counters = 0
 
-    def run(self, h, x, counts):
+    def run(self, h, x, counts, add=True):
         M, ff = x.shape[0], self.spec.ff
         a = torch.empty(M, ops.pad8(ff), dtype=h.dtype, device=h.device)
         ops.linear(self.up, h, M, ff, self.D, ops.store(a, a.shape[1], ff, self.spec.act, self.p, self.q))
-        ops.linear(self.down, a, M, self.D, ff, ops.add(x))
+        ops.linear(self.down, a, M, self.D, ff, ops.sublayer_output(x, add))
         return None
 
 
@@ -134,7 +295,7 @@ class ExpertsFF:
     def counters(self):
         return self.spec.experts
 
-    def run(self, h, x, counts):
+    def run(self, h, x, counts, add=True):
         sp, M, D, dev = self.spec, x.shape[0], self.D, x.device
         E, fs = sp.experts, sp.shared_ff
         logits = torch.empty(M, E, dtype=torch.float32, device=dev)
@@ -149,5 +310,7 @@ class ExpertsFF:
         ops.linear(self.down, u, M * sp.top, D, sp.ff, ops.store(y, D, D, out_type=ops.OUT_F32), groups=E,
                    gsw=D * self.down.shape[2], counts=counts)
         if fs:
-            ops.linear(self.shared_down, a, M, D, fs, ops.add(x))
+            ops.linear(self.shared_down, a, M, D, fs, ops.sublayer_output(x, add))
+        elif not add:
+            x.zero_()
         return y, place, weight

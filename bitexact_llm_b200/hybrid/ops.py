@@ -10,8 +10,9 @@ import torch
 from .. import _native as nv
 
 DTYPES = {"bfloat16": (torch.bfloat16, 0), "float32": (torch.float32, 1)}
-ACTS = {"none": 0, "relu2": 1, "xielu": 2}
-STORE, ADD, ROPE, GATE = 0, 1, 2, 3
+ACTS = {"none": 0, "relu2": 1, "xielu": 2, "gelu": 3, "softcap": 4, "scale": 5}
+STORE, ADD, ROPE, GATE, GLU = 0, 1, 2, 3, 4
+DECAY_CHANNEL, DECAY_HEAD = 0, 1
 OUT_T, OUT_F32, OUT_I64 = 0, 1, 2
 
 
@@ -37,15 +38,31 @@ def linear(w, x, M, N, K, epi, groups=1, gsw=0, ldx=None, gsx=0, counts=None, ti
     nv.check(rc, "bxf_linear")
 
 
-def store(out, ldo, n, act="none", act_p=0.0, act_q=0.0, out_type=OUT_T, gso=0, side=None, bias=None):
+def store(out, ldo, n, act="none", act_p=0.0, act_q=0.0, out_type=OUT_T, gso=0, side=None, bias=None,
+          main_bias=None):
     """Epilogue of a plain product: channels below n to `out`, the others (with bias) to the float tensor `side`."""
     return nv.Epilogue(kind=STORE, out_type=out_type, act=ACTS[act], n_main=n, act_p=act_p, act_q=act_q,
                        out=out.data_ptr(), ldo=ldo, gso=gso, side=nv.ptr(side), lds=0 if side is None else side.stride(0),
-                       bias=nv.ptr(bias))
+                       bias=nv.ptr(bias), main_bias=nv.ptr(main_bias))
 
 
 def add(x):
     return nv.Epilogue(kind=ADD, out=x.data_ptr(), ldo=x.stride(0))
+
+
+def sublayer_output(x, add_to):
+    """Epilogue of a sublayer's last product: x float [M, D] += it, or x = it."""
+    return add(x) if add_to else store(x, x.stride(0), x.shape[1], out_type=OUT_F32)
+
+
+def glu(out, act):
+    """Epilogue of a product whose rows 2 i and 2 i + 1 are a gate and its value: out[m, i] = act(gate) * value."""
+    return nv.Epilogue(kind=GLU, act=ACTS[act], out=out.data_ptr(), ldo=out.stride(0))
+
+
+def interleave(gate, up):
+    """[N, K] twice -> [2 N, K], a row of each in turn."""
+    return torch.stack([gate, up], 1).reshape(-1, gate.shape[1])
 
 
 def norm(x, w, b, eps, h=None, ids=None, embed=None, experts=None, zero=None):
@@ -142,4 +159,98 @@ def latent_attention(q, spec, cache, bt, seq, pos, sink, tiles=None, variant=0):
                                   0 if tiles is None else tiles.shape[0], spec.window, nv.ptr(sink), spec.scale,
                                   out.data_ptr(), out.shape[2], nv.ptr(scratch), need, variant, nv.stream())
     nv.check(rc, "bxf_latent_attention")
+    return out
+
+
+def streams(x, eps, start=None, update=None, mix_in=None, w=None, h=None, total=None):
+    """Residual streams x float [M, S, D]. start = (ids, embed): every stream is the embedding; update = (y, out, mix): the
+    streams after a sublayer with output y. Then h T [M, pad8(D)] = RMS norm (weight w) of the streams weighted by mix_in,
+    or total float [M, D] = their sum."""
+    M, S, D = x.shape
+    ids, embed = start if start is not None else (None, None)
+    y, out, mix = update if update is not None else (None, None, None)
+    p = nv.StreamsStep(x=x.data_ptr(), ids=nv.ptr(ids), embed=nv.ptr(embed), vocab=0 if embed is None else embed.shape[0],
+                       y=nv.ptr(y), out=nv.ptr(out), mix=nv.ptr(mix), in_=nv.ptr(mix_in), w=nv.ptr(w), h=nv.ptr(h),
+                       ldh=0 if h is None else h.stride(0), sum=nv.ptr(total), eps=eps, streams=S, D=D)
+    t = h if h is not None else embed
+    nv.check(nv.float_lib().bxf_streams(0 if t is None else code(t), ctypes.byref(p), M, nv.stream()), "bxf_streams")
+
+
+def angles(freq, pos):
+    """freq double [half] -> (cos, sin) of pos * freq, float [M, half, 2]."""
+    cs = torch.empty(pos.shape[0], freq.shape[0], 2, dtype=torch.float32, device=pos.device)
+    rc = nv.float_lib().bxf_angles(freq.data_ptr(), freq.shape[0], pos.data_ptr(), cs.data_ptr(), pos.shape[0], nv.stream())
+    nv.check(rc, "bxf_angles")
+    return cs
+
+
+def gqa_prepare(y, spec, q_norm, k_norm, cs, slot, cache):
+    """y T [M, >= q | k | v] -> queries T [kv_heads, M, heads per group, pad8(dim)]; the tokens' cache rows are written."""
+    M, G = y.shape[0], spec.kv_heads
+    q = torch.empty(G, M, spec.heads // G, pad8(spec.dim), dtype=y.dtype, device=y.device)
+    p = nv.GqaRows(y=y.data_ptr(), ldy=y.stride(0), heads=spec.heads, kv_heads=G, dim=spec.dim, vdim=spec.vdim,
+                   rot_dims=spec.rot_dims, page=cache.shape[2], q_norm=nv.ptr(q_norm), k_norm=nv.ptr(k_norm), cs=nv.ptr(cs),
+                   slot=slot.data_ptr(), q=q.data_ptr(), ldq=q.shape[3], cache=cache.data_ptr(), ldc=cache.shape[3],
+                   voff=pad8(spec.dim), eps=spec.eps)
+    nv.check(nv.float_lib().bxf_gqa_prepare(code(y), ctypes.byref(p), M, nv.stream()), "bxf_gqa_prepare")
+    return q
+
+
+def gqa_attention(q, spec, cache, bt, seq, pos, sink, tiles=None, variant=0):
+    """q T [kv_heads, M, heads per group, ldq] against the paged cache T [blocks, kv_heads, bs, ldc] -> T [M, pad8(heads vdim)]."""
+    G, M, per, ldq = q.shape
+    lib, H = nv.float_lib(), spec.heads
+    out = torch.empty(M, pad8(H * spec.vdim), dtype=q.dtype, device=q.device)
+    need = lib.bxf_gqa_attention_scratch(M, H, G, spec.vdim)
+    scratch = torch.empty(need, dtype=torch.uint8, device=q.device) if need else None
+    assert bt.dtype in (torch.int32, torch.int64) and bt.stride(1) == 1 and q.is_contiguous() and cache.is_contiguous()
+    rc = lib.bxf_gqa_attention(code(q), q.data_ptr(), ldq, M, H, G, spec.dim, spec.vdim, cache.data_ptr(), cache.shape[3],
+                               pad8(spec.dim), cache.shape[2], cache.shape[0], bt.data_ptr(), int(bt.dtype == torch.int64),
+                               bt.stride(0), bt.shape[1], seq.data_ptr(), pos.data_ptr(), nv.ptr(tiles),
+                               0 if tiles is None else tiles.shape[0], spec.window, nv.ptr(sink), spec.scale, out.data_ptr(),
+                               out.shape[1], nv.ptr(scratch), need, variant, nv.stream())
+    nv.check(rc, "bxf_gqa_attention")
+    return out
+
+
+def conv_of(u, w, b, state, step):
+    """bxf_conv of inputs u T [M, channels] (a view into wider rows), w float [channels, taps]."""
+    return nv.Conv(u=u.data_ptr(), ldu=u.stride(0), w=w.data_ptr(), b=b.data_ptr(), state=state.data_ptr(),
+                   flags=step.flags.data_ptr(), seq=step.seq.data_ptr(), pos=step.pos.data_ptr(), channels=w.shape[0],
+                   taps=w.shape[1])
+
+
+def causal_conv(conv, M, like):
+    """-> silu(convolution) T [M, pad8(channels)]."""
+    out = torch.empty(M, pad8(conv.channels), dtype=like.dtype, device=like.device)
+    rc = nv.float_lib().bxf_causal_conv(code(like), ctypes.byref(conv), out.data_ptr(), out.stride(0), M, nv.stream())
+    nv.check(rc, "bxf_causal_conv")
+    return out
+
+
+def recurrence(kind, y, side, state, step, groups, columns, conv=None, a2=None, a2_b=None, inv_tau=0.0, q_scale=1.0,
+               A_log=None, skip=None):
+    """state float [slots, heads, K, V] is advanced by the rows of y; columns = where q, k, v begin in y -> outputs T
+    [M, pad8(heads V)]."""
+    M, (_, H, K, V) = y.shape[0], state.shape
+    out = torch.empty(M, pad8(H * V), dtype=y.dtype, device=y.device)
+    p = nv.RecurrenceRows(kind=kind, heads=H, groups=groups, K=K, V=V, rank=0 if a2 is None else a2.shape[1], q0=columns[0],
+                          k0=columns[1], v0=columns[2], y=y.data_ptr(), ldy=y.stride(0), side=side.data_ptr(),
+                          lds=side.stride(0), a2=nv.ptr(a2), a2_b=nv.ptr(a2_b), inv_tau=inv_tau, q_scale=q_scale,
+                          A_log=nv.ptr(A_log), skip=nv.ptr(skip), state=state.data_ptr(), flags=step.flags.data_ptr(),
+                          seq=step.seq.data_ptr(), out=out.data_ptr(), ldo=out.stride(0))
+    if conv is not None:
+        p.conv = conv
+    nv.check(nv.float_lib().bxf_recurrence(code(y), ctypes.byref(p), M, nv.stream()), "bxf_recurrence")
+    return out
+
+
+def gated_norm(o, z, n, parts, w, eps, gate_first, conv=None):
+    """o, z T [M, >= n] -> T [M, pad8(n)]: RMS norm of `parts` equal parts and the gate silu(z), before or after the norm."""
+    out = torch.empty(o.shape[0], pad8(n), dtype=o.dtype, device=o.device)
+    p = nv.GateRows(o=o.data_ptr(), z=z.data_ptr(), ldo=o.stride(0), ldz=z.stride(0), w=w.data_ptr(), out=out.data_ptr(),
+                    ldout=out.stride(0), n=n, parts=parts, wn=w.shape[0], gate_first=int(gate_first), eps=eps)
+    if conv is not None:
+        p.conv = conv
+    nv.check(nv.float_lib().bxf_gated_norm(code(o), ctypes.byref(p), o.shape[0], nv.stream()), "bxf_gated_norm")
     return out

@@ -24,9 +24,49 @@ class LatentAttentionSpec:
 
 
 @dataclass(frozen=True)
+class AttentionSpec:
+    """Grouped-query attention; biases, query / key norms and sinks are there when the weights have them."""
+    heads: int
+    kv_heads: int
+    dim: int                # query / key entries per head
+    vdim: int
+    rot_dims: int           # rotated entries per head (the first ones, halves paired)
+    rot_base: float
+    scale: float
+    window: int             # 0: all before it
+    eps: float              # of the query and key norms
+
+
+@dataclass(frozen=True)
+class Mamba2Spec:
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    taps: int
+    norm_groups: int
+    eps: float              # of the gated norm
+
+
+@dataclass(frozen=True)
+class GLASpec:
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    eps: float              # of the output norm
+
+
+@dataclass(frozen=True)
 class DenseSpec:
     ff: int
     act: str = "xielu"
+
+
+@dataclass(frozen=True)
+class GatedSpec:
+    ff: int
+    act: str = "gelu"
 
 
 @dataclass(frozen=True)
@@ -41,8 +81,8 @@ class ExpertsSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: object           # MinGRUSpec or LatentAttentionSpec
-    ff: object              # DenseSpec, ExpertsSpec or None
+    mixer: object           # MinGRUSpec, LatentAttentionSpec, AttentionSpec, Mamba2Spec or GLASpec
+    ff: object              # DenseSpec, GatedSpec, ExpertsSpec or None
 
 
 @dataclass(frozen=True)
@@ -51,3 +91,7 @@ class ModelSpec:
     width: int
     eps: float
     layers: tuple
+    runs: tuple = None          # the layers in the order they run (a layer may run several times); None: each once
+    streams: int = 0            # residual streams (hyper-connections, RMS norms); 0: one residual, layer norms with bias
+    logit_scale: float = 1.0
+    logit_softcap: float = 0.0  # 0: none

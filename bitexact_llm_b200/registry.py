@@ -2,6 +2,7 @@
 `engine_base`, so the decode loop, the command line and the trace runner treat all of them alike.
 
   Fedatar            hybrid.fedatar   dtype bfloat16 (default) or float32
+  Veredra            hybrid.veredra   dtype bfloat16 (default) or float32
   LlamaForCausalLM   integer engines  dtype exact (default: original bf16 weights as limbs) or int8
 
 A folder holds config.json and model.safetensors; the integer engines also take constants.bx (`constfile`), which
@@ -38,6 +39,13 @@ class FedatarFamily:
         return fedatar.load(cfg, _tensors(folder), dev, dtype)
 
 
+class VeredraFamily(FedatarFamily):
+    @staticmethod
+    def load(folder, cfg, dev, dtype, max_len):
+        from .hybrid import veredra
+        return veredra.load(cfg, _tensors(folder), dev, dtype)
+
+
 class LlamaFamily:
     dtypes, libraries = ("exact", "int8"), ("integer",)
     serving_dtype = "exact"
@@ -62,7 +70,7 @@ class LlamaFamily:
         return IntEngine(c, dev)
 
 
-FAMILIES = {"Fedatar": FedatarFamily, "LlamaForCausalLM": LlamaFamily}
+FAMILIES = {"Fedatar": FedatarFamily, "Veredra": VeredraFamily, "LlamaForCausalLM": LlamaFamily}
 
 
 def read_config(folder):

@@ -21,6 +21,9 @@ extern "C" {
 
 #define BXF_MAX_TOP 32          /* experts per token */
 #define BXF_MAX_EXPERTS 1024
+#define BXF_MAX_STREAMS 8       /* residual streams */
+#define BXF_MAX_TAPS 16         /* of a causal convolution */
+#define BXF_MAX_STATE 512       /* key channels of a matrix-valued recurrent state */
 
 /* Row flags (bxf_row_flags): first / last row of its sequence in this step, first token of the sequence, padding. */
 #define BXF_ROW_FIRST 1
@@ -29,10 +32,11 @@ extern "C" {
 #define BXF_ROW_PAD 8
 
 /* What a product does with its accumulators. */
-#define BXF_EPI_STORE 0         /* out[m, n] = act(acc); rows n >= n_main go to side[m, n - n_main] = acc + bias (float) */
+#define BXF_EPI_STORE 0         /* out[m, n] = act(acc + main_bias[n]); rows n >= n_main go to side[m, n - n_main] = acc + bias (float) */
 #define BXF_EPI_ADD 1           /* out (float) [m, n] += acc */
 #define BXF_EPI_ROPE 2          /* n < n_main: out[m, n] = acc; the others are rotated pairs, see rot_* */
 #define BXF_EPI_GATE 3          /* out[m, n] = acc * gate[m, group] */
+#define BXF_EPI_GLU 4           /* rows 2 i and 2 i + 1 are a pair: out (T) [m, i] = act(acc[2 i]) * acc[2 i + 1]; N even */
 
 #define BXF_OUT_T 0
 #define BXF_OUT_F32 1
@@ -41,6 +45,9 @@ extern "C" {
 #define BXF_ACT_NONE 0
 #define BXF_ACT_RELU2 1         /* max(z, 0)^2 */
 #define BXF_ACT_XIELU 2         /* z > 0: act_p z^2 + z / 2; else act_q (e^z - 1 - z) + z / 2 */
+#define BXF_ACT_GELU 3          /* tanh form */
+#define BXF_ACT_SOFTCAP 4       /* act_q tanh(act_p z) */
+#define BXF_ACT_SCALE 5         /* act_p z */
 
 typedef struct {
   int kind, out_type, act, n_main;
@@ -57,6 +64,7 @@ typedef struct {
   int64_t ldr, hsr;
   int rot_dim;
   int pad_;
+  const float* main_bias;       /* BXF_EPI_STORE: [n_main] or NULL */
 } bxf_epilogue;
 
 /* The recurrence of a minGRU layer after its three products (update, candidate, output gate). */
@@ -68,6 +76,102 @@ typedef struct {
   void* out;                    /* T [M, ldo]: state * silu(gate) */
   int64_t ldo;
 } bxf_gru;
+
+/* Residual streams x float [M, streams, D] (hyper-connections). In this order: ids != NULL: every stream = embed[ids]; else,
+ * with y (a sublayer's output, float [M, D]), x_t = sum_s mix[s, t] x_s + out[t] y. Then u = sum_s in[s] x_s (in NULL: the plain
+ * sum) goes to h (T [M, ldh]) as u / sqrt(mean(u^2) + eps) * w and, with sum, to sum float [M, D]. Without h the streams
+ * themselves are left as they were. */
+typedef struct {
+  float* x;
+  const int64_t* ids;
+  const void* embed;            /* T [vocab, D] */
+  int64_t vocab;
+  const float *y, *out, *mix;   /* mix [streams, streams] = [from, to] */
+  const float* in;
+  const float* w;               /* [D] */
+  void* h;
+  int64_t ldh;
+  float* sum;
+  float eps;
+  int streams, D, pad_;
+} bxf_streams_step;
+
+/* After the projection of a grouped-query attention layer, y T [M, ldy] = [q: heads dim | k: kv_heads dim | v: kv_heads vdim]:
+ * q and k each divided by the root mean square of all their rows (times q_norm / k_norm; NULL: no norm), the first rot_dims
+ * entries of every head turned by cs (entry i with i + rot_dims / 2), q to T [kv_heads, M, heads / kv_heads, ldq], k and v to
+ * the cache row of the token's slot: T [pages, kv_heads, page, ldc] with the value from entry voff on. */
+typedef struct {
+  const void* y;
+  int64_t ldy;
+  int heads, kv_heads, dim, vdim, rot_dims, page;
+  const float *q_norm, *k_norm; /* [heads dim], [kv_heads dim] */
+  const float* cs;              /* bxf_angles */
+  const int64_t* slot;          /* [M]; negative: row 0 */
+  void* q;
+  int64_t ldq;
+  void* cache;
+  int64_t ldc, voff;
+  float eps;
+  int pad_;
+} bxf_gqa_rows;
+
+/* A causal convolution per channel over the rows of a sequence, followed by silu: c[m, ch] = silu(b[ch] + sum_j w[ch, j]
+ * u[m - taps + 1 + j, ch]); rows before the step come from the sequence's state (its last taps - 1 inputs, oldest first),
+ * rows before the sequence are zero. */
+typedef struct {
+  const void* u;                /* T [M, ldu] */
+  int64_t ldu;
+  const float *w, *b;           /* [channels, taps], [channels] */
+  void* state;                  /* T [slots, taps - 1, channels] */
+  const int* flags;             /* [M] row flags */
+  const int64_t *seq, *pos;     /* [M] */
+  int channels, taps;
+} bxf_conv;
+
+#define BXF_DECAY_CHANNEL 0     /* one decay per key channel */
+#define BXF_DECAY_HEAD 1        /* one decay per head */
+
+/* Linear recurrence with a matrix state per head: S_t = diag(a_t) S_(t-1) + k_t v_t^T (K x V), o_t = S_t^T q_t.
+ * q, k, v are columns of y (T [M, ldy]) from q0, k0, v0 on: q and k by group (K entries each; head h uses group
+ * h / (heads / groups)), v by head.
+ *   BXF_DECAY_CHANNEL (groups = heads): side float [M, lds] holds `rank` entries; z = a2 side + a2_b (a2 float [heads K, rank]),
+ *     a = sigmoid(z)^inv_tau; q is multiplied by q_scale.
+ *   BXF_DECAY_HEAD: side float [M, lds] holds the step sizes before softplus; dt = softplus(side), a = exp(-exp(A_log) dt),
+ *     k is multiplied by dt, and skip[h] v_t is added to o_t.
+ * conv.w != NULL: y's columns are the inputs of a causal convolution with silu and q, k, v its results (conv.u = column 0 of
+ * q0, k0, v0; its state is read only, see bxf_gated_norm). With chunks the columns must be convolved already.
+ * state float [slots, heads, K, V] is advanced by the rows of every sequence; out T [M, ldo] = o (heads concatenated). */
+typedef struct {
+  int kind, heads, groups, K, V, rank, q0, k0, v0, pad_;
+  const void* y;
+  int64_t ldy;
+  const float* side;
+  int64_t lds;
+  const float *a2, *a2_b;
+  float inv_tau, q_scale;
+  const float *A_log, *skip;
+  bxf_conv conv;
+  float* state;
+  const int* flags;
+  const int64_t* seq;
+  void* out;
+  int64_t ldo;
+} bxf_recurrence_rows;
+
+/* Gate and norm of a recurrent layer's output o (T [M, ldo], n entries in `parts` equal parts), z T [M, ldz]:
+ * gate_first: out = rms(o silu(z)) w, else out = rms(o) w silu(z); every part by its own root mean square, w float [wn] used
+ * periodically. With conv.w the convolution's state is advanced over the rows of the step. */
+typedef struct {
+  const void *o, *z;
+  int64_t ldo, ldz;
+  const float* w;
+  void* out;
+  int64_t ldout;
+  int n, parts, wn, gate_first;
+  float eps;
+  int pad_;
+  bxf_conv conv;
+} bxf_gate_rows;
 
 int bxf_version(void);
 long long bxf_launch_count(void);
@@ -139,6 +243,25 @@ int bxf_latent_attention(int dtype, const void* q, int64_t ldq, int M, int heads
                          int nblk, const int64_t* seq, const int64_t* pos, const int* tiles, int ntiles, int window,
                          const float* sink, float scale, void* out, int64_t ldo, void* scratch, size_t scratch_bytes,
                          int variant, void* stream);
+
+/* cs float [M, half, 2] = (cos, sin) of pos * freq[i] (freq double [half], angles reduced in double). */
+int bxf_angles(const double* freq, int half, const int64_t* pos, float* cs, int M, void* stream);
+int bxf_gqa_prepare(int dtype, const bxf_gqa_rows* rows, int M, void* stream);
+
+/* Grouped-query attention over a paged cache of [key | value] rows (T [nb, kv_heads, bs, ldc], value from entry voff on, a
+ * multiple of 8 in bf16), otherwise like bxf_latent_attention. q T [kv_heads, M, heads / kv_heads, ldq]; out T [M, ldo] =
+ * heads concatenated; tiles as above with bxf_latent_attention_tile(heads / kv_heads) rows. */
+size_t bxf_gqa_attention_scratch(int M, int heads, int kv_heads, int vdim);
+int bxf_gqa_attention(int dtype, const void* q, int64_t ldq, int M, int heads, int kv_heads, int dim, int vdim,
+                      const void* cache, int64_t ldc, int64_t voff, int bs, int nb, const void* bt, int bt_is64,
+                      int64_t bt_stride, int nblk, const int64_t* seq, const int64_t* pos, const int* tiles, int ntiles,
+                      int window, const float* sink, float scale, void* out, int64_t ldo, void* scratch,
+                      size_t scratch_bytes, int variant, void* stream);
+
+int bxf_streams(int dtype, const bxf_streams_step* step, int M, void* stream);
+int bxf_causal_conv(int dtype, const bxf_conv* conv, void* out, int64_t ldo, int M, void* stream);
+int bxf_recurrence(int dtype, const bxf_recurrence_rows* rows, int M, void* stream);
+int bxf_gated_norm(int dtype, const bxf_gate_rows* rows, int M, void* stream);
 
 #ifdef __cplusplus
 }

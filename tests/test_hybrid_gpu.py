@@ -369,7 +369,7 @@ def test_latent_attention_layer(name, layer, dtype):
         for k in cuts:
             st = steps(dtype, [(0, at, k)], 16, 12, 1)
             tt = eng.tile_table([(0, 0, k, at + k)], 16)
-            st.tiles = None if tt is None or k == 1 else tt.cuda()
+            st.tiles = None if tt is None or k == 1 else tt.to("cuda")
             mixer.run(st, packed(h[at:at + k], dtype), x[at:at + k], cache)
             at += k
         close(x.cpu(), want, dtype)
