@@ -2,7 +2,7 @@
 """Benchmark of the exact-mode decode path: random-init Llama-3.2-1B, 512-token prompts, batched decode.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--repeats R] [--batch B] [--prompt P] [--mode exact|int8]
-                    [--impl reference] [--workload llama|hybrid]
+                    [--impl reference] [--workload llama|hybrid|veredra]
 
 `--workload hybrid` measures the hybrid float models beside the integer Llama instead (bench_hybrid.py). Otherwise:
 A step is one decode step of the whole batch: 16 layers (4 limb GEMMs, RoPE/KV store, paged attention, attention
@@ -48,7 +48,7 @@ def parse():
     ap.add_argument("--mode", default="exact", choices=["exact", "int8"],
                     help="exact: original bf16 weights as 3 limbs (the headline); int8: int8 weights, 2-limb activations")
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
-    ap.add_argument("--workload", default="llama", choices=["llama", "hybrid"],
+    ap.add_argument("--workload", default="llama", choices=["llama", "hybrid", "veredra"],
                     help="hybrid: prefill and decode throughput of the hybrid float models beside the integer Llama")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-int8-extra", action="store_true", help="skip the int8-mode pass reported under `extra`")
@@ -733,7 +733,7 @@ def main():
     if args.impl == "reference":
         run_reference(args, rank)
         return
-    if args.workload == "hybrid":
+    if args.workload in ("hybrid", "veredra"):
         import bench_hybrid
         if rank == 0:
             bench_hybrid.run(args)

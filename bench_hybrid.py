@@ -1,10 +1,11 @@
-"""Throughput of the hybrid float models beside the framework's closest existing one: `python bench.py --workload hybrid`.
+"""Throughput of the hybrid float models: Fedatar beside the integer Llama, `python bench.py --workload hybrid`, and Veredra
+beside Fedatar, `python bench.py --workload veredra`.
 
 Three sizes that resemble a real model's layers (random weights): 16 layers of width 2048 and of width 1024, 4 layers of
 width 4096; minGRU and latent-attention layers alternate, the first feed-forward is dense, the others have 8 experts (two
 per token) and a shared one, sized so that a token's active weights per layer are those of a Llama layer of that width
-(three matrices of 4 x width; at 4096 the integer kernels' limit, 14336). The closest existing model is the integer Llama of the same width, depth and vocabulary,
-in exact mode and in int8 mode. Prompts: 4 x 2048 tokens through `Session.prefill`; decoding: batches of 1, 16 and 256
+(three matrices of 4 x width; at 4096 the integer kernels' limit, 14336). Beside it the integer Llama of the same width, depth
+and vocabulary, in exact mode and in int8 mode. Veredra: `veredra_config` (a gated feed-forward of the same weights). Prompts: 4 x 2048 tokens through `Session.prefill`; decoding: batches of 1, 16 and 256
 after 512-token prompts, the whole step (forward, head, sampler at T = 0.7) replayed from one CUDA graph.
 Every number is device time from CUDA events after warm-up; the weights exceed L2. One JSON line per model and size."""
 
@@ -87,6 +88,74 @@ def random_weights(cfg, dev, seed=0):
     return t
 
 
+def veredra_config(width, layers, vocab=VOCAB):
+    """Gated linear attention, attention and Mamba-2 in turn, two streams, no layer repeated; a gated feed-forward of 4 x width."""
+    mixers = [("gla", {"heads": max(1, width // 256), "dim": 128, "vdim": 256, "tau": 16.0}),
+              ("attention", {"heads": width // 128, "kv_heads": width // 512, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                             "rot": {"base": 1e6, "dims": 128}, "mask": {"size": 1024}}),
+              ("mamba2", {"heads": width // 32, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8})]
+    out = [{"type": mixers[i % 3][0], "mixer": mixers[i % 3][1], "mlp": {"kind": "dense", "ff": 4 * width}} for i in range(layers)]
+    return {"architecture": "Veredra", "vocab": vocab, "width": width, "streams": 2, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
+            "logit_softcap": 30.0, "loop": None, "layers": out}
+
+
+def veredra_weights(cfg, dev, seed=0):
+    """bf16 tensors under the design's names, generated on the device."""
+    import torch
+    g = torch.Generator(device=dev).manual_seed(seed)
+    D, S, t = cfg["width"], cfg["streams"], {}
+
+    def mat(name, n, k):
+        t[name] = (torch.randn(n, k, generator=g, device=dev) * k ** -0.5).to(torch.bfloat16)
+
+    def vec(name, n, mean=0.0):
+        t[name] = (mean + 0.1 * torch.randn(n, generator=g, device=dev)).to(torch.bfloat16)
+
+    mat("embed", cfg["vocab"], D)
+    mat("head", cfg["vocab"], D)
+    vec("final.norm", D)
+    for i, ly in enumerate(cfg["layers"]):
+        p, m, ff = f"l{i}.", ly["mixer"], ly["mlp"]["ff"]
+        for q in (1, 2):
+            vec(f"{p}norm{q}", D)
+            vec(f"{p}hc{q}.in", S, 1.0 / S)
+            vec(f"{p}hc{q}.out", S, 0.7)
+            t[f"{p}hc{q}.mix"] = torch.eye(S, device=dev).to(torch.bfloat16)
+        for n, a, b in (("gate", ff, D), ("up", ff, D), ("down", D, ff)):
+            mat(f"{p}mlp.{n}", a, b)
+        p += "mix."
+        H = m["heads"]
+        if ly["type"] == "attention":
+            for n, rows in (("q", H * m["dim"]), ("k", m["kv_heads"] * m["dim"]), ("v", m["kv_heads"] * m["vdim"])):
+                mat(p + n, rows, D)
+                vec(f"{p}{n}.b", rows)
+                if n != "v":
+                    vec(f"{p}{n}.norm", rows, 1.0)
+            vec(p + "sink", H)
+            mat(p + "o", D, H * m["vdim"])
+        elif ly["type"] == "gla":
+            nk, nv = H * m["dim"], H * m["vdim"]
+            for n, rows, k in (("q", nk, D), ("k", nk, D), ("v", nv, D), ("g", nv, D), ("a1", 16, D), ("a2", nk, 16)):
+                mat(p + n, rows, k)
+            vec(p + "a2.b", nk, 2.0)
+            vec(p + "norm", m["vdim"], 1.0)
+            mat(p + "o", D, nv)
+        else:
+            inner, bc = H * m["vdim"], 2 * m["groups"] * m["state"]
+            mat(p + "in", 2 * inner + bc + H, D)
+            mat(p + "conv", inner + bc, m["conv"])
+            for n, size, mean in (("conv.b", inner + bc, 0.0), ("dt_bias", H, -3.0), ("A_log", H, 0.0), ("D", H, 1.0), ("norm", inner, 1.0)):
+                vec(p + n, size, mean)
+            mat(p + "o", D, inner)
+    return t
+
+
+def veredra_engine(width, layers, dev="cuda"):
+    from bitexact_llm_b200.hybrid import veredra
+    cfg = veredra_config(width, layers)
+    return veredra.load(cfg, veredra_weights(cfg, dev), dev, "bfloat16")
+
+
 def hybrid_engine(width, layers, dev="cuda"):
     from bitexact_llm_b200.hybrid import fedatar
     cfg = hybrid_config(width, layers)
@@ -158,13 +227,14 @@ def run(args):
     for target in build.TARGETS:
         build.build(target=target)
     for name, (width, layers) in SIZES.items():
-        for model, make in (("Fedatar bf16", lambda: hybrid_engine(width, layers)),
-                            ("Llama exact", lambda: llama_engine(width, layers, "exact")),
-                            ("Llama int8", lambda: llama_engine(width, layers, "int8"))):
+        models = {"Veredra bf16": lambda: veredra_engine(width, layers), "Fedatar bf16": lambda: hybrid_engine(width, layers),
+                  "Llama exact": lambda: llama_engine(width, layers, "exact"),
+                  "Llama int8": lambda: llama_engine(width, layers, "int8")}
+        for model, make in list(models.items())[:2] if args.workload == "veredra" else list(models.items())[1:]:
             eng = make()
             torch.cuda.empty_cache()
             r = measure(eng, args.steps, args.warmup)
-            print(json.dumps({"workload": "hybrid", "size": name, "width": width, "layers": layers, "model": model,
+            print(json.dumps({"workload": args.workload, "size": name, "width": width, "layers": layers, "model": model,
                               "data": "synthetic", **r}), flush=True)
             del eng
             torch.cuda.empty_cache()

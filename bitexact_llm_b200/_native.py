@@ -157,6 +157,9 @@ _FLOAT_SIGNATURES = {
     "bxf_streams": (I, [I, ctypes.POINTER(StreamsStep), I, P]),
     "bxf_causal_conv": (I, [I, ctypes.POINTER(Conv), P, L, I, P]),
     "bxf_recurrence": (I, [I, ctypes.POINTER(RecurrenceRows), I, P]),
+    "bxf_recurrence_chunk_rows": (I, [I, I, I]),
+    "bxf_recurrence_chunk_scratch": (Z, [I, I, I, I, I]),
+    "bxf_recurrence_chunks": (I, [I, ctypes.POINTER(RecurrenceRows), P, I, P, I, P, Z, I, P]),
     "bxf_gated_norm": (I, [I, ctypes.POINTER(GateRows), I, P]),
 }
 

@@ -30,14 +30,66 @@ __device__ __forceinline__ float conv_at(const bxf_conv& c, int m, int ch) {
   return silu<T>(acc);
 }
 
-constexpr int CONV_ROWS = 16;
+constexpr int CONV_ROWS = 16, CONV_THREADS = 128;
+
+// Prompts: a thread walks CONV_ROWS rows of 8 channels with the last TAPS inputs in registers.
+template <int TAPS>
+__global__ void __launch_bounds__(CONV_THREADS) fl_causal_conv_rows_kernel(const bxf_conv c, bf16* __restrict__ out, i64 ldo, int M) {
+  launch_next();
+  const int ch = (blockIdx.x * CONV_THREADS + threadIdx.x) * 8;
+  if (ch >= c.channels) return;
+  float w[TAPS][8], b[8], win[TAPS][8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    b[i] = c.b[ch + i];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j][i] = c.w[(ch + i) * TAPS + j];
+  }
+  wait_previous();
+  const int m0 = blockIdx.y * CONV_ROWS, m1 = min(M, m0 + CONV_ROWS);
+  const bf16* u = static_cast<const bf16*>(c.u) + ch;
+  for (int m = m0; m < m1; ++m) {
+    const int f = c.flags[m];
+    if (f & BXF_ROW_PAD) continue;
+    if (m == m0 || (f & BXF_ROW_FIRST)) {                // the inputs before this row: rows of the step, the state, zeros
+      int first = (f & BXF_ROW_FIRST) ? 0 : -1;
+#pragma unroll
+      for (int back = 1; back < TAPS; ++back) {
+        float (&v)[8] = win[TAPS - 1 - back];
+        if (back > c.pos[m]) {
+#pragma unroll
+          for (int i = 0; i < 8; ++i) v[i] = 0.0f;
+        } else if (first < 0) {
+          load_v<8>(u + (i64)(m - back) * c.ldu, v);
+          if (c.flags[m - back] & BXF_ROW_FIRST) first = back;
+        } else {
+          load_v<8>(static_cast<const bf16*>(c.state) + (c.seq[m] * (TAPS - 1) + first - back + TAPS - 1) * c.channels + ch, v);
+        }
+      }
+    }
+    load_v<8>(u + (i64)m * c.ldu, win[TAPS - 1]);
+    float o[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      o[i] = b[i];
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) o[i] = fmaf(w[j][i], win[j][i], o[i]);
+      o[i] = silu<bf16>(o[i]);
+    }
+    store_v<8>(out + m * ldo + ch, o);
+#pragma unroll
+    for (int j = 0; j + 1 < TAPS; ++j)
+#pragma unroll
+      for (int i = 0; i < 8; ++i) win[j][i] = win[j + 1][i];
+  }
+}
 
 template <class T>
-__global__ void __launch_bounds__(128) fl_causal_conv_kernel(const bxf_conv c, T* __restrict__ out, i64 ldo, int M) {
+__global__ void __launch_bounds__(CONV_THREADS) fl_causal_conv_kernel(const bxf_conv c, T* __restrict__ out, i64 ldo, int M) {
   launch_next();
   wait_previous();
   for (int k = 0; k < 2; ++k) {
-    const int ch = blockIdx.x * 256 + k * 128 + threadIdx.x;
+    const int ch = blockIdx.x * 2 * CONV_THREADS + k * CONV_THREADS + threadIdx.x;
     if (ch >= c.channels) return;
     for (int m = blockIdx.y * CONV_ROWS; m < min(M, (int)(blockIdx.y + 1) * CONV_ROWS); ++m)
       if (!(c.flags[m] & BXF_ROW_PAD)) st(out + m * ldo + ch, conv_at<T>(c, m, ch));

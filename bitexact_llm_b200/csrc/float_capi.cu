@@ -10,7 +10,7 @@
 #include "fl_attention_tc.cuh"
 #include "fl_gemm.cuh"
 #include "fl_gemm_simt.cuh"
-#include "fl_recurrence.cuh"
+#include "fl_recurrence_chunks.cuh"
 #include "fl_stages.cuh"
 #include "fl_streams.cuh"
 
@@ -18,7 +18,10 @@ namespace {
 
 using namespace bxf;
 
-static_assert(sizeof(bxf_epilogue) == 136 && sizeof(bxf_gru) == 56, "layouts of the callers' structs");
+static_assert(sizeof(bxf_epilogue) == 136 && sizeof(bxf_gru) == 56 && sizeof(bxf_streams_step) == 112 &&
+                  sizeof(bxf_gqa_rows) == 120 && sizeof(bxf_conv) == 72 && sizeof(bxf_recurrence_rows) == 224 &&
+                  sizeof(bxf_gate_rows) == 152,
+              "layouts of the callers' structs");
 
 inline cudaStream_t stream_of(void* s) { return static_cast<cudaStream_t>(s); }
 inline bool dtype_ok(int d) { return d == BXF_BF16 || d == BXF_F32; }
@@ -359,6 +362,45 @@ int launch_recurrence(const bxf_recurrence_rows& p, int M, cudaStream_t st) {
   return p.kind == BXF_DECAY_CHANNEL ? go(std::true_type{}) : go(std::false_type{});
 }
 
+// The chunk kernel takes bf16 rows whose key and value sizes are multiples of 8.
+bool chunks_fit(int dtype, int K, int V) { return dtype == BXF_BF16 && K % 8 == 0 && V % 8 == 0 && K <= RC_MAX_K; }
+
+struct ChunkScratch {
+  size_t planes, edge, masks, bytes;
+};
+
+ChunkScratch chunk_scratch(int M, int chunks, int heads, int K) {
+  const auto up = [](size_t n) { return (n + 255) / 256 * 256; };
+  ChunkScratch s;
+  s.planes = up((size_t)4 * M * heads * K * 2);
+  s.edge = up((size_t)M * heads * K * 4);
+  s.masks = up((size_t)chunks * heads * 8);
+  s.bytes = s.planes + s.edge + s.masks;
+  return s;
+}
+
+template <bool CHANNEL, int KT, int NW>
+int launch_chunks_as(const bxf_recurrence_rows& p, const ChunkArgs& a, int nruns, cudaStream_t st) {
+  using Cfg = ChunkCfg<CHANNEL, KT, NW>;
+  static PerDevice configured;
+  if (once_per_device(configured, [] {
+        return cudaFuncSetAttribute(fl_recurrence_chunk_kernel<CHANNEL, KT, NW>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                    Cfg::SMEM);
+      }) != BX_OK)
+    return BX_ELAUNCH;
+  return launch_chained(fl_recurrence_chunk_kernel<CHANNEL, KT, NW>, dim3(nruns, p.heads, ceil_div(p.V, Cfg::VS)), 32 * NW,
+                        Cfg::SMEM, st, 0, p, a);
+}
+
+template <bool CHANNEL>
+int launch_chunks(const bxf_recurrence_rows& p, const ChunkArgs& a, int nruns, cudaStream_t st) {
+  const int kt = ceil_div(p.K, 16);
+  if (kt <= 2) return launch_chunks_as<CHANNEL, 2, 4>(p, a, nruns, st);
+  if (kt <= 4) return launch_chunks_as<CHANNEL, 4, 4>(p, a, nruns, st);
+  if (kt <= 8) return launch_chunks_as<CHANNEL, 8, 4>(p, a, nruns, st);
+  return launch_chunks_as<CHANNEL, 16, 4>(p, a, nruns, st);
+}
+
 template <class T>
 int launch_gated_norm(const bxf_gate_rows& p, int M, cudaStream_t st) {
   const int size = p.n / p.parts;
@@ -591,10 +633,18 @@ int bxf_causal_conv(int dtype, const bxf_conv* c, void* out, int64_t ldo, int M,
   if (!dtype_ok(dtype) || !conv_ok(c) || !out || ldo < c->channels || M < 0) return BX_EARG;
   if (M == 0) return BX_OK;
   if (ceil_div(M, CONV_ROWS) > 65535) return BX_ELIMIT;
-  const dim3 grid(ceil_div(c->channels, 256), ceil_div(M, CONV_ROWS));
+  const dim3 grid(ceil_div(c->channels, 2 * CONV_THREADS), ceil_div(M, CONV_ROWS));
+  cudaStream_t st = stream_of(stream);
   if (dtype == BXF_F32)
-    return launch_chained(fl_causal_conv_kernel<float>, grid, 128, 0, stream_of(stream), 0, *c, static_cast<float*>(out), ldo, M);
-  return launch_chained(fl_causal_conv_kernel<bf16>, grid, 128, 0, stream_of(stream), 0, *c, static_cast<bf16*>(out), ldo, M);
+    return launch_chained(fl_causal_conv_kernel<float>, grid, CONV_THREADS, 0, st, 0, *c, static_cast<float*>(out), ldo, M);
+  if (c->taps >= 2 && c->taps <= 4 && c->channels % 8 == 0 && c->ldu % 8 == 0 && ldo % 8 == 0 && aligned16(c->u) &&
+      aligned16(out) && aligned16(c->state)) {
+    const dim3 wide(ceil_div(c->channels, 8 * CONV_THREADS), ceil_div(M, CONV_ROWS));
+    return launch_chained(c->taps == 2 ? fl_causal_conv_rows_kernel<2> : c->taps == 3 ? fl_causal_conv_rows_kernel<3>
+                                                                                      : fl_causal_conv_rows_kernel<4>,
+                          wide, CONV_THREADS, 0, st, 0, *c, static_cast<bf16*>(out), ldo, M);
+  }
+  return launch_chained(fl_causal_conv_kernel<bf16>, grid, CONV_THREADS, 0, st, 0, *c, static_cast<bf16*>(out), ldo, M);
 }
 
 int bxf_recurrence(int dtype, const bxf_recurrence_rows* p, int M, void* stream) {
@@ -602,6 +652,43 @@ int bxf_recurrence(int dtype, const bxf_recurrence_rows* p, int M, void* stream)
   if (p->K > BXF_MAX_STATE || p->heads > 65535 || ceil_div(p->V, REC_COLS) > 65535) return BX_ELIMIT;
   if (M == 0) return BX_OK;
   return dtype == BXF_F32 ? launch_recurrence<float>(*p, M, stream_of(stream)) : launch_recurrence<bf16>(*p, M, stream_of(stream));
+}
+
+int bxf_recurrence_chunk_rows(int dtype, int K, int V) { return chunks_fit(dtype, K, V) ? RC_ROWS : 0; }
+
+size_t bxf_recurrence_chunk_scratch(int kind, int M, int chunks, int heads, int K) {
+  return kind == BXF_DECAY_CHANNEL && M > 0 && chunks > 0 && heads > 0 && K > 0 ? chunk_scratch(M, chunks, heads, K).bytes : 0;
+}
+
+int bxf_recurrence_chunks(int dtype, const bxf_recurrence_rows* p, const int* runs, int nruns, const int* chunks, int nchunks,
+                          void* scratch, size_t scratch_bytes, int M, void* stream) {
+  if (!recurrence_ok(p) || p->conv.w || M < 0 || !runs || !chunks || nruns < 0 || nchunks < nruns) return BX_EARG;
+  if (!chunks_fit(dtype, p->K, p->V) || p->heads > 65535) return BX_ELIMIT;
+  if (p->ldy % 8 || p->q0 % 8 || p->k0 % 8 || p->v0 % 8 || p->ldo % 2 || !aligned16(p->y)) return BX_EARG;
+  if (M == 0 || nruns == 0) return BX_OK;
+  cudaStream_t st = stream_of(stream);
+  ChunkArgs a{runs, nullptr, nullptr, nullptr, M};
+  if (p->kind == BXF_DECAY_HEAD) return launch_chunks<false>(*p, a, nruns, st);
+  const ChunkScratch s = chunk_scratch(M, nchunks, p->heads, p->K);
+  if (!scratch || !aligned16(scratch) || scratch_bytes < s.bytes) return BX_EARG;
+  const int smem = decay_prepare_smem(p->K, p->rank);
+  if (smem > 200 * 1024) return BX_ELIMIT;
+  static PerDevice configured;
+  if (once_per_device(configured, [] {
+        return cudaFuncSetAttribute(fl_decay_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+      }) != BX_OK)
+    return BX_ELAUNCH;
+  uint8_t* base = static_cast<uint8_t*>(scratch);
+  bf16* planes = reinterpret_cast<bf16*>(base);
+  float* edge = reinterpret_cast<float*>(base + s.planes);
+  unsigned long long* masks = reinterpret_cast<unsigned long long*>(base + s.planes + s.edge);
+  const int rc = launch_chained(fl_decay_prepare_kernel, dim3(nchunks, p->heads), RP_THREADS, smem, st, 0, *p, chunks, planes, edge,
+                                masks, M);
+  if (rc != BX_OK) return rc;
+  a.planes = planes;
+  a.edge = edge;
+  a.masks = masks;
+  return launch_chunks<true>(*p, a, nruns, st);
 }
 
 int bxf_gated_norm(int dtype, const bxf_gate_rows* p, int M, void* stream) {

@@ -36,20 +36,32 @@ class Step:
 
 class Tiles:
     """What the tile kernels of a prompt portion walk: attention tiles int32 [T, 3] (table row, first row, rows) by their
-    number of tokens, and the runs int32 [R, 2] (first row, rows) of its sequences."""
+    number of tokens; the runs int32 [R, 3] (first row, rows, first chunk) of its sequences and their chunks int32 [C, 2]
+    (first row, rows) for the recurrences."""
 
-    def __init__(self, attention, runs):
-        self.attention, self.runs = attention, runs
+    CHUNK = 64
+
+    def __init__(self, attention, runs, chunks):
+        self.attention, self.runs, self.chunks = attention, runs, chunks
 
     @classmethod
     def of(cls, runs, sizes):
         """runs = [(table row, first token row, tokens, context length)], sizes: the tile heights in use."""
         table = lambda n: torch.tensor([[r, t0 + s, min(n, ql - s)] for r, t0, ql, _ in runs for s in range(0, ql, n)],
                                        dtype=torch.int32).reshape(-1, 3)
-        return cls({n: table(n) for n in sizes}, torch.tensor([[t0, ql] for _, t0, ql, _ in runs], dtype=torch.int32).reshape(-1, 2))
+        per_run, chunks = [], []
+        for _, t0, ql, _ in runs:
+            per_run.append([t0, ql, len(chunks)])
+            chunks += [[t0 + s, min(cls.CHUNK, ql - s)] for s in range(0, ql, cls.CHUNK)]
+        return cls({n: table(n) for n in sizes}, torch.tensor(per_run, dtype=torch.int32).reshape(-1, 3),
+                   torch.tensor(chunks, dtype=torch.int32).reshape(-1, 2))
 
     def to(self, dev):
-        return Tiles({n: t.to(dev) for n, t in self.attention.items()}, self.runs.to(dev))
+        return Tiles({n: t.to(dev) for n, t in self.attention.items()}, self.runs.to(dev), self.chunks.to(dev))
+
+    def chunked(self, K, V, rows):
+        """Whether a recurrence of these sizes runs in chunks: portions of a few rows are shorter row by row."""
+        return rows >= 16 * self.runs.shape[0] and nv.float_lib().bxf_recurrence_chunk_rows(0, K, V) == self.CHUNK
 
     def for_heads(self, heads):
         return self.attention.get(nv.float_lib().bxf_latent_attention_tile(heads))
@@ -201,7 +213,8 @@ class GLA:
         a1 = torch.empty(M, self.rank, dtype=torch.float32, device=x.device)
         ops.linear(self.first, h, M, n + self.rank, self.D, ops.store(y, y.shape[1], n, side=a1))
         o = ops.recurrence(ops.DECAY_CHANNEL, y, a1, cache, step, sp.heads, (0, nk, 2 * nk), a2=self.a2, a2_b=self.a2_b,
-                           inv_tau=1.0 / sp.tau, q_scale=sp.dim ** -0.5)
+                           inv_tau=1.0 / sp.tau, q_scale=sp.dim ** -0.5,
+                           tiles=step.tiles if step.tiles is not None and step.tiles.chunked(sp.dim, sp.vdim, M) else None)
         o = ops.gated_norm(o, y[:, 2 * nk + nv_:], nv_, sp.heads, self.norm, sp.eps, gate_first=False)
         ops.linear(self.o, o, M, self.D, nv_, ops.sublayer_output(x, add))
 
@@ -234,8 +247,12 @@ class Mamba2:
         dt = torch.empty(M, sp.heads, dtype=torch.float32, device=x.device)
         ops.linear(self.first, h, M, n + sp.heads, self.D, ops.store(y, y.shape[1], n, side=dt, bias=self.dt_bias))
         conv = ops.conv_of(y[:, inner:], self.conv, self.conv_b, cache[1], step)
-        o = ops.recurrence(ops.DECAY_HEAD, y, dt, cache[0], step, sp.groups, (2 * inner + gn, 2 * inner, inner), conv=conv,
-                           A_log=self.A_log, skip=self.skip)
+        if step.tiles is not None and inner % 8 == 0 and step.tiles.chunked(sp.state, sp.vdim, M):
+            o = ops.recurrence(ops.DECAY_HEAD, ops.causal_conv(conv, M, y), dt, cache[0], step, sp.groups, (inner + gn, inner, 0),
+                               A_log=self.A_log, skip=self.skip, tiles=step.tiles)
+        else:
+            o = ops.recurrence(ops.DECAY_HEAD, y, dt, cache[0], step, sp.groups, (2 * inner + gn, 2 * inner, inner), conv=conv,
+                               A_log=self.A_log, skip=self.skip)
         o = ops.gated_norm(o, y, inner, sp.norm_groups, self.norm, sp.eps, gate_first=True, conv=conv)
         ops.linear(self.o, o, M, self.D, inner, ops.sublayer_output(x, add))
 

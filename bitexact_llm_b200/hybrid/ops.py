@@ -229,9 +229,9 @@ def causal_conv(conv, M, like):
 
 
 def recurrence(kind, y, side, state, step, groups, columns, conv=None, a2=None, a2_b=None, inv_tau=0.0, q_scale=1.0,
-               A_log=None, skip=None):
+               A_log=None, skip=None, tiles=None):
     """state float [slots, heads, K, V] is advanced by the rows of y; columns = where q, k, v begin in y -> outputs T
-    [M, pad8(heads V)]."""
+    [M, pad8(heads V)]. tiles: the chunk kernels walk its runs, else the rows go one by one."""
     M, (_, H, K, V) = y.shape[0], state.shape
     out = torch.empty(M, pad8(H * V), dtype=y.dtype, device=y.device)
     p = nv.RecurrenceRows(kind=kind, heads=H, groups=groups, K=K, V=V, rank=0 if a2 is None else a2.shape[1], q0=columns[0],
@@ -241,7 +241,16 @@ def recurrence(kind, y, side, state, step, groups, columns, conv=None, a2=None, 
                           seq=step.seq.data_ptr(), out=out.data_ptr(), ldo=out.stride(0))
     if conv is not None:
         p.conv = conv
-    nv.check(nv.float_lib().bxf_recurrence(code(y), ctypes.byref(p), M, nv.stream()), "bxf_recurrence")
+    lib = nv.float_lib()
+    if tiles is None:
+        nv.check(lib.bxf_recurrence(code(y), ctypes.byref(p), M, nv.stream()), "bxf_recurrence")
+        return out
+    chunks = tiles.chunks.shape[0]
+    need = lib.bxf_recurrence_chunk_scratch(kind, M, chunks, H, K)
+    scratch = torch.empty(need, dtype=torch.uint8, device=y.device) if need else None
+    rc = lib.bxf_recurrence_chunks(code(y), ctypes.byref(p), tiles.runs.data_ptr(), tiles.runs.shape[0], tiles.chunks.data_ptr(),
+                                   chunks, nv.ptr(scratch), need, M, nv.stream())
+    nv.check(rc, "bxf_recurrence_chunks")
     return out
 
 

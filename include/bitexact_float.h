@@ -139,7 +139,7 @@ typedef struct {
  *   BXF_DECAY_HEAD: side float [M, lds] holds the step sizes before softplus; dt = softplus(side), a = exp(-exp(A_log) dt),
  *     k is multiplied by dt, and skip[h] v_t is added to o_t.
  * conv.w != NULL: y's columns are the inputs of a causal convolution with silu and q, k, v its results (conv.u = column 0 of
- * q0, k0, v0; its state is read only, see bxf_gated_norm). With chunks the columns must be convolved already.
+ * q0, k0, v0; its state is read only, see bxf_gated_norm).
  * state float [slots, heads, K, V] is advanced by the rows of every sequence; out T [M, ldo] = o (heads concatenated). */
 typedef struct {
   int kind, heads, groups, K, V, rank, q0, k0, v0, pad_;
@@ -261,6 +261,14 @@ int bxf_gqa_attention(int dtype, const void* q, int64_t ldq, int M, int heads, i
 int bxf_streams(int dtype, const bxf_streams_step* step, int M, void* stream);
 int bxf_causal_conv(int dtype, const bxf_conv* conv, void* out, int64_t ldo, int M, void* stream);
 int bxf_recurrence(int dtype, const bxf_recurrence_rows* rows, int M, void* stream);
+/* The same over prompts, in chunks of up to 64 rows on the tensor cores. bxf_recurrence_chunk_rows: rows of a chunk, 0 when the
+ * sizes or the element type do not fit (bxf_recurrence takes those). runs int32 [nruns, 3] = (first row, rows, first chunk) of
+ * every sequence of the step; chunks int32 [nchunks, 2] = (first row, rows), cut from every run at multiples of the chunk
+ * rows, in the order of the runs. q0, k0, v0, ldy multiples of 8; conv unused. */
+int bxf_recurrence_chunk_rows(int dtype, int K, int V);
+size_t bxf_recurrence_chunk_scratch(int kind, int M, int chunks, int heads, int K);
+int bxf_recurrence_chunks(int dtype, const bxf_recurrence_rows* rows, const int* runs, int nruns, const int* chunks,
+                          int nchunks, void* scratch, size_t scratch_bytes, int M, void* stream);
 int bxf_gated_norm(int dtype, const bxf_gate_rows* rows, int M, void* stream);
 
 #ifdef __cplusplus

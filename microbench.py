@@ -8,10 +8,12 @@
     python microbench.py prompt [--batch 4] [--ctx 2048] [--chunk 4096] [--iters 3]
     python microbench.py bmm [--ctx 2048] [--iters 5]
     python microbench.py hybrid [--m 1,16,256,4096] [--iters 10]
+    python microbench.py veredra [--m 1,16,256,8192] [--iters 10]
 
 hybrid: every kernel of the hybrid float models at the sizes of bench_hybrid.py's w2048 (bytes and FLOPs of the algorithm,
       inputs beyond L2; fractions of the copy bandwidth and of the bf16 GEMM rate in MEASURED_PEAKS.json, else of
       6.65 TB/s and 1.59 PFLOP/s).
+veredra: the same for the Veredra design at the sizes of bench_hybrid.py's w2048.
 gemm: the exact-mode fused linear on the projection shapes of one Llama-3.2-1B layer and the LM head
       (int8-equivalent ops = 2 * 9 * M * N * K; algorithmic bytes = 3 N K + 4 M K + 8 M N).
 gemmr: the fused projections of one layer with REAL constants (bf16 weights from N(0, 0.02^2), decomposed into limbs
@@ -436,17 +438,9 @@ def peaks():
     return 6.65e12, 1.59e15
 
 
-def hybrid(args):
-    from types import SimpleNamespace
-
-    from bitexact_llm_b200.hybrid import ops
-    from bitexact_llm_b200.hybrid.spec import LatentAttentionSpec
-    dev, D, BF = "cuda", 2048, torch.bfloat16
+def reporter(args):
     hbm, mma = peaks()
     only = set(args.proj.split(",")) if args.proj else None
-    W = lambda *s: torch.randn(*s, device=dev, dtype=BF) * 0.02
-    X = lambda *s: torch.randn(*s, device=dev, dtype=BF)
-    F = lambda *s: torch.randn(*s, device=dev)
 
     def report(name, M, make, flops, byts, per_set):
         """make() -> a call on a fresh set of inputs, which must keep every tensor alive whose address it passes on;
@@ -460,6 +454,139 @@ def hybrid(args):
                "roofline_us": round(max(flops / mma, byts / hbm) * 1e6, 2)}
         rec["frac"] = round(rec["roofline_us"] / us, 3)
         print(json.dumps(rec), flush=True)
+    return report
+
+
+def veredra(args):
+    """Sizes of bench_hybrid.veredra_config(2048, ..). M <= 256: a decoding batch of M sequences; else 4 prompts."""
+    from bitexact_llm_b200.hybrid import ops
+    from bitexact_llm_b200.hybrid.layers import Step, Tiles
+    from bitexact_llm_b200.hybrid.spec import AttentionSpec
+    dev, D, BF = "cuda", 2048, torch.bfloat16
+    W = lambda *s: torch.randn(*s, device=dev, dtype=BF) * 0.02
+    X = lambda *s: torch.randn(*s, device=dev, dtype=BF)
+    F = lambda *s: torch.randn(*s, device=dev)
+    report = reporter(args)
+
+    def linear(name, M, N, K, kind, side=0):
+        def make():
+            w, x, b = W(N + side, K), X(M, K), F(N)
+            s = F(M, side) if side else None
+            out = torch.empty(M, N // 2 if kind == "glu" else N, device=dev,
+                              dtype={"glu": BF, "bf16": BF, "bias": BF, "f32": torch.float32, "i64": torch.long}[kind])
+            epi = {"glu": lambda: ops.glu(out, "gelu"), "bf16": lambda: ops.store(out, N, N, side=s),
+                   "bias": lambda: ops.store(out, N, N, main_bias=b), "f32": lambda: ops.store(out, N, N, out_type=ops.OUT_F32),
+                   "i64": lambda: ops.store(out, N, N, "softcap", 0.1, 15.0, out_type=ops.OUT_I64)}[kind]()
+            return lambda: (out, b, s, ops.linear(w, x, M, N + side, K, epi))
+        byts = 2.0 * (N + side) * K + 2.0 * M * K + {"glu": 1, "bf16": 2, "bias": 2, "f32": 4, "i64": 8}[kind] * M * N + 4.0 * M * side
+        report(name, M, make, 2.0 * M * (N + side) * K, byts, byts)
+
+    def step_of(M, first):
+        B = M if M <= 256 else 4
+        n = M // B
+        seq = torch.arange(B, device=dev).repeat_interleave(n)
+        pos = torch.arange(first, first + n, device=dev).repeat(B)
+        tiles = Tiles.of([(b, b * n, n, first + n) for b in range(B)], {32}).to(dev) if n > 1 else None
+        return B, n, Step(pos, pos, seq, None, ops.row_flags(seq, pos, pos), tiles)
+
+    def attention(name, B, ctx, n, window, H=16, G=4, d=128):
+        sp = AttentionSpec(H, G, d, d, 0, 1.0, 0.1, window, 1e-6)
+        M, bs = B * n, 64
+        nblk = (ctx + bs - 1) // bs
+
+        def make():
+            cache = X(1 + B * nblk, G, bs, 2 * d)
+            bt = (torch.randperm(B * nblk, device=dev) + 1).view(B, nblk).int()
+            seq = torch.arange(B, device=dev).repeat_interleave(n)
+            pos = torch.arange(ctx - n, ctx, device=dev).repeat(B)
+            q, sink = X(G, M, H // G, d), F(H)
+            tiles = Tiles.of([(b, b * n, n, ctx) for b in range(B)], {32}).to(dev).attention[32] if n > 1 else None
+            return lambda: ops.gqa_attention(q, sp, cache, bt, seq, pos, sink, tiles)
+        keys = sum(min(p + 1, window or p + 1) for p in range(ctx - n, ctx)) * B
+        kv = B * min(ctx, (window or ctx) + n - 1) * G * 4.0 * d
+        report(name, M, make, 4.0 * keys * H * d, kv + 4.0 * M * H * d, kv + 4.0 * M * H * d)
+
+    def recurrence(name, M, kind, H, G, K, V, rank):
+        inner, gk = H * V, G * K
+        B, n, st = step_of(M, 512 if M <= 256 else 0)
+        n_state = B * H * K * V * 8.0 if M <= 256 else 0.0
+
+        def make():
+            state = torch.zeros(B, H, K, V, device=dev)
+            if kind == ops.DECAY_CHANNEL:
+                y, side, a2, b = X(M, 2 * gk + inner), F(M, rank), F(gk, rank) * 0.3, F(gk) + 2.0
+                return lambda: ops.recurrence(kind, y, side, state, st, G, (0, gk, 2 * gk), a2=a2, a2_b=b, inv_tau=1 / 16.0,
+                                              q_scale=K ** -0.5, tiles=st.tiles)
+            u, side, A, s = X(M, inner + 2 * gk), F(M, H) - 2.0, F(H), F(H)
+            w, b, cs = F(inner + 2 * gk, 4) * 0.5, F(inner + 2 * gk), torch.zeros(B, 3, inner + 2 * gk, device=dev, dtype=BF)
+            if st.tiles is None:
+                return lambda: ops.recurrence(kind, u, side, state, st, G, (inner + gk, inner, 0), conv=ops.conv_of(u, w, b, cs, st),
+                                              A_log=A, skip=s)
+            return lambda: ops.recurrence(kind, ops.causal_conv(ops.conv_of(u, w, b, cs, st), M, u), side, state, st, G,
+                                          (inner + gk, inner, 0), A_log=A, skip=s, tiles=st.tiles)
+        flops = M * H * (4.0 * K * V + (2.0 * 32 * (K + V) if M > 256 else 0))
+        byts = n_state + M * (2.0 * (2 * gk + inner) + 2.0 * inner + 4.0 * (rank or H))
+        report(name, M, make, flops, byts, byts)
+        if kind == ops.DECAY_HEAD and M > 256:
+            def conv():
+                u, w, b = X(M, inner + 2 * gk), F(inner + 2 * gk, 4) * 0.5, F(inner + 2 * gk)
+                cs = torch.zeros(B, 3, inner + 2 * gk, device=dev, dtype=BF)
+                return lambda: (w, b, cs, ops.causal_conv(ops.conv_of(u, w, b, cs, st), M, u))
+            report("causal_conv", M, conv, 0, 4.0 * M * (inner + 2 * gk), 4.0 * M * (inner + 2 * gk))
+
+    def gated_norm(name, M, n, parts, wn, first):
+        def make():
+            o, z, w = X(M, n), X(M, n), F(wn)
+            return lambda: ops.gated_norm(o, z, n, parts, w, 1e-6, first)
+        report(name, M, make, 0, 6.0 * M * n, 6.0 * M * n)
+
+    for M in [int(v) for v in args.m.split(",")]:
+        linear("gate_up", M, 8 * D, D, "glu")
+        linear("down", M, D, 4 * D, "f32")
+        linear("qkv", M, 3072, D, "bias")
+        linear("gla_first", M, 6144, D, "bf16", side=16)
+        linear("mamba_in", M, 4 * D + 2 * 8 * 128, D, "bf16", side=64)
+        linear("out_2048", M, D, D, "f32")
+        linear("out_4096", M, D, 2 * D, "f32")
+        if M <= 256:
+            linear("head", M, 128256, D, "i64")
+            attention("attention_decode", M, 1040, 1, 1024)
+            attention("attention_decode_8k", M, 8192, 1, 0)
+        else:
+            attention("attention_prompt", 4, M // 4, M // 4, 1024)
+            attention("attention_prompt_full", 4, M // 4, M // 4, 0)
+        recurrence("gla", M, ops.DECAY_CHANNEL, 8, 8, 128, 256, 16)
+        recurrence("mamba2", M, ops.DECAY_HEAD, 64, 8, 128, 64, 0)
+        gated_norm("gla_norm", M, 2048, 8, 256, False)
+        gated_norm("mamba_norm", M, 4096, 8, 4096, True)
+        for S in (2, 4):
+            def streams():
+                x, y, h, w = F(M, S, D), F(M, D), X(M, D), F(D)
+                a, b, c = F(S), F(S), torch.eye(S, device=dev)
+                return lambda: (w, a, b, c, ops.streams(x, 1e-6, None, (y, b, c), a, w, h))
+            report(f"streams_{S}", M, streams, 0, M * D * (8.0 * S + 6), M * D * (8 * S + 6))
+
+        def prepare():
+            sp = AttentionSpec(16, 4, 128, 128, 128, 1e6, 0.1, 1024, 1e-6)
+            y, cache = X(M, 3072), X(M // 64 + 2, 4, 64, 256)
+            a, b, cs = F(2048), F(512), F(M, 64, 2)
+            pos = torch.arange(M, device=dev)
+            return lambda: (cs, ops.gqa_prepare(y, sp, a, b, cs, pos, cache))
+        report("gqa_prepare", M, prepare, 0, M * (4.0 * 3072 + 512), M * 12800)
+    if nv.float_device_status() != 0:
+        raise SystemExit("device-side wait timed out")
+
+
+def hybrid(args):
+    from types import SimpleNamespace
+
+    from bitexact_llm_b200.hybrid import ops
+    from bitexact_llm_b200.hybrid.spec import LatentAttentionSpec
+    dev, D, BF = "cuda", 2048, torch.bfloat16
+    W = lambda *s: torch.randn(*s, device=dev, dtype=BF) * 0.02
+    X = lambda *s: torch.randn(*s, device=dev, dtype=BF)
+    F = lambda *s: torch.randn(*s, device=dev)
+    report = reporter(args)
 
     def linear(name, M, N, K, kind, groups=1, act="none"):
         def make():
@@ -585,7 +712,7 @@ def hybrid(args):
 
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("what", choices=["gemm", "gemmr", "gemm8", "attn", "stages", "prefill", "prompt", "bmm", "hybrid"])
+    ap.add_argument("what", choices=["gemm", "gemmr", "gemm8", "attn", "stages", "prefill", "prompt", "bmm", "hybrid", "veredra"])
     ap.add_argument("--m", default="1,16,256,4096")
     ap.add_argument("--tile", type=int, default=0)
     ap.add_argument("--iters", type=int, default=10)
@@ -596,12 +723,12 @@ def main():
     ap.add_argument("--variant", type=int, default=0)
     ap.add_argument("--no-scratch", action="store_true", help="attn: no scratch buffer (long contexts: cluster kernels)")
     ap.add_argument("--fixed", action="store_true", help="attn: every request has exactly --ctx keys")
-    ap.add_argument("--proj", default="", help="gemmr / gemm8: only this projection (wqkv, wo, wgu, wd, lm); hybrid: only these kernels")
+    ap.add_argument("--proj", default="", help="gemmr / gemm8: only this projection (wqkv, wo, wgu, wd, lm); hybrid, veredra: only these kernels")
     ap.add_argument("--eager", action="store_true", help="gemmr / gemm8: one plain launch per weight set, no timing")
     ap.add_argument("--chunk", type=int, default=4096, help="prompt: token rows per forward call")
     args = ap.parse_args()
     {"gemm": gemm, "gemmr": gemmr, "gemm8": gemm8, "attn": attn, "stages": stages, "prefill": prefill, "prompt": prompt, "bmm": bmm_bench,
-     "hybrid": hybrid}[args.what](args)
+     "hybrid": hybrid, "veredra": veredra}[args.what](args)
     if nv.device_status() != 0:
         raise SystemExit("device-side wait timed out")
 
