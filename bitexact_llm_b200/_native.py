@@ -120,9 +120,14 @@ class Conv(ctypes.Structure):
 class RecurrenceRows(ctypes.Structure):
     """bxf_recurrence_rows."""
     _fields_ = [("kind", I), ("heads", I), ("groups", I), ("K", I), ("V", I), ("rank", I), ("q0", I), ("k0", I), ("v0", I),
-                ("pad_", I), ("y", P), ("ldy", L), ("side", P), ("lds", L), ("a2", P), ("a2_b", P), ("inv_tau", R),
-                ("q_scale", R), ("A_log", P), ("skip", P), ("conv", Conv), ("state", P), ("flags", P), ("seq", P), ("out", P),
-                ("ldo", L)]
+                ("batch", I), ("y", P), ("ldy", L), ("side", P), ("lds", L), ("a2", P), ("a2_b", P), ("inv_tau", R),
+                ("q_scale", R), ("A_log", P), ("skip", P), ("state", P), ("flags", P), ("seq", P), ("out", P), ("ldo", L)]
+
+
+class ChunkTable(ctypes.Structure):
+    """bxf_chunk_table."""
+    _fields_ = [("runs", P), ("chunks", P), ("segments", P), ("spans", P), ("nruns", I), ("nchunks", I), ("nsegments", I),
+                ("pad_", I)]
 
 
 class GateRows(ctypes.Structure):
@@ -158,8 +163,8 @@ _FLOAT_SIGNATURES = {
     "bxf_causal_conv": (I, [I, ctypes.POINTER(Conv), P, L, I, P]),
     "bxf_recurrence": (I, [I, ctypes.POINTER(RecurrenceRows), I, P]),
     "bxf_recurrence_chunk_rows": (I, [I, I, I]),
-    "bxf_recurrence_chunk_scratch": (Z, [I, I, I, I, I]),
-    "bxf_recurrence_chunks": (I, [I, ctypes.POINTER(RecurrenceRows), P, I, P, I, P, Z, I, P]),
+    "bxf_recurrence_chunk_scratch": (Z, [I, I, I, I, I, I, I]),
+    "bxf_recurrence_chunks": (I, [I, ctypes.POINTER(RecurrenceRows), ctypes.POINTER(ChunkTable), P, Z, I, P]),
     "bxf_gated_norm": (I, [I, ctypes.POINTER(GateRows), I, P]),
 }
 

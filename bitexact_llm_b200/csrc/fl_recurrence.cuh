@@ -25,62 +25,73 @@ __device__ __forceinline__ float conv_at(const bxf_conv& c, int m, int ch) {
     } else {
       v = ld(static_cast<const T*>(c.state) + (c.seq[m] * (c.taps - 1) + first - back + c.taps - 1) * c.channels + ch);
     }
-    acc = fmaf(c.w[ch * c.taps + c.taps - 1 - back], v, acc);
+    acc = fmaf(c.w[(i64)(c.taps - 1 - back) * c.channels + ch], v, acc);
   }
   return silu<T>(acc);
 }
 
-constexpr int CONV_ROWS = 16, CONV_THREADS = 128;
+constexpr int CONV_ROWS = 16, CONV_THREADS = 128, CONV_BATCH = 4;
 
-// Prompts: a thread walks CONV_ROWS rows of 8 channels with the last TAPS inputs in registers.
+// A thread walks up to CONV_ROWS rows (`rows`) of 8 channels with the last TAPS inputs in registers; the rows are read ahead
+// a few at a time.
 template <int TAPS>
-__global__ void __launch_bounds__(CONV_THREADS) fl_causal_conv_rows_kernel(const bxf_conv c, bf16* __restrict__ out, i64 ldo, int M) {
+__global__ void __launch_bounds__(CONV_THREADS)
+fl_causal_conv_rows_kernel(const bxf_conv c, bf16* __restrict__ out, i64 ldo, int M, int rows) {
   launch_next();
   const int ch = (blockIdx.x * CONV_THREADS + threadIdx.x) * 8;
   if (ch >= c.channels) return;
   float w[TAPS][8], b[8], win[TAPS][8];
+  load_v<8>(c.b + ch, b);
 #pragma unroll
-  for (int i = 0; i < 8; ++i) {
-    b[i] = c.b[ch + i];
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) w[j][i] = c.w[(ch + i) * TAPS + j];
-  }
+  for (int j = 0; j < TAPS; ++j) load_v<8>(c.w + (i64)j * c.channels + ch, w[j]);
   wait_previous();
-  const int m0 = blockIdx.y * CONV_ROWS, m1 = min(M, m0 + CONV_ROWS);
+  const int m0 = blockIdx.y * rows, m1 = min(M, m0 + rows);
   const bf16* u = static_cast<const bf16*>(c.u) + ch;
-  for (int m = m0; m < m1; ++m) {
-    const int f = c.flags[m];
-    if (f & BXF_ROW_PAD) continue;
-    if (m == m0 || (f & BXF_ROW_FIRST)) {                // the inputs before this row: rows of the step, the state, zeros
-      int first = (f & BXF_ROW_FIRST) ? 0 : -1;
+  for (int at = m0; at < m1; at += CONV_BATCH) {
+    uint4 raw[CONV_BATCH];
+    int flags[CONV_BATCH];
 #pragma unroll
-      for (int back = 1; back < TAPS; ++back) {
-        float (&v)[8] = win[TAPS - 1 - back];
-        if (back > c.pos[m]) {
+    for (int r = 0; r < CONV_BATCH; ++r)
+      if (at + r < m1) {
+        raw[r] = *reinterpret_cast<const uint4*>(u + (i64)(at + r) * c.ldu);
+        flags[r] = c.flags[at + r];
+      }
 #pragma unroll
-          for (int i = 0; i < 8; ++i) v[i] = 0.0f;
-        } else if (first < 0) {
-          load_v<8>(u + (i64)(m - back) * c.ldu, v);
-          if (c.flags[m - back] & BXF_ROW_FIRST) first = back;
-        } else {
-          load_v<8>(static_cast<const bf16*>(c.state) + (c.seq[m] * (TAPS - 1) + first - back + TAPS - 1) * c.channels + ch, v);
+    for (int r = 0; r < CONV_BATCH; ++r) {
+      const int m = at + r, f = flags[r];
+      if (m >= m1 || (f & BXF_ROW_PAD)) continue;
+      if (m == m0 || (f & BXF_ROW_FIRST)) {              // the inputs before this row: rows of the step, the state, zeros
+        const i64 pos = c.pos[m], slot = c.seq[m];
+        int first = (f & BXF_ROW_FIRST) ? 0 : -1;
+#pragma unroll
+        for (int back = 1; back < TAPS; ++back) {
+          float (&v)[8] = win[TAPS - 1 - back];
+          if (back > pos) {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) v[i] = 0.0f;
+          } else if (first < 0) {
+            load_v<8>(u + (i64)(m - back) * c.ldu, v);
+            if (c.flags[m - back] & BXF_ROW_FIRST) first = back;
+          } else {
+            load_v<8>(static_cast<const bf16*>(c.state) + (slot * (TAPS - 1) + first - back + TAPS - 1) * c.channels + ch, v);
+          }
         }
       }
+      load_v<8>(raw[r], win[TAPS - 1]);
+      float o[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        o[i] = b[i];
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) o[i] = fmaf(w[j][i], win[j][i], o[i]);
+        o[i] = silu<bf16>(o[i]);
+      }
+      store_v<8>(out + m * ldo + ch, o);
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS; ++j)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) win[j][i] = win[j + 1][i];
     }
-    load_v<8>(u + (i64)m * c.ldu, win[TAPS - 1]);
-    float o[8];
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      o[i] = b[i];
-#pragma unroll
-      for (int j = 0; j < TAPS; ++j) o[i] = fmaf(w[j][i], win[j][i], o[i]);
-      o[i] = silu<bf16>(o[i]);
-    }
-    store_v<8>(out + m * ldo + ch, o);
-#pragma unroll
-    for (int j = 0; j + 1 < TAPS; ++j)
-#pragma unroll
-      for (int i = 0; i < 8; ++i) win[j][i] = win[j + 1][i];
   }
 }
 
@@ -110,37 +121,46 @@ __device__ __forceinline__ void conv_advance(const bxf_conv& c, int m) {
 }
 
 // ---- the recurrence row by row: decoding, short portions, 32-bit, any sizes ----
-// One CTA per (sequence of the step, head, 32 value columns) walks the sequence's rows with its part of the state in
-// registers: thread = 4 columns x every 32nd key channel. Rows are prepared in shared memory a few at a time.
-constexpr int REC_THREADS = 256, REC_COLS = 32, REC_LANES = 32, REC_ROWS = 8;
+// One CTA per (sequence of the step, head, 4 CW value columns) walks the sequence's rows with its part of the state in
+// registers: thread = 4 columns x every (256 / CW)th key channel. Rows are prepared in shared memory ROWS at a time (one for
+// decoding). Wide
+// slices share the preparation, narrow ones spread a small batch over more SMs.
+constexpr int REC_THREADS = 256, REC_ROWS = 8, REC_RANK = 16;   // REC_ROWS: most rows at a time
 
-__host__ __device__ constexpr int recurrence_smem(int K, bool channel) {
-  return (REC_ROWS * K * (channel ? 3 : 2) + REC_ROWS * REC_COLS * 9 + REC_ROWS * 2) * 4;
+__host__ __device__ constexpr int recurrence_smem(int K, int CW, bool channel, int rows) {
+  return (rows * K * (channel ? 3 : 2) + rows * 4 * CW * 9 + 2 * REC_ROWS) * 4;
 }
 
-template <class T, bool CHANNEL, int KR>
-__global__ void __launch_bounds__(REC_THREADS) fl_recurrence_kernel(const bxf_recurrence_rows p, int M) {
+template <class T, bool CHANNEL, int CW, int KR, int ROWS>
+__global__ void __launch_bounds__(REC_THREADS, CHANNEL || KR > 8 ? 1 : KR <= 4 ? 4 : 3) fl_recurrence_kernel(const bxf_recurrence_rows p, int M) {
   launch_next();
-  wait_previous();
   extern __shared__ float rec_smem[];
-  const int m0 = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * REC_COLS, tid = threadIdx.x;
+  constexpr int COLS = 4 * CW, LANES = REC_THREADS / CW;
+  const int m0 = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * COLS, tid = threadIdx.x;
+  float w2[REC_RANK];                                    // the decay projection's weights of channel tid, entries 0 .. 15
+  if (CHANNEL) {
+#pragma unroll
+    for (int j = 0; j < REC_RANK; ++j) w2[j] = tid < p.K && j < p.rank ? p.a2[((i64)j * p.heads + h) * p.K + tid] : 0.0f;
+  }
+  wait_previous();
   const int f0 = p.flags[m0];
+  const i64 slot = p.seq[m0];
   if ((f0 & (BXF_ROW_FIRST | BXF_ROW_PAD)) != BXF_ROW_FIRST) return;
   const int K = p.K, V = p.V, g = h / (p.heads / p.groups);
-  float* sv = rec_smem;                                  // [rows][32]
-  float* red = sv + REC_ROWS * REC_COLS;                 // [rows][8 warps][32]
-  float* s_dt = red + REC_ROWS * 8 * REC_COLS;           // [rows] step size and decay of the head
+  float* sv = rec_smem;                                  // [rows][COLS]
+  float* red = sv + ROWS * COLS;                     // [rows][8 warps][COLS]
+  float* s_dt = red + ROWS * 8 * COLS;               // [rows] step size and decay of the head
   float* s_dec = s_dt + REC_ROWS;
   float* sq = s_dec + REC_ROWS;                          // [rows][K]
-  float* sk = sq + REC_ROWS * K;
-  float* sa = sk + REC_ROWS * K;                         // CHANNEL: decays
-  const int cx = (tid & 7) * 4, kl = tid >> 3, col = c0 + cx;
-  float* state = p.state + ((p.seq[m0] * p.heads + h) * K) * (i64)V + col;
+  float* sk = sq + ROWS * K;
+  float* sa = sk + ROWS * K;                         // CHANNEL: decays
+  const int cx = (tid % CW) * 4, kl = tid / CW, col = c0 + cx;
+  float* state = p.state + ((slot * p.heads + h) * K) * (i64)V + col;
   const bool fresh = f0 & BXF_ROW_START, wide = V % 4 == 0 && col < V;
   float s[KR][4];
 #pragma unroll
   for (int j = 0; j < KR; ++j) {
-    const int k = j * REC_LANES + kl;
+    const int k = j * LANES + kl;
 #pragma unroll
     for (int i = 0; i < 4; ++i) s[j][i] = 0.0f;
     if (fresh || k >= K) continue;
@@ -152,38 +172,45 @@ __global__ void __launch_bounds__(REC_THREADS) fl_recurrence_kernel(const bxf_re
         if (col + i < V) s[j][i] = state[(i64)k * V + i];
     }
   }
-  const auto value = [&](int m, int column) {
-    return !CHANNEL && p.conv.w ? conv_at<T>(p.conv, m, column - min(p.q0, min(p.k0, p.v0)))
-                                : ld(static_cast<const T*>(p.y) + m * p.ldy + column);
-  };
+  const T* y = static_cast<const T*>(p.y);
   for (int m = m0;;) {
     int n = 0;
     bool end = false;
-    while (n < REC_ROWS && !end) end = p.flags[m + n++] & BXF_ROW_LAST;
-    for (int at = tid; at < n * K; at += REC_THREADS) {
-      const int r = at / K, k = at % K;
-      sq[r * K + k] = value(m + r, p.q0 + g * K + k) * (CHANNEL ? p.q_scale : 1.0f);
-      sk[r * K + k] = value(m + r, p.k0 + g * K + k);
-    }
-    for (int at = tid; at < n * REC_COLS; at += REC_THREADS) {
-      const int c = at % REC_COLS;
-      sv[at] = c0 + c < V ? value(m + at / REC_COLS, p.v0 + h * V + c0 + c) : 0.0f;
+    while (n < ROWS && !end) end = p.flags[m + n++] & BXF_ROW_LAST;
+    for (int r = 0; r < n; ++r) {
+      const T* row = y + (i64)(m + r) * p.ldy;
+      for (int k = tid; k < K; k += REC_THREADS) {
+        sq[r * K + k] = ld(row + p.q0 + g * K + k) * (CHANNEL ? p.q_scale : 1.0f);
+        sk[r * K + k] = ld(row + p.k0 + g * K + k);
+      }
+      if (tid < COLS) sv[r * COLS + tid] = c0 + tid < V ? ld(row + p.v0 + (i64)h * V + c0 + tid) : 0.0f;
     }
     if (CHANNEL) {
       for (int k = tid; k < K; k += REC_THREADS) {
-        const float* a2 = p.a2 + ((i64)h * K + k) * p.rank;
+        const float* a2 = p.a2 + h * K + k;
         const float b = p.a2_b[h * K + k];
-        float z[REC_ROWS];
+        float z[ROWS];
 #pragma unroll
-        for (int r = 0; r < REC_ROWS; ++r) z[r] = b;
-        for (int j = 0; j < p.rank; ++j) {
-          const float w = a2[j];
+        for (int r = 0; r < ROWS; ++r) z[r] = b;
+        for (int j0 = 0; j0 < p.rank; j0 += REC_RANK) {
+          float w[REC_RANK];
 #pragma unroll
-          for (int r = 0; r < REC_ROWS; ++r)
-            if (r < n) z[r] = fmaf(w, p.side[(m + r) * p.lds + j], z[r]);
+          for (int j = 0; j < REC_RANK; ++j) w[j] = w2[j];
+          if (k != tid || j0 > 0) {
+#pragma unroll
+            for (int j = 0; j < REC_RANK; ++j) w[j] = j0 + j < p.rank ? a2[(i64)(j0 + j) * p.heads * K] : 0.0f;
+          }
+#pragma unroll
+          for (int r = 0; r < ROWS; ++r) {
+            if (r >= n) break;
+            const float* side = p.side + (m + r) * p.lds + j0;
+#pragma unroll
+            for (int j = 0; j < REC_RANK; ++j)
+              if (j0 + j < p.rank) z[r] = fmaf(w[j], side[j], z[r]);
+          }
         }
 #pragma unroll
-        for (int r = 0; r < REC_ROWS; ++r)
+        for (int r = 0; r < ROWS; ++r)
           if (r < n) sa[r * K + k] = expf(-softplus(-z[r]) * p.inv_tau);
       }
     } else if (tid < n) {
@@ -193,13 +220,13 @@ __global__ void __launch_bounds__(REC_THREADS) fl_recurrence_kernel(const bxf_re
     }
     __syncthreads();
     for (int r = 0; r < n; ++r) {
-      const float4 x = *reinterpret_cast<const float4*>(sv + r * REC_COLS + cx);
+      const float4 x = *reinterpret_cast<const float4*>(sv + r * COLS + cx);
       const float dt = CHANNEL ? 1.0f : s_dt[r], dec = CHANNEL ? 1.0f : s_dec[r];
       const float v[4] = {x.x * dt, x.y * dt, x.z * dt, x.w * dt};
       float o[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
       for (int j = 0; j < KR; ++j) {
-        const int k = j * REC_LANES + kl;
+        const int k = j * LANES + kl;
         if (k < K) {
           const float a = CHANNEL ? sa[r * K + k] : dec, kv = sk[r * K + k], qv = sq[r * K + k];
 #pragma unroll
@@ -210,37 +237,38 @@ __global__ void __launch_bounds__(REC_THREADS) fl_recurrence_kernel(const bxf_re
         }
       }
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        o[i] += __shfl_xor_sync(0xffffffffu, o[i], 8);
-        o[i] += __shfl_xor_sync(0xffffffffu, o[i], 16);
+      for (int d = CW; d < 32; d *= 2)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) o[i] += __shfl_xor_sync(0xffffffffu, o[i], d);
+      if ((tid & 31) < CW) store_v<4>(red + (r * 8 + (tid >> 5)) * COLS + cx, o);
+    }
+    if (end) {
+#pragma unroll
+      for (int j = 0; j < KR; ++j) {
+        const int k = j * LANES + kl;
+        if (k >= K) continue;
+        if (wide) {
+          store_v<4>(state + (i64)k * V, s[j]);
+        } else {
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+            if (col + i < V) state[(i64)k * V + i] = s[j][i];
+        }
       }
-      if ((tid & 31) < 8) store_v<4>(red + (r * 8 + (tid >> 5)) * REC_COLS + cx, o);
     }
     __syncthreads();
-    for (int at = tid; at < n * REC_COLS; at += REC_THREADS) {
-      const int r = at / REC_COLS, c = at % REC_COLS;
+    for (int at = tid; at < n * COLS; at += REC_THREADS) {
+      const int r = at / COLS, c = at % COLS;
       if (c0 + c >= V) continue;
       float o = 0.0f;
 #pragma unroll
-      for (int w = 0; w < 8; ++w) o += red[(r * 8 + w) * REC_COLS + c];
+      for (int w = 0; w < 8; ++w) o += red[(r * 8 + w) * COLS + c];
       if (!CHANNEL) o = fmaf(p.skip[h], sv[at], o);
       st(static_cast<T*>(p.out) + (m + r) * p.ldo + (i64)h * V + c0 + c, o);
     }
     if (end) break;
     m += n;
     __syncthreads();                                     // the next rows overwrite sv
-  }
-#pragma unroll
-  for (int j = 0; j < KR; ++j) {
-    const int k = j * REC_LANES + kl;
-    if (k >= K) continue;
-    if (wide) {
-      store_v<4>(state + (i64)k * V, s[j]);
-    } else {
-#pragma unroll
-      for (int i = 0; i < 4; ++i)
-        if (col + i < V) state[(i64)k * V + i] = s[j][i];
-    }
   }
 }
 

@@ -2,7 +2,9 @@
 // c_t the sum of the log decays of the rows after its first one up to t,
 //   o_t = (q_t e^(c_t)) S' + sum_(s <= t) (q_t e^(c_t)) . (k_s e^(-c_s)) v_s,     S' = diag(a_first) S,
 //   S  <- diag(e^(c_last)) (S' + sum_s (k_s e^(-c_s)) v_s^T).
-// One CTA per (run of rows, head, slice of value columns) walks the chunks of its run; a warp holds the state of 16 value
+// One CTA per (run of rows, head, slice of value columns) walks the chunks of its run. Long runs are cut into segments that are
+// walked side by side: a first pass makes every segment's own contribution to the state and its decays, a small kernel
+// chains them to the states the segments start from, and the second pass produces the outputs. A warp holds the state of 16 value
 // columns in registers, 32-bit, transposed (accumulators of V^T K), so that it is at the same time the B operand of Q S.
 // Products are bf16 mma with 32-bit accumulation; whatever carries a decay, a step size or a state is split into two bf16
 // terms (high and low part, about 17 bits), so only q, k, v themselves have bf16 precision.
@@ -10,7 +12,7 @@
 // BXF_DECAY_HEAD: q, k enter the scores unscaled and every score gets its factor e^(c_t - c_s) <= 1 in 32-bit.
 // BXF_DECAY_CHANNEL: the factors belong to the contraction index, so q e^c and k e^-c are made beforehand, by
 // fl_decay_prepare_kernel, in high and low parts. e^-c must not overflow: a chunk whose channels decay by more than e^-40
-// is cut into shorter segments there, down to single rows (c = 0), whatever the decays are.
+// is cut into shorter pieces there, down to single rows (c = 0), whatever the decays are.
 #pragma once
 
 #include "fl_recurrence.cuh"
@@ -48,9 +50,9 @@ __device__ __forceinline__ void copy16(bf16* to, const bf16* from, bool there) {
 }
 __device__ __forceinline__ void copies_done() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
-// ---- decays per channel: log decays, segments, scaled queries and keys ----
+// ---- decays per channel: log decays, pieces, scaled queries and keys ----
 // One CTA per (chunk, head). planes bf16 [4][M][heads K] = q high, q low, k high, k low; edge float [M][heads K]: in a
-// segment's first row its decays, in its last row (of several) e^(c_last); masks [chunks][heads]: bit t = row t starts a segment.
+// piece's first row its decays, in its last row (of several) e^(c_last); masks [chunks][heads]: bit t = row t starts a piece.
 constexpr int RP_THREADS = 256, RP_RANK = 16;
 
 __host__ __device__ constexpr int decay_prepare_smem(int K, int rank) { return (RC_ROWS * K + RC_ROWS * rank) * 4; }
@@ -69,13 +71,13 @@ fl_decay_prepare_kernel(const bxf_recurrence_rows p, const int* __restrict__ chu
   __syncthreads();
   const int lanes = RP_THREADS / K, t0 = tid / K, k = tid % K;
   if (t0 < lanes) {
-    const float* a2 = p.a2 + ((i64)h * K + k) * p.rank;
+    const float* a2 = p.a2 + h * K + k;
     const float bias = p.a2_b[h * K + k];
     for (int j0 = 0; j0 < p.rank; j0 += RP_RANK) {
       float w[RP_RANK];
       const int nj = min(RP_RANK, p.rank - j0);
 #pragma unroll
-      for (int j = 0; j < RP_RANK; ++j) w[j] = j < nj ? a2[j0 + j] : 0.0f;
+      for (int j = 0; j < RP_RANK; ++j) w[j] = j < nj ? a2[(j0 + j) * HK] : 0.0f;
       for (int t = t0; t < n; t += lanes) {
         float z = j0 == 0 ? bias : la[t * K + k];
 #pragma unroll
@@ -87,16 +89,31 @@ fl_decay_prepare_kernel(const bxf_recurrence_rows p, const int* __restrict__ chu
   }
   __syncthreads();
   float sum = 0.0f;
-  if (tid < K)
+  if (tid < K) {
+#pragma unroll 8
     for (int t = 1; t < n; ++t) sum += la[t * K + tid];
+  }
   const bool one = __syncthreads_and(sum >= -RC_RANGE);
   unsigned long long mask = 1;
   float c = 0.0f;
   int start = 0;
   float* e = edge + (i64)row0 * HK + h * K + tid;
-  for (int t = 0; t < n; ++t) {
+  if (one && tid < K) {
+    e[0] = expf(la[tid]);
+    for (int t = 0; t < n; t += 8) {
+      float l[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) l[i] = t + i > 0 && t + i < n ? la[(t + i) * K + tid] : 0.0f;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        c += l[i];
+        if (t + i < n) la[(t + i) * K + tid] = c;
+      }
+    }
+  }
+  for (int t = 0; t < n && !one; ++t) {
     const float l = tid < K ? la[t * K + tid] : 0.0f;
-    const bool cut = t > 0 && !one && __syncthreads_or(c + l < -RC_RANGE);
+    const bool cut = t > 0 && __syncthreads_or(c + l < -RC_RANGE);
     if (cut) {
       if (tid < K && t - 1 > start) e[(i64)(t - 1) * HK] = expf(c);
       mask |= 1ull << t;
@@ -125,8 +142,9 @@ fl_decay_prepare_kernel(const bxf_recurrence_rows p, const int* __restrict__ chu
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const float c0 = la[t * K + d + 2 * i], c1 = la[t * K + d + 2 * i + 1];
-      split_pair(q[2 * i] * p.q_scale * expf(c0), q[2 * i + 1] * p.q_scale * expf(c1), o[0][i], o[1][i]);
-      split_pair(kk[2 * i] * expf(-c0), kk[2 * i + 1] * expf(-c1), o[2][i], o[3][i]);
+      const float e0 = expf(c0), e1 = expf(c1);          // e^-40 at the least: the reciprocals stay finite
+      split_pair(q[2 * i] * p.q_scale * e0, q[2 * i + 1] * p.q_scale * e1, o[0][i], o[1][i]);
+      split_pair(kk[2 * i] / e0, kk[2 * i + 1] / e1, o[2][i], o[3][i]);
     }
 #pragma unroll
     for (int j = 0; j < 4; ++j)
@@ -136,12 +154,16 @@ fl_decay_prepare_kernel(const bxf_recurrence_rows p, const int* __restrict__ chu
 
 // ---- the chunk kernel ----
 struct ChunkArgs {
-  const int* runs;               // [runs, 3] (first row, rows, first chunk)
+  const int* runs;               // [runs, 3] (first row, rows, first chunk) of what a CTA walks
   const bf16* planes;            // BXF_DECAY_CHANNEL: of fl_decay_prepare_kernel
   const float* edge;
   const unsigned long long* masks;
+  float* states;                 // segments: [segments][heads][K][V] contributions, then the states they start from
+  float* decays;                 // segments: [segments][heads][K] of the whole segment
   int M;
 };
+
+enum ChunkPass { WHOLE_RUN, CONTRIBUTION, OUTPUTS };
 
 template <bool CHANNEL, int KT, int NW>
 struct ChunkCfg {
@@ -151,7 +173,7 @@ struct ChunkCfg {
   static constexpr int CTAS = SMEM * 3 <= 224 * 1024 && KT <= 8 && NW <= 4 ? 3 : SMEM * 2 <= 224 * 1024 && KT <= 8 ? 2 : 1;
 };
 
-template <bool CHANNEL, int KT, int NW>
+template <bool CHANNEL, int KT, int NW, ChunkPass PASS>
 __global__ void __launch_bounds__(32 * NW, ChunkCfg<CHANNEL, KT, NW>::CTAS)
 fl_recurrence_chunk_kernel(const bxf_recurrence_rows p, const ChunkArgs a) {
   using Cfg = ChunkCfg<CHANNEL, KT, NW>;
@@ -163,7 +185,7 @@ fl_recurrence_chunk_kernel(const bxf_recurrence_rows p, const ChunkArgs a) {
   bf16* ks = qs + Cfg::PARTS * Cfg::QK;
   bf16* vs = ks + Cfg::PARTS * Cfg::QK;                  // [64][LDV]
   bf16* as = vs + Cfg::V;                                // [2][64][72] scores, high and low parts
-  float* first = reinterpret_cast<float*>(as + 2 * Cfg::A);   // [KP] decays of the segment's first row
+  float* first = reinterpret_cast<float*>(as + 2 * Cfg::A);   // [KP] decays of the piece's first row
   float* last = first + KP;                              // [KP] e^(c_last)
   float* cum = last + KP;                                // [64] BXF_DECAY_HEAD: sums of the log decays
   float* dts = cum + RC_ROWS;                            // [64] step sizes
@@ -178,9 +200,15 @@ fl_recurrence_chunk_kernel(const bxf_recurrence_rows p, const ChunkArgs a) {
   const int lm = lane & 7, b1 = (lane >> 3) & 1, b2 = lane >> 4;
 
   // the state, transposed: value column v0 + lrow (+ 8), key channel 8 j + 2 quad (+ 1)
-  float* state = p.state + ((p.seq[row0] * p.heads + h) * K) * (i64)V;
+  float* state = (PASS == WHOLE_RUN ? p.state + ((p.seq[row0] * p.heads + h) * K) * (i64)V
+                                    : a.states + (((i64)blockIdx.x * p.heads + h) * K) * V);
   float S[2 * KT][4];
-  const bool fresh = p.flags[row0] & BXF_ROW_START;
+  const bool fresh = PASS == CONTRIBUTION || (PASS == WHOLE_RUN && (p.flags[row0] & BXF_ROW_START));
+  float total[PASS == CONTRIBUTION && CHANNEL ? 2 * KT : 1][2], total_log = 0.0f;       // decays of the segment
+  if (PASS == CONTRIBUTION && CHANNEL) {
+#pragma unroll
+    for (int j = 0; j < 2 * KT; ++j) total[j][0] = total[j][1] = 1.0f;
+  }
 #pragma unroll
   for (int j = 0; j < 2 * KT; ++j)
 #pragma unroll
@@ -196,23 +224,36 @@ fl_recurrence_chunk_kernel(const bxf_recurrence_rows p, const ChunkArgs a) {
       if (ahead) n = min(n, __ffsll(ahead));
     }
     const i64 m0 = row0 + r0;
-    // ---- rows into shared memory, zeros beyond the segment and the sizes ----
+    // ---- rows into shared memory, zeros beyond the piece and the sizes ----
+    {
+      constexpr int PER = KP / 8, STEP = THREADS / PER;                   // 16-byte pieces of a row, rows at a time
+      static_assert(THREADS % PER == 0 && RC_ROWS % STEP == 0, "a thread keeps its columns");
+      const int t0 = tid / PER, d = tid % PER * 8;
+      const int col = d < K ? d : 0;
+      const i64 ld = CHANNEL ? HK : p.ldy;
+      const bf16* q = CHANNEL ? a.planes + (m0 + t0) * HK + h * K + col : y + (m0 + t0) * p.ldy + p.q0 + g * K + col;
+      const bf16* k = CHANNEL ? q + 2 * plane : y + (m0 + t0) * p.ldy + p.k0 + g * K + col;
 #pragma unroll
-    for (int part = 0; part < Cfg::PARTS; ++part)
-      for (int at = tid; at < RC_ROWS * (KP / 8); at += THREADS) {
-        const int t = at / (KP / 8), d = at % (KP / 8) * 8;
-        const bool there = t < n && d < K;
-        const i64 m = there ? m0 + t : m0;
-        const int col = there ? d : 0;
-        const bf16* q = CHANNEL ? a.planes + part * plane + m * HK + h * K + col : y + m * p.ldy + p.q0 + g * K + col;
-        const bf16* k = CHANNEL ? a.planes + (2 + part) * plane + m * HK + h * K + col : y + m * p.ldy + p.k0 + g * K + col;
-        copy16(qs + part * Cfg::QK + t * LDK + d, q, there);
-        copy16(ks + part * Cfg::QK + t * LDK + d, k, there);
+      for (int i = 0; i < RC_ROWS / STEP; ++i) {
+        const bool there = t0 + i * STEP < n && d < K;
+        const i64 off = there ? i * STEP * ld : -t0 * ld;                 // the segment's first row stands in for none
+#pragma unroll
+        for (int part = 0; part < Cfg::PARTS; ++part) {
+          const int to = part * Cfg::QK + (t0 + i * STEP) * LDK + d;
+          if (PASS != CONTRIBUTION) copy16(qs + to, q + part * plane + off, there);
+          copy16(ks + to, k + part * plane + off, there);
+        }
       }
-    for (int at = tid; at < RC_ROWS * (Cfg::VS / 8); at += THREADS) {
-      const int t = at / (Cfg::VS / 8), d = at % (Cfg::VS / 8) * 8;
-      const bool there = t < n && c0 + d < V;
-      copy16(vs + t * LDV + d, y + (there ? m0 + t : m0) * p.ldy + p.v0 + (i64)h * V + (there ? c0 + d : 0), there);
+    }
+    {
+      constexpr int PER = Cfg::VS / 8, STEP = THREADS / PER;
+      const int t0 = tid / PER, d = tid % PER * 8;
+      const bf16* v = y + (m0 + t0) * p.ldy + p.v0 + (i64)h * V + (c0 + d < V ? c0 + d : 0);
+#pragma unroll
+      for (int i = 0; i < RC_ROWS / STEP; ++i) {
+        const bool there = t0 + i * STEP < n && c0 + d < V;
+        copy16(vs + (t0 + i * STEP) * LDV + d, v + (there ? i * STEP : -t0) * p.ldy, there);
+      }
     }
     if (CHANNEL) {
       for (int k = tid; k < KP; k += THREADS) {
@@ -238,7 +279,7 @@ fl_recurrence_chunk_kernel(const bxf_recurrence_rows p, const ChunkArgs a) {
     __syncthreads();
 
     // ---- scores: warp = 16 rows x 64 (32) columns ----
-    {
+    if (PASS != CONTRIBUTION) {
       constexpr int NT = NW == 8 ? 4 : 8;
       const int rb = warp & 3, cb = NW == 8 ? (warp >> 2) * 4 : 0;
       float acc[NT][4];
@@ -293,89 +334,93 @@ fl_recurrence_chunk_kernel(const bxf_recurrence_rows p, const ChunkArgs a) {
 #pragma unroll
         for (int i = 0; i < 4; ++i) S[j][i] *= first[8 * j + 2 * quad + (i & 1)];
     }
-    __syncthreads();
+    if (PASS != CONTRIBUTION) {
+      __syncthreads();
 
-    // ---- outputs of this warp's 16 columns: state, then scores ----
-    float o[4][2][4];
+      // ---- outputs of this warp's 16 columns: state, then scores ----
+      float o[4][2][4];
 #pragma unroll
-    for (int mt = 0; mt < 4; ++mt)
+      for (int mt = 0; mt < 4; ++mt)
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt)
+        for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) o[mt][nt][i] = 0.0f;
+          for (int i = 0; i < 4; ++i) o[mt][nt][i] = 0.0f;
 #pragma unroll
-    for (int kt = 0; kt < KT; ++kt) {
-      uint32_t hi[2][2], lo[2][2];
+      for (int kt = 0; kt < KT; ++kt) {
+        uint32_t hi[2][2], lo[2][2];
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt)
+        for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-        for (int b = 0; b < 2; ++b) split_pair(S[2 * kt + b][2 * nt], S[2 * kt + b][2 * nt + 1], hi[nt][b], lo[nt][b]);
+          for (int b = 0; b < 2; ++b) split_pair(S[2 * kt + b][2 * nt], S[2 * kt + b][2 * nt + 1], hi[nt][b], lo[nt][b]);
 #pragma unroll
-      for (int mt = 0; mt < 4; ++mt) {
-        uint32_t q[4];
-        const int at_q = (mt * 16 + b1 * 8 + lm) * LDK + kt * 16 + b2 * 8;
-        ldsm4(q, qs + at_q);
+        for (int mt = 0; mt < 4; ++mt) {
+          uint32_t q[4];
+          const int at_q = (mt * 16 + b1 * 8 + lm) * LDK + kt * 16 + b2 * 8;
+          ldsm4(q, qs + at_q);
 #pragma unroll
-        for (int nt = 0; nt < 2; ++nt) {
-          mma16816(o[mt][nt], q, hi[nt][0], hi[nt][1]);
-          mma16816(o[mt][nt], q, lo[nt][0], lo[nt][1]);
-        }
-        if (CHANNEL) {
-          ldsm4(q, qs + Cfg::QK + at_q);
-#pragma unroll
-          for (int nt = 0; nt < 2; ++nt) mma16816(o[mt][nt], q, hi[nt][0], hi[nt][1]);
-        }
-      }
-    }
-    if (!CHANNEL) {
-#pragma unroll
-      for (int mt = 0; mt < 4; ++mt) {
-        const float e0 = __expf(cum[mt * 16 + lrow]), e1 = __expf(cum[mt * 16 + lrow + 8]);
-#pragma unroll
-        for (int nt = 0; nt < 2; ++nt) {
-          o[mt][nt][0] *= e0;
-          o[mt][nt][1] *= e0;
-          o[mt][nt][2] *= e1;
-          o[mt][nt][3] *= e1;
-        }
-      }
-    }
-#pragma unroll
-    for (int sk = 0; sk < 4; ++sk) {
-      uint32_t v[4];
-      ldsm4_t(v, vs + (sk * 16 + b1 * 8 + lm) * LDV + warp * 16 + b2 * 8);
-#pragma unroll
-      for (int mt = sk; mt < 4; ++mt)
-#pragma unroll
-        for (int part = 0; part < 2; ++part) {
-          uint32_t s[4];
-          ldsm4(s, as + part * Cfg::A + (mt * 16 + b1 * 8 + lm) * RC_LDA + sk * 16 + b2 * 8);
-          mma16816(o[mt][0], s, v[0], v[1]);
-          mma16816(o[mt][1], s, v[2], v[3]);
-        }
-    }
-#pragma unroll
-    for (int mt = 0; mt < 4; ++mt)
-#pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int t = mt * 16 + lrow + half * 8;
-        if (t >= n) continue;
-        bf16* out = static_cast<bf16*>(p.out) + (m0 + t) * p.ldo + (i64)h * V;
-#pragma unroll
-        for (int nt = 0; nt < 2; ++nt) {
-          const int col = v0 + nt * 8 + 2 * quad;
-          if (col >= V) continue;
-          float x0 = o[mt][nt][2 * half], x1 = o[mt][nt][2 * half + 1];
-          if (!CHANNEL) {
-            const uint32_t x = *reinterpret_cast<const uint32_t*>(vs + t * LDV + warp * 16 + nt * 8 + 2 * quad);
-            x0 = fmaf(skip, __uint_as_float(x << 16), x0);
-            x1 = fmaf(skip, __uint_as_float(x & 0xffff0000u), x1);
+          for (int nt = 0; nt < 2; ++nt) {
+            mma16816(o[mt][nt], q, hi[nt][0], hi[nt][1]);
+            mma16816(o[mt][nt], q, lo[nt][0], lo[nt][1]);
           }
-          *reinterpret_cast<uint32_t*>(out + col) = pack_bf16(x0, x1);
+          if (CHANNEL) {
+            ldsm4(q, qs + Cfg::QK + at_q);
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt) mma16816(o[mt][nt], q, hi[nt][0], hi[nt][1]);
+          }
         }
       }
+      if (!CHANNEL) {
+#pragma unroll
+        for (int mt = 0; mt < 4; ++mt) {
+          const float e0 = __expf(cum[mt * 16 + lrow]), e1 = __expf(cum[mt * 16 + lrow + 8]);
+#pragma unroll
+          for (int nt = 0; nt < 2; ++nt) {
+            o[mt][nt][0] *= e0;
+            o[mt][nt][1] *= e0;
+            o[mt][nt][2] *= e1;
+            o[mt][nt][3] *= e1;
+          }
+        }
+      }
+#pragma unroll
+      for (int sk = 0; sk < 4; ++sk) {
+        uint32_t v[4];
+        ldsm4_t(v, vs + (sk * 16 + b1 * 8 + lm) * LDV + warp * 16 + b2 * 8);
+#pragma unroll
+        for (int mt = sk; mt < 4; ++mt)
+#pragma unroll
+          for (int part = 0; part < 2; ++part) {
+            uint32_t s[4];
+            ldsm4(s, as + part * Cfg::A + (mt * 16 + b1 * 8 + lm) * RC_LDA + sk * 16 + b2 * 8);
+            mma16816(o[mt][0], s, v[0], v[1]);
+            mma16816(o[mt][1], s, v[2], v[3]);
+          }
+      }
+#pragma unroll
+      for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int t = mt * 16 + lrow + half * 8;
+          if (t >= n) continue;
+          bf16* out = static_cast<bf16*>(p.out) + (m0 + t) * p.ldo + (i64)h * V;
+#pragma unroll
+          for (int nt = 0; nt < 2; ++nt) {
+            const int col = v0 + nt * 8 + 2 * quad;
+            if (col >= V) continue;
+            float x0 = o[mt][nt][2 * half], x1 = o[mt][nt][2 * half + 1];
+            if (!CHANNEL) {
+              const uint32_t x = *reinterpret_cast<const uint32_t*>(vs + t * LDV + warp * 16 + nt * 8 + 2 * quad);
+              x0 = fmaf(skip, __uint_as_float(x << 16), x0);
+              x1 = fmaf(skip, __uint_as_float(x & 0xffff0000u), x1);
+            }
+            *reinterpret_cast<uint32_t*>(out + col) = pack_bf16(x0, x1);
+          }
+        }
 
-    // ---- the state after the segment ----
+    }
+
+    // ---- the state after the piece ----
+    if (PASS == CONTRIBUTION && !CHANNEL) total_log += cum[RC_ROWS - 1];
     if (!CHANNEL) {
       const float e = __expf(cum[RC_ROWS - 1]);
 #pragma unroll
@@ -421,8 +466,27 @@ fl_recurrence_chunk_kernel(const bxf_recurrence_rows p, const ChunkArgs a) {
       for (int j = 0; j < 2 * KT; ++j)
 #pragma unroll
         for (int i = 0; i < 4; ++i) S[j][i] *= last[8 * j + 2 * quad + (i & 1)];
+      if (PASS == CONTRIBUTION) {
+#pragma unroll
+        for (int j = 0; j < 2 * KT; ++j)
+#pragma unroll
+          for (int i = 0; i < 2; ++i) total[j][i] *= first[8 * j + 2 * quad + i] * last[8 * j + 2 * quad + i];
+      }
     }
-    __syncthreads();                                     // the next segment overwrites the operands
+    __syncthreads();                                     // the next piece overwrites the operands
+  }
+  if (PASS == OUTPUTS) return;
+  if (PASS == CONTRIBUTION && blockIdx.z == 0) {
+    float* decays = a.decays + ((i64)blockIdx.x * p.heads + h) * K;
+    if (CHANNEL) {
+#pragma unroll
+      for (int j = 0; j < 2 * KT; ++j)
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+          if (warp == 0 && lrow == 0 && 8 * j + 2 * quad + i < K) decays[8 * j + 2 * quad + i] = total[j][i];
+    } else {
+      for (int k = tid; k < K; k += THREADS) decays[k] = expf(total_log);
+    }
   }
 #pragma unroll
   for (int j = 0; j < 2 * KT; ++j)
@@ -431,6 +495,39 @@ fl_recurrence_chunk_kernel(const bxf_recurrence_rows p, const ChunkArgs a) {
       const int k = 8 * j + 2 * quad + (i & 1), v = v0 + lrow + (i >> 1) * 8;
       if (k < K && v < V) state[(i64)k * V + v] = S[j][i];
     }
+}
+
+// The states that the segments of a run start from, in place of their contributions, and the state after the run. spans
+// [runs, 3] (first row, first segment, segments). Thread = 4 consecutive values.
+__global__ void __launch_bounds__(256) fl_recurrence_chain_kernel(const bxf_recurrence_rows p, const int* spans, float* states,
+                                                                  const float* decays) {
+  launch_next();
+  wait_previous();
+  const int row0 = spans[blockIdx.x * 3], seg0 = spans[blockIdx.x * 3 + 1], segs = spans[blockIdx.x * 3 + 2], h = blockIdx.y;
+  const int at = (blockIdx.z * 256 + threadIdx.x) * 4, k = at / p.V;
+  const i64 size = (i64)p.K * p.V;
+  if (at >= size) return;
+  float* state = p.state + (p.seq[row0] * p.heads + h) * size + at;
+  float S[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+  if (!(p.flags[row0] & BXF_ROW_START)) load_v<4>(state, S);
+  for (int s0 = 0; s0 < segs; s0 += 4) {                 // four segments' contributions in flight
+    float c[4][4], d[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (s0 + j < segs) {
+        const i64 n = (i64)(seg0 + s0 + j) * p.heads + h;
+        load_v<4>(states + n * size + at, c[j]);
+        d[j] = decays[n * p.K + k];
+      }
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (s0 + j < segs) {
+        store_v<4>(states + ((i64)(seg0 + s0 + j) * p.heads + h) * size + at, S);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) S[i] = fmaf(d[j], S[i], c[j][i]);
+      }
+  }
+  store_v<4>(state, S);
 }
 
 }  // namespace bxf

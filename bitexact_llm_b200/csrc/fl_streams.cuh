@@ -9,15 +9,19 @@ namespace bxf {
 
 // V consecutive values: 16-byte accesses for V = 8 (the address is aligned), single ones for V = 1.
 template <int V>
+__device__ __forceinline__ void load_v(const uint4& u, float (&v)[V]) {
+  static_assert(V == 8, "eight bf16 values");
+  const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    v[2 * i] = __uint_as_float(w[i] << 16);
+    v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+  }
+}
+template <int V>
 __device__ __forceinline__ void load_v(const bf16* p, float (&v)[V]) {
   if constexpr (V == 8) {
-    const uint4 u = *reinterpret_cast<const uint4*>(p);
-    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      v[2 * i] = __uint_as_float(w[i] << 16);
-      v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
-    }
+    load_v<8>(*reinterpret_cast<const uint4*>(p), v);
   } else {
 #pragma unroll
     for (int i = 0; i < V; ++i) v[i] = ld(p + i);
@@ -185,7 +189,7 @@ __global__ void __launch_bounds__(PREP_THREADS) fl_gqa_prepare_kernel(const bxf_
   T* rows = static_cast<T*>(p.cache) + (slot / p.page * p.kv_heads * p.page + slot % p.page) * p.ldc;   // of group 0
   const i64 group_stride = p.page * p.ldc;
   const int half = p.rot_dims / 2;
-  const float2* cs = reinterpret_cast<const float2*>(p.cs) + m * half;
+  const float* cs = p.cs + m * half * 2;
   for (int e = threadIdx.x * V; e < nq + nk; e += PREP_THREADS * V) {
     const bool is_q = e < nq;
     const float r = is_q ? rq : rk;
@@ -198,8 +202,7 @@ __global__ void __launch_bounds__(PREP_THREADS) fl_gqa_prepare_kernel(const bxf_
       for (int i = 0; i < V; ++i) o[i] *= r;
       if (w) {
         float g[V];
-#pragma unroll
-        for (int i = 0; i < V; ++i) g[i] = w[at + i];
+        load_v<V>(w + at, g);
 #pragma unroll
         for (int i = 0; i < V; ++i) o[i] *= g[i];
       }
@@ -208,11 +211,15 @@ __global__ void __launch_bounds__(PREP_THREADS) fl_gqa_prepare_kernel(const bxf_
     if (d < p.rot_dims) {
       float o[V];
       normed(d < half ? e + half : e - half, o);
-#pragma unroll
-      for (int i = 0; i < V; ++i) {
-        const float2 c = cs[(d < half ? d : d - half) + i];
-        v[i] = d < half ? v[i] * c.x - o[i] * c.y : v[i] * c.x + o[i] * c.y;
+      float c[2 * V];
+      if constexpr (V == 8) {
+        load_v<16>(cs + (d < half ? d : d - half) * 2, c);
+      } else {
+        c[0] = cs[(d < half ? d : d - half) * 2];
+        c[1] = cs[(d < half ? d : d - half) * 2 + 1];
       }
+#pragma unroll
+      for (int i = 0; i < V; ++i) v[i] = d < half ? v[i] * c[2 * i] - o[i] * c[2 * i + 1] : v[i] * c[2 * i] + o[i] * c[2 * i + 1];
     }
     T* to = is_q ? static_cast<T*>(p.q) + (((i64)(h / per) * M + m) * per + h % per) * p.ldq + d : rows + h * group_stride + d;
     store_v<V>(to, v);

@@ -19,8 +19,8 @@ namespace {
 using namespace bxf;
 
 static_assert(sizeof(bxf_epilogue) == 136 && sizeof(bxf_gru) == 56 && sizeof(bxf_streams_step) == 112 &&
-                  sizeof(bxf_gqa_rows) == 120 && sizeof(bxf_conv) == 72 && sizeof(bxf_recurrence_rows) == 224 &&
-                  sizeof(bxf_gate_rows) == 152,
+                  sizeof(bxf_gqa_rows) == 120 && sizeof(bxf_conv) == 72 && sizeof(bxf_recurrence_rows) == 152 &&
+                  sizeof(bxf_gate_rows) == 152 && sizeof(bxf_chunk_table) == 48,
               "layouts of the callers' structs");
 
 inline cudaStream_t stream_of(void* s) { return static_cast<cudaStream_t>(s); }
@@ -335,29 +335,37 @@ bool recurrence_ok(const bxf_recurrence_rows* p) {
   return p->kind == BXF_DECAY_HEAD && p->A_log && p->skip;
 }
 
-template <class T, bool CHANNEL, int KR>
-int launch_recurrence_as(const bxf_recurrence_rows& p, int M, cudaStream_t st) {
-  const int smem = recurrence_smem(p.K, CHANNEL);
+template <class T, bool CHANNEL, int CW, int KR, int ROWS>
+int launch_recurrence_rows(const bxf_recurrence_rows& p, int M, cudaStream_t st) {
+  const int smem = recurrence_smem(p.K, CW, CHANNEL, ROWS);
   static PerDevice configured;
   if (once_per_device(configured, [] {
-        return cudaFuncSetAttribute(fl_recurrence_kernel<T, CHANNEL, KR>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                    recurrence_smem(REC_LANES * KR, CHANNEL));
+        return cudaFuncSetAttribute(fl_recurrence_kernel<T, CHANNEL, CW, KR, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                    recurrence_smem(REC_THREADS / CW * KR, CW, CHANNEL, ROWS));
       }) != BX_OK)
     return BX_ELAUNCH;
-  return launch_chained(fl_recurrence_kernel<T, CHANNEL, KR>, dim3(M, p.heads, ceil_div(p.V, REC_COLS)), REC_THREADS, smem, st, 0,
-                        p, M);
+  return launch_chained(fl_recurrence_kernel<T, CHANNEL, CW, KR, ROWS>, dim3(M, p.heads, ceil_div(p.V, 4 * CW)), REC_THREADS,
+                        smem, st, 0, p, M);
+}
+
+template <class T, bool CHANNEL, int CW, int KR>
+int launch_recurrence_as(const bxf_recurrence_rows& p, int M, cudaStream_t st) {
+  if (std::is_same<T, bf16>::value && p.batch == 1) return launch_recurrence_rows<T, CHANNEL, CW, KR, 1>(p, M, st);
+  return launch_recurrence_rows<T, CHANNEL, CW, KR, REC_ROWS>(p, M, st);
 }
 
 template <class T>
 int launch_recurrence(const bxf_recurrence_rows& p, int M, cudaStream_t st) {
-  const int kr = ceil_div(p.K, REC_LANES);
   auto go = [&](auto channel) {
     constexpr bool C = decltype(channel)::value;
-    if (kr <= 1) return launch_recurrence_as<T, C, 1>(p, M, st);
-    if (kr <= 2) return launch_recurrence_as<T, C, 2>(p, M, st);
-    if (kr <= 4) return launch_recurrence_as<T, C, 4>(p, M, st);
-    if (kr <= 8) return launch_recurrence_as<T, C, 8>(p, M, st);
-    return launch_recurrence_as<T, C, 16>(p, M, st);
+    if (p.V >= 64 && p.K <= 128 && (i64)M * p.heads * ceil_div(p.V, 64) >= 4 * 148)
+      return p.K <= 64 ? launch_recurrence_as<T, C, 16, 4>(p, M, st) : launch_recurrence_as<T, C, 16, 8>(p, M, st);
+    const int kr = ceil_div(p.K, 32);
+    if (kr <= 1) return launch_recurrence_as<T, C, 8, 1>(p, M, st);
+    if (kr <= 2) return launch_recurrence_as<T, C, 8, 2>(p, M, st);
+    if (kr <= 4) return launch_recurrence_as<T, C, 8, 4>(p, M, st);
+    if (kr <= 8) return launch_recurrence_as<T, C, 8, 8>(p, M, st);
+    return launch_recurrence_as<T, C, 8, 16>(p, M, st);
   };
   return p.kind == BXF_DECAY_CHANNEL ? go(std::true_type{}) : go(std::false_type{});
 }
@@ -366,39 +374,56 @@ int launch_recurrence(const bxf_recurrence_rows& p, int M, cudaStream_t st) {
 bool chunks_fit(int dtype, int K, int V) { return dtype == BXF_BF16 && K % 8 == 0 && V % 8 == 0 && K <= RC_MAX_K; }
 
 struct ChunkScratch {
-  size_t planes, edge, masks, bytes;
+  size_t planes, edge, masks, states, decays, bytes;     // sizes, in this order
 };
 
-ChunkScratch chunk_scratch(int M, int chunks, int heads, int K) {
+ChunkScratch chunk_scratch(int kind, int M, int chunks, int segments, int heads, int K, int V) {
   const auto up = [](size_t n) { return (n + 255) / 256 * 256; };
+  const size_t channel = kind == BXF_DECAY_CHANNEL ? 1 : 0;
   ChunkScratch s;
-  s.planes = up((size_t)4 * M * heads * K * 2);
-  s.edge = up((size_t)M * heads * K * 4);
-  s.masks = up((size_t)chunks * heads * 8);
-  s.bytes = s.planes + s.edge + s.masks;
+  s.planes = up(channel * 4 * M * heads * K * 2);
+  s.edge = up(channel * M * heads * K * 4);
+  s.masks = up(channel * chunks * heads * 8);
+  s.states = up((size_t)segments * heads * K * V * 4);
+  s.decays = up((size_t)segments * heads * K * 4);
+  s.bytes = s.planes + s.edge + s.masks + s.states + s.decays;
   return s;
 }
 
-template <bool CHANNEL, int KT, int NW>
-int launch_chunks_as(const bxf_recurrence_rows& p, const ChunkArgs& a, int nruns, cudaStream_t st) {
+template <bool CHANNEL, int KT, int NW, ChunkPass PASS>
+int launch_chunk_pass(const bxf_recurrence_rows& p, const ChunkArgs& a, int n, cudaStream_t st) {
   using Cfg = ChunkCfg<CHANNEL, KT, NW>;
   static PerDevice configured;
   if (once_per_device(configured, [] {
-        return cudaFuncSetAttribute(fl_recurrence_chunk_kernel<CHANNEL, KT, NW>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                    Cfg::SMEM);
+        return cudaFuncSetAttribute(fl_recurrence_chunk_kernel<CHANNEL, KT, NW, PASS>,
+                                    cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM);
       }) != BX_OK)
     return BX_ELAUNCH;
-  return launch_chained(fl_recurrence_chunk_kernel<CHANNEL, KT, NW>, dim3(nruns, p.heads, ceil_div(p.V, Cfg::VS)), 32 * NW,
+  return launch_chained(fl_recurrence_chunk_kernel<CHANNEL, KT, NW, PASS>, dim3(n, p.heads, ceil_div(p.V, Cfg::VS)), 32 * NW,
                         Cfg::SMEM, st, 0, p, a);
 }
 
+// nsegs = 0: every CTA walks a whole run.
+template <bool CHANNEL, int KT>
+int launch_chunks_as(const bxf_recurrence_rows& p, ChunkArgs a, int nruns, const int* segs, int nsegs, const int* spans,
+                     cudaStream_t st) {
+  if (nsegs == 0) return launch_chunk_pass<CHANNEL, KT, 4, WHOLE_RUN>(p, a, nruns, st);
+  a.runs = segs;
+  int rc = launch_chunk_pass<CHANNEL, KT, 4, CONTRIBUTION>(p, a, nsegs, st);
+  if (rc != BX_OK) return rc;
+  rc = launch_chained(fl_recurrence_chain_kernel, dim3(nruns, p.heads, ceil_div(p.K * p.V, 1024)), 256, 0, st, 0, p, spans, a.states,
+                      a.decays);
+  return rc != BX_OK ? rc : launch_chunk_pass<CHANNEL, KT, 4, OUTPUTS>(p, a, nsegs, st);
+}
+
 template <bool CHANNEL>
-int launch_chunks(const bxf_recurrence_rows& p, const ChunkArgs& a, int nruns, cudaStream_t st) {
+int launch_chunks(const bxf_recurrence_rows& p, const ChunkArgs& a, int nruns, const int* segs, int nsegs, const int* spans,
+                  cudaStream_t st) {
   const int kt = ceil_div(p.K, 16);
-  if (kt <= 2) return launch_chunks_as<CHANNEL, 2, 4>(p, a, nruns, st);
-  if (kt <= 4) return launch_chunks_as<CHANNEL, 4, 4>(p, a, nruns, st);
-  if (kt <= 8) return launch_chunks_as<CHANNEL, 8, 4>(p, a, nruns, st);
-  return launch_chunks_as<CHANNEL, 16, 4>(p, a, nruns, st);
+  if (kt <= 2) return launch_chunks_as<CHANNEL, 2>(p, a, nruns, segs, nsegs, spans, st);
+  if (kt <= 4) return launch_chunks_as<CHANNEL, 4>(p, a, nruns, segs, nsegs, spans, st);
+  if (kt <= 8) return launch_chunks_as<CHANNEL, 8>(p, a, nruns, segs, nsegs, spans, st);
+  return launch_chunks_as<CHANNEL, 16>(p, a, nruns, segs, nsegs, spans, st);
 }
 
 template <class T>
@@ -638,39 +663,54 @@ int bxf_causal_conv(int dtype, const bxf_conv* c, void* out, int64_t ldo, int M,
   if (dtype == BXF_F32)
     return launch_chained(fl_causal_conv_kernel<float>, grid, CONV_THREADS, 0, st, 0, *c, static_cast<float*>(out), ldo, M);
   if (c->taps >= 2 && c->taps <= 4 && c->channels % 8 == 0 && c->ldu % 8 == 0 && ldo % 8 == 0 && aligned16(c->u) &&
-      aligned16(out) && aligned16(c->state)) {
-    const dim3 wide(ceil_div(c->channels, 8 * CONV_THREADS), ceil_div(M, CONV_ROWS));
+      aligned16(out) && aligned16(c->state) && aligned16(c->w) && aligned16(c->b)) {
+    const int rows = M <= 512 ? 1 : CONV_ROWS;
+    const dim3 wide(ceil_div(c->channels, 8 * CONV_THREADS), ceil_div(M, rows));
     return launch_chained(c->taps == 2 ? fl_causal_conv_rows_kernel<2> : c->taps == 3 ? fl_causal_conv_rows_kernel<3>
                                                                                       : fl_causal_conv_rows_kernel<4>,
-                          wide, CONV_THREADS, 0, st, 0, *c, static_cast<bf16*>(out), ldo, M);
+                          wide, CONV_THREADS, 0, st, 0, *c, static_cast<bf16*>(out), ldo, M, rows);
   }
   return launch_chained(fl_causal_conv_kernel<bf16>, grid, CONV_THREADS, 0, st, 0, *c, static_cast<bf16*>(out), ldo, M);
 }
 
 int bxf_recurrence(int dtype, const bxf_recurrence_rows* p, int M, void* stream) {
-  if (!dtype_ok(dtype) || !recurrence_ok(p) || M < 0 || (p->conv.w && !conv_ok(&p->conv))) return BX_EARG;
-  if (p->K > BXF_MAX_STATE || p->heads > 65535 || ceil_div(p->V, REC_COLS) > 65535) return BX_ELIMIT;
+  if (!dtype_ok(dtype) || !recurrence_ok(p) || M < 0) return BX_EARG;
+  if (p->K > BXF_MAX_STATE || p->heads > 65535 || ceil_div(p->V, 32) > 65535) return BX_ELIMIT;
   if (M == 0) return BX_OK;
   return dtype == BXF_F32 ? launch_recurrence<float>(*p, M, stream_of(stream)) : launch_recurrence<bf16>(*p, M, stream_of(stream));
 }
 
 int bxf_recurrence_chunk_rows(int dtype, int K, int V) { return chunks_fit(dtype, K, V) ? RC_ROWS : 0; }
 
-size_t bxf_recurrence_chunk_scratch(int kind, int M, int chunks, int heads, int K) {
-  return kind == BXF_DECAY_CHANNEL && M > 0 && chunks > 0 && heads > 0 && K > 0 ? chunk_scratch(M, chunks, heads, K).bytes : 0;
+size_t bxf_recurrence_chunk_scratch(int kind, int M, int chunks, int segments, int heads, int K, int V) {
+  if (M < 1 || chunks < 1 || segments < 0 || heads < 1 || K < 1 || V < 1) return 0;
+  return chunk_scratch(kind, M, chunks, segments, heads, K, V).bytes;
 }
 
-int bxf_recurrence_chunks(int dtype, const bxf_recurrence_rows* p, const int* runs, int nruns, const int* chunks, int nchunks,
-                          void* scratch, size_t scratch_bytes, int M, void* stream) {
-  if (!recurrence_ok(p) || p->conv.w || M < 0 || !runs || !chunks || nruns < 0 || nchunks < nruns) return BX_EARG;
-  if (!chunks_fit(dtype, p->K, p->V) || p->heads > 65535) return BX_ELIMIT;
-  if (p->ldy % 8 || p->q0 % 8 || p->k0 % 8 || p->v0 % 8 || p->ldo % 2 || !aligned16(p->y)) return BX_EARG;
-  if (M == 0 || nruns == 0) return BX_OK;
+int bxf_recurrence_chunks(int dtype, const bxf_recurrence_rows* p, const bxf_chunk_table* t, void* scratch,
+                          size_t scratch_bytes, int M, void* stream) {
+  if (!recurrence_ok(p) || !t || M < 0 || !t->runs || !t->chunks || t->nruns < 0 || t->nchunks < t->nruns || t->nsegments < 0 ||
+      (t->nsegments > 0 && (!t->segments || !t->spans)))
+    return BX_EARG;
+  if (!chunks_fit(dtype, p->K, p->V) || p->heads > 65535 || ceil_div(p->K * p->V, 1024) > 65535) return BX_ELIMIT;
+  if (p->ldy % 8 || p->q0 % 8 || p->k0 % 8 || p->v0 % 8 || p->ldo % 2 || !aligned16(p->y) || !aligned16(p->state)) return BX_EARG;
+  if (M == 0 || t->nruns == 0) return BX_OK;
+  const ChunkScratch s = chunk_scratch(p->kind, M, t->nchunks, t->nsegments, p->heads, p->K, p->V);
+  if (s.bytes > 0 && (!scratch || !aligned16(scratch) || scratch_bytes < s.bytes)) return BX_EARG;
+  uint8_t* at = static_cast<uint8_t*>(scratch);
+  const auto take = [&](size_t bytes) {
+    uint8_t* r = at;
+    at += bytes;
+    return r;
+  };
+  bf16* planes = reinterpret_cast<bf16*>(take(s.planes));
+  float* edge = reinterpret_cast<float*>(take(s.edge));
+  auto* masks = reinterpret_cast<unsigned long long*>(take(s.masks));
+  float* states = reinterpret_cast<float*>(take(s.states));
+  float* decays = reinterpret_cast<float*>(take(s.decays));
+  const ChunkArgs a{t->runs, planes, edge, masks, states, decays, M};
   cudaStream_t st = stream_of(stream);
-  ChunkArgs a{runs, nullptr, nullptr, nullptr, M};
-  if (p->kind == BXF_DECAY_HEAD) return launch_chunks<false>(*p, a, nruns, st);
-  const ChunkScratch s = chunk_scratch(M, nchunks, p->heads, p->K);
-  if (!scratch || !aligned16(scratch) || scratch_bytes < s.bytes) return BX_EARG;
+  if (p->kind == BXF_DECAY_HEAD) return launch_chunks<false>(*p, a, t->nruns, t->segments, t->nsegments, t->spans, st);
   const int smem = decay_prepare_smem(p->K, p->rank);
   if (smem > 200 * 1024) return BX_ELIMIT;
   static PerDevice configured;
@@ -678,17 +718,9 @@ int bxf_recurrence_chunks(int dtype, const bxf_recurrence_rows* p, const int* ru
         return cudaFuncSetAttribute(fl_decay_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
       }) != BX_OK)
     return BX_ELAUNCH;
-  uint8_t* base = static_cast<uint8_t*>(scratch);
-  bf16* planes = reinterpret_cast<bf16*>(base);
-  float* edge = reinterpret_cast<float*>(base + s.planes);
-  unsigned long long* masks = reinterpret_cast<unsigned long long*>(base + s.planes + s.edge);
-  const int rc = launch_chained(fl_decay_prepare_kernel, dim3(nchunks, p->heads), RP_THREADS, smem, st, 0, *p, chunks, planes, edge,
-                                masks, M);
-  if (rc != BX_OK) return rc;
-  a.planes = planes;
-  a.edge = edge;
-  a.masks = masks;
-  return launch_chunks<true>(*p, a, nruns, st);
+  const int rc = launch_chained(fl_decay_prepare_kernel, dim3(t->nchunks, p->heads), RP_THREADS, smem, st, 0, *p, t->chunks, planes,
+                                edge, masks, M);
+  return rc != BX_OK ? rc : launch_chunks<true>(*p, a, t->nruns, t->segments, t->nsegments, t->spans, st);
 }
 
 int bxf_gated_norm(int dtype, const bxf_gate_rows* p, int M, void* stream) {

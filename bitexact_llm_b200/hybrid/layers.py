@@ -36,28 +36,33 @@ class Step:
 
 class Tiles:
     """What the tile kernels of a prompt portion walk: attention tiles int32 [T, 3] (table row, first row, rows) by their
-    number of tokens; the runs int32 [R, 3] (first row, rows, first chunk) of its sequences and their chunks int32 [C, 2]
-    (first row, rows) for the recurrences."""
+    number of tokens; for the recurrences the runs int32 [R, 3] (first row, rows, first chunk) of its sequences, their chunks
+    int32 [C, 2] (first row, rows), the segments [S, 3] (like runs) that long runs are cut into and the spans [R, 3] (first row,
+    first segment, segments) of the runs."""
 
-    CHUNK = 64
+    CHUNK, SEGMENT = 64, 512    # a segment costs two passes over the states: short ones only where rows are few
 
-    def __init__(self, attention, runs, chunks):
-        self.attention, self.runs, self.chunks = attention, runs, chunks
+    def __init__(self, attention, runs, chunks, segments, spans):
+        self.attention, self.runs, self.chunks, self.segments, self.spans = attention, runs, chunks, segments, spans
 
     @classmethod
     def of(cls, runs, sizes):
         """runs = [(table row, first token row, tokens, context length)], sizes: the tile heights in use."""
         table = lambda n: torch.tensor([[r, t0 + s, min(n, ql - s)] for r, t0, ql, _ in runs for s in range(0, ql, n)],
                                        dtype=torch.int32).reshape(-1, 3)
-        per_run, chunks = [], []
+        size = cls.SEGMENT if sum(ql for _, _, ql, _ in runs) >= 4096 else cls.SEGMENT // 2
+        per_run, chunks, segments, spans = [], [], [], []
         for _, t0, ql, _ in runs:
             per_run.append([t0, ql, len(chunks)])
+            spans.append([t0, len(segments), (ql + size - 1) // size])
+            segments += [[t0 + s, min(size, ql - s), len(chunks) + s // cls.CHUNK] for s in range(0, ql, size)]
             chunks += [[t0 + s, min(cls.CHUNK, ql - s)] for s in range(0, ql, cls.CHUNK)]
-        return cls({n: table(n) for n in sizes}, torch.tensor(per_run, dtype=torch.int32).reshape(-1, 3),
-                   torch.tensor(chunks, dtype=torch.int32).reshape(-1, 2))
+        tensor = lambda rows, n: torch.tensor(rows, dtype=torch.int32).reshape(-1, n)
+        return cls({n: table(n) for n in sizes}, tensor(per_run, 3), tensor(chunks, 2), tensor(segments, 3), tensor(spans, 3))
 
     def to(self, dev):
-        return Tiles({n: t.to(dev) for n, t in self.attention.items()}, self.runs.to(dev), self.chunks.to(dev))
+        return Tiles({n: t.to(dev) for n, t in self.attention.items()},
+                     *(t.to(dev) for t in (self.runs, self.chunks, self.segments, self.spans)))
 
     def chunked(self, K, V, rows):
         """Whether a recurrence of these sizes runs in chunks: portions of a few rows are shorter row by row."""
@@ -198,7 +203,7 @@ class GLA:
         self.spec, self.D = spec, D
         self.first = ops.pack(torch.cat([w["q"], w["k"], w["v"], w["g"], w["a1"]]), dtype, dev)
         self.rank = w["a1"].shape[0]
-        self.a2, self.a2_b, self.norm = (_vec(w[n], dev) for n in ("a2", "a2.b", "norm"))
+        self.a2, self.a2_b, self.norm = _vec(w["a2"].t(), dev), _vec(w["a2.b"], dev), _vec(w["norm"], dev)
         self.o = ops.pack(w["o"], dtype, dev)
 
     def new_cache(self, n_seqs, n_blocks, bs):
@@ -229,9 +234,10 @@ class Mamba2:
         self.conv, self.conv_b, self.dt_bias, self.A_log, self.skip, self.norm = (
             _vec(w[n], dev) for n in ("conv", "conv.b", "dt_bias", "A_log", "D", "norm"))
         self.o = ops.pack(w["o"], dtype, dev)
-        self.channels = self.conv.shape[0]
+        self.channels, taps = self.conv.shape
+        self.conv = self.conv.t().contiguous()
         inner = spec.heads * spec.vdim
-        if self.channels != inner + 2 * spec.groups * spec.state or self.conv.shape[1] != spec.taps or inner % spec.norm_groups:
+        if self.channels != inner + 2 * spec.groups * spec.state or taps != spec.taps or inner % spec.norm_groups:
             raise ValueError("mamba2: sizes of the convolution or the norm groups do not fit")
 
     def new_cache(self, n_seqs, n_blocks, bs):
@@ -247,12 +253,9 @@ class Mamba2:
         dt = torch.empty(M, sp.heads, dtype=torch.float32, device=x.device)
         ops.linear(self.first, h, M, n + sp.heads, self.D, ops.store(y, y.shape[1], n, side=dt, bias=self.dt_bias))
         conv = ops.conv_of(y[:, inner:], self.conv, self.conv_b, cache[1], step)
-        if step.tiles is not None and inner % 8 == 0 and step.tiles.chunked(sp.state, sp.vdim, M):
-            o = ops.recurrence(ops.DECAY_HEAD, ops.causal_conv(conv, M, y), dt, cache[0], step, sp.groups, (inner + gn, inner, 0),
-                               A_log=self.A_log, skip=self.skip, tiles=step.tiles)
-        else:
-            o = ops.recurrence(ops.DECAY_HEAD, y, dt, cache[0], step, sp.groups, (2 * inner + gn, 2 * inner, inner), conv=conv,
-                               A_log=self.A_log, skip=self.skip)
+        o = ops.recurrence(ops.DECAY_HEAD, ops.causal_conv(conv, M, y), dt, cache[0], step, sp.groups, (inner + gn, inner, 0),
+                           A_log=self.A_log, skip=self.skip,
+                           tiles=step.tiles if step.tiles is not None and step.tiles.chunked(sp.state, sp.vdim, M) else None)
         o = ops.gated_norm(o, y, inner, sp.norm_groups, self.norm, sp.eps, gate_first=True, conv=conv)
         ops.linear(self.o, o, M, self.D, inner, ops.sublayer_output(x, add))
 

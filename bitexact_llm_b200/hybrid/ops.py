@@ -214,10 +214,10 @@ def gqa_attention(q, spec, cache, bt, seq, pos, sink, tiles=None, variant=0):
 
 
 def conv_of(u, w, b, state, step):
-    """bxf_conv of inputs u T [M, channels] (a view into wider rows), w float [channels, taps]."""
+    """bxf_conv of inputs u T [M, channels] (a view into wider rows), w float [taps, channels]."""
     return nv.Conv(u=u.data_ptr(), ldu=u.stride(0), w=w.data_ptr(), b=b.data_ptr(), state=state.data_ptr(),
-                   flags=step.flags.data_ptr(), seq=step.seq.data_ptr(), pos=step.pos.data_ptr(), channels=w.shape[0],
-                   taps=w.shape[1])
+                   flags=step.flags.data_ptr(), seq=step.seq.data_ptr(), pos=step.pos.data_ptr(), channels=w.shape[1],
+                   taps=w.shape[0])
 
 
 def causal_conv(conv, M, like):
@@ -228,28 +228,28 @@ def causal_conv(conv, M, like):
     return out
 
 
-def recurrence(kind, y, side, state, step, groups, columns, conv=None, a2=None, a2_b=None, inv_tau=0.0, q_scale=1.0,
+def recurrence(kind, y, side, state, step, groups, columns, a2=None, a2_b=None, inv_tau=0.0, q_scale=1.0,
                A_log=None, skip=None, tiles=None):
     """state float [slots, heads, K, V] is advanced by the rows of y; columns = where q, k, v begin in y -> outputs T
     [M, pad8(heads V)]. tiles: the chunk kernels walk its runs, else the rows go one by one."""
     M, (_, H, K, V) = y.shape[0], state.shape
     out = torch.empty(M, pad8(H * V), dtype=y.dtype, device=y.device)
-    p = nv.RecurrenceRows(kind=kind, heads=H, groups=groups, K=K, V=V, rank=0 if a2 is None else a2.shape[1], q0=columns[0],
-                          k0=columns[1], v0=columns[2], y=y.data_ptr(), ldy=y.stride(0), side=side.data_ptr(),
+    p = nv.RecurrenceRows(kind=kind, heads=H, groups=groups, K=K, V=V, rank=0 if a2 is None else a2.shape[0], q0=columns[0],
+                          k0=columns[1], v0=columns[2], batch=int(step.tiles is None), y=y.data_ptr(), ldy=y.stride(0), side=side.data_ptr(),
                           lds=side.stride(0), a2=nv.ptr(a2), a2_b=nv.ptr(a2_b), inv_tau=inv_tau, q_scale=q_scale,
                           A_log=nv.ptr(A_log), skip=nv.ptr(skip), state=state.data_ptr(), flags=step.flags.data_ptr(),
                           seq=step.seq.data_ptr(), out=out.data_ptr(), ldo=out.stride(0))
-    if conv is not None:
-        p.conv = conv
     lib = nv.float_lib()
     if tiles is None:
         nv.check(lib.bxf_recurrence(code(y), ctypes.byref(p), M, nv.stream()), "bxf_recurrence")
         return out
-    chunks = tiles.chunks.shape[0]
-    need = lib.bxf_recurrence_chunk_scratch(kind, M, chunks, H, K)
+    segments = tiles.segments if tiles.segments.shape[0] > tiles.runs.shape[0] else None
+    t = nv.ChunkTable(runs=tiles.runs.data_ptr(), chunks=tiles.chunks.data_ptr(), segments=nv.ptr(segments),
+                      spans=tiles.spans.data_ptr(), nruns=tiles.runs.shape[0], nchunks=tiles.chunks.shape[0],
+                      nsegments=0 if segments is None else segments.shape[0])
+    need = lib.bxf_recurrence_chunk_scratch(kind, M, t.nchunks, t.nsegments, H, K, V)
     scratch = torch.empty(need, dtype=torch.uint8, device=y.device) if need else None
-    rc = lib.bxf_recurrence_chunks(code(y), ctypes.byref(p), tiles.runs.data_ptr(), tiles.runs.shape[0], tiles.chunks.data_ptr(),
-                                   chunks, nv.ptr(scratch), need, M, nv.stream())
+    rc = lib.bxf_recurrence_chunks(code(y), ctypes.byref(p), ctypes.byref(t), nv.ptr(scratch), need, M, nv.stream())
     nv.check(rc, "bxf_recurrence_chunks")
     return out
 

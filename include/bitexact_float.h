@@ -115,13 +115,13 @@ typedef struct {
   int pad_;
 } bxf_gqa_rows;
 
-/* A causal convolution per channel over the rows of a sequence, followed by silu: c[m, ch] = silu(b[ch] + sum_j w[ch, j]
+/* A causal convolution per channel over the rows of a sequence, followed by silu: c[m, ch] = silu(b[ch] + sum_j w[j, ch]
  * u[m - taps + 1 + j, ch]); rows before the step come from the sequence's state (its last taps - 1 inputs, oldest first),
  * rows before the sequence are zero. */
 typedef struct {
   const void* u;                /* T [M, ldu] */
   int64_t ldu;
-  const float *w, *b;           /* [channels, taps], [channels] */
+  const float *w, *b;           /* [taps, channels], [channels] */
   void* state;                  /* T [slots, taps - 1, channels] */
   const int* flags;             /* [M] row flags */
   const int64_t *seq, *pos;     /* [M] */
@@ -134,15 +134,14 @@ typedef struct {
 /* Linear recurrence with a matrix state per head: S_t = diag(a_t) S_(t-1) + k_t v_t^T (K x V), o_t = S_t^T q_t.
  * q, k, v are columns of y (T [M, ldy]) from q0, k0, v0 on: q and k by group (K entries each; head h uses group
  * h / (heads / groups)), v by head.
- *   BXF_DECAY_CHANNEL (groups = heads): side float [M, lds] holds `rank` entries; z = a2 side + a2_b (a2 float [heads K, rank]),
+ *   BXF_DECAY_CHANNEL (groups = heads): side float [M, lds] holds `rank` entries; z = a2 side + a2_b (a2 float [rank, heads K]),
  *     a = sigmoid(z)^inv_tau; q is multiplied by q_scale.
  *   BXF_DECAY_HEAD: side float [M, lds] holds the step sizes before softplus; dt = softplus(side), a = exp(-exp(A_log) dt),
  *     k is multiplied by dt, and skip[h] v_t is added to o_t.
- * conv.w != NULL: y's columns are the inputs of a causal convolution with silu and q, k, v its results (conv.u = column 0 of
- * q0, k0, v0; its state is read only, see bxf_gated_norm).
  * state float [slots, heads, K, V] is advanced by the rows of every sequence; out T [M, ldo] = o (heads concatenated). */
 typedef struct {
-  int kind, heads, groups, K, V, rank, q0, k0, v0, pad_;
+  int kind, heads, groups, K, V, rank, q0, k0, v0;
+  int batch;                    /* bxf_recurrence, bf16: 1 = sequences of one row (decoding) are the usual case */
   const void* y;
   int64_t ldy;
   const float* side;
@@ -150,7 +149,6 @@ typedef struct {
   const float *a2, *a2_b;
   float inv_tau, q_scale;
   const float *A_log, *skip;
-  bxf_conv conv;
   float* state;
   const int* flags;
   const int64_t* seq;
@@ -262,13 +260,19 @@ int bxf_streams(int dtype, const bxf_streams_step* step, int M, void* stream);
 int bxf_causal_conv(int dtype, const bxf_conv* conv, void* out, int64_t ldo, int M, void* stream);
 int bxf_recurrence(int dtype, const bxf_recurrence_rows* rows, int M, void* stream);
 /* The same over prompts, in chunks of up to 64 rows on the tensor cores. bxf_recurrence_chunk_rows: rows of a chunk, 0 when the
- * sizes or the element type do not fit (bxf_recurrence takes those). runs int32 [nruns, 3] = (first row, rows, first chunk) of
- * every sequence of the step; chunks int32 [nchunks, 2] = (first row, rows), cut from every run at multiples of the chunk
- * rows, in the order of the runs. q0, k0, v0, ldy multiples of 8; conv unused. */
+ * sizes or the element type do not fit (bxf_recurrence takes those). q0, k0, v0, ldy multiples of 8. */
+typedef struct {
+  const int* runs;              /* int32 [nruns, 3] = (first row, rows, first chunk) of every sequence of the step */
+  const int* chunks;            /* int32 [nchunks, 2] = (first row, rows): every run cut at multiples of the chunk rows, in order */
+  const int* segments;          /* int32 [nsegments, 3] = (first row, rows, first chunk): every run cut at multiples of chunks;
+                                   they are computed side by side. nsegments 0: one CTA walks a whole run */
+  const int* spans;             /* int32 [nruns, 3] = (first row, first segment, segments) */
+  int nruns, nchunks, nsegments, pad_;
+} bxf_chunk_table;
 int bxf_recurrence_chunk_rows(int dtype, int K, int V);
-size_t bxf_recurrence_chunk_scratch(int kind, int M, int chunks, int heads, int K);
-int bxf_recurrence_chunks(int dtype, const bxf_recurrence_rows* rows, const int* runs, int nruns, const int* chunks,
-                          int nchunks, void* scratch, size_t scratch_bytes, int M, void* stream);
+size_t bxf_recurrence_chunk_scratch(int kind, int M, int chunks, int segments, int heads, int K, int V);
+int bxf_recurrence_chunks(int dtype, const bxf_recurrence_rows* rows, const bxf_chunk_table* table, void* scratch,
+                          size_t scratch_bytes, int M, void* stream);
 int bxf_gated_norm(int dtype, const bxf_gate_rows* rows, int M, void* stream);
 
 #ifdef __cplusplus

@@ -514,22 +514,19 @@ def veredra(args):
         def make():
             state = torch.zeros(B, H, K, V, device=dev)
             if kind == ops.DECAY_CHANNEL:
-                y, side, a2, b = X(M, 2 * gk + inner), F(M, rank), F(gk, rank) * 0.3, F(gk) + 2.0
+                y, side, a2, b = X(M, 2 * gk + inner), F(M, rank), F(rank, gk) * 0.3, F(gk) + 2.0
                 return lambda: ops.recurrence(kind, y, side, state, st, G, (0, gk, 2 * gk), a2=a2, a2_b=b, inv_tau=1 / 16.0,
                                               q_scale=K ** -0.5, tiles=st.tiles)
             u, side, A, s = X(M, inner + 2 * gk), F(M, H) - 2.0, F(H), F(H)
-            w, b, cs = F(inner + 2 * gk, 4) * 0.5, F(inner + 2 * gk), torch.zeros(B, 3, inner + 2 * gk, device=dev, dtype=BF)
-            if st.tiles is None:
-                return lambda: ops.recurrence(kind, u, side, state, st, G, (inner + gk, inner, 0), conv=ops.conv_of(u, w, b, cs, st),
-                                              A_log=A, skip=s)
+            w, b, cs = F(4, inner + 2 * gk) * 0.5, F(inner + 2 * gk), torch.zeros(B, 3, inner + 2 * gk, device=dev, dtype=BF)
             return lambda: ops.recurrence(kind, ops.causal_conv(ops.conv_of(u, w, b, cs, st), M, u), side, state, st, G,
                                           (inner + gk, inner, 0), A_log=A, skip=s, tiles=st.tiles)
         flops = M * H * (4.0 * K * V + (2.0 * 32 * (K + V) if M > 256 else 0))
         byts = n_state + M * (2.0 * (2 * gk + inner) + 2.0 * inner + 4.0 * (rank or H))
         report(name, M, make, flops, byts, byts)
-        if kind == ops.DECAY_HEAD and M > 256:
+        if kind == ops.DECAY_HEAD:
             def conv():
-                u, w, b = X(M, inner + 2 * gk), F(inner + 2 * gk, 4) * 0.5, F(inner + 2 * gk)
+                u, w, b = X(M, inner + 2 * gk), F(4, inner + 2 * gk) * 0.5, F(inner + 2 * gk)
                 cs = torch.zeros(B, 3, inner + 2 * gk, device=dev, dtype=BF)
                 return lambda: (w, b, cs, ops.causal_conv(ops.conv_of(u, w, b, cs, st), M, u))
             report("causal_conv", M, conv, 0, 4.0 * M * (inner + 2 * gk), 4.0 * M * (inner + 2 * gk))

@@ -68,6 +68,11 @@ def test_tables_of_a_portion():
     assert t.runs.tolist() == [[0, 130, 0], [130, 1, 3], [131, 64, 4]]
     assert t.chunks.tolist() == [[0, 64], [64, 64], [128, 2], [130, 1], [131, 64]]
     assert t.attention[50].tolist() == [[4, 0, 50], [4, 50, 50], [4, 100, 30], [2, 130, 1], [0, 131, 50], [0, 181, 14]]
+    assert t.segments.tolist() == t.runs.tolist() and t.spans.tolist() == [[0, 0, 1], [130, 1, 1], [131, 2, 1]]
+    long = Tiles.of([(0, 0, 600, 600), (1, 600, 3, 3)], ())
+    assert long.segments.tolist() == [[0, 256, 0], [256, 256, 4], [512, 88, 8], [600, 3, 10]]
+    assert long.spans.tolist() == [[0, 0, 3], [600, 3, 1]]
+    assert Tiles.of([(0, 0, 5000, 5000)], ()).segments[1].tolist() == [512, 512, 8]
     assert len(t.attention[16]) == 9 + 1 + 4 and Tiles.of([(0, 0, 2, 2)], ()).attention == {}
 
 
@@ -76,7 +81,7 @@ def test_library_checks_its_arguments():
     from bitexact_llm_b200 import build
     build.build(target="float")
     lib = nv.float_lib()
-    sizes = {nv.StreamsStep: 112, nv.GqaRows: 120, nv.Conv: 72, nv.RecurrenceRows: 224, nv.GateRows: 152}
+    sizes = {nv.StreamsStep: 112, nv.GqaRows: 120, nv.Conv: 72, nv.RecurrenceRows: 152, nv.ChunkTable: 48, nv.GateRows: 152}
     assert all(ctypes.sizeof(c) == n for c, n in sizes.items())                  # as asserted in float_capi.cu
     ref = ctypes.byref
     p = nv.StreamsStep(x=16, streams=9, D=8, sum=16)
@@ -90,7 +95,10 @@ def test_library_checks_its_arguments():
     assert lib.bxf_recurrence(0, ref(r), 1, None) == nv.BX_EARG                  # channel decays have a key per head
     r.groups, r.K = 2, 513
     assert lib.bxf_recurrence(0, ref(r), 1, None) == nv.BX_ELIMIT
-    assert lib.bxf_recurrence_chunks(0, ref(r), 16, 1, 16, 1, 16, 1 << 20, 1, None) == nv.BX_ELIMIT
+    t = nv.ChunkTable(runs=16, chunks=16, nruns=1, nchunks=1)
+    assert lib.bxf_recurrence_chunks(0, ref(r), ref(t), 16, 1 << 20, 1, None) == nv.BX_ELIMIT
+    r.K, t.nsegments = 8, 2
+    assert lib.bxf_recurrence_chunks(0, ref(r), ref(t), 16, 1 << 20, 1, None) == nv.BX_EARG             # segments without a table
     assert [lib.bxf_recurrence_chunk_rows(*a) for a in ((0, 128, 64), (0, 12, 64), (0, 16, 12), (0, 264, 8), (1, 128, 64))] == [64, 0, 0, 0, 0]
     epi = nv.Epilogue(kind=4, out=16)
     assert lib.bxf_linear(0, 16, 8, 0, 16, 8, 0, 1, 1, 7, 8, None, ref(epi), 0, None) == nv.BX_EARG    # pairs

@@ -303,14 +303,14 @@ def recurrence_inputs(kind, H, G, K, V, rank, rng, T, dtype, hard=False):
     """(rows y, side, keyword arguments of ops.recurrence, oracle q, k, v, decay, skip)."""
     y = rounded(rng.randn(T, 2 * G * K + H * V), dtype)
     q, k, v = y[:, :G * K].reshape(T, G, K), y[:, G * K:2 * G * K].reshape(T, G, K), y[:, 2 * G * K:].reshape(T, H, V)
-    f32 = lambda a: torch.tensor(a, dtype=torch.float32).cuda()
+    f32 = lambda a: torch.tensor(np.ascontiguousarray(a), dtype=torch.float32).cuda()
     if kind == 0:
         side = rng.randn(T, rank).astype(np.float32)
         a2, b = (rng.randn(H * K, rank) * 0.7).astype(np.float32), (2.0 + rng.randn(H * K)).astype(np.float32)
         if hard:                                                      # rows whose decays reach from none to e^-200
             side[::7] *= 12.0
             side[5::31] -= 40.0
-        kw = dict(a2=f32(a2), a2_b=f32(b), inv_tau=1.0 if hard else 0.125, q_scale=0.3)
+        kw = dict(a2=f32(a2.T), a2_b=f32(b), inv_tau=1.0 if hard else 0.125, q_scale=0.3)
         z = side.astype(np.float64) @ a2.astype(np.float64).T + b
         decay = np.exp(-oh.softplus(-z) * kw["inv_tau"]).reshape(T, H, K)
         return y, side, kw, q * 0.3, k, v, decay, None
@@ -338,7 +338,7 @@ def test_recurrence(kind, H, G, K, V, rank, hard, dtype):
     """Row by row and in chunks, in portions of several sizes of three sequences side by side, slots that held other states."""
     from bitexact_llm_b200.hybrid import ops
     rng = np.random.RandomState(K + V)
-    for cuts in ([200], [2, 3, 1, 64, 65, 1, 64], [130, 70]):
+    for cuts in ([200], [2, 3, 1, 64, 65, 1, 64], [130, 70], [3, 600]):
         T = sum(cuts)
         seqs, first = (3, 1, 2), {}
         for s in seqs:
@@ -347,7 +347,7 @@ def test_recurrence(kind, H, G, K, V, rank, hard, dtype):
         if kind == 0:                                                 # one layer: the same weights for every sequence
             for s in seqs[1:]:
                 y, side, _, q, k, v, _, _ = first[s]
-                z = side.astype(np.float64) @ kw["a2"].double().cpu().numpy().T + kw["a2_b"].double().cpu().numpy()
+                z = side.astype(np.float64) @ kw["a2"].double().cpu().numpy() + kw["a2_b"].double().cpu().numpy()
                 first[s] = (y, side, kw, q, k, v, np.exp(-oh.softplus(-z) * kw["inv_tau"]).reshape(T, H, K), None)
         else:
             A, sk = kw["A_log"].double().cpu().numpy(), kw["skip"].double().cpu().numpy()
@@ -366,7 +366,7 @@ def test_recurrence(kind, H, G, K, V, rank, hard, dtype):
             got, at = {s: [] for s in seqs}, 0
             for n in cuts:
                 runs = [(s, at, n) for s in seqs]
-                st = steps(dtype, runs, 8, 1 + 4 * 30, 4)
+                st = steps(dtype, runs, 8, 1 + 4 * 80, 4)
                 Y = packed(np.concatenate([first[s][0][at:at + n] for s in seqs]), dtype)
                 side = torch.tensor(np.concatenate([first[s][1][at:at + n] for s in seqs])).cuda()
                 o = ops.recurrence(kind, Y, side, state, st, G, (0, G * K, 2 * G * K), tiles=tiles_of(runs) if use_tiles else None, **kw)
@@ -391,7 +391,7 @@ def test_a_state_lasts_over_a_long_pause(dtype):
     decay = np.ones((T, 1, K)) / (1 + np.exp(-9.0))
     o, _ = ov.linear_recurrence(y[:, None, :K], y[:, None, K:2 * K], y[:, None, 2 * K:], decay)
     assert abs(o[-1]).max() > 0.1
-    kw = dict(a2=torch.zeros(K, 1, device="cuda"), a2_b=torch.full((K,), 9.0, device="cuda"), inv_tau=1.0)
+    kw = dict(a2=torch.zeros(1, K, device="cuda"), a2_b=torch.full((K,), 9.0, device="cuda"), inv_tau=1.0)
     for cuts, tiles in (([T], False), ([300, 1, 799], False), ([T], True), ([65, 1035], True)):
         if tiles and dtype == "float32":
             continue
@@ -413,7 +413,7 @@ def test_causal_convolution(taps, channels, dtype):
     rng = np.random.RandomState(taps + channels)
     n_all = 60
     w, b = rng.randn(channels, taps).astype(np.float32), rng.randn(channels).astype(np.float32)
-    W, Bv = torch.tensor(w).cuda(), torch.tensor(b).cuda()
+    W, Bv = torch.tensor(w.T.copy()).cuda(), torch.tensor(b).cuda()
     us = {s: rounded(rng.randn(n_all, channels), dtype) for s in (2, 0)}
     want = {s: oh.silu(ov.causal_conv(u, w.astype(np.float64), b.astype(np.float64))) for s, u in us.items()}
     for cuts in ([60], [1] * 60, [2] * 30, [1, 2, 3, 20, 34]):
