@@ -121,7 +121,7 @@ class RecurrenceRows(ctypes.Structure):
     """bxf_recurrence_rows."""
     _fields_ = [("kind", I), ("heads", I), ("groups", I), ("K", I), ("V", I), ("rank", I), ("q0", I), ("k0", I), ("v0", I),
                 ("batch", I), ("y", P), ("ldy", L), ("side", P), ("lds", L), ("a2", P), ("a2_b", P), ("inv_tau", R),
-                ("q_scale", R), ("A_log", P), ("skip", P), ("state", P), ("flags", P), ("seq", P), ("out", P), ("ldo", L)]
+                ("q_scale", R), ("decays", P), ("A_log", P), ("skip", P), ("state", P), ("flags", P), ("seq", P), ("out", P), ("ldo", L)]
 
 
 class ChunkTable(ctypes.Structure):

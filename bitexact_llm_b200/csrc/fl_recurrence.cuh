@@ -120,28 +120,59 @@ __device__ __forceinline__ void conv_advance(const bxf_conv& c, int m) {
       state[(i64)e * c.channels + ch] = e < R - n ? state[(i64)(e + n) * c.channels + ch] : u[(i64)(m - (R - 1 - e)) * c.ldu + ch];
 }
 
+// ---- decays per channel, a thread each for a few rows ----
+constexpr int DECAY_RANK = 16, DECAY_ROWS = 8;
+
+// sigmoid(z)^inv_tau, its logarithm first.
+__device__ __forceinline__ float log_decay(float z, float inv_tau) { return -softplus(-z) * inv_tau; }
+
+__global__ void __launch_bounds__(256) fl_decay_rows_kernel(const bxf_recurrence_rows p, int M, int rows) {
+  launch_next();
+  const i64 HK = (i64)p.heads * p.K;
+  const int c = blockIdx.x * 256 + threadIdx.x, m0 = blockIdx.y * rows, m1 = min(M, m0 + rows);
+  if (c >= HK) return;
+  const float bias = p.a2_b[c];
+  float z[DECAY_ROWS];
+#pragma unroll
+  for (int r = 0; r < DECAY_ROWS; ++r) z[r] = bias;
+  bool waited = false;
+  for (int j0 = 0; j0 < p.rank; j0 += DECAY_RANK) {
+    float w[DECAY_RANK];
+#pragma unroll
+    for (int j = 0; j < DECAY_RANK; ++j) w[j] = j0 + j < p.rank ? p.a2[(j0 + j) * HK + c] : 0.0f;
+    if (!waited) wait_previous();
+    waited = true;
+#pragma unroll
+    for (int r = 0; r < DECAY_ROWS; ++r) {
+      if (m0 + r >= m1) break;
+      const float* side = p.side + (m0 + r) * p.lds + j0;
+#pragma unroll
+      for (int j = 0; j < DECAY_RANK; ++j)
+        if (j0 + j < p.rank) z[r] = fmaf(w[j], side[j], z[r]);
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < DECAY_ROWS; ++r)
+    if (m0 + r < m1) p.decays[(m0 + r) * HK + c] = expf(log_decay(z[r], p.inv_tau));
+}
+
 // ---- the recurrence row by row: decoding, short portions, 32-bit, any sizes ----
 // One CTA per (sequence of the step, head, 4 CW value columns) walks the sequence's rows with its part of the state in
 // registers: thread = 4 columns x every (256 / CW)th key channel. Rows are prepared in shared memory ROWS at a time (one for
 // decoding). Wide
 // slices share the preparation, narrow ones spread a small batch over more SMs.
-constexpr int REC_THREADS = 256, REC_ROWS = 8, REC_RANK = 16;   // REC_ROWS: most rows at a time
+constexpr int REC_THREADS = 256, REC_ROWS = 8;   // REC_ROWS: most rows at a time
 
 __host__ __device__ constexpr int recurrence_smem(int K, int CW, bool channel, int rows) {
   return (rows * K * (channel ? 3 : 2) + rows * 4 * CW * 9 + 2 * REC_ROWS) * 4;
 }
 
 template <class T, bool CHANNEL, int CW, int KR, int ROWS>
-__global__ void __launch_bounds__(REC_THREADS, CHANNEL || KR > 8 ? 1 : KR <= 4 ? 4 : 3) fl_recurrence_kernel(const bxf_recurrence_rows p, int M) {
+__global__ void __launch_bounds__(REC_THREADS, KR > 8 ? 1 : KR <= 4 ? 4 : 3) fl_recurrence_kernel(const bxf_recurrence_rows p, int M) {
   launch_next();
   extern __shared__ float rec_smem[];
   constexpr int COLS = 4 * CW, LANES = REC_THREADS / CW;
   const int m0 = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * COLS, tid = threadIdx.x;
-  float w2[REC_RANK];                                    // the decay projection's weights of channel tid, entries 0 .. 15
-  if (CHANNEL) {
-#pragma unroll
-    for (int j = 0; j < REC_RANK; ++j) w2[j] = tid < p.K && j < p.rank ? p.a2[((i64)j * p.heads + h) * p.K + tid] : 0.0f;
-  }
   wait_previous();
   const int f0 = p.flags[m0];
   const i64 slot = p.seq[m0];
@@ -182,38 +213,11 @@ __global__ void __launch_bounds__(REC_THREADS, CHANNEL || KR > 8 ? 1 : KR <= 4 ?
       for (int k = tid; k < K; k += REC_THREADS) {
         sq[r * K + k] = ld(row + p.q0 + g * K + k) * (CHANNEL ? p.q_scale : 1.0f);
         sk[r * K + k] = ld(row + p.k0 + g * K + k);
+        if (CHANNEL) sa[r * K + k] = p.decays[((i64)(m + r) * p.heads + h) * K + k];
       }
       if (tid < COLS) sv[r * COLS + tid] = c0 + tid < V ? ld(row + p.v0 + (i64)h * V + c0 + tid) : 0.0f;
     }
-    if (CHANNEL) {
-      for (int k = tid; k < K; k += REC_THREADS) {
-        const float* a2 = p.a2 + h * K + k;
-        const float b = p.a2_b[h * K + k];
-        float z[ROWS];
-#pragma unroll
-        for (int r = 0; r < ROWS; ++r) z[r] = b;
-        for (int j0 = 0; j0 < p.rank; j0 += REC_RANK) {
-          float w[REC_RANK];
-#pragma unroll
-          for (int j = 0; j < REC_RANK; ++j) w[j] = w2[j];
-          if (k != tid || j0 > 0) {
-#pragma unroll
-            for (int j = 0; j < REC_RANK; ++j) w[j] = j0 + j < p.rank ? a2[(i64)(j0 + j) * p.heads * K] : 0.0f;
-          }
-#pragma unroll
-          for (int r = 0; r < ROWS; ++r) {
-            if (r >= n) break;
-            const float* side = p.side + (m + r) * p.lds + j0;
-#pragma unroll
-            for (int j = 0; j < REC_RANK; ++j)
-              if (j0 + j < p.rank) z[r] = fmaf(w[j], side[j], z[r]);
-          }
-        }
-#pragma unroll
-        for (int r = 0; r < ROWS; ++r)
-          if (r < n) sa[r * K + k] = expf(-softplus(-z[r]) * p.inv_tau);
-      }
-    } else if (tid < n) {
+    if (!CHANNEL && tid < n) {
       const float dt = softplus(p.side[(m + tid) * p.lds + h]);
       s_dt[tid] = dt;
       s_dec[tid] = expf(-expf(p.A_log[h]) * dt);

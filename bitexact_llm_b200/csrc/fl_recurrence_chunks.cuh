@@ -83,7 +83,7 @@ fl_decay_prepare_kernel(const bxf_recurrence_rows p, const int* __restrict__ chu
 #pragma unroll
         for (int j = 0; j < RP_RANK; ++j)
           if (j < nj) z = fmaf(w[j], side[t * p.rank + j0 + j], z);
-        la[t * K + k] = j0 + RP_RANK >= p.rank ? -softplus(-z) * p.inv_tau : z;
+        la[t * K + k] = j0 + RP_RANK >= p.rank ? log_decay(z, p.inv_tau) : z;
       }
     }
   }

@@ -19,7 +19,7 @@ namespace {
 using namespace bxf;
 
 static_assert(sizeof(bxf_epilogue) == 136 && sizeof(bxf_gru) == 56 && sizeof(bxf_streams_step) == 112 &&
-                  sizeof(bxf_gqa_rows) == 120 && sizeof(bxf_conv) == 72 && sizeof(bxf_recurrence_rows) == 152 &&
+                  sizeof(bxf_gqa_rows) == 120 && sizeof(bxf_conv) == 72 && sizeof(bxf_recurrence_rows) == 160 &&
                   sizeof(bxf_gate_rows) == 152 && sizeof(bxf_chunk_table) == 48,
               "layouts of the callers' structs");
 
@@ -676,7 +676,15 @@ int bxf_causal_conv(int dtype, const bxf_conv* c, void* out, int64_t ldo, int M,
 int bxf_recurrence(int dtype, const bxf_recurrence_rows* p, int M, void* stream) {
   if (!dtype_ok(dtype) || !recurrence_ok(p) || M < 0) return BX_EARG;
   if (p->K > BXF_MAX_STATE || p->heads > 65535 || ceil_div(p->V, 32) > 65535) return BX_ELIMIT;
+  if (p->kind == BXF_DECAY_CHANNEL && !p->decays) return BX_EARG;
   if (M == 0) return BX_OK;
+  if (p->kind == BXF_DECAY_CHANNEL) {
+    const int rows = M <= 64 ? 1 : DECAY_ROWS;
+    if (ceil_div(M, rows) > 65535) return BX_ELIMIT;
+    const int rc = launch_chained(fl_decay_rows_kernel, dim3(ceil_div(p->heads * p->K, 256), ceil_div(M, rows)), 256, 0,
+                                  stream_of(stream), 0, *p, M, rows);
+    if (rc != BX_OK) return rc;
+  }
   return dtype == BXF_F32 ? launch_recurrence<float>(*p, M, stream_of(stream)) : launch_recurrence<bf16>(*p, M, stream_of(stream));
 }
 

@@ -241,6 +241,9 @@ def recurrence(kind, y, side, state, step, groups, columns, a2=None, a2_b=None, 
                           seq=step.seq.data_ptr(), out=out.data_ptr(), ldo=out.stride(0))
     lib = nv.float_lib()
     if tiles is None:
+        if kind == DECAY_CHANNEL:
+            decays = torch.empty(M, H * K, dtype=torch.float32, device=y.device)
+            p.decays = decays.data_ptr()
         nv.check(lib.bxf_recurrence(code(y), ctypes.byref(p), M, nv.stream()), "bxf_recurrence")
         return out
     segments = tiles.segments if tiles.segments.shape[0] > tiles.runs.shape[0] else None

@@ -148,6 +148,7 @@ typedef struct {
   int64_t lds;
   const float *a2, *a2_b;
   float inv_tau, q_scale;
+  float* decays;                /* bxf_recurrence, BXF_DECAY_CHANNEL: scratch float [M, heads K] */
   const float *A_log, *skip;
   float* state;
   const int* flags;

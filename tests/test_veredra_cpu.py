@@ -81,7 +81,7 @@ def test_library_checks_its_arguments():
     from bitexact_llm_b200 import build
     build.build(target="float")
     lib = nv.float_lib()
-    sizes = {nv.StreamsStep: 112, nv.GqaRows: 120, nv.Conv: 72, nv.RecurrenceRows: 152, nv.ChunkTable: 48, nv.GateRows: 152}
+    sizes = {nv.StreamsStep: 112, nv.GqaRows: 120, nv.Conv: 72, nv.RecurrenceRows: 160, nv.ChunkTable: 48, nv.GateRows: 152}
     assert all(ctypes.sizeof(c) == n for c, n in sizes.items())                  # as asserted in float_capi.cu
     ref = ctypes.byref
     p = nv.StreamsStep(x=16, streams=9, D=8, sum=16)
