@@ -165,29 +165,32 @@ struct ChunkArgs {
 
 enum ChunkPass { WHOLE_RUN, CONTRIBUTION, OUTPUTS };
 
-template <bool CHANNEL, int KT, int NW>
+template <bool CHANNEL, int KT, int NW, ChunkPass PASS>
 struct ChunkCfg {
   static constexpr int KP = 16 * KT, LDK = KP + 8, VS = 16 * NW, LDV = VS + 8, PARTS = CHANNEL ? 2 : 1;
-  static constexpr int QK = RC_ROWS * LDK, V = RC_ROWS * LDV, A = RC_ROWS * RC_LDA;     // bf16 elements
-  static constexpr int SMEM = (2 * PARTS * QK + V + 2 * A) * 2 + (2 * KP + 2 * RC_ROWS) * 4;
-  static constexpr int CTAS = SMEM * 3 <= 224 * 1024 && KT <= 8 && NW <= 4 ? 3 : SMEM * 2 <= 224 * 1024 && KT <= 8 ? 2 : 1;
+  static constexpr int QK = RC_ROWS * LDK, V = RC_ROWS * LDV;             // bf16 elements
+  static constexpr int Q = PASS == CONTRIBUTION ? 0 : PARTS * QK, A = PASS == CONTRIBUTION ? 0 : RC_ROWS * RC_LDA;
+  static constexpr int SMEM = (Q + PARTS * QK + V + 2 * A) * 2 + (3 * KP + 2 * RC_ROWS) * 4;
+  static constexpr int FIT = 224 * 1024 / SMEM;
+  static constexpr int CTAS = KT > 8 || FIT < 2 ? 1 : FIT < 3 ? 2 : PASS == CONTRIBUTION && FIT >= 4 ? 4 : 3;
 };
 
 template <bool CHANNEL, int KT, int NW, ChunkPass PASS>
-__global__ void __launch_bounds__(32 * NW, ChunkCfg<CHANNEL, KT, NW>::CTAS)
+__global__ void __launch_bounds__(32 * NW, ChunkCfg<CHANNEL, KT, NW, PASS>::CTAS)
 fl_recurrence_chunk_kernel(const bxf_recurrence_rows p, const ChunkArgs a) {
-  using Cfg = ChunkCfg<CHANNEL, KT, NW>;
+  using Cfg = ChunkCfg<CHANNEL, KT, NW, PASS>;
   constexpr int LDK = Cfg::LDK, LDV = Cfg::LDV, KP = Cfg::KP, THREADS = 32 * NW;
   launch_next();
   wait_previous();
   extern __shared__ __align__(16) uint8_t rc_smem[];
   bf16* qs = reinterpret_cast<bf16*>(rc_smem);           // [PARTS][64][LDK]
-  bf16* ks = qs + Cfg::PARTS * Cfg::QK;
+  bf16* ks = qs + Cfg::Q;
   bf16* vs = ks + Cfg::PARTS * Cfg::QK;                  // [64][LDV]
   bf16* as = vs + Cfg::V;                                // [2][64][72] scores, high and low parts
   float* first = reinterpret_cast<float*>(as + 2 * Cfg::A);   // [KP] decays of the piece's first row
   float* last = first + KP;                              // [KP] e^(c_last)
-  float* cum = last + KP;                                // [64] BXF_DECAY_HEAD: sums of the log decays
+  float* total = last + KP;                              // [KP] decays of the segment so far
+  float* cum = total + KP;                               // [64] BXF_DECAY_HEAD: sums of the log decays
   float* dts = cum + RC_ROWS;                            // [64] step sizes
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, quad = lane & 3, lrow = lane >> 2;
   const int h = blockIdx.y, K = p.K, V = p.V, c0 = blockIdx.z * Cfg::VS, v0 = c0 + warp * 16;
@@ -204,11 +207,9 @@ fl_recurrence_chunk_kernel(const bxf_recurrence_rows p, const ChunkArgs a) {
                                     : a.states + (((i64)blockIdx.x * p.heads + h) * K) * V);
   float S[2 * KT][4];
   const bool fresh = PASS == CONTRIBUTION || (PASS == WHOLE_RUN && (p.flags[row0] & BXF_ROW_START));
-  float total[PASS == CONTRIBUTION && CHANNEL ? 2 * KT : 1][2], total_log = 0.0f;       // decays of the segment
-  if (PASS == CONTRIBUTION && CHANNEL) {
-#pragma unroll
-    for (int j = 0; j < 2 * KT; ++j) total[j][0] = total[j][1] = 1.0f;
-  }
+  float total_log = 0.0f;
+  if (PASS == CONTRIBUTION && CHANNEL)
+    for (int k = tid; k < KP; k += THREADS) total[k] = 1.0f;
 #pragma unroll
   for (int j = 0; j < 2 * KT; ++j)
 #pragma unroll
@@ -259,6 +260,7 @@ fl_recurrence_chunk_kernel(const bxf_recurrence_rows p, const ChunkArgs a) {
       for (int k = tid; k < KP; k += THREADS) {
         first[k] = k < K ? a.edge[m0 * HK + h * K + k] : 0.0f;
         last[k] = k < K && n > 1 ? a.edge[(m0 + n - 1) * HK + h * K + k] : 1.0f;
+        if (PASS == CONTRIBUTION) total[k] *= first[k] * last[k];         // always this thread's
       }
     } else if (warp == 0) {
       const int t = 2 * lane;
@@ -352,21 +354,25 @@ fl_recurrence_chunk_kernel(const bxf_recurrence_rows p, const ChunkArgs a) {
         for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
           for (int b = 0; b < 2; ++b) split_pair(S[2 * kt + b][2 * nt], S[2 * kt + b][2 * nt + 1], hi[nt][b], lo[nt][b]);
+        uint32_t q[4][4];
+        const int at_q = (b1 * 8 + lm) * LDK + kt * 16 + b2 * 8;
 #pragma unroll
-        for (int mt = 0; mt < 4; ++mt) {
-          uint32_t q[4];
-          const int at_q = (mt * 16 + b1 * 8 + lm) * LDK + kt * 16 + b2 * 8;
-          ldsm4(q, qs + at_q);
+        for (int mt = 0; mt < 4; ++mt) ldsm4(q[mt], qs + at_q + mt * 16 * LDK);
 #pragma unroll
-          for (int nt = 0; nt < 2; ++nt) {
-            mma16816(o[mt][nt], q, hi[nt][0], hi[nt][1]);
-            mma16816(o[mt][nt], q, lo[nt][0], lo[nt][1]);
-          }
-          if (CHANNEL) {
-            ldsm4(q, qs + Cfg::QK + at_q);
+        for (int mt = 0; mt < 4; ++mt)
 #pragma unroll
-            for (int nt = 0; nt < 2; ++nt) mma16816(o[mt][nt], q, hi[nt][0], hi[nt][1]);
-          }
+          for (int nt = 0; nt < 2; ++nt) mma16816(o[mt][nt], q[mt], hi[nt][0], hi[nt][1]);
+#pragma unroll
+        for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+          for (int nt = 0; nt < 2; ++nt) mma16816(o[mt][nt], q[mt], lo[nt][0], lo[nt][1]);
+        if (CHANNEL) {
+#pragma unroll
+          for (int mt = 0; mt < 4; ++mt) ldsm4(q[mt], qs + Cfg::QK + at_q + mt * 16 * LDK);
+#pragma unroll
+          for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt) mma16816(o[mt][nt], q[mt], hi[nt][0], hi[nt][1]);
         }
       }
       if (!CHANNEL) {
@@ -466,27 +472,13 @@ fl_recurrence_chunk_kernel(const bxf_recurrence_rows p, const ChunkArgs a) {
       for (int j = 0; j < 2 * KT; ++j)
 #pragma unroll
         for (int i = 0; i < 4; ++i) S[j][i] *= last[8 * j + 2 * quad + (i & 1)];
-      if (PASS == CONTRIBUTION) {
-#pragma unroll
-        for (int j = 0; j < 2 * KT; ++j)
-#pragma unroll
-          for (int i = 0; i < 2; ++i) total[j][i] *= first[8 * j + 2 * quad + i] * last[8 * j + 2 * quad + i];
-      }
     }
     __syncthreads();                                     // the next piece overwrites the operands
   }
   if (PASS == OUTPUTS) return;
   if (PASS == CONTRIBUTION && blockIdx.z == 0) {
     float* decays = a.decays + ((i64)blockIdx.x * p.heads + h) * K;
-    if (CHANNEL) {
-#pragma unroll
-      for (int j = 0; j < 2 * KT; ++j)
-#pragma unroll
-        for (int i = 0; i < 2; ++i)
-          if (warp == 0 && lrow == 0 && 8 * j + 2 * quad + i < K) decays[8 * j + 2 * quad + i] = total[j][i];
-    } else {
-      for (int k = tid; k < K; k += THREADS) decays[k] = expf(total_log);
-    }
+    for (int k = tid; k < K; k += THREADS) decays[k] = CHANNEL ? total[k] : expf(total_log);
   }
 #pragma unroll
   for (int j = 0; j < 2 * KT; ++j)

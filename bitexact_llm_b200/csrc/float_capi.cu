@@ -392,7 +392,7 @@ ChunkScratch chunk_scratch(int kind, int M, int chunks, int segments, int heads,
 
 template <bool CHANNEL, int KT, int NW, ChunkPass PASS>
 int launch_chunk_pass(const bxf_recurrence_rows& p, const ChunkArgs& a, int n, cudaStream_t st) {
-  using Cfg = ChunkCfg<CHANNEL, KT, NW>;
+  using Cfg = ChunkCfg<CHANNEL, KT, NW, PASS>;
   static PerDevice configured;
   if (once_per_device(configured, [] {
         return cudaFuncSetAttribute(fl_recurrence_chunk_kernel<CHANNEL, KT, NW, PASS>,
