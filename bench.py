@@ -4,7 +4,8 @@
     python bench.py [--gpus N] [--steps K] [--warmup W] [--repeats R] [--batch B] [--prompt P] [--mode exact|int8]
                     [--impl reference] [--workload llama|hybrid|veredra]
 
-`--workload hybrid` measures the hybrid float models beside the integer Llama instead (bench_hybrid.py). Otherwise:
+`--workload hybrid` measures the hybrid float models beside the integer Llama instead, `--workload veredra` the Veredra design
+beside Fedatar (bench_hybrid.py). Otherwise:
 A step is one decode step of the whole batch: 16 layers (4 limb GEMMs, RoPE/KV store, paged attention, attention
 division, two RMSNorms, SiLU per layer), final norm, LM head and the integer Gumbel-max sampler at T = 0.7.
 One process per GPU; with N > 1 (torchrun) every rank decodes its own B sequences (sequence sharding, no
@@ -49,7 +50,8 @@ def parse():
                     help="exact: original bf16 weights as 3 limbs (the headline); int8: int8 weights, 2-limb activations")
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--workload", default="llama", choices=["llama", "hybrid", "veredra"],
-                    help="hybrid: prefill and decode throughput of the hybrid float models beside the integer Llama")
+                    help="hybrid: prefill and decode throughput of the hybrid float models beside the integer Llama; veredra: of "
+                         "the Veredra design beside Fedatar")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-int8-extra", action="store_true", help="skip the int8-mode pass reported under `extra`")
     ap.add_argument("--no-column-sharded", action="store_true",
