@@ -664,7 +664,7 @@ int bxf_causal_conv(int dtype, const bxf_conv* c, void* out, int64_t ldo, int M,
     return launch_chained(fl_causal_conv_kernel<float>, grid, CONV_THREADS, 0, st, 0, *c, static_cast<float*>(out), ldo, M);
   if (c->taps >= 2 && c->taps <= 4 && c->channels % 8 == 0 && c->ldu % 8 == 0 && ldo % 8 == 0 && aligned16(c->u) &&
       aligned16(out) && aligned16(c->state) && aligned16(c->w) && aligned16(c->b)) {
-    const int rows = M <= 512 ? 1 : CONV_ROWS;
+    const int rows = M <= 64 ? 1 : M <= 1024 ? CONV_BATCH : CONV_ROWS;
     const dim3 wide(ceil_div(c->channels, 8 * CONV_THREADS), ceil_div(M, rows));
     return launch_chained(c->taps == 2 ? fl_causal_conv_rows_kernel<2> : c->taps == 3 ? fl_causal_conv_rows_kernel<3>
                                                                                       : fl_causal_conv_rows_kernel<4>,

@@ -560,6 +560,23 @@ def test_the_batch_changes_nothing_beyond_rounding(name):
     assert np.abs(logits(eng, both) - alone).max() < 1e-4 * np.abs(alone).max()
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["looped", "wide"])
+def test_large_decoding_batch(name, dtype):
+    """Eighty sequences of unequal lengths step together: one row each, neighbours in the kernels' row groups."""
+    cfg, _, eng = model(name, dtype)
+    n, more = 80, 3
+    toks = {s: hm.tokens(cfg, 1 + s % 7 + more, 100 + s) for s in range(n)}
+    ses = session(eng, n, 32)
+    order = [(7 * s) % n for s in range(n)]
+    got = {s: [x] for s, x in zip(order, ses.feed([(s, toks[s][:-more]) for s in order]))}
+    for k in range(more):
+        for s, x in zip(order, ses.feed([(s, [toks[s][k - more]]) for s in order])):
+            got[s].append(x)
+    for s in (0, 1, 5, 6, 7, 33, 63, 64, 79):
+        mostly(logits(eng, torch.cat(got[s])), want_logits(name, toks[s]), dtype)
+
+
 @pytest.mark.parametrize("name", list(vm.CONFIGS))
 def test_greedy_generation_of_an_unequal_batch(name):
     from bitexact_llm_b200.decode import generate
