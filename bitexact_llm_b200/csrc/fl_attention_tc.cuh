@@ -8,9 +8,10 @@
 // the softmax warps leave it as bf16 in place of the scores. TMEM: two score buffers of 64 columns, then the output
 // accumulator (256 columns; a wider latent is cut into value slices over blockIdx.z).
 //
-// Warp 0 = TMA, warp 1 = MMA, warps 2 .. 17 = softmax: a query row is shared by four threads (one per warp of its TMEM lane
-// quarter), 16 of the 64 keys each; a decoding tile fills one quarter only, and a single warp per row would be bound by its
-// own latency. The running maximum starts at the sink (denominator 1); the accumulator is rescaled only when the maximum
+// Warp 0 = TMA, warp 1 = MMA, the others = softmax: a query row is shared by PARTS threads (one per warp of its TMEM lane
+// quarter), 64 / PARTS of the 64 keys each; a decoding tile fills one quarter only, and a single warp per row would be bound
+// by its own latency. PARTS = 4: one CTA per SM. PARTS = 2 for values of up to 128 entries: half the TMEM and half the threads,
+// so that two CTAs share an SM and the scores -> softmax -> values chain of one tile runs beside the other's. The running maximum starts at the sink (denominator 1); the accumulator is rescaled only when the maximum
 // grows by more than 2^8 since the last time. Few tiles (decoding): the keys of a tile are split over blockIdx.y, and a
 // second kernel joins the parts.
 #pragma once
@@ -20,7 +21,7 @@
 
 namespace bxf {
 
-constexpr int LT_KEYS = 64, LT_THREADS = 64 + 512, LT_MAX_STAGES = 4, LT_MAX_SPLIT = 8, LT_VCOLS = 256;
+constexpr int LT_KEYS = 64, LT_MAX_STAGES = 4, LT_MAX_SPLIT = 8, LT_VCOLS = 256;
 constexpr int LT_O = 2 * LT_KEYS;                        // first TMEM column of the output accumulator
 constexpr float LT_LOG2E = 1.4426950408889634f;
 constexpr float LT_GROWTH = 8.0f;
@@ -47,8 +48,12 @@ __device__ __forceinline__ float exp2_fast(float v) {
   return r;
 }
 
-// The four warps of a lane quarter.
-__device__ __forceinline__ void quarter_barrier(int quarter) { asm volatile("bar.sync %0, 128;" ::"r"(1 + quarter) : "memory"); }
+// The PARTS warps of a lane quarter.
+template <int PARTS>
+__device__ __forceinline__ void quarter_barrier(int quarter) {
+  asm volatile("bar.sync %0, %1;" ::"r"(1 + quarter), "n"(32 * PARTS) : "memory");
+}
+__host__ __device__ constexpr int lt_threads(int parts) { return 64 + 128 * parts; }
 
 // D (+)= A[tmem] * B[smem]; A: bf16 pairs, one row per lane.
 __device__ __forceinline__ void umma_bf16_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t b_desc, uint32_t idesc,
@@ -71,9 +76,11 @@ __device__ __forceinline__ uint64_t umma_desc_mn(uint32_t addr) {
   return d | static_cast<uint64_t>((LT_KEYS * 128) >> 4) << 16;
 }
 
-__global__ void __launch_bounds__(LT_THREADS, 1)
+template <int PARTS>
+__global__ void __launch_bounds__(lt_threads(PARTS), PARTS == 2 ? 2 : 1)
 fl_paged_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mc,
                              const PagedAttn a, const LatentTc c) {
+  constexpr int TCOLS = PARTS == 2 ? 256 : 512;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* qs = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int q_box = c.qrows * 128;                       // bytes of a column block of the queries
@@ -117,7 +124,7 @@ fl_paged_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gri
     }
     for (int i = 0; i < 2; ++i) {
       mbar_init(&sh->s_full[i], 1);
-      mbar_init(&sh->p_full[i], 4 * quarters);
+      mbar_init(&sh->p_full[i], PARTS * quarters);
       mbar_init(&sh->pv_done[i], 1);
     }
     sh->abort_flag = *reinterpret_cast<volatile int*>(&g_wait_timeouts) != 0;
@@ -127,7 +134,7 @@ fl_paged_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gri
   }
   __syncthreads();
   if (warp == 1) {
-    tmem_alloc(&sh->tmem_base, 512);
+    tmem_alloc(&sh->tmem_base, TCOLS);
     tmem_relinquish();
   }
   tc_fence_before();
@@ -221,7 +228,7 @@ fl_paged_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gri
     }
   } else if ((warp & 3) < quarters) {
     // ---- softmax. A wait that gives up is remembered and the loop goes on (the quarter's barriers count every warp) ----
-    constexpr int KW = LT_KEYS / 4;
+    constexpr int KW = LT_KEYS / PARTS;
     const int quarter = warp & 3, part = (warp - 2) >> 2, r = quarter * 32 + lane;
     const bool live = r < rows;
     const int flat = row0 + (live ? r : 0), token = tok0 + flat / a.H, head = group * a.H + flat % a.H;
@@ -238,7 +245,8 @@ fl_paged_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gri
       __syncwarp();
       tc_fence_after();
       uint32_t u[KW];
-      tmem_ld16(tmem + lanes + buf * LT_KEYS + part * KW, u);
+#pragma unroll
+      for (int k = 0; k < KW; k += 16) tmem_ld16(tmem + lanes + buf * LT_KEYS + part * KW + k, *reinterpret_cast<uint32_t(*)[16]>(u + k));
       tmem_ld_wait();
       const int k0 = (b0 + i) * LT_KEYS + part * KW;
       float s[KW], mx = -INFINITY;
@@ -257,9 +265,10 @@ fl_paged_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gri
       }
       sh->row_max[buf][part][r] = mx;
       tc_fence_before();
-      quarter_barrier(quarter);                            // the quarter's scores are in registers: P may replace them
+      quarter_barrier<PARTS>(quarter);                     // the quarter's scores are in registers: P may replace them
       tc_fence_after();
-      mx = fmaxf(fmaxf(sh->row_max[buf][0][r], sh->row_max[buf][1][r]), fmaxf(sh->row_max[buf][2][r], sh->row_max[buf][3][r]));
+#pragma unroll
+      for (int k = 0; k < PARTS; ++k) mx = fmaxf(mx, sh->row_max[buf][k][r]);
       float f = 1.0f;
       if (mx > ref + LT_GROWTH || ref == -INFINITY) {
         f = ref == -INFINITY ? 0.0f : exp2_fast(ref - mx);
@@ -272,7 +281,7 @@ fl_paged_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gri
           ok = ok && mbar_wait(&sh->pv_done[buf ^ 1], ((i - 1) >> 1) & 1);
           __syncwarp();
           tc_fence_after();
-          for (int q = part * 16; q < vn; q += 64) {
+          for (int q = part * 16; q < vn; q += 16 * PARTS) {
             uint32_t o[16];
             tmem_ld16(tmem + lanes + LT_O + q, o);
             tmem_ld_wait();
@@ -293,7 +302,9 @@ fl_paged_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gri
         w[k] = pack_bf16(e0, e1);
       }
       den += d0 + d1;
-      tmem_st8(tmem + lanes + buf * LT_KEYS + part * (KW / 2), w);
+#pragma unroll
+      for (int k = 0; k < KW / 2; k += 8)
+        tmem_st8(tmem + lanes + buf * LT_KEYS + part * (KW / 2) + k, *reinterpret_cast<const uint32_t(*)[8]>(w + k));
       tmem_st_wait();
       tc_fence_before();
       __syncwarp();
@@ -302,8 +313,10 @@ fl_paged_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gri
     if (nb > 0) ok = ok && mbar_wait(&sh->o_done, 0);
     ok = __all_sync(0xffffffffu, ok);
     sh->row_den[part][r] = den;
-    quarter_barrier(quarter);
-    den = (sh->row_den[0][r] + sh->row_den[1][r]) + (sh->row_den[2][r] + sh->row_den[3][r]);
+    quarter_barrier<PARTS>(quarter);
+    den = 0.0f;
+#pragma unroll
+    for (int k = 0; k < PARTS; ++k) den += sh->row_den[k][r];
     if (!ok) {
       if (lane == 0) fail();
     } else {
@@ -312,7 +325,7 @@ fl_paged_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gri
       const float inv = 1.0f / den;
       float* acc = c.part + (blockIdx.y * n + at) * a.R + v0;
       bf16* out = static_cast<bf16*>(a.out) + token * a.out_tok + head * a.out_head + v0;
-      for (int q = part * 16; q < vn; q += 64) {
+      for (int q = part * 16; q < vn; q += 16 * PARTS) {
         uint32_t u[16] = {};
         if (nb > 0) {
           tmem_ld16(tmem + lanes + LT_O + q, u);
@@ -339,7 +352,7 @@ fl_paged_attention_tc_kernel(const __grid_constant__ CUtensorMap mq, const __gri
   if (warp == 1) {
     __syncwarp();
     tc_fence_after();
-    tmem_dealloc(tmem, 512);
+    tmem_dealloc(tmem, TCOLS);
   }
 }
 

@@ -244,6 +244,15 @@ bool paged_tc_fits(int dtype, const PagedAttn& a) {
          a.ldq % 8 == 0 && a.ldc % 8 == 0 && a.voff % 8 == 0;
 }
 
+// Two CTAs per SM: values in half of the TMEM columns, two key stages in half of the shared memory.
+constexpr int LT_PAIR_SMEM = 113 * 1024;
+
+bool paged_pair_fits(const PagedAttn& a) {
+  const int kcols = ceil_div(a.W, 64), cols = kcols + (a.voff > 0 ? ceil_div(a.R, 64) : 0);
+  const int rows = (a.tiles ? bxf_latent_attention_tile(a.H) : 1) * a.H, qrows = rows >= 128 ? 128 : ceil_div(rows, 8) * 8;
+  return a.R <= 128 && 1024 + kcols * qrows * 128 + (int)sizeof(LatentShared) + 2 * cols * LT_KEYS * 128 <= LT_PAIR_SMEM;
+}
+
 size_t attention_scratch(i64 rows, int R, int splits) { return (size_t)splits * rows * (R + 2) * sizeof(float); }
 
 // Key splits only happen while the query tiles leave SMs idle (148 of them).
@@ -253,11 +262,12 @@ size_t attention_scratch_for(int M, int groups, int heads, int R) {
   return attention_scratch((i64)M * groups * heads, R, splits);
 }
 
+template <int PARTS>
 int launch_paged_tc(const PagedAttn& a, void* scratch, size_t scratch_bytes, cudaStream_t st) {
-  constexpr int SMEM_MAX = 227 * 1024;
+  constexpr int SMEM_MAX = PARTS == 2 ? LT_PAIR_SMEM : 227 * 1024;
   static PerDevice configured;
   if (once_per_device(configured, [] {
-        return cudaFuncSetAttribute(fl_paged_attention_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MAX);
+        return cudaFuncSetAttribute(fl_paged_attention_tc_kernel<PARTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MAX);
       }) != BX_OK)
     return BX_ELAUNCH;
   LatentTc c = {};
@@ -288,7 +298,7 @@ int launch_paged_tc(const PagedAttn& a, void* scratch, size_t scratch_bytes, cud
                      a.bs < LT_KEYS ? a.bs : LT_KEYS, 1))
     return BX_ELAUNCH;
   const dim3 grid(tiles, c.splits, c.row_blocks * c.vsplit * a.G);
-  const int rc = launch_chained(fl_paged_attention_tc_kernel, grid, LT_THREADS, fixed + c.stages * c.cols * LT_KEYS * 128, st,
+  const int rc = launch_chained(fl_paged_attention_tc_kernel<PARTS>, grid, lt_threads(PARTS), fixed + c.stages * c.cols * LT_KEYS * 128, st,
                                 0, mq, mc, a, c);
   if (rc != BX_OK || c.splits == 1) return rc;
   return launch_chained(fl_attention_join_kernel, dim3((unsigned)(a.M * a.H * a.G)), 128, 0, st, 0, a, c.part, c.splits);
@@ -299,7 +309,8 @@ int run_attention(int dtype, const PagedAttn& a, void* scratch, size_t scratch_b
   if (g_status_seen.load() != 0) return BX_EDEVICE;
   if (a.M == 0) return BX_OK;
   if (variant == 2 && !paged_tc_fits(dtype, a)) return BX_ELIMIT;
-  if (variant != 1 && paged_tc_fits(dtype, a) && (!a.tiles || a.ntiles > 0)) return launch_paged_tc(a, scratch, scratch_bytes, st);
+  if (variant != 1 && paged_tc_fits(dtype, a) && (!a.tiles || a.ntiles > 0))
+    return paged_pair_fits(a) ? launch_paged_tc<2>(a, scratch, scratch_bytes, st) : launch_paged_tc<4>(a, scratch, scratch_bytes, st);
   const dim3 grid(a.M, a.H * a.G);
   if (dtype == BXF_F32) fl_paged_attention_kernel<float><<<grid, LA_THREADS, a.W * 4, st>>>(a);
   else fl_paged_attention_kernel<bf16><<<grid, LA_THREADS, a.W * 4, st>>>(a);
