@@ -55,7 +55,8 @@ __device__ __forceinline__ void copies_done() { asm volatile("cp.async.wait_all;
 // piece's first row its decays, in its last row (of several) e^(c_last); masks [chunks][heads]: bit t = row t starts a piece.
 constexpr int RP_THREADS = 256, RP_RANK = 16;
 
-__host__ __device__ constexpr int decay_prepare_smem(int K, int rank) { return (RC_ROWS * K + RC_ROWS * rank) * 4; }
+__host__ __device__ constexpr int decay_ranks(int rank) { return (rank + RP_RANK - 1) / RP_RANK * RP_RANK; }
+__host__ __device__ constexpr int decay_prepare_smem(int K, int rank) { return RC_ROWS * (K + decay_ranks(rank)) * 4; }
 
 __global__ void __launch_bounds__(RP_THREADS)
 fl_decay_prepare_kernel(const bxf_recurrence_rows p, const int* __restrict__ chunks, bf16* __restrict__ planes,
@@ -66,8 +67,10 @@ fl_decay_prepare_kernel(const bxf_recurrence_rows p, const int* __restrict__ chu
   const int K = p.K, h = blockIdx.y, tid = threadIdx.x, row0 = chunks[blockIdx.x * 2], n = chunks[blockIdx.x * 2 + 1];
   const i64 HK = (i64)p.heads * K;
   float* la = rp_smem;                                   // [64][K] log decays, then c
-  float* side = la + RC_ROWS * K;                        // [64][rank]
-  for (int at = tid; at < n * p.rank; at += RP_THREADS) side[at] = p.side[(row0 + at / p.rank) * p.lds + at % p.rank];
+  float* side = la + RC_ROWS * K;                        // [64][rank], zeros up to a multiple of RP_RANK
+  const int R = decay_ranks(p.rank);
+  for (int at = tid; at < n * R; at += RP_THREADS)
+    side[at] = at % R < p.rank ? p.side[(row0 + at / R) * p.lds + at % R] : 0.0f;
   __syncthreads();
   const int lanes = RP_THREADS / K, t0 = tid / K, k = tid % K;
   if (t0 < lanes) {
@@ -75,14 +78,14 @@ fl_decay_prepare_kernel(const bxf_recurrence_rows p, const int* __restrict__ chu
     const float bias = p.a2_b[h * K + k];
     for (int j0 = 0; j0 < p.rank; j0 += RP_RANK) {
       float w[RP_RANK];
-      const int nj = min(RP_RANK, p.rank - j0);
 #pragma unroll
-      for (int j = 0; j < RP_RANK; ++j) w[j] = j < nj ? a2[(j0 + j) * HK] : 0.0f;
+      for (int j = 0; j < RP_RANK; ++j) w[j] = j0 + j < p.rank ? a2[(j0 + j) * HK] : 0.0f;
       for (int t = t0; t < n; t += lanes) {
         float z = j0 == 0 ? bias : la[t * K + k];
+        float s[RP_RANK];
+        load_v<RP_RANK>(side + t * R + j0, s);
 #pragma unroll
-        for (int j = 0; j < RP_RANK; ++j)
-          if (j < nj) z = fmaf(w[j], side[t * p.rank + j0 + j], z);
+        for (int j = 0; j < RP_RANK; ++j) z = fmaf(w[j], s[j], z);
         la[t * K + k] = j0 + RP_RANK >= p.rank ? log_decay(z, p.inv_tau) : z;
       }
     }
@@ -144,7 +147,7 @@ fl_decay_prepare_kernel(const bxf_recurrence_rows p, const int* __restrict__ chu
       const float c0 = la[t * K + d + 2 * i], c1 = la[t * K + d + 2 * i + 1];
       const float e0 = expf(c0), e1 = expf(c1);          // e^-40 at the least: the reciprocals stay finite
       split_pair(q[2 * i] * p.q_scale * e0, q[2 * i + 1] * p.q_scale * e1, o[0][i], o[1][i]);
-      split_pair(kk[2 * i] / e0, kk[2 * i + 1] / e1, o[2][i], o[3][i]);
+      split_pair(__fdividef(kk[2 * i], e0), __fdividef(kk[2 * i + 1], e1), o[2][i], o[3][i]);
     }
 #pragma unroll
     for (int j = 0; j < 4; ++j)

@@ -6,6 +6,7 @@ and adds its output to the rows x, or stores it there. A feed-forward's `run(h, 
 what is still due to x (the experts' outputs, folded into the next norm) or None. Weights arrive as a dict name -> tensor with the
 mechanism's own names ('z', 'dq.norm', 'e0.up', ...)."""
 
+import functools
 import math
 from dataclasses import dataclass, field
 
@@ -76,12 +77,10 @@ def _vec(t, dev):
     return t.to(dev).float().contiguous()
 
 
-def _frequencies(base, dims, dev, made={}):
+@functools.lru_cache(maxsize=None)
+def _frequencies(base, dims, dev):
     """base^(-2 i / dims) in double; layers with the same rotation share the tensor."""
-    key = (base, dims, str(dev))
-    if key not in made:
-        made[key] = torch.tensor([base ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64, device=dev)
-    return made[key]
+    return torch.tensor([base ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64, device=dev)
 
 
 class MinGRU:

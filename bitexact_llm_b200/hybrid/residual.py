@@ -7,10 +7,7 @@ returns the residual float [M, D]. `sub` is what `prepare` made of the sublayer'
 import torch
 
 from . import ops
-
-
-def _vec(t, dev):
-    return t.to(dev).float().contiguous()
+from .layers import _vec
 
 
 class LayerNormResidual:
